@@ -546,9 +546,9 @@ __global__ void __launch_bounds__(THREADS, BLOCKS_PER_SM) k_decode_attn(AttnArgs
  * query slots (16 / G rows x the G heads of the kv group) over the whole key range, so there are no partial states,
  * no workspace and no merge launch: the warp normalises and writes its bf16 outputs itself.
  *
- * The arithmetic differs from the decode kernel's, because here the tensor pipe, not HBM, is the limit, and on this
- * architecture every mma.sync with e4m3 operands costs four extra fp32 adds and operand shuffling around the MMA
- * itself (measured: 546 instructions per page for 32 of them). So the page's bytes are widened to f16 in registers
+ * The arithmetic differs from the decode kernel's, because here the tensor pipe, not HBM, is the limit, and the
+ * instruction counter shows e4m3 mma.sync to be expensive here (546 instructions per page for 32 MMAs with their
+ * fragment loads). So the page's bytes are widened to f16 in registers
  * (exact: e4m3 is a subset of f16) and both contractions run as m16n8k16 f16 MMAs with the QUERY SLOTS as the M
  * dimension: scores S = Q K^T come out as (slot, key) tiles whose accumulator layout is already the A operand layout
  * of P V, so probabilities need no shuffles, and queries (bf16, exact in f16 after a power-of-two scale) and
