@@ -57,6 +57,36 @@ enum {
 
 const char *ncb_status_string(int status);
 
+/*
+ * GEMMs around a residual stream kept in fp32 (entry points *_rs of decode_step, stream_gemm, tile_gemm, and gemm_f32).
+ * The stream is three buffers per row: h fp32 [N], x = h * gain of the norm that reads it (bf16; fp32 in gemm_f32), and
+ * partial sums of squares ss of h. A GEMM that reads the stream multiplies x and scales its fp32 product by the row's
+ * scale / sqrt(sum(ss) / norm_count + eps), which is the RMS norm with a gain; a GEMM that writes the stream adds
+ * mult * product to h, writes x for the next norm's gain and its own partial sums. No norm launch in between.
+ *   epilogue 0: y [rows][ldy] = product; 3: fp32 y [rows][ldy]; both store columns below n_store only.
+ *   epilogue 5: features 2 j and 2 j + 1 are a gate and its value: y[row][j] = gelu_tanh(gate) * value (N / 2 columns).
+ *   epilogue 6: h [rows][N] += mult * product; x_next [rows][N] = h * gain[N]; ss_next [rows][parts] with a count of partial
+ *               sums per row that depends on the entry point (see their declarations).
+ */
+typedef struct {
+    const void *x;      /* [rows][K] */
+    const void *w;      /* [N][K] */
+    void *y;            /* epilogues 0, 3, 5 */
+    long long rows, ldy;
+    int N, K, n_store, epilogue;
+    const float *ss;    /* [rows][ss_parts] or NULL: the product is only multiplied by `scale` */
+    int ss_parts, norm_count;
+    float eps, scale;
+    float *h;           /* epilogue 6 */
+    const float *gain;
+    void *x_next;
+    float *ss_next;
+    float mult;
+    const void *next_w; /* stream_gemm_rs: see stream_gemm */
+    long long next_bytes;
+    int *status;
+} ncb_gemm_rs;
+
 /* ---- library kv_append -------------------------------------------------------------------------------------- */
 
 /* Bytes of one layer's cache for n_slots sequences of at most max_len positions (rounded up to whole pages). */
@@ -318,11 +348,11 @@ int greedy_choice(const void *logits, void *tokens, void *pos, int rows, int voc
  * raw logits; otherwise logits are capped (softcap * tanh(s / softcap), softcap 0: none), optionally cut to the
  * nucleus of mass top_p (keep e >= e*, the least e whose cumulative mass from below exceeds (1 - top_p) of the
  * total; bisection on IEEE bits) and sampled by Gumbel-max with Philox4x32-10 noise at counter (token id,
- * pos - first), key seed. Ties to the lowest id; `allow` (uint32 [rows][vocab / 32], may be NULL) masks tokens.
+ * pos - first), key seed. Ties to the lowest id; `allow` (uint32 [rows][ceil(vocab / 32)], may be NULL) masks tokens.
  * tokens[row] = choice (-1 if the mask allows nothing; embed_norm reads a token outside the vocabulary as token 0),
  * pos[row] += 1, trace as greedy_choice; idle rows (pos[row] < 0) are left alone.
  * logits fp32 [rows][vocab]; probs fp32 [rows][vocab] scratch; temperature, top_p fp32 [rows]; seed uint64 [rows];
- * first int32 [rows]; vocab a multiple of 32.
+ * first int32 [rows].
  */
 int sample_choice(const void *logits, void *probs, const void *temperature, const void *top_p, const void *seed,
                   const void *first, const void *allow, float softcap, void *tokens, void *pos, int rows, int vocab,
@@ -384,6 +414,84 @@ int tile_gemm(const void *x, const void *w, const void *resid, void *y, long lon
  */
 int tile_gemm_form(const void *x, const void *w, const void *resid, void *y, long long rows, int N, int K, int epilogue,
                    int form, int *status, void *stream);
+
+/* ---- library gla ---------------------------------------------------------------------------------------------------
+ * Gated linear attention with a decay per key channel (csrc/gla.cu has the recurrence). proj, out: bf16, or fp32 when
+ * the entry point's f32 is not 0. proj rows hold q, k [heads dim], v, gate [heads vdim] and the low-rank decay input
+ * [rank] at the given element offsets; dim and vdim multiples of 16 (zero-padded channels stay zero), norm_count the
+ * vdim that counts in the norm. state fp32 [n_slots][heads][dim][vdim]. Rows of a segment are consecutive, of one slot
+ * and at ascending positions; a row at position 0 starts from a zero state; a segment whose first position is negative
+ * is idle. out NULL: only the state is advanced.
+ *   gla_step     token by token; seg_first NULL: every row is a segment.
+ *   gla_chunked  segments cut into chunks of at most gla_chunk_tokens(dim) rows (= chunk): chunk_first / chunk_count
+ *                [n_chunks], seg_chunk [n_segments + 1] (a segment's first chunk). Scratch: decay fp32 [rows][heads dim],
+ *                chunk_decay fp32 [n_chunks][heads dim], states fp32 [n_chunks][heads][dim][vdim], raw fp32
+ *                [rows][heads][vdim]. Four launches. */
+typedef struct {
+    const void *proj;
+    void *out;
+    long long rows, ldp, ldo;
+    int off_q, off_k, off_v, off_g, off_a;
+    int heads, dim, vdim, rank, norm_count, n_slots;
+    float q_scale, inv_tau, eps;
+    const float *a2, *a2_bias, *norm; /* fp32 [heads dim][rank], [heads dim], [vdim] */
+    float *state;
+    const int *pos, *slot_map;        /* per row; slot_map NULL: row r is slot r */
+    const int *seg_first, *seg_count, *seg_chunk, *chunk_first, *chunk_count;
+    int n_segments, n_chunks, chunk;
+    float *decay, *chunk_decay, *states, *raw;
+    int *status;
+} ncb_gla;
+int gla_chunk_tokens(int dim);
+int gla_step(const ncb_gla *args, int f32, void *stream);
+int gla_chunked(const ncb_gla *args, int f32, void *stream);
+
+/* ---- library latent_attn -------------------------------------------------------------------------------------------
+ * Latent attention over a cache of [latent | rotated key] rows (csrc/latent_attn.cu has the mathematics and the layout).
+ * proj, q_abs, cache, w_*, out: bf16, or fp32 when the entry point's f32 is not 0. proj rows hold per head [dim | rot] of q
+ * at off_q, [rank | rot] at off_kv and the gate [heads vdim] at off_g. dim and rank multiples of 32, rot and vdim of 16
+ * (zero-padded values stay zero; rotated pairs are i and i + rot / 2); norm_count the latent values that count in the norm.
+ * cos, sin fp32 [table_len][rot / 2] by absolute position. cache [n_slots][capacity][rank + rot]. Rows with a negative
+ * position are idle: nothing appended, a zero output row; rows outside the cache are skipped and flagged.
+ *   latent_append  norm, rotate, append; with rotate_q also rotates proj's q in place (expanded form)
+ *   latent_query   the same append, and q_abs [rows][heads][rank + rot] = [w_uk_t q | rotated q]; w_uk_t [heads][rank][dim]
+ *   latent_split   states of chunks of at most chunk_tiles tiles of NCB_LATENT_TILE positions: parts fp32
+ *                  [rows][heads][max_chunks][rank + 4]; max_len bounds every position + 1
+ *   latent_out     out [rows][ldo] = sigmoid(gate) * w_uv merged(states); w_uv [heads][vdim][rank]; sink fp32 [heads] or
+ *                  NULL; gated 0: no gate */
+#define NCB_LATENT_TILE 32
+typedef struct {
+    void *proj;
+    void *q_abs, *cache, *out;
+    const void *w_uk_t, *w_uv;
+    long long rows, ldp, ldo;
+    int off_q, off_kv, off_g, gated, rotate_q;
+    int heads, dim, rot, vdim, rank, norm_count;
+    int n_slots, capacity, table_len, max_len, chunk_tiles, max_chunks;
+    float scale, eps;
+    const float *norm, *cos, *sin, *sink;
+    const int *pos, *slot_map; /* per row; slot_map NULL: row r is slot r */
+    float *parts;
+    int *status;
+} ncb_latent;
+int latent_append(const ncb_latent *args, int f32, void *stream);
+int latent_query(const ncb_latent *args, int f32, void *stream);
+int latent_split(const ncb_latent *args, int f32, void *stream);
+int latent_out(const ncb_latent *args, int f32, void *stream);
+
+/* ---- GEMMs around an fp32 residual stream (ncb_gemm_rs above) ------------------------------------------------
+ * Shapes as for the plain entry points: skinny_gemm_rs at most 16 rows, K as skinny_gemm without norm, N a multiple of 8,
+ * N / 8 partial sums; stream_gemm_rs at most 256 rows, N a multiple of 128, K of 64, N / 128 partial sums; tile_gemm_rs
+ * any rows, same multiples, N / 32 partial sums; gemm_f32_rs (library gemm_f32: x, w, y, x_next fp32, plain FMA
+ * arithmetic) any rows, N and K multiples of 64, N / 64 partial sums. */
+int skinny_gemm_rs(const ncb_gemm_rs *args, void *stream);
+int stream_gemm_rs(const ncb_gemm_rs *args, void *stream);
+int tile_gemm_rs(const ncb_gemm_rs *args, void *stream);
+int gemm_f32_rs(const ncb_gemm_rs *args, void *stream);
+/* The stream's first rows: h fp32 [rows][C] = embed[tokens], x = h * gain, ss fp32 [rows] (one partial sum per row).
+ * embed, x: bf16, or fp32 with f32 != 0; C columns are read, all of them written. A token outside [0, vocab) reads row 0. */
+int embed_rs(const void *embed, const void *tokens, void *h, const void *gain, void *x, void *ss, long long rows, int C,
+             int vocab, int f32, void *stream);
 
 #ifdef __cplusplus
 }

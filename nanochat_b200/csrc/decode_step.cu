@@ -24,15 +24,14 @@
  * These kernels wait for their predecessor with griddepcontrol.wait and are launched with programmatic stream
  * serialisation, so inside a captured step the launch of each overlaps the tail of the one before.
  */
-#include "ncb_common.cuh"
+#include "gemm_rs.cuh"
 
 constexpr int GEMM_WARPS = 8;
 constexpr int GEMM_THREADS = GEMM_WARPS * 32;
 constexpr int TILE_N = 8;         /* output features per block */
 constexpr int MAX_ROWS = 16;
-constexpr int MAX_K_ITERS = 20;   /* 32 k-values per iteration and warp: K <= 8 * 20 * 32 = 5120 */
 
-enum { EPI_STORE = 0, EPI_RESID = 1, EPI_RELU2 = 2, EPI_F32 = 3, EPI_MIX = 4 };
+enum { EPI_STORE = 0, EPI_RESID = 1, EPI_RELU2 = 2, EPI_F32 = 3, EPI_MIX = 4, EPI_GEGLU = 5, EPI_STREAM = 6 };
 
 struct GemmArgs {
     const bf16 *x;     /* [rows][K] */
@@ -42,6 +41,9 @@ struct GemmArgs {
     int rows, N, K, norm_input;
     const bf16 *x0;    /* EPI_MIX: [rows][N], the first normed embedding rows */
     float l1, l2;      /* EPI_MIX: the next layer's (resid_lambda, x0_lambda) */
+    long long ldy;     /* row stride of y for EPI_STORE, EPI_F32 and EPI_GEGLU */
+    int n_store;       /* columns below this are stored (EPI_STORE, EPI_F32) */
+    StreamIO rs;       /* row scale of the product, EPI_STREAM's outputs */
 };
 
 /* The per-layer stream mix of the reference's model (inference/modeling_nanochat.py:170-171; decode.cu:430-432):
@@ -156,6 +158,14 @@ __global__ void __launch_bounds__(GEMM_THREADS, ITERS > 8 ? 2 : 1) k_skinny_gemm
             if (HI) xhi[i] = scale_bf16x8(xhi[i], r_hi);
         }
     }
+    if (!NORM) { /* row scales from the stream's partial sums: 16 threads per row (first read behind a barrier) */
+        const int row = tid >> 4;
+        float s = 0.f;
+        if (a.rs.ss && row < a.rows)
+            for (int i = tid & 15; i < a.rs.ss_parts; i += 16) s += a.rs.ss[(size_t)row * a.rs.ss_parts + i];
+        for (int o = 8; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+        if ((tid & 15) == 0) rstd[row] = row_scale(a.rs, s);
+    }
     for (; tile < tiles; tile += gridDim.x) {
         float acc[4] = {0.f, 0.f, 0.f, 0.f}, acc2[4] = {0.f, 0.f, 0.f, 0.f}; /* two chains: MMA latency overlaps */
 #pragma unroll
@@ -194,13 +204,31 @@ __global__ void __launch_bounds__(GEMM_THREADS, ITERS > 8 ? 2 : 1) k_skinny_gemm
         __syncthreads();
         if (tid < 16 * TILE_N) {
             const int row = tid / TILE_N, col = tid % TILE_N;
-            if (row < a.rows) {
-                float v = 0.f;
+            float v = 0.f;
 #pragma unroll
-                for (int w = 0; w < GEMM_WARPS; w++) v += part[w][row][col];
-                const size_t at = (size_t)row * a.N + (size_t)tile * TILE_N + col;
-                if (EPI == EPI_F32) {
-                    reinterpret_cast<float *>(a.y)[at] = v;
+            for (int w = 0; w < GEMM_WARPS; w++) v += part[w][row][col];
+            if (!NORM) v *= rstd[row];
+            const size_t at = (size_t)row * a.N + (size_t)tile * TILE_N + col;
+            if (EPI == EPI_GEGLU) {
+                const float up = __shfl_xor_sync(0xffffffffu, v, 1);
+                if (row < a.rows && (col & 1) == 0)
+                    reinterpret_cast<bf16 *>(a.y)[row * a.ldy + tile * (TILE_N / 2) + col / 2] = __float2bfloat16_rn(gelu_tanh(v) * up);
+            } else if (EPI == EPI_STREAM) {
+                float hv = 0.f;
+                if (row < a.rows) {
+                    hv = stream_add(a.rs, at, v);
+                    reinterpret_cast<bf16 *>(a.rs.x_next)[at] = __float2bfloat16_rn(hv * a.rs.gain[tile * TILE_N + col]);
+                }
+                float q = hv * hv;
+                for (int o = 1; o < TILE_N; o <<= 1) q += __shfl_xor_sync(0xffffffffu, q, o);
+                if (row < a.rows && col == 0) a.rs.ss_next[(size_t)row * tiles + tile] = q;
+            } else if (row < a.rows) {
+                if (EPI == EPI_F32 || EPI == EPI_STORE) {
+                    const int c = tile * TILE_N + col;
+                    if (c < a.n_store) {
+                        if (EPI == EPI_F32) reinterpret_cast<float *>(a.y)[row * a.ldy + c] = v;
+                        else reinterpret_cast<bf16 *>(a.y)[row * a.ldy + c] = __float2bfloat16_rn(v);
+                    }
                 } else {
                     bf16 out = __float2bfloat16_rn(v);
                     if (EPI == EPI_RESID || EPI == EPI_MIX)
@@ -243,6 +271,31 @@ __global__ void __launch_bounds__(128) k_embed_norm(const bf16 *embed, const lon
         }
         *reinterpret_cast<uint4 *>(h + (size_t)row * C + i) = v;
     }
+}
+
+/* The first rows of an fp32 residual stream: h = embed[token], x = h * gain for the first norm, one sum of squares. */
+constexpr int EMBED_THREADS = 128;
+template <typename T>
+__global__ void __launch_bounds__(EMBED_THREADS) k_embed_rs(const T *embed, const long long *tokens, float *h, const float *gain,
+                                                            T *x, float *ss, int C, int vocab) {
+    __shared__ float warp_sums[EMBED_THREADS / 32];
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    long long token = tokens[blockIdx.x];
+    if (token < 0 || token >= vocab) token = 0;
+    const T *e = embed + (size_t)token * C;
+    const size_t base = (size_t)blockIdx.x * C;
+    float s = 0.f;
+    for (int i = threadIdx.x; i < C; i += EMBED_THREADS) {
+        const float v = (float)e[i];
+        h[base + i] = v;
+        x[base + i] = (T)(v * gain[i]);
+        s += v * v;
+    }
+    for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+    if ((threadIdx.x & 31) == 0) warp_sums[threadIdx.x >> 5] = s;
+    __syncthreads();
+    if (threadIdx.x == 0) ss[blockIdx.x] = (warp_sums[0] + warp_sums[1]) + (warp_sums[2] + warp_sums[3]);
 }
 
 /* h[row] += y[row] (bf16 add, skipped when y is NULL), n[row] = rms_norm(h[row]); one block of 256 threads per row,
@@ -402,7 +455,7 @@ struct SampleArgs {
     const float *temperature, *top_p; /* [rows] */
     const unsigned long long *seed;   /* [rows] */
     const int32_t *first;      /* [rows]: the position of each row's first generated token's input (step = pos - first) */
-    const uint32_t *allow;     /* [rows][vocab / 32] or NULL */
+    const uint32_t *allow;     /* [rows][ceil(vocab / 32)] or NULL */
     long long *tokens;
     int32_t *pos;
     long long *trace;
@@ -420,7 +473,7 @@ __global__ void __launch_bounds__(SAMPLE_THREADS) k_sample(SampleArgs a) {
     if (a.pos[b] < 0) return; /* an idle row (the whole block leaves): no choice, no advance */
     const float *s = a.logits + (size_t)b * V;
     float *e = a.probs + (size_t)b * V;
-    const uint32_t *allow = a.allow ? a.allow + (size_t)b * (V / 32) : nullptr;
+    const uint32_t *allow = a.allow ? a.allow + (size_t)b * ((V + 31) / 32) : nullptr;
     const float T = a.temperature[b], top_p = a.top_p[b];
     const bool sampled = T > 0.f, nucleus = sampled && top_p < 1.f;
     const int step = a.pos[b] - a.first[b];
@@ -535,8 +588,13 @@ template <int ITERS, bool HI, bool NORM> static int launch_gemm_epi(const GemmAr
     case EPI_RELU2: { auto k = k_skinny_gemm<ITERS, HI, EPI_RELU2, NORM>; return launch_pdl(k, dim3(grid_for(k, tiles, ITERS <= 8)), block, stream, a); }
     case EPI_F32: { auto k = k_skinny_gemm<ITERS, HI, EPI_F32, NORM>; return launch_pdl(k, dim3(grid_for(k, tiles, ITERS <= 8)), block, stream, a); }
     case EPI_MIX: { auto k = k_skinny_gemm<ITERS, HI, EPI_MIX, NORM>; return launch_pdl(k, dim3(grid_for(k, tiles, ITERS <= 8)), block, stream, a); }
-    default: return NCB_ERR_ARG;
+    default: break;
     }
+    if constexpr (!NORM) { /* the residual-stream forms scale by row instead of norming their input */
+        if (epilogue == EPI_GEGLU) { auto k = k_skinny_gemm<ITERS, HI, EPI_GEGLU, false>; return launch_pdl(k, dim3(grid_for(k, tiles, ITERS <= 8)), block, stream, a); }
+        if (epilogue == EPI_STREAM) { auto k = k_skinny_gemm<ITERS, HI, EPI_STREAM, false>; return launch_pdl(k, dim3(grid_for(k, tiles, ITERS <= 8)), block, stream, a); }
+    }
+    return NCB_ERR_ARG;
 }
 
 template <int ITERS> static int launch_gemm_rows(const GemmArgs &a, int epilogue, cudaStream_t stream) {
@@ -563,7 +621,7 @@ static int launch_skinny(const GemmArgs &a, int epilogue, cudaStream_t s) {
     if (rows < 0 || rows > MAX_ROWS || N <= 0 || K <= 0 || N % TILE_N || K % (GEMM_WARPS * 32)) return NCB_ERR_ARG;
     if (!skinny_depth_ok(K)) return NCB_ERR_UNSUPPORTED;
     if (rows == 0) return NCB_OK;
-    if (!a.x || !a.w || !a.y || ((epilogue == EPI_RESID || epilogue == EPI_MIX) && !a.resid) ||
+    if (!a.x || !a.w || (!a.y && epilogue != EPI_STREAM) || ((epilogue == EPI_RESID || epilogue == EPI_MIX) && !a.resid) ||
         (epilogue == EPI_MIX && !a.x0))
         return NCB_ERR_ARG;
     if (((uintptr_t)a.x | (uintptr_t)a.w) % 16 || (uintptr_t)a.y % 4) return NCB_ERR_ALIGN;
@@ -602,7 +660,8 @@ int skinny_gemm_supported(int rows, int N, int K, int norm_input) {
 int skinny_gemm(const void *x, const void *w, const void *resid, void *y, int rows, int N, int K, int norm_input,
                 int epilogue, void *stream) {
     if (epilogue < EPI_STORE || epilogue > EPI_F32) return NCB_ERR_ARG;
-    const GemmArgs a = {(const bf16 *)x, (const bf16 *)w, (const bf16 *)resid, y, rows, N, K, norm_input, nullptr, 1.f, 0.f};
+    const GemmArgs a = {(const bf16 *)x, (const bf16 *)w, (const bf16 *)resid, y, rows, N, K, norm_input, nullptr, 1.f, 0.f,
+                        N, N, no_stream()};
     return launch_skinny(a, epilogue, (cudaStream_t)stream);
 }
 
@@ -610,8 +669,33 @@ int skinny_gemm(const void *x, const void *w, const void *resid, void *y, int ro
  * y = bf16(l1 * bf16(resid + bf16(x . W^T)) + l2 * x0), x0 bf16 [rows][N]. */
 int skinny_gemm_mix(const void *x, const void *w, const void *resid, const void *x0, float l1, float l2, void *y, int rows,
                     int N, int K, int norm_input, void *stream) {
-    const GemmArgs a = {(const bf16 *)x, (const bf16 *)w, (const bf16 *)resid, y, rows, N, K, norm_input, (const bf16 *)x0, l1, l2};
+    const GemmArgs a = {(const bf16 *)x, (const bf16 *)w, (const bf16 *)resid, y, rows, N, K, norm_input, (const bf16 *)x0, l1, l2,
+                        N, N, no_stream()};
     return launch_skinny(a, EPI_MIX, (cudaStream_t)stream);
+}
+
+/* skinny_gemm on a residual stream kept in fp32 (ncb_gemm_rs): the input's norm is a row scale of the product, epilogues
+ * store, fp32 store, gated unit, stream update. */
+int skinny_gemm_rs(const ncb_gemm_rs *g, void *stream) {
+    if (!g || g->rows > MAX_ROWS) return NCB_ERR_ARG;
+    const int rc = check_rs(*g);
+    if (rc != NCB_OK) return rc;
+    const GemmArgs a = {(const bf16 *)g->x, (const bf16 *)g->w, nullptr, g->y, (int)g->rows, g->N, g->K, 0, nullptr, 1.f, 0.f,
+                        g->ldy, g->n_store, stream_io(*g)};
+    return launch_skinny(a, g->epilogue, (cudaStream_t)stream);
+}
+
+int embed_rs(const void *embed, const void *tokens, void *h, const void *gain, void *x, void *ss, long long rows, int C,
+             int vocab, int f32, void *stream) {
+    if (rows < 0 || rows > 0x7fffffffLL || C <= 0 || vocab <= 0) return NCB_ERR_ARG;
+    if (rows == 0) return NCB_OK;
+    if (!embed || !tokens || !h || !gain || !x || !ss) return NCB_ERR_ARG;
+    const dim3 grid((unsigned)rows), block(EMBED_THREADS);
+    if (f32)
+        return launch_pdl(k_embed_rs<float>, grid, block, (cudaStream_t)stream, (const float *)embed, (const long long *)tokens,
+                          (float *)h, (const float *)gain, (float *)x, (float *)ss, C, vocab);
+    return launch_pdl(k_embed_rs<bf16>, grid, block, (cudaStream_t)stream, (const bf16 *)embed, (const long long *)tokens,
+                      (float *)h, (const float *)gain, (bf16 *)x, (float *)ss, C, vocab);
 }
 
 static int launch_embed(const void *embed, const void *tokens, void *h, void *x0, float l1, float l2, int mix, int rows,
@@ -684,13 +768,13 @@ int greedy_choice(const void *logits, void *tokens, void *pos, int rows, int voc
  * tokens[row] = the reference's choice for logits fp32 [rows][vocab] (see "sampling" above); pos[row] += 1; the
  * choice is logged in trace like greedy_choice does (-1 when the mask allows no token).
  *   temperature, top_p fp32 [rows]; seed uint64 [rows]; first int32 [rows] (step = pos - first picks the noise);
- *   allow uint32 [rows][vocab / 32] or NULL; probs fp32 [rows][vocab] scratch (used when top_p < 1);
- *   softcap: the logit cap c applied to sampled rows (0: none). vocab a multiple of 32.
+ *   allow uint32 [rows][ceil(vocab / 32)] or NULL; probs fp32 [rows][vocab] scratch (used when top_p < 1);
+ *   softcap: the logit cap c applied to sampled rows (0: none). allow rows are ceil(vocab / 32) words.
  */
 int sample_choice(const void *logits, void *probs, const void *temperature, const void *top_p, const void *seed,
                   const void *first, const void *allow, float softcap, void *tokens, void *pos, int rows, int vocab,
                   void *trace, int trace_stride, void *stream) {
-    if (rows < 0 || vocab <= 0 || vocab % 32 || softcap < 0.f) return NCB_ERR_ARG;
+    if (rows < 0 || vocab <= 0 || softcap < 0.f) return NCB_ERR_ARG;
     if (rows == 0) return NCB_OK;
     if (!logits || !probs || !temperature || !top_p || !seed || !first || !tokens || !pos) return NCB_ERR_ARG;
     const SampleArgs a = {(const float *)logits, (float *)probs, (const float *)temperature, (const float *)top_p,

@@ -22,6 +22,7 @@
  * Every mbarrier wait is bounded; on expiry NCB_DEV_WAIT_TIMEOUT is flagged and the block still walks through both
  * cluster barriers and frees its tensor memory.
  */
+#include "gemm_rs.cuh"
 #include "umma.cuh"
 
 #include <cooperative_groups.h>
@@ -36,7 +37,7 @@ constexpr int RING_KB_SMALL = 100;               /* ring of the <= 128-row shape
 constexpr int THREADS = 128;
 constexpr int MAX_SPLIT = 8;                     /* portable cluster size */
 
-enum { EPI_STORE = 0, EPI_RESID = 1, EPI_RELU2 = 2, EPI_F32 = 3, EPI_MIX = 4 };
+enum { EPI_STORE = 0, EPI_RESID = 1, EPI_RELU2 = 2, EPI_F32 = 3, EPI_MIX = 4, EPI_GEGLU = 5, EPI_STREAM = 6 };
 
 template <int NP> struct Shape {
     /* A stage holds KSUB consecutive boxes of W and the matching boxes of x. Wider stages (2 or 4 boxes, i.e. 256
@@ -65,6 +66,9 @@ struct GemmArgs {
     int *status;
     const bf16 *x0; /* EPI_MIX: [rows][N], the first normed embedding rows */
     float l1, l2;   /* EPI_MIX: the next layer's (resid_lambda, x0_lambda) */
+    long long ldy;  /* row stride of y for EPI_STORE, EPI_F32 and EPI_GEGLU */
+    int n_store;    /* columns below this are stored (EPI_STORE, EPI_F32) */
+    StreamIO rs;    /* row scale of the product (norm_input == 0), EPI_STREAM's outputs */
 };
 
 __device__ __forceinline__ float sumsq_bf16x8(const uint4 &u) {
@@ -192,6 +196,14 @@ __global__ void __launch_bounds__(THREADS) k_stream_gemm(const __grid_constant__
         }
     }
     if (tid != 0) asm volatile("griddepcontrol.wait;" ::: "memory");
+    if (warp >= 2 && !a.norm_input) { /* row scales from the stream's partial sums; every block needs every row's */
+        for (int r = tid - 64; r < a.rows; r += 64) {
+            float v = 0.f;
+            if (a.rs.ss)
+                for (int i = 0; i < a.rs.ss_parts; i++) v += a.rs.ss[(size_t)r * a.rs.ss_parts + i];
+            sumsq[r] = row_scale(a.rs, v);
+        }
+    }
     if (warp >= 2 && a.norm_input) {
         /* Sums of squares of x[:, this block's K slice] from the staged x boxes: warp 2 takes the lower half of the
          * rows, warp 3 the upper; 8 lanes read one row's 128 bytes (the swizzle only permutes 16-byte chunks inside
@@ -265,13 +277,38 @@ __global__ void __launch_bounds__(THREADS) k_stream_gemm(const __grid_constant__
                 const int r = c * 32 + j;
                 res[j] = HAS_RESID && r < a.rows ? __bfloat162float(a.resid[(size_t)r * a.N + col]) : 0.f;
                 if (EPI == EPI_MIX) mix[j] = r < a.rows ? __bfloat162float(a.x0[(size_t)r * a.N + col]) : 0.f;
-                if (a.norm_input) v[j] *= rsqrtf(sumsq[r] * inv_k + FLT_EPSILON);
+                if (r < a.rows) v[j] *= a.norm_input ? rsqrtf(sumsq[r] * inv_k + FLT_EPSILON) : sumsq[r];
             }
 #pragma unroll
             for (int j = 0; j < 32; j++) {
                 const int r = c * 32 + j;
-                if (r < a.rows) finish(v[j], res[j], EPI == EPI_MIX ? mix[j] : 0.f, (size_t)r * a.N + col);
+                if (EPI == EPI_GEGLU) { /* gate and value are neighbouring features, so neighbouring lanes */
+                    const float up = __shfl_down_sync(0xffffffffu, v[j], 1);
+                    if (r < a.rows && (tid & 1) == 0)
+                        reinterpret_cast<bf16 *>(a.y)[r * a.ldy + (col >> 1)] = __float2bfloat16_rn(gelu_tanh(v[j]) * up);
+                } else if (EPI == EPI_STREAM) {
+                    const size_t at = (size_t)r * a.N + col;
+                    float h = 0.f;
+                    if (r < a.rows) {
+                        h = stream_add(a.rs, at, v[j]);
+                        reinterpret_cast<bf16 *>(a.rs.x_next)[at] = __float2bfloat16_rn(h * a.rs.gain[col]);
+                    }
+                    h *= h;
+                    for (int o = 16; o > 0; o >>= 1) h += __shfl_xor_sync(0xffffffffu, h, o);
+                    if (lane == 0) park[warp * NP + r] = h; /* the ring is free: every staged box has been consumed */
+                } else if (r < a.rows) {
+                    if (EPI == EPI_STORE || EPI == EPI_F32) {
+                        if ((int)col < a.n_store) finish(v[j], 0.f, 0.f, (size_t)r * a.ldy + col);
+                    } else {
+                        finish(v[j], res[j], EPI == EPI_MIX ? mix[j] : 0.f, (size_t)r * a.N + col);
+                    }
+                }
             }
+        }
+        if (EPI == EPI_STREAM) {
+            __syncthreads();
+            for (int r = tid; r < a.rows; r += THREADS)
+                a.rs.ss_next[(size_t)r * gridDim.y + tile] = (park[r] + park[NP + r]) + (park[2 * NP + r] + park[3 * NP + r]);
         }
         asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
         __syncthreads();
@@ -307,6 +344,7 @@ __global__ void __launch_bounds__(THREADS) k_stream_gemm(const __grid_constant__
         float4 pv[RB][MAX_SPLIT];
         float ps[RB][MAX_SPLIT];
         uint2 res[RB], mix[RB];
+        float4 hold[EPI == EPI_STREAM ? RB : 1];
 #pragma unroll
         for (int i = 0; i < RB; i++) {
             const int r = r0 + i * 4 * S;
@@ -317,6 +355,8 @@ __global__ void __launch_bounds__(THREADS) k_stream_gemm(const __grid_constant__
                 ps[i][s] = ok && s < S && a.norm_input ? peer_sumsq[s][r] : 0.f;
             }
             res[i] = HAS_RESID && ok ? *reinterpret_cast<const uint2 *>(a.resid + (size_t)r * a.N + col4) : make_uint2(0u, 0u);
+            if (EPI == EPI_STREAM)
+                hold[i] = ok ? *reinterpret_cast<const float4 *>(a.rs.h + (size_t)r * a.N + col4) : make_float4(0.f, 0.f, 0.f, 0.f);
             mix[i] = EPI == EPI_MIX && ok ? *reinterpret_cast<const uint2 *>(a.x0 + (size_t)r * a.N + col4) : make_uint2(0u, 0u);
         }
 #pragma unroll
@@ -332,11 +372,46 @@ __global__ void __launch_bounds__(THREADS) k_stream_gemm(const __grid_constant__
             if (a.norm_input) {
                 const float rstd = rsqrtf(ss * inv_k + FLT_EPSILON);
                 v.x *= rstd, v.y *= rstd, v.z *= rstd, v.w *= rstd;
+            } else if (r < a.rows) {
+                const float f = sumsq[r];
+                v.x *= f, v.y *= f, v.z *= f, v.w *= f;
+            }
+            if (EPI == EPI_STREAM) { /* a warp holds the whole row of this tile (r is the same for its lanes) */
+                float4 h = hold[i];
+                h.x += a.rs.mult * v.x, h.y += a.rs.mult * v.y, h.z += a.rs.mult * v.z, h.w += a.rs.mult * v.w;
+                float q = h.x * h.x + h.y * h.y + h.z * h.z + h.w * h.w;
+                for (int o = 16; o > 0; o >>= 1) q += __shfl_xor_sync(0xffffffffu, q, o);
+                if (r < a.rows) {
+                    const size_t at = (size_t)r * a.N + col4;
+                    const float4 g = *reinterpret_cast<const float4 *>(a.rs.gain + col4);
+                    *reinterpret_cast<float4 *>(a.rs.h + at) = h;
+                    uint2 out;
+                    __nv_bfloat162 *oo = reinterpret_cast<__nv_bfloat162 *>(&out);
+                    oo[0] = __floats2bfloat162_rn(h.x * g.x, h.y * g.y);
+                    oo[1] = __floats2bfloat162_rn(h.z * g.z, h.w * g.w);
+                    *reinterpret_cast<uint2 *>(reinterpret_cast<bf16 *>(a.rs.x_next) + at) = out;
+                    if (lane == 0) a.rs.ss_next[(size_t)r * gridDim.y + tile] = q;
+                }
+                continue;
             }
             if (r >= a.rows) continue;
             const size_t at = (size_t)r * a.N + col4;
-            if (EPI == EPI_F32) {
-                *reinterpret_cast<float4 *>(reinterpret_cast<float *>(a.y) + at) = v;
+            if (EPI == EPI_GEGLU) {
+                *reinterpret_cast<__nv_bfloat162 *>(reinterpret_cast<bf16 *>(a.y) + (size_t)r * a.ldy + (col4 >> 1)) =
+                    __floats2bfloat162_rn(gelu_tanh(v.x) * v.y, gelu_tanh(v.z) * v.w);
+            } else if ((EPI == EPI_STORE || EPI == EPI_F32) && ((int)col4 + 4 > a.n_store || (a.ldy & 3))) {
+                const float e[4] = {v.x, v.y, v.z, v.w}; /* the last stored columns, or rows without vector alignment */
+#pragma unroll
+                for (int j = 0; j < 4; j++)
+                    if ((int)col4 + j < a.n_store) finish(e[j], 0.f, 0.f, (size_t)r * a.ldy + col4 + j);
+            } else if (EPI == EPI_F32) {
+                *reinterpret_cast<float4 *>(reinterpret_cast<float *>(a.y) + (size_t)r * a.ldy + col4) = v;
+            } else if (EPI == EPI_STORE) {
+                uint2 out;
+                __nv_bfloat162 *oo = reinterpret_cast<__nv_bfloat162 *>(&out);
+                oo[0] = __floats2bfloat162_rn(v.x, v.y);
+                oo[1] = __floats2bfloat162_rn(v.z, v.w);
+                *reinterpret_cast<uint2 *>(reinterpret_cast<bf16 *>(a.y) + (size_t)r * a.ldy + col4) = out;
             } else {
                 const __nv_bfloat162 *rr = reinterpret_cast<const __nv_bfloat162 *>(&res[i]);
                 const __nv_bfloat162 *mm = reinterpret_cast<const __nv_bfloat162 *>(&mix[i]);
@@ -407,6 +482,8 @@ int launch_epi(const CUtensorMap &map_w, const CUtensorMap &map_x, const GemmArg
     case EPI_RELU2: return launch<NP, EPI_RELU2>(map_w, map_x, a, split, stream);
     case EPI_F32: return launch<NP, EPI_F32>(map_w, map_x, a, split, stream);
     case EPI_MIX: return launch<NP, EPI_MIX>(map_w, map_x, a, split, stream);
+    case EPI_GEGLU: return launch<NP, EPI_GEGLU>(map_w, map_x, a, split, stream);
+    case EPI_STREAM: return launch<NP, EPI_STREAM>(map_w, map_x, a, split, stream);
     default: return NCB_ERR_ARG;
     }
 }
@@ -426,12 +503,12 @@ int stream_gemm_split(int rows, int N, int K) {
 /* The checks and the launch shared by stream_gemm and stream_gemm_mix. */
 static int run_stream_gemm(const void *x, const void *w, const void *resid, void *y, int rows, int N, int K, int norm_input,
                            int epilogue, int split, const void *next_w, long long next_bytes, int *status, void *stream,
-                           const void *x0, float l1, float l2) {
+                           const void *x0, float l1, float l2, long long ldy, int n_store, const StreamIO &rs) {
     if (rows < 0 || rows > 256 || N <= 0 || K <= 0 || N % TILE_F || K % KBLK) return NCB_ERR_ARG;
-    if (epilogue < EPI_STORE || epilogue > EPI_MIX || split < 0 || split > MAX_SPLIT || split > K / KBLK) return NCB_ERR_ARG;
+    if (epilogue < EPI_STORE || epilogue > EPI_STREAM || split < 0 || split > MAX_SPLIT || split > K / KBLK) return NCB_ERR_ARG;
     if (rows == 0) return NCB_OK;
     const bool has_resid = epilogue == EPI_RESID || epilogue == EPI_MIX;
-    if (!x || !w || !y || (has_resid && !resid) || (epilogue == EPI_MIX && !x0)) return NCB_ERR_ARG;
+    if (!x || !w || (!y && epilogue != EPI_STREAM) || (has_resid && !resid) || (epilogue == EPI_MIX && !x0)) return NCB_ERR_ARG;
     if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)y | (uintptr_t)resid | (uintptr_t)x0) % 16) return NCB_ERR_ALIGN;
     if (next_w && ((uintptr_t)next_w % 16 || next_bytes % 16 || next_bytes < 0)) return NCB_ERR_ALIGN;
     if (split == 0) split = auto_split(rows, N / TILE_F, K / KBLK);
@@ -439,7 +516,8 @@ static int run_stream_gemm(const void *x, const void *w, const void *resid, void
     CUtensorMap map_w, map_x;
     if (!tensor_map(w, N, K, TILE_F, &map_w) || !tensor_map(x, rows, K, np, &map_x)) return NCB_ERR_LAUNCH;
     const GemmArgs a = {(const bf16 *)x, (const bf16 *)resid, y, rows, N, K, norm_input,
-                        next_bytes > 0 ? (const uint8_t *)next_w : nullptr, next_bytes, status, (const bf16 *)x0, l1, l2};
+                        next_bytes > 0 ? (const uint8_t *)next_w : nullptr, next_bytes, status, (const bf16 *)x0, l1, l2,
+                        ldy, n_store, rs};
     cudaStream_t s = (cudaStream_t)stream;
     switch (np) {
     case 32: return launch_epi<32>(map_w, map_x, a, epilogue, split, s);
@@ -464,9 +542,9 @@ extern "C" {
  */
 int stream_gemm(const void *x, const void *w, const void *resid, void *y, int rows, int N, int K, int norm_input,
                 int epilogue, int split, const void *next_w, long long next_bytes, int *status, void *stream) {
-    if (epilogue == EPI_MIX) return NCB_ERR_ARG;
+    if (epilogue > EPI_F32) return NCB_ERR_ARG;
     return run_stream_gemm(x, w, resid, y, rows, N, K, norm_input, epilogue, split, next_w, next_bytes, status, stream,
-                           nullptr, 1.f, 0.f);
+                           nullptr, 1.f, 0.f, N, N, no_stream());
 }
 
 /* stream_gemm with the residual epilogue followed by the NEXT layer's stream mix:
@@ -475,7 +553,16 @@ int stream_gemm_mix(const void *x, const void *w, const void *resid, const void 
                     int N, int K, int norm_input, int split, const void *next_w, long long next_bytes, int *status,
                     void *stream) {
     return run_stream_gemm(x, w, resid, y, rows, N, K, norm_input, EPI_MIX, split, next_w, next_bytes, status, stream, x0,
-                           l1, l2);
+                           l1, l2, N, N, no_stream());
+}
+
+/* stream_gemm on a residual stream kept in fp32 (ncb_gemm_rs). */
+int stream_gemm_rs(const ncb_gemm_rs *g, void *stream) {
+    if (!g || g->rows > 256) return NCB_ERR_ARG;
+    const int rc = check_rs(*g);
+    if (rc != NCB_OK) return rc;
+    return run_stream_gemm(g->x, g->w, nullptr, g->y, (int)g->rows, g->N, g->K, 0, g->epilogue, 0, g->next_w, g->next_bytes,
+                           g->status, stream, nullptr, 1.f, 0.f, g->ldy, g->n_store, stream_io(*g));
 }
 
 } /* extern "C" */

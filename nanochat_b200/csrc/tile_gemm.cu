@@ -22,6 +22,7 @@
  * Every mbarrier wait is bounded; on expiry NCB_DEV_WAIT_TIMEOUT is flagged, every role abandons its remaining tiles
  * and the block still frees its tensor memory.
  */
+#include "gemm_rs.cuh"
 #include "umma.cuh"
 
 namespace {
@@ -30,7 +31,7 @@ constexpr int BM = 128;          /* rows per tile = MMA M */
 constexpr int THREADS = 192;     /* producer warp, MMA warp, four epilogue warps */
 constexpr int A_BYTES = BM * KBLK * 2;
 
-enum { EPI_STORE = 0, EPI_RESID = 1, EPI_RELU2 = 2, EPI_F32 = 3 };
+enum { EPI_STORE = 0, EPI_RESID = 1, EPI_RELU2 = 2, EPI_F32 = 3, EPI_GEGLU = 5, EPI_STREAM = 6 };
 
 template <int BN> struct Tile {
     static constexpr int B_BYTES = BN * KBLK * 2;
@@ -47,7 +48,20 @@ struct TileArgs {
     int rows, N, K;
     int *status;
     int split_from; /* tiles from this index on are worked on as two half-width units each (= tiles: none) */
+    long long ldy;  /* row stride of y for EPI_STORE, EPI_F32 and EPI_GEGLU */
+    int n_store;    /* columns below this are stored (EPI_STORE, EPI_F32) */
+    StreamIO rs;    /* row scale of the product, EPI_STREAM's outputs */
 };
+
+/* The factor of a row's products: the stream's partial sums of squares are summed once per tile. */
+static __device__ __forceinline__ float scale_of_row(const TileArgs &a, int row) {
+    float s = 0.f;
+    if (a.rs.ss && row < a.rows) {
+        const float *p = a.rs.ss + (size_t)row * a.rs.ss_parts;
+        for (int i = 0; i < a.rs.ss_parts; i++) s += p[i];
+    }
+    return row_scale(a.rs, s);
+}
 
 /* A unit of work: a tile, or half of one. */
 struct Unit {
@@ -66,9 +80,51 @@ static __device__ __forceinline__ Unit unit_of(int u, int n_tiles, int split_fro
     return {(t / n_tiles) * BM, (t % n_tiles) * BN + (h & 1) * (BN / 2), BN / 2};
 }
 
-/* The epilogue on 32 consecutive fp32 products of one row, written at element offset `at` of y. */
-template <int EPI> static __device__ __forceinline__ void store_columns(const TileArgs &a, size_t at, const float *v) {
-    if (EPI == EPI_F32) {
+/* The epilogue on 32 consecutive fp32 products of one row, columns n .. n + 31; `v` is scaled by the row's factor. */
+template <int EPI> static __device__ __forceinline__ void store_columns(const TileArgs &a, int row, int n, float *v, float factor) {
+    const size_t at = (size_t)row * (EPI == EPI_STORE || EPI == EPI_F32 ? a.ldy : (long long)a.N) + n;
+#pragma unroll
+    for (int j = 0; j < 32; j++) v[j] *= factor;
+    if (EPI == EPI_GEGLU) {
+        uint4 packed[2];
+        __nv_bfloat162 *o = reinterpret_cast<__nv_bfloat162 *>(packed);
+#pragma unroll
+        for (int j = 0; j < 8; j++)
+            o[j] = __floats2bfloat162_rn(gelu_tanh(v[4 * j]) * v[4 * j + 1], gelu_tanh(v[4 * j + 2]) * v[4 * j + 3]);
+        uint4 *dst = reinterpret_cast<uint4 *>(reinterpret_cast<bf16 *>(a.y) + (size_t)row * a.ldy + (n >> 1));
+        dst[0] = packed[0], dst[1] = packed[1];
+    } else if (EPI == EPI_STREAM) {
+        float4 *h = reinterpret_cast<float4 *>(a.rs.h + at);
+        const float4 *gain = reinterpret_cast<const float4 *>(a.rs.gain + n);
+        uint4 packed[4];
+        __nv_bfloat162 *o = reinterpret_cast<__nv_bfloat162 *>(packed);
+        float4 hv[8];
+#pragma unroll
+        for (int j = 0; j < 8; j++) hv[j] = h[j];
+        float q = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; j++) {
+            float4 x = hv[j];
+            x.x += a.rs.mult * v[4 * j], x.y += a.rs.mult * v[4 * j + 1];
+            x.z += a.rs.mult * v[4 * j + 2], x.w += a.rs.mult * v[4 * j + 3];
+            q += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+            h[j] = x;
+            const float4 g = gain[j];
+            o[2 * j] = __floats2bfloat162_rn(x.x * g.x, x.y * g.y);
+            o[2 * j + 1] = __floats2bfloat162_rn(x.z * g.z, x.w * g.w);
+        }
+        uint4 *dst = reinterpret_cast<uint4 *>(reinterpret_cast<bf16 *>(a.rs.x_next) + at);
+#pragma unroll
+        for (int j = 0; j < 4; j++) dst[j] = packed[j];
+        a.rs.ss_next[(size_t)row * (a.N >> 5) + (n >> 5)] = q;
+    } else if ((EPI == EPI_STORE || EPI == EPI_F32) && (n + 32 > a.n_store || (a.ldy & 7))) {
+#pragma unroll
+        for (int j = 0; j < 32; j++) /* the last stored columns, or rows without vector alignment */
+            if (n + j < a.n_store) {
+                if (EPI == EPI_F32) reinterpret_cast<float *>(a.y)[at + j] = v[j];
+                else reinterpret_cast<bf16 *>(a.y)[at + j] = __float2bfloat16_rn(v[j]);
+            }
+    } else if (EPI == EPI_F32) {
         float4 *out = reinterpret_cast<float4 *>(reinterpret_cast<float *>(a.y) + at);
 #pragma unroll
         for (int j = 0; j < 8; j++) out[j] = make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
@@ -213,6 +269,7 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm(const __grid_constant_
             const uint32_t buf = it & 1;
             const Unit un = unit_of<BN>(u, n_tiles, split_from);
             const int m0 = un.m0, n0 = un.n0;
+            const float factor = scale_of_row(a, m0 + quarter * 32 + lane);
             if (*failed || !mbar_wait(acc_full(buf), (it >> 1) & 1)) {
                 if (!*failed && lane == 0) flag(a.status, NCB_DEV_WAIT_TIMEOUT);
                 *failed = 1;
@@ -221,13 +278,12 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm(const __grid_constant_
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const int row = m0 + quarter * 32 + lane;
             const bool live = row < a.rows;
-            const size_t base = (size_t)row * a.N + n0;
 #pragma unroll 1
             for (int c = 0; c < un.width / 32; c++) {
                 float v[32];
                 tmem_load32(tmem + ((uint32_t)(quarter * 32) << 16) + buf * BN + c * 32, v);
                 if (!live) continue;
-                store_columns<EPI>(a, base + c * 32, v);
+                store_columns<EPI>(a, row, n0 + c * 32, v, factor);
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             __syncwarp();
@@ -456,6 +512,7 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm_pair(const __grid_cons
             const uint32_t buf = acc_of(it);
             const Unit un = pair_unit_of<WIDTH>(u, n_tiles, split_from);
             const int m0 = un.m0 + (int)rank * BM, n0 = un.n0;
+            const float factor = scale_of_row(a, m0 + quarter * 32 + lane);
             if (*failed || !mbar_wait(acc_full(buf), use_of(it) & 1)) {
                 if (!*failed && lane == 0) flag(a.status, NCB_DEV_WAIT_TIMEOUT);
                 *failed = 1;
@@ -464,13 +521,12 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm_pair(const __grid_cons
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const int row = m0 + quarter * 32 + lane;
             const bool live = row < a.rows;
-            const size_t base = (size_t)row * a.N + n0;
 #pragma unroll 1
             for (int c = 0; c < un.width / 32; c++) {
                 float v[32];
                 tmem_load32(tmem + ((uint32_t)(quarter * 32) << 16) + buf * WIDTH + c * 32, v);
                 if (!live) continue;
-                store_columns<EPI>(a, base + c * 32, v);
+                store_columns<EPI>(a, row, n0 + c * 32, v, factor);
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             __syncwarp();
@@ -534,6 +590,8 @@ int launch_epi(const CUtensorMap &map_x, const CUtensorMap &map_w, const CUtenso
     case EPI_RESID: return launch<BN, EPI_RESID>(map_x, map_w, map_w_half, a, stream);
     case EPI_RELU2: return launch<BN, EPI_RELU2>(map_x, map_w, map_w_half, a, stream);
     case EPI_F32: return launch<BN, EPI_F32>(map_x, map_w, map_w_half, a, stream);
+    case EPI_GEGLU: return launch<BN, EPI_GEGLU>(map_x, map_w, map_w_half, a, stream);
+    case EPI_STREAM: return launch<BN, EPI_STREAM>(map_x, map_w, map_w_half, a, stream);
     default: return NCB_ERR_ARG;
     }
 }
@@ -621,6 +679,8 @@ int launch_pair_epi(const CUtensorMap &map_x, const CUtensorMap &map_w, const CU
     case EPI_RESID: return launch_pair<NMMA, NSUB, EPI_RESID>(map_x, map_w, map_w_half, a, pairs, stream);
     case EPI_RELU2: return launch_pair<NMMA, NSUB, EPI_RELU2>(map_x, map_w, map_w_half, a, pairs, stream);
     case EPI_F32: return launch_pair<NMMA, NSUB, EPI_F32>(map_x, map_w, map_w_half, a, pairs, stream);
+    case EPI_GEGLU: return launch_pair<NMMA, NSUB, EPI_GEGLU>(map_x, map_w, map_w_half, a, pairs, stream);
+    case EPI_STREAM: return launch_pair<NMMA, NSUB, EPI_STREAM>(map_x, map_w, map_w_half, a, pairs, stream);
     default: return NCB_ERR_ARG;
     }
 }
@@ -636,6 +696,33 @@ double pair_cost(int rows, int N, int width, bool can_split, int pairs) {
 }
 
 } /* namespace */
+
+/* The checks that depend on the kernel form, the choice of the form, and the launch. */
+static int run_tile_gemm(const void *x, const void *w, TileArgs a, int epilogue, int form, cudaStream_t stream) {
+    const int rows = a.rows, N = a.N, K = a.K;
+    CUtensorMap map_x, map_w, map_w_half;
+    const bool wide_ok = N % 320 == 0, std_ok = N % 256 == 0;
+    if ((form == 2 || (form == 0 && PAIR_BY_DEFAULT && rows > BM)) && (wide_ok || std_ok)) {
+        const int pairs = resident_pairs();
+        if (pairs > 0) {
+            const bool wide = wide_ok && (!std_ok || pair_cost(rows, N, 320, false, pairs) < pair_cost(rows, N, 256, true, pairs));
+            const int nmma = wide ? 160 : 256;
+            if (!tensor_map(x, rows, K, BM, &map_x) || !tensor_map(w, N, K, nmma / 2, &map_w) ||
+                !tensor_map(w, N, K, nmma / 4, &map_w_half))
+                return NCB_ERR_LAUNCH;
+            return wide ? launch_pair_epi<160, 2>(map_x, map_w, map_w_half, a, epilogue, pairs, stream)
+                        : launch_pair_epi<256, 1>(map_x, map_w, map_w_half, a, epilogue, pairs, stream);
+        }
+        if (form == 2) return NCB_ERR_UNSUPPORTED;
+    } else if (form == 2) {
+        return NCB_ERR_UNSUPPORTED;
+    }
+    const int bn = N % 256 == 0 ? 256 : 128;
+    if (!tensor_map(x, rows, K, BM, &map_x) || !tensor_map(w, N, K, bn, &map_w) || !tensor_map(w, N, K, bn / 2, &map_w_half))
+        return NCB_ERR_LAUNCH;
+    return bn == 256 ? launch_epi<256>(map_x, map_w, map_w_half, a, epilogue, stream)
+                     : launch_epi<128>(map_x, map_w, map_w_half, a, epilogue, stream);
+}
 
 extern "C" {
 
@@ -657,30 +744,18 @@ int tile_gemm_form(const void *x, const void *w, const void *resid, void *y, lon
     if (rows == 0) return NCB_OK;
     if (!x || !w || !y || (epilogue == EPI_RESID && !resid)) return NCB_ERR_ARG;
     if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)y | (uintptr_t)resid) % 16) return NCB_ERR_ALIGN;
-    const TileArgs a = {(const bf16 *)resid, y, (int)rows, N, K, status, 0};
-    CUtensorMap map_x, map_w, map_w_half;
-    const bool wide_ok = N % 320 == 0, std_ok = N % 256 == 0;
-    if ((form == 2 || (form == 0 && PAIR_BY_DEFAULT && rows > BM)) && (wide_ok || std_ok)) {
-        const int pairs = resident_pairs();
-        if (pairs > 0) {
-            const bool wide = wide_ok && (!std_ok || pair_cost((int)rows, N, 320, false, pairs) < pair_cost((int)rows, N, 256, true, pairs));
-            const int nmma = wide ? 160 : 256;
-            if (!tensor_map(x, (int)rows, K, BM, &map_x) || !tensor_map(w, N, K, nmma / 2, &map_w) ||
-                !tensor_map(w, N, K, nmma / 4, &map_w_half))
-                return NCB_ERR_LAUNCH;
-            return wide ? launch_pair_epi<160, 2>(map_x, map_w, map_w_half, a, epilogue, pairs, (cudaStream_t)stream)
-                        : launch_pair_epi<256, 1>(map_x, map_w, map_w_half, a, epilogue, pairs, (cudaStream_t)stream);
-        }
-        if (form == 2) return NCB_ERR_UNSUPPORTED;
-    } else if (form == 2) {
-        return NCB_ERR_UNSUPPORTED;
-    }
-    const int bn = N % 256 == 0 ? 256 : 128;
-    if (!tensor_map(x, (int)rows, K, BM, &map_x) || !tensor_map(w, N, K, bn, &map_w) ||
-        !tensor_map(w, N, K, bn / 2, &map_w_half))
-        return NCB_ERR_LAUNCH;
-    return bn == 256 ? launch_epi<256>(map_x, map_w, map_w_half, a, epilogue, (cudaStream_t)stream)
-                     : launch_epi<128>(map_x, map_w, map_w_half, a, epilogue, (cudaStream_t)stream);
+    const TileArgs a = {(const bf16 *)resid, y, (int)rows, N, K, status, 0, N, N, no_stream()};
+    return run_tile_gemm(x, w, a, epilogue, form, (cudaStream_t)stream);
+}
+
+/* tile_gemm on a residual stream kept in fp32 (ncb_gemm_rs). */
+int tile_gemm_rs(const ncb_gemm_rs *g, void *stream) {
+    if (!g || g->rows > 0x7fffff00LL || g->N % 128 || g->K % KBLK) return NCB_ERR_ARG;
+    const int rc = check_rs(*g);
+    if (rc != NCB_OK || g->rows == 0) return rc;
+    if (g->epilogue == EPI_GEGLU && g->ldy % 8) return NCB_ERR_ALIGN;
+    const TileArgs a = {nullptr, g->y, (int)g->rows, g->N, g->K, g->status, 0, g->ldy, g->n_store, stream_io(*g)};
+    return run_tile_gemm(g->x, g->w, a, g->epilogue, 0, (cudaStream_t)stream);
 }
 
 int tile_gemm(const void *x, const void *w, const void *resid, void *y, long long rows, int N, int K, int epilogue,

@@ -174,7 +174,10 @@ def slot_bytes(cfg: DecoderConfig) -> int:
     """Device bytes one more slot costs a decoder of this shape: its pages in every layer's cache plus its rows of the
     step's buffers (hidden, qkv, attention output, MLP, x0, normed rows in bf16; fp32 logits and sampling
     probabilities; the int64 token trace), each rounded up to 256 bytes as the allocator rounds them. The reference
-    sums its per-slot buffers the same way (slot_buffers / padded, decode.cu:977-979)."""
+    sums its per-slot buffers the same way (slot_buffers / padded, decode.cu:977-979). A configuration of another kind
+    of model brings its own count."""
+    if hasattr(cfg, "slot_bytes"):
+        return cfg.slot_bytes()
     from .kv_cache import PAGE_BYTES, cache_pages
 
     def padded(n: int) -> int:
@@ -201,8 +204,25 @@ def slots_that_fit(cfg: DecoderConfig, free_bytes: int, max_slots: int = MAX_SLO
     return int(n)
 
 
-class Decoder:
-    """Greedy decoding of up to n_slots sequences with an fp8 KV cache per layer."""
+class StepDecoder:
+    """What every model's decoder shares: slots with caches, prefill in row passes, the captured decode step with its greedy
+    or sampled choice, generation, and portions of a sequence fed from outside. A model provides `cfg` (with vocab), `caches`,
+    `capacity`, `store`, `status`, and
+
+        fill_rows(tokens, pos, slot_map, max_kv_len, host_rows)             run prompt rows for their caches alone
+        place_logits(tokens, pos, slot_map, max_kv_len, host_rows, places)  the same rows, fp32 logits of some of them
+        step_buffers(batch), run_step(tokens, pos, slot_map, buf)           one token per slot, logits in buf["logits"]
+        planned_chunk(positions, steps)                                     optional: the step's attention chunk size"""
+
+    softcap = 0.0
+    chunk_pages = 0  # attention chunk size of decode steps; 0: the library's choice for full-length slots
+
+    def _start(self, cfg, weights, n_slots: int, device: "torch.device | str", softcap: float) -> None:
+        self.softcap = float(softcap)
+        self.cfg, self.w, self.n_slots, self.device = cfg, weights, n_slots, torch.device(device)
+        self.status = torch.zeros(1, dtype=torch.int32, device=device)
+        self._graphs: dict[tuple, tuple] = {}
+        self._graph_tensors: dict[tuple, tuple] = {}
 
     @classmethod
     def sized_for_free_memory(cls, cfg: DecoderConfig, weights: DecoderWeights, device: "torch.device | str" = "cuda",
@@ -212,26 +232,226 @@ class Decoder:
         free, _ = torch.cuda.mem_get_info(torch.device(device))
         return cls(cfg, weights, slots_that_fit(cfg, max(free - reserve_bytes, 0), max_slots), device, **kwargs)
 
+    # ---- prefill ----------------------------------------------------------------------------------------------
+
+    @torch.no_grad()
+    def prefill(self, prompts: list[list[int]], slots: list[int], rows_per_pass: int = 4096) -> None:
+        """Cache positions 0 .. len - 2 of every prompt (its last token is the first decode input). Sequences are
+        processed in passes of at most rows_per_pass rows; a pass holds whole position ranges in order, so every row
+        finds the earlier positions of its sequence either in the cache or earlier in its own pass."""
+        import numpy as np
+
+        counts = [len(p) - 1 for p in prompts]
+        total = sum(counts)
+        if total == 0:
+            return
+        # the rows of all passes as arrays (a prompt of thousands of tokens must not cost a Python loop per row)
+        slot_rows = np.repeat(np.asarray(slots, dtype=np.int32), counts)
+        pos_rows = np.concatenate([np.arange(n, dtype=np.int32) for n in counts])
+        token_rows = np.concatenate([np.asarray(p[:-1], dtype=np.int64) for p in prompts])
+        for at in range(0, total, rows_per_pass):
+            part = slice(at, min(at + rows_per_pass, total))
+            n = part.stop - part.start
+            # tokens, positions and slots of the pass cross to the device in ONE copy
+            packed = np.empty(2 * n, dtype=np.int64)
+            packed[:n] = token_rows[part]
+            packed[n:].view(np.int32)[:n] = pos_rows[part]
+            packed[n:].view(np.int32)[n:] = slot_rows[part]
+            dev = torch.from_numpy(packed).to(self.device, non_blocking=True)
+            tokens, small = dev[:n], dev[n:].view(torch.int32)
+            self.fill_rows(tokens, small[:n], small[n:], int(pos_rows[part].max()) + 1, (slot_rows[part], pos_rows[part]))
+
+    @torch.no_grad()
+    def feed(self, slot: int, tokens: list[int], start: int, want: list[int], rows_per_pass: int = 4096) -> Tensor:
+        """Run `tokens` at positions start .. of `slot`, whose cache and state hold the positions before, and return the
+        fp32 logits (len(want), V) at the places `want` among them. One token runs as a captured decode step, several as
+        row passes: what generation runs for a new token and for a prompt."""
+        import numpy as np
+
+        n = len(tokens)
+        if n < 1 or start < 0 or start + n > self.capacity or not 0 <= slot < self.n_slots:
+            raise ValueError(f"{n} tokens at position {start} of slot {slot}: the cache holds {self.n_slots} slots of {self.capacity}")
+        if n == 1:
+            graph, side, dev_tokens, pos, logits, trace, ctl = self._step_graph(1)
+            slot_map = self._graph_tensors[(1, False, 0, False)][0]
+            side.wait_stream(torch.cuda.current_stream(self.device))
+            with torch.cuda.stream(side):
+                dev_tokens.fill_(tokens[0])
+                pos.fill_(start)
+                slot_map.fill_(slot)
+                graph.replay()
+                out = logits[[0] * len(want)]
+            torch.cuda.current_stream(self.device).wait_stream(side)
+            return out
+        found = []
+        for at in range(0, n, rows_per_pass):
+            m = min(rows_per_pass, n - at)
+            positions = np.arange(start + at, start + at + m, dtype=np.int32)
+            slots = np.full(m, slot, dtype=np.int32)
+            dev = torch.tensor(tokens[at:at + m], dtype=torch.long).to(self.device)
+            small = torch.from_numpy(np.concatenate([positions, slots])).to(self.device)
+            places = [w - at for w in want if at <= w < at + m]
+            args = (dev, small[:m], small[m:], int(positions[-1]) + 1, (slots, positions))
+            if places:
+                found.append(self.place_logits(*args, places))
+            else:
+                self.fill_rows(*args)
+        return torch.cat(found) if found else torch.empty((0, self.cfg.vocab), dtype=torch.float32, device=self.device)
+
+    # ---- decode -----------------------------------------------------------------------------------------------
+
+    def _step_graph(self, batch: int, sampled: bool = False, chunk_pages: int = 0, masked: bool = False):
+        """The captured step for `batch` slots 0 .. batch - 1: tokens, pos (device) -> chosen tokens; pos += 1; every
+        choice is logged at its position in a (batch, capacity + 1) trace. `sampled` steps choose by temperature /
+        nucleus / Gumbel-max (sample_choice) from per-slot controls, the others take the argmax. `chunk_pages` is
+        the attention chunk size baked into the graph (0: the library's choice for full-length slots). `masked`
+        (sampled steps only) adds per-slot allowed-token bit masks, ctl["allow"] int32 (batch, ceil(vocab / 32)), all ones
+        until a caller writes a row."""
+        key = (batch, sampled, chunk_pages, masked)
+        if key in self._graphs:
+            return self._graphs[key]
+        self.chunk_pages = chunk_pages
+        dev, lib, V = self.device, cuda_library("decode_step"), self.cfg.vocab
+        tokens = torch.zeros(batch, dtype=torch.long, device=dev)
+        pos = torch.zeros(batch, dtype=torch.int32, device=dev)
+        slot_map = torch.arange(batch, dtype=torch.int32, device=dev)
+        buf = self.step_buffers(batch)
+        logits, trace = buf["logits"], buf["trace"]
+        ctl = None
+        if sampled:
+            ctl = {"temperature": torch.zeros(batch, dtype=torch.float32, device=dev),
+                   "top_p": torch.ones(batch, dtype=torch.float32, device=dev),
+                   "seed": torch.zeros(batch, dtype=torch.long, device=dev),
+                   "first": torch.zeros(batch, dtype=torch.int32, device=dev),
+                   "probs": torch.empty((batch, V), dtype=torch.float32, device=dev)}
+            if masked:
+                ctl["allow"] = torch.full((batch, (V + 31) // 32), -1, dtype=torch.int32, device=dev)
+
+        def body():
+            self.run_step(tokens, pos, slot_map, buf)
+            if sampled:
+                check(lib.sample_choice(pointer(logits), pointer(ctl["probs"]), pointer(ctl["temperature"]),
+                                        pointer(ctl["top_p"]), pointer(ctl["seed"]), pointer(ctl["first"]),
+                                        pointer(ctl.get("allow")),
+                                        self.softcap, pointer(tokens), pointer(pos), batch, V, pointer(trace),
+                                        trace.shape[1], stream()), "sample_choice")
+            else:
+                check(lib.greedy_choice(pointer(logits), pointer(tokens), pointer(pos), batch, V, pointer(trace),
+                                        trace.shape[1], stream()), "greedy_choice")
+
+        side = torch.cuda.Stream(dev)
+        side.wait_stream(torch.cuda.current_stream(dev))
+        with torch.cuda.stream(side):
+            # eager warm-up (first-use set-up has to happen outside capture) with every slot idle: a negative position
+            # appends nothing, attends nothing and advances nothing, so caches that already hold sequences (decode_from
+            # with a key not captured yet) are left as they are
+            pos.fill_(-1)
+            body()
+            pos.zero_()
+            tokens.zero_()
+            side.synchronize()
+            graph = torch.cuda.CUDAGraph()
+            with no_collection(), torch.cuda.graph(graph, stream=side):
+                body()
+        self.chunk_pages = 0
+        # the graph holds raw pointers: every tensor its kernels touch must stay alive as long as the graph does
+        self._graph_tensors[key] = (slot_map, buf, ctl)
+        self._graphs[key] = (graph, side, tokens, pos, logits, trace, ctl)
+        return self._graphs[key]
+
+    def planned_chunk(self, positions: list[int], steps: int) -> int:
+        """The attention chunk size (in the model's own unit) for `steps` decode steps starting at these positions,
+        baked into the captured step; 0: the model's choice for full-length slots."""
+        return 0
+
+    @torch.no_grad()
+    def decode_from(self, first_tokens: list[int], positions: list[int], steps: int, temperature: float = 0.0,
+                    top_p: float = 1.0, seeds: list[int] | None = None) -> tuple[list[list[int]], float]:
+        """`steps` steps for slots 0 .. B - 1 whose caches already hold positions 0 .. positions[b] - 1: slot b's
+        next input is first_tokens[b] at position positions[b]. Greedy at temperature 0, else sampled as the
+        reference samples (capped logits / temperature, nucleus top_p, Gumbel-max noise keyed by seeds[b] and the
+        step; the cap is the decoder's `softcap`). Returns the chosen tokens and the seconds the steps took on the
+        device. Stream-ordered after work queued on the current stream."""
+        B = len(first_tokens)
+        assert B <= self.n_slots and max(positions) + steps <= self.capacity
+        sampled = temperature > 0.0
+        key = (B, sampled, self.planned_chunk(positions, steps), False)
+        graph, side, tokens, pos, logits, trace, ctl = self._step_graph(*key)
+        # The step's rows are the slots in descending order of length: the attention kernel's blocks start in row
+        # order, and a ragged batch that starts with its longest sequences leaves the shortest tail of idle SMs.
+        # (A row is computed from its own slot alone, so the order changes no result.)
+        order = sorted(range(B), key=lambda b: (-positions[b], b))
+        row_of = {b: r for r, b in enumerate(order)}
+        slot_map = self._graph_tensors[key][0]
+        begin, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        side.wait_stream(torch.cuda.current_stream(self.device))
+        with torch.cuda.stream(side):
+            slot_map.copy_(torch.tensor(order, dtype=torch.int32))
+            tokens.copy_(torch.tensor([first_tokens[b] for b in order], dtype=torch.long))
+            pos.copy_(torch.tensor([positions[b] for b in order], dtype=torch.int32))
+            first = pos.clone()
+            if sampled:
+                seeds = seeds if seeds is not None else list(range(B))
+                ctl["temperature"].fill_(temperature)
+                ctl["top_p"].fill_(top_p)
+                ctl["seed"].copy_(torch.tensor([seeds[b] for b in order], dtype=torch.long))
+                ctl["first"].copy_(first)
+            begin.record()
+            for _ in range(steps):
+                graph.replay()
+            end.record()
+            at = first.long()[:, None] + 1 + torch.arange(steps, device=self.device)[None, :]
+            out = trace.gather(1, at)  # every choice was logged at its position: one gather at the end
+        side.synchronize()
+        code = int(self.status.item())
+        if code:
+            raise RuntimeError(f"device status {code:#x} (NCB_DEV_* bits)")
+        rows = out.tolist()
+        return [rows[row_of[b]] for b in range(B)], begin.elapsed_time(end) * 1e-3
+
+    @torch.no_grad()
+    def generate(self, prompts: list[list[int]], max_new_tokens: int, temperature: float = 0.0, top_p: float = 1.0,
+                 seeds: list[int] | None = None) -> tuple[list[list[int]], dict]:
+        """Continuation of every prompt (slot b = prompt b), greedy or sampled (see decode_from). Returns the new
+        tokens and timings: prefill seconds, decode seconds (the max_new_tokens steps), tokens per second of the
+        decode phase."""
+        B = len(prompts)
+        assert B <= self.n_slots and all(len(p) >= 1 for p in prompts)
+        assert max(len(p) for p in prompts) - 1 + max_new_tokens <= self.capacity
+        # capture (and its warm-up step) before the caches are filled
+        self._step_graph(B, temperature > 0.0, self.planned_chunk([len(p) - 1 for p in prompts], max_new_tokens))
+        start, mid = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        start.record()
+        missing = [b for b in range(B) if self.store is None or not self.store.load(b, prompts[b])]
+        self.prefill([prompts[b] for b in missing], missing)
+        if self.store is not None:
+            for b in missing:
+                self.store.save(b, prompts[b])
+        mid.record()
+        out, decode_s = self.decode_from([p[-1] for p in prompts], [len(p) - 1 for p in prompts], max_new_tokens,
+                                         temperature, top_p, seeds)
+        return out, {"prefill_s": start.elapsed_time(mid) * 1e-3, "decode_s": decode_s,
+                     "tokens_per_s": B * max_new_tokens / decode_s}
+
+
+class Decoder(StepDecoder):
+    """Greedy decoding of up to n_slots sequences with an fp8 KV cache per layer."""
+
     def __init__(self, cfg: DecoderConfig, weights: DecoderWeights, n_slots: int, device: "torch.device | str" = "cuda",
                  prompt_store: int = 0, softcap: float = 0.0):
         """prompt_store: positions of pinned host memory for prompts already prefilled (0: none); a prompt seen
         again is copied back into its slot instead of being prefilled (inference/decoder.py:193-232). softcap: the
         output-logit cap c applied (c tanh(z / c)) before sampling; greedy choices need none (decode.cu:195)."""
-        self.softcap = float(softcap)
-        self.cfg, self.w, self.n_slots, self.device = cfg, weights, n_slots, torch.device(device)
+        self._start(cfg, weights, n_slots, device, softcap)
         self.caches = [Fp8KVCache(n_slots, cfg.n_kv_heads, cfg.max_len, device=device) for _ in range(cfg.n_layers)]
         self.store = PromptStore(self.caches, prompt_store) if prompt_store > 0 else None
         self.capacity = self.caches[0].capacity
         self.cos, self.sin = ops.rotary_table(self.capacity, cfg.rope_theta, device=device)
-        self.status = torch.zeros(1, dtype=torch.int32, device=device)
         self.windows = cfg.windows or [0] * cfg.n_layers
         self.use_fused = True  # decode steps of <= 64 rows run on this package's GEMM kernels when the shapes allow
         self.use_stream_gemm = True  # ... of 17 to 64 rows on the tcgen05 stream_gemm (else the row path)
         self.use_tile_gemm = True  # row passes (prefill, steps above 64 rows) on the tiled tcgen05 GEMM, not torch's
-        self.chunk_pages = 0  # attention chunk size of decode steps; 0: the library's choice for full-length slots
         self.prefetch_next = True  # stream_gemm also pulls the next GEMM's weights into L2 (d32-class step: -1.3 %)
-        self._graphs: dict[int, tuple] = {}
-        self._graph_tensors: dict[int, tuple] = {}
         self._workspaces: dict[tuple[int, int], Tensor] = {}
 
     # ---- one pass over `rows` tokens -------------------------------------------------------------------------
@@ -469,103 +689,27 @@ class Decoder:
                                     pointer(buf["trace"]), buf["trace"].shape[1], s), "greedy_choice")
         return buf["logits"]
 
-    # ---- prefill ----------------------------------------------------------------------------------------------
+    # ---- what StepDecoder drives ---------------------------------------------------------------------------------
 
-    @torch.no_grad()
-    def prefill(self, prompts: list[list[int]], slots: list[int], rows_per_pass: int = 4096) -> None:
-        """Cache positions 0 .. len - 2 of every prompt (its last token is the first decode input). Sequences are
-        processed in passes of at most rows_per_pass rows; a pass holds whole position ranges in order, so every row
-        finds the earlier positions of its sequence either in the cache or earlier in its own pass."""
-        import numpy as np
+    def fill_rows(self, tokens: Tensor, pos: Tensor, slot_map: Tensor, max_kv_len: int, host_rows: tuple) -> None:
+        self.hidden_rows(tokens, pos, slot_map, max_kv_len, attend_last_layer=False, host_rows=host_rows)
 
-        counts = [len(p) - 1 for p in prompts]
-        total = sum(counts)
-        if total == 0:
-            return
-        # the rows of all passes as arrays (a prompt of thousands of tokens must not cost a Python loop per row)
-        slot_rows = np.repeat(np.asarray(slots, dtype=np.int32), counts)
-        pos_rows = np.concatenate([np.arange(n, dtype=np.int32) for n in counts])
-        token_rows = np.concatenate([np.asarray(p[:-1], dtype=np.int64) for p in prompts])
-        for at in range(0, total, rows_per_pass):
-            part = slice(at, min(at + rows_per_pass, total))
-            n = part.stop - part.start
-            # tokens, positions and slots of the pass cross to the device in ONE copy
-            packed = np.empty(2 * n, dtype=np.int64)
-            packed[:n] = token_rows[part]
-            packed[n:].view(np.int32)[:n] = pos_rows[part]
-            packed[n:].view(np.int32)[n:] = slot_rows[part]
-            dev = torch.from_numpy(packed).to(self.device, non_blocking=True)
-            tokens, small = dev[:n], dev[n:].view(torch.int32)
-            self.hidden_rows(tokens, small[:n], small[n:], int(pos_rows[part].max()) + 1, attend_last_layer=False,
-                             host_rows=(slot_rows[part], pos_rows[part]))
+    def place_logits(self, tokens: Tensor, pos: Tensor, slot_map: Tensor, max_kv_len: int, host_rows: tuple,
+                     places: list[int]) -> Tensor:
+        return self.head(self.hidden_rows(tokens, pos, slot_map, max_kv_len, host_rows=host_rows)[places])
 
-    # ---- decode -----------------------------------------------------------------------------------------------
+    def step_buffers(self, batch: int) -> dict[str, Tensor]:
+        if self.use_fused and self.fused_supported(batch):
+            return self.fused_buffers(batch)
+        return {"logits": torch.empty((batch, self.cfg.vocab), dtype=torch.float32, device=self.device),
+                "trace": torch.zeros((batch, self.capacity + 1), dtype=torch.long, device=self.device)}
 
-    def _step_graph(self, batch: int, sampled: bool = False, chunk_pages: int = 0, masked: bool = False):
-        """The captured step for `batch` slots 0 .. batch - 1: tokens, pos (device) -> chosen tokens; pos += 1; every
-        choice is logged at its position in a (batch, capacity + 1) trace. `sampled` steps choose by temperature /
-        nucleus / Gumbel-max (sample_choice) from per-slot controls, the others take the argmax. `chunk_pages` is
-        the attention chunk size baked into the graph (0: the library's choice for full-length slots). `masked`
-        (sampled steps only) adds per-slot allowed-token bit masks, ctl["allow"] int32 (batch, vocab / 32), all ones
-        until a caller writes a row."""
-        key = (batch, sampled, chunk_pages, masked)
-        if key in self._graphs:
-            return self._graphs[key]
-        self.chunk_pages = chunk_pages
-        dev, lib, V = self.device, cuda_library("decode_step"), self.cfg.vocab
-        tokens = torch.zeros(batch, dtype=torch.long, device=dev)
-        pos = torch.zeros(batch, dtype=torch.int32, device=dev)
-        slot_map = torch.arange(batch, dtype=torch.int32, device=dev)
-        fused = self.use_fused and self.fused_supported(batch)
-        buf = self.fused_buffers(batch) if fused else {
-            "logits": torch.empty((batch, V), dtype=torch.float32, device=dev),
-            "trace": torch.zeros((batch, self.capacity + 1), dtype=torch.long, device=dev)}
-        logits, trace = buf["logits"], buf["trace"]
-        ctl = None
-        if sampled:
-            assert V % 32 == 0, "sampling needs a vocabulary that is a multiple of 32"
-            ctl = {"temperature": torch.zeros(batch, dtype=torch.float32, device=dev),
-                   "top_p": torch.ones(batch, dtype=torch.float32, device=dev),
-                   "seed": torch.zeros(batch, dtype=torch.long, device=dev),
-                   "first": torch.zeros(batch, dtype=torch.int32, device=dev),
-                   "probs": torch.empty((batch, V), dtype=torch.float32, device=dev)}
-            if masked:
-                ctl["allow"] = torch.full((batch, V // 32), -1, dtype=torch.int32, device=dev)
-
-        def body():
-            if fused:
-                self.fused_step(tokens, pos, slot_map, self.capacity, buf, choose=False, slots=list(range(batch)))
-            else:
-                logits.copy_(self.head(self.hidden_rows(tokens, pos, slot_map, self.capacity, distinct_slots=True)))
-            if sampled:
-                check(lib.sample_choice(pointer(logits), pointer(ctl["probs"]), pointer(ctl["temperature"]),
-                                        pointer(ctl["top_p"]), pointer(ctl["seed"]), pointer(ctl["first"]),
-                                        pointer(ctl.get("allow")),
-                                        self.softcap, pointer(tokens), pointer(pos), batch, V, pointer(trace),
-                                        trace.shape[1], stream()), "sample_choice")
-            else:
-                check(lib.greedy_choice(pointer(logits), pointer(tokens), pointer(pos), batch, V, pointer(trace),
-                                        trace.shape[1], stream()), "greedy_choice")
-
-        side = torch.cuda.Stream(dev)
-        side.wait_stream(torch.cuda.current_stream(dev))
-        with torch.cuda.stream(side):
-            # eager warm-up (first-use set-up has to happen outside capture) with every slot idle: a negative position
-            # appends nothing, attends nothing and advances nothing, so caches that already hold sequences (decode_from
-            # with a key not captured yet) are left as they are
-            pos.fill_(-1)
-            body()
-            pos.zero_()
-            tokens.zero_()
-            side.synchronize()
-            graph = torch.cuda.CUDAGraph()
-            with no_collection(), torch.cuda.graph(graph, stream=side):
-                body()
-        self.chunk_pages = 0
-        # the graph holds raw pointers: every tensor its kernels touch must stay alive as long as the graph does
-        self._graph_tensors[key] = (slot_map, buf, ctl)
-        self._graphs[key] = (graph, side, tokens, pos, logits, trace, ctl)
-        return self._graphs[key]
+    def run_step(self, tokens: Tensor, pos: Tensor, slot_map: Tensor, buf: dict[str, Tensor]) -> None:
+        rows = tokens.shape[0]
+        if self.use_fused and self.fused_supported(rows):
+            self.fused_step(tokens, pos, slot_map, self.capacity, buf, choose=False, slots=list(range(rows)))
+        else:
+            buf["logits"].copy_(self.head(self.hidden_rows(tokens, pos, slot_map, self.capacity, distinct_slots=True)))
 
     def planned_chunk(self, positions: list[int], steps: int) -> int:
         """The attention chunk size for `steps` decode steps starting at these positions: the library's block-fill
@@ -573,72 +717,3 @@ class Decoder:
         captured step)."""
         lens = [min(p + 1 + steps // 2, self.capacity) for p in positions]
         return ops.plan_chunk_pages(lens, self.cfg.n_kv_heads, self.capacity)
-
-    @torch.no_grad()
-    def decode_from(self, first_tokens: list[int], positions: list[int], steps: int, temperature: float = 0.0,
-                    top_p: float = 1.0, seeds: list[int] | None = None) -> tuple[list[list[int]], float]:
-        """`steps` steps for slots 0 .. B - 1 whose caches already hold positions 0 .. positions[b] - 1: slot b's
-        next input is first_tokens[b] at position positions[b]. Greedy at temperature 0, else sampled as the
-        reference samples (capped logits / temperature, nucleus top_p, Gumbel-max noise keyed by seeds[b] and the
-        step; the cap is the decoder's `softcap`). Returns the chosen tokens and the seconds the steps took on the
-        device. Stream-ordered after work queued on the current stream."""
-        B = len(first_tokens)
-        assert B <= self.n_slots and max(positions) + steps <= self.capacity
-        sampled = temperature > 0.0
-        key = (B, sampled, self.planned_chunk(positions, steps), False)
-        graph, side, tokens, pos, logits, trace, ctl = self._step_graph(*key)
-        # The step's rows are the slots in descending order of length: the attention kernel's blocks start in row
-        # order, and a ragged batch that starts with its longest sequences leaves the shortest tail of idle SMs.
-        # (A row is computed from its own slot alone, so the order changes no result.)
-        order = sorted(range(B), key=lambda b: (-positions[b], b))
-        row_of = {b: r for r, b in enumerate(order)}
-        slot_map = self._graph_tensors[key][0]
-        begin, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        side.wait_stream(torch.cuda.current_stream(self.device))
-        with torch.cuda.stream(side):
-            slot_map.copy_(torch.tensor(order, dtype=torch.int32))
-            tokens.copy_(torch.tensor([first_tokens[b] for b in order], dtype=torch.long))
-            pos.copy_(torch.tensor([positions[b] for b in order], dtype=torch.int32))
-            first = pos.clone()
-            if sampled:
-                seeds = seeds if seeds is not None else list(range(B))
-                ctl["temperature"].fill_(temperature)
-                ctl["top_p"].fill_(top_p)
-                ctl["seed"].copy_(torch.tensor([seeds[b] for b in order], dtype=torch.long))
-                ctl["first"].copy_(first)
-            begin.record()
-            for _ in range(steps):
-                graph.replay()
-            end.record()
-            at = first.long()[:, None] + 1 + torch.arange(steps, device=self.device)[None, :]
-            out = trace.gather(1, at)  # every choice was logged at its position: one gather at the end
-        side.synchronize()
-        code = int(self.status.item())
-        if code:
-            raise RuntimeError(f"device status {code:#x} (NCB_DEV_* bits)")
-        rows = out.tolist()
-        return [rows[row_of[b]] for b in range(B)], begin.elapsed_time(end) * 1e-3
-
-    @torch.no_grad()
-    def generate(self, prompts: list[list[int]], max_new_tokens: int, temperature: float = 0.0, top_p: float = 1.0,
-                 seeds: list[int] | None = None) -> tuple[list[list[int]], dict]:
-        """Continuation of every prompt (slot b = prompt b), greedy or sampled (see decode_from). Returns the new
-        tokens and timings: prefill seconds, decode seconds (the max_new_tokens steps), tokens per second of the
-        decode phase."""
-        B = len(prompts)
-        assert B <= self.n_slots and all(len(p) >= 1 for p in prompts)
-        assert max(len(p) for p in prompts) - 1 + max_new_tokens <= self.capacity
-        # capture (and its warm-up step) before the caches are filled
-        self._step_graph(B, temperature > 0.0, self.planned_chunk([len(p) - 1 for p in prompts], max_new_tokens))
-        start, mid = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        start.record()
-        missing = [b for b in range(B) if self.store is None or not self.store.load(b, prompts[b])]
-        self.prefill([prompts[b] for b in missing], missing)
-        if self.store is not None:
-            for b in missing:
-                self.store.save(b, prompts[b])
-        mid.record()
-        out, decode_s = self.decode_from([p[-1] for p in prompts], [len(p) - 1 for p in prompts], max_new_tokens,
-                                         temperature, top_p, seeds)
-        return out, {"prefill_s": start.elapsed_time(mid) * 1e-3, "decode_s": decode_s,
-                     "tokens_per_s": B * max_new_tokens / decode_s}

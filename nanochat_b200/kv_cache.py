@@ -1,4 +1,5 @@
-"""The paged fp8 (e4m3) KV cache of one layer and the index arithmetic of its page layout.
+"""The caches of one layer: the paged fp8 (e4m3) KV cache with the index arithmetic of its page layout, and, for models
+that mix kinds of layers, the cache of latent rows and the recurrent state.
 
 Replaces the reference's bf16 cache `kc, vc [B][L][max_len][C]` (model/kernels/decode.cu:726, addressed at
 decode.cu:562,578-579). A page is NCB_PAGE_BYTES = 16,896 bytes holding 64 positions of one (slot, kv head): K rows
@@ -58,6 +59,11 @@ class Fp8KVCache:
     def nbytes(self) -> int:
         return self.pages.numel()
 
+    @staticmethod
+    def pages_for(positions: int) -> int:
+        """Pages of a slot that hold its first `positions` positions (per kv head)."""
+        return cache_pages(positions)
+
     def _flat(self, slot: int) -> tuple[torch.Tensor, torch.Tensor]:
         """(bytes [kv_heads, pages * PAGE_BYTES], floats [kv_heads, pages * PAGE_BYTES / 4]) views of a slot."""
         b = self.pages[slot].view(self.kv_heads, -1)
@@ -93,6 +99,51 @@ class Fp8KVCache:
         v = flat[:, (base + v_off[j]).reshape(-1)].view(self.kv_heads, n, HEAD_DIM)
         fbase = page * (PAGE_BYTES // 4) + j
         return k, floats[:, fbase + PAGE_KS // 4], v, floats[:, fbase + PAGE_VS // 4]
+
+
+class LatentCache:
+    """One latent-attention layer's cache: a row of `width` values (normed latent, then the rotated key part) per position,
+    T [n_slots, capacity, width]. `pages` is the same memory in the unit the prompt store copies: 64 positions of a slot."""
+
+    def __init__(self, n_slots: int, width: int, max_len: int, dtype: torch.dtype, device: "torch.device | str" = "cuda"):
+        self.n_slots, self.width = n_slots, width
+        self.pages_per_slot = cache_pages(max_len)
+        self.capacity = self.pages_per_slot * PAGE_TOKENS
+        self.rows = torch.zeros((n_slots, self.capacity, width), dtype=dtype, device=device)
+        self.pages = self.rows.view(torch.uint8).view(n_slots, 1, self.pages_per_slot, -1)
+
+    @property
+    def device(self) -> torch.device:
+        return self.rows.device
+
+    def nbytes(self) -> int:
+        return self.pages.numel()
+
+    @staticmethod
+    def pages_for(positions: int) -> int:
+        return cache_pages(positions)
+
+
+class StateCache:
+    """One recurrent layer's state: fp32 [n_slots, heads, dim, vdim], carried from token to token. A row at position 0
+    starts from zero whatever its slot holds, so a slot that is used again needs no clearing. As `pages`, a slot is a
+    single page: the state after the last position that was run."""
+
+    def __init__(self, n_slots: int, heads: int, dim: int, vdim: int, device: "torch.device | str" = "cuda"):
+        self.n_slots = n_slots
+        self.state = torch.zeros((n_slots, heads, dim, vdim), dtype=torch.float32, device=device)
+        self.pages = self.state.view(n_slots, 1, 1, -1).view(torch.uint8)
+
+    @property
+    def device(self) -> torch.device:
+        return self.state.device
+
+    def nbytes(self) -> int:
+        return self.pages.numel()
+
+    @staticmethod
+    def pages_for(positions: int) -> int:
+        return 1 if positions > 0 else 0
 
 
 def native_cache_bytes(n_slots: int, kv_heads: int, max_len: int) -> int:

@@ -1,0 +1,270 @@
+"""Token mixers of models whose layers differ in kind: weights prepared for the kernels, the cache or state each needs, and
+the launches between the input projection and the output projection. A mixer is built from its sizes and a dict of
+checkpoint tensors, so any model whose layers use it can share it; models/hybrid decoders only see
+
+    w_in, w_out                    fused input projection [in_width, C], output projection [C, out_width]
+    new_cache(n_slots, max_len)    one layer's cache
+    run(proj, cache, rows, out)    proj [rows, in_width] -> out [rows, out_width]; out None: only fill the cache
+
+Sizes the kernels want as multiples (of 16, 32 or 128) are reached by zero-padding weights here: padded values are zero
+everywhere they appear, so they change nothing, and no kernel has ragged edges."""
+
+from dataclasses import dataclass, field
+
+import numpy as np
+import torch
+from torch import Tensor
+
+from .kv_cache import LatentCache, StateCache
+from .native import Gla, Latent, check, cuda_library, stream
+from .rotary import half_tables
+
+LATENT_TILE = 32  # NCB_LATENT_TILE
+SM_COUNT = 148
+
+
+def up(n: int, multiple: int) -> int:
+    return (n + multiple - 1) // multiple * multiple
+
+
+def pad_to(t: Tensor, *shape: int) -> Tensor:
+    """t with zeros appended to each axis up to `shape`."""
+    out = torch.zeros(shape, dtype=t.dtype, device=t.device)
+    out[tuple(slice(0, n) for n in t.shape)] = t
+    return out
+
+
+def split_halves(t: Tensor, padded: int) -> Tensor:
+    """Rows of a rotated part [.., dims, C] -> [.., padded, C] with each half at the start of its padded half."""
+    half = t.shape[-2] // 2
+    out = torch.zeros((*t.shape[:-2], padded, t.shape[-1]), dtype=t.dtype, device=t.device)
+    out[..., :half, :] = t[..., :half, :]
+    out[..., padded // 2:padded // 2 + half, :] = t[..., half:, :]
+    return out
+
+
+def stack_fields(fields: list[Tensor], width: int, columns: int) -> tuple[Tensor, list[int]]:
+    """Fields [n_i, C] stacked into [width multiple, columns], each starting at a multiple of 8 rows; their offsets."""
+    offsets, at = [], 0
+    for f in fields:
+        offsets.append(at)
+        at += up(f.shape[0], 8)
+    out = torch.zeros((up(at, width), columns), dtype=fields[0].dtype, device=fields[0].device)
+    for f, o in zip(fields, offsets):
+        out[o:o + f.shape[0], :f.shape[1]] = f
+    return out, offsets
+
+
+class RowPlan:
+    """The segments of one prefill pass (runs of rows of one slot at ascending positions) and their chunks for recurrent
+    layers, on the device. Built once per pass, shared by the layers."""
+
+    def __init__(self, slots, positions, device):
+        slots, positions = np.asarray(slots, dtype=np.int32), np.asarray(positions, dtype=np.int32)
+        n = len(slots)
+        cut = np.ones(n, dtype=bool)
+        cut[1:] = (slots[1:] != slots[:-1]) | (positions[1:] != positions[:-1] + 1)
+        first = np.flatnonzero(cut).astype(np.int32)
+        self.first, self.count = first, np.diff(np.append(first, n)).astype(np.int32)
+        self.slots, self.starts, self.device = slots[first], positions[first], device
+        self._on_device: dict = {}
+
+    @property
+    def n_segments(self) -> int:
+        return len(self.first)
+
+    @property
+    def longest(self) -> int:
+        return int(self.count.max())
+
+    def upload(self, key, arrays: list[np.ndarray]) -> list[Tensor]:
+        """The arrays on the device (one copy), kept under `key` for the pass's other layers."""
+        if key not in self._on_device:
+            flat = torch.from_numpy(np.concatenate([np.asarray(a, dtype=np.int32) for a in arrays])).to(self.device)
+            self._on_device[key] = list(flat.split([len(a) for a in arrays]))
+        return self._on_device[key]
+
+    def segments(self) -> list[Tensor]:
+        return self.upload("segments", [self.first, self.count])
+
+    def chunks(self, size: int) -> tuple[list[Tensor], int]:
+        """([segment's first chunk (n + 1), chunk's first row, chunk's rows], number of chunks) for chunks of `size` rows."""
+        per = (self.count + size - 1) // size
+        base = np.concatenate([[0], np.cumsum(per)]).astype(np.int32)
+        within = np.arange(base[-1], dtype=np.int32) - np.repeat(base[:-1], per)
+        rows = np.repeat(self.first, per) + within * size
+        count = np.minimum(size, np.repeat(self.first + self.count, per) - rows)
+        return self.upload(("chunks", size), [base, rows, count]), int(base[-1])
+
+
+@dataclass
+class Rows:
+    """The rows of one pass or decode step: positions and slots on the device, a bound of every position + 1, and the
+    segments (None: a decode step, every row a slot of its own)."""
+    n: int
+    pos: Tensor
+    slot_map: Tensor
+    max_len: int
+    status: Tensor
+    plan: "RowPlan | None" = None
+    chunk_tiles: int = 0
+    scratch: dict = field(default_factory=dict)  # name -> tensor, reused by the layers of one pass
+
+    def buffer(self, name: str, numel: int, dtype: torch.dtype, device) -> Tensor:
+        t = self.scratch.get((name, dtype))
+        if t is None or t.numel() < numel:
+            t = self.scratch[(name, dtype)] = torch.empty(numel, dtype=dtype, device=device)
+        return t
+
+
+class GatedLinearAttention:
+    """Linear attention with a decay per key channel, per-head output norm and silu gate (csrc/gla.cu).
+    sizes: heads, dim, vdim, tau. tensors: q, k, v, g, o, a1, a2, a2.b, norm."""
+
+    CHUNKED_FROM = 24  # shorter segments run token by token
+
+    def __init__(self, sizes: dict, tensors: dict, eps: float, columns: int, dtype: torch.dtype, device):
+        H, D, V = int(sizes["heads"]), int(sizes["dim"]), int(sizes["vdim"])
+        self.heads, self.true_vdim, self.eps, self.dtype, self.device = H, V, float(eps), dtype, torch.device(device)
+        self.dim, self.vdim = up(D, 16), up(V, 16)
+        self.q_scale, self.inv_tau = float(D) ** -0.5, 1.0 / float(sizes["tau"])
+        t = {k: v.to(device) for k, v in tensors.items()}
+        C = t["q"].shape[1]
+
+        def per_head(w: Tensor, n: int, padded: int) -> Tensor:
+            return pad_to(w.reshape(H, n, C), H, padded, C).reshape(H * padded, C).to(dtype)
+
+        self.rank = t["a1"].shape[0]
+        fields = [per_head(t["q"], D, self.dim), per_head(t["k"], D, self.dim), per_head(t["v"], V, self.vdim),
+                  per_head(t["g"], V, self.vdim), t["a1"].to(dtype)]
+        self.w_in, self.offsets = stack_fields(fields, 128, columns)
+        self.a2 = pad_to(t["a2"].float().reshape(H, D, self.rank), H, self.dim, self.rank).contiguous()
+        self.a2_bias = pad_to(t["a2.b"].float().reshape(H, D), H, self.dim).contiguous()
+        self.norm = pad_to(t["norm"].float(), self.vdim)
+        o = pad_to(t["o"].reshape(-1, H, V), columns, H, self.vdim).reshape(columns, H * self.vdim)
+        self.out_width = up(H * self.vdim, 128)
+        self.w_out = pad_to(o, columns, self.out_width).to(dtype)
+        self.in_width = self.w_in.shape[0]
+        self.chunk = cuda_library("gla").gla_chunk_tokens(self.dim)
+
+    def new_cache(self, n_slots: int, max_len: int) -> StateCache:
+        return StateCache(n_slots, self.heads, self.dim, self.vdim, device=self.device)
+
+    @staticmethod
+    def cache_bytes(sizes: dict, max_len: int, itemsize: int) -> int:
+        return int(sizes["heads"]) * up(int(sizes["dim"]), 16) * up(int(sizes["vdim"]), 16) * 4
+
+    def run(self, proj: Tensor, cache: StateCache, rows: Rows, out: "Tensor | None") -> None:
+        n, f32 = rows.n, int(self.dtype == torch.float32)
+        a = Gla(proj=proj.data_ptr(), out=None if out is None else out.data_ptr(), rows=n, ldp=proj.stride(0),
+                ldo=0 if out is None else out.stride(0), heads=self.heads, dim=self.dim, vdim=self.vdim, rank=self.rank,
+                norm_count=self.true_vdim, n_slots=cache.n_slots, q_scale=self.q_scale, inv_tau=self.inv_tau, eps=self.eps,
+                a2=self.a2.data_ptr(), a2_bias=self.a2_bias.data_ptr(), norm=self.norm.data_ptr(),
+                state=cache.state.data_ptr(), pos=rows.pos.data_ptr(), slot_map=rows.slot_map.data_ptr(),
+                status=rows.status.data_ptr())
+        a.off_q, a.off_k, a.off_v, a.off_g, a.off_a = self.offsets
+        lib, plan = cuda_library("gla"), rows.plan
+        if plan is not None:
+            first, count = plan.segments()
+            a.seg_first, a.seg_count, a.n_segments = first.data_ptr(), count.data_ptr(), plan.n_segments
+        if plan is None or self.chunk == 0 or plan.longest < self.CHUNKED_FROM:
+            check(lib.gla_step(pointer_to(a), f32, stream()), "gla_step")
+            return
+        (seg_chunk, chunk_first, chunk_count), n_chunks = plan.chunks(self.chunk)
+        HD, HV, f = self.heads * self.dim, self.heads * self.vdim, torch.float32
+        a.seg_chunk, a.chunk_first, a.chunk_count = seg_chunk.data_ptr(), chunk_first.data_ptr(), chunk_count.data_ptr()
+        a.n_chunks, a.chunk = n_chunks, self.chunk
+        a.decay = rows.buffer("gla_decay", n * HD, f, self.device).data_ptr()
+        a.chunk_decay = rows.buffer("gla_chunk_decay", n_chunks * HD, f, self.device).data_ptr()
+        a.states = rows.buffer("gla_states", n_chunks * HD * self.vdim, f, self.device).data_ptr()
+        a.raw = rows.buffer("gla_raw", n * HV, f, self.device).data_ptr()
+        check(lib.gla_chunked(pointer_to(a), f32, stream()), "gla_chunked")
+
+
+class LatentAttention:
+    """Attention over a cache of latent rows shared by the heads (csrc/latent_attn.cu).
+    sizes: heads, dim, rot_dim, vdim, kv_rank, scale, rot (dims, base, scaling). tensors: q, dkv, dkv.norm, uk, uv, o and
+    optionally g (output gate) and sink."""
+
+    def __init__(self, sizes: dict, tensors: dict, eps: float, columns: int, dtype: torch.dtype, device):
+        H, D, R = int(sizes["heads"]), int(sizes["dim"]), int(sizes["rot_dim"])
+        V, rank, rot = int(sizes["vdim"]), int(sizes["kv_rank"]), sizes["rot"]
+        if int(rot["dims"]) != R or R % 2:
+            raise ValueError(f"the rotated part has {R} dimensions, rot.dims is {rot['dims']}: they have to be equal and even")
+        self.heads, self.rank_count, self.rot, self.rot_spec = H, rank, up(R, 16), rot
+        self.dim, self.vdim, self.rank = up(D, 32), up(V, 16), up(rank, 32)
+        self.scale, self.eps, self.dtype, self.device = float(sizes["scale"]), float(eps), dtype, torch.device(device)
+        t = {k: v.to(device) for k, v in tensors.items()}
+        C = t["q"].shape[1]
+        q = t["q"].reshape(H, D + R, C)
+        q = torch.cat([pad_to(q[:, :D], H, self.dim, C), split_halves(q[:, D:], self.rot)], 1).reshape(-1, C)
+        kv = torch.cat([pad_to(t["dkv"][:rank], self.rank, C), split_halves(t["dkv"][rank:], self.rot)], 0)
+        fields = [q.to(dtype), kv.to(dtype)]
+        self.gated = "g" in t
+        if self.gated:
+            fields.append(pad_to(t["g"].reshape(H, V, C), H, self.vdim, C).reshape(-1, C).to(dtype))
+        self.w_in, offsets = stack_fields(fields, 128, columns)
+        self.off_q, self.off_kv, self.off_g = offsets[0], offsets[1], offsets[2] if self.gated else 0
+        self.norm = pad_to(t["dkv.norm"].float(), self.rank)
+        uk = pad_to(t["uk"].reshape(H, D, rank), H, self.dim, self.rank)
+        uv = pad_to(t["uv"].reshape(H, V, rank), H, self.vdim, self.rank)
+        self.w_uk_t = uk.transpose(1, 2).contiguous().to(dtype)
+        self.w_uv = uv.contiguous().to(dtype)
+        self.sink = t["sink"].float().contiguous() if "sink" in t else None
+        o = pad_to(t["o"].reshape(-1, H, V), columns, H, self.vdim).reshape(columns, H * self.vdim)
+        self.out_width = up(H * self.vdim, 128)
+        self.w_out = pad_to(o, columns, self.out_width).to(dtype)
+        self.in_width = self.w_in.shape[0]
+        self.tables: "tuple[Tensor, Tensor] | None" = None
+
+    def new_cache(self, n_slots: int, max_len: int) -> LatentCache:
+        cache = LatentCache(n_slots, self.rank + self.rot, max_len, self.dtype, device=self.device)
+        if self.tables is None or self.tables[0].shape[0] < cache.capacity:
+            self.tables = half_tables(cache.capacity, int(self.rot_spec["dims"]), float(self.rot_spec["base"]),
+                                      self.rot_spec.get("scaling"), self.rot, self.device)
+        return cache
+
+    @staticmethod
+    def cache_bytes(sizes: dict, max_len: int, itemsize: int) -> int:
+        return up(max_len, 64) * (up(int(sizes["kv_rank"]), 32) + up(int(sizes["rot_dim"]), 16)) * itemsize
+
+    def default_chunk(self, rows: int, max_len: int) -> int:
+        """Tiles per chunk of the split kernel for `rows` rows of at most max_len positions: about two blocks per SM, at
+        least two tiles (a chunk's state has to be merged again) and at most 128 chunks."""
+        tiles, blocks = (max_len + LATENT_TILE - 1) // LATENT_TILE, rows * ((self.heads + 15) // 16)
+        wanted = max(1, (2 * SM_COUNT) // blocks)
+        return max(2, (tiles + wanted - 1) // wanted, (tiles + 127) // 128)
+
+    def run(self, proj: Tensor, cache: LatentCache, rows: Rows, out: "Tensor | None") -> None:
+        n, f32, lib = rows.n, int(self.dtype == torch.float32), cuda_library("latent_attn")
+        cos, sin = self.tables
+        a = Latent(proj=proj.data_ptr(), cache=cache.rows.data_ptr(), rows=n, ldp=proj.stride(0), off_q=self.off_q,
+                   off_kv=self.off_kv, off_g=self.off_g, gated=int(self.gated), rotate_q=0, heads=self.heads, dim=self.dim,
+                   rot=self.rot, vdim=self.vdim, rank=self.rank, norm_count=self.rank_count, n_slots=cache.n_slots,
+                   capacity=cache.capacity, table_len=cos.shape[0], scale=self.scale, eps=self.eps,
+                   norm=self.norm.data_ptr(), cos=cos.data_ptr(), sin=sin.data_ptr(),
+                   sink=None if self.sink is None else self.sink.data_ptr(), pos=rows.pos.data_ptr(),
+                   slot_map=rows.slot_map.data_ptr(), status=rows.status.data_ptr())
+        if out is None:
+            check(lib.latent_append(pointer_to(a), f32, stream()), "latent_append")
+            return
+        max_len = min(rows.max_len, cache.capacity)
+        tiles = (max_len + LATENT_TILE - 1) // LATENT_TILE
+        a.max_len, a.chunk_tiles = max_len, rows.chunk_tiles or self.default_chunk(n, max_len)
+        a.max_chunks = (tiles + a.chunk_tiles - 1) // a.chunk_tiles
+        a.out, a.ldo, a.w_uk_t, a.w_uv = out.data_ptr(), out.stride(0), self.w_uk_t.data_ptr(), self.w_uv.data_ptr()
+        a.q_abs = rows.buffer("latent_q", n * self.heads * (self.rank + self.rot), self.dtype, self.device).data_ptr()
+        a.parts = rows.buffer("latent_parts", n * self.heads * a.max_chunks * (self.rank + 4), torch.float32,
+                              self.device).data_ptr()
+        check(lib.latent_query(pointer_to(a), f32, stream()), "latent_query")
+        check(lib.latent_split(pointer_to(a), f32, stream()), "latent_split")
+        check(lib.latent_out(pointer_to(a), f32, stream()), "latent_out")
+
+
+def pointer_to(struct):
+    import ctypes
+
+    return ctypes.byref(struct)
+
+
+MIXERS = {"latent_attention": LatentAttention, "gla": GatedLinearAttention}

@@ -22,9 +22,42 @@ KERNELS = PACKAGE / "csrc"
 INCLUDE = PACKAGE.parent / "include"
 NATIVE = PACKAGE / "_native"
 HEAD_DIM = 128
-LIBRARIES = ("kv_append", "decode_attn", "decode_step", "stream_gemm", "tile_gemm")
+LIBRARIES = ("kv_append", "decode_attn", "decode_step", "stream_gemm", "tile_gemm", "gemm_f32", "latent_attn", "gla")
 
 c_ptr, c_int, c_ll, c_float = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong, ctypes.c_float
+
+
+class GemmRs(ctypes.Structure):
+    """ncb_gemm_rs of include/nanochat_b200.h, field for field."""
+    _fields_ = [("x", c_ptr), ("w", c_ptr), ("y", c_ptr), ("rows", c_ll), ("ldy", c_ll), ("N", c_int), ("K", c_int),
+                ("n_store", c_int), ("epilogue", c_int), ("ss", c_ptr), ("ss_parts", c_int), ("norm_count", c_int),
+                ("eps", c_float), ("scale", c_float), ("h", c_ptr), ("gain", c_ptr), ("x_next", c_ptr), ("ss_next", c_ptr),
+                ("mult", c_float), ("next_w", c_ptr), ("next_bytes", c_ll), ("status", c_ptr)]
+
+
+class Latent(ctypes.Structure):
+    """ncb_latent of include/nanochat_b200.h, field for field."""
+    _fields_ = [("proj", c_ptr), ("q_abs", c_ptr), ("cache", c_ptr), ("out", c_ptr), ("w_uk_t", c_ptr), ("w_uv", c_ptr),
+                ("rows", c_ll), ("ldp", c_ll), ("ldo", c_ll)] + \
+               [(n, c_int) for n in ("off_q", "off_kv", "off_g", "gated", "rotate_q", "heads", "dim", "rot", "vdim", "rank",
+                                     "norm_count", "n_slots", "capacity", "table_len", "max_len", "chunk_tiles",
+                                     "max_chunks")] + \
+               [("scale", c_float), ("eps", c_float)] + \
+               [(n, c_ptr) for n in ("norm", "cos", "sin", "sink", "pos", "slot_map", "parts", "status")]
+
+
+class Gla(ctypes.Structure):
+    """ncb_gla of include/nanochat_b200.h, field for field."""
+    _fields_ = [("proj", c_ptr), ("out", c_ptr), ("rows", c_ll), ("ldp", c_ll), ("ldo", c_ll)] + \
+               [(n, c_int) for n in ("off_q", "off_k", "off_v", "off_g", "off_a", "heads", "dim", "vdim", "rank",
+                                     "norm_count", "n_slots")] + \
+               [(n, c_float) for n in ("q_scale", "inv_tau", "eps")] + \
+               [(n, c_ptr) for n in ("a2", "a2_bias", "norm", "state", "pos", "slot_map", "seg_first", "seg_count",
+                                     "seg_chunk", "chunk_first", "chunk_count")] + \
+               [(n, c_int) for n in ("n_segments", "n_chunks", "chunk")] + \
+               [(n, c_ptr) for n in ("decay", "chunk_decay", "states", "raw", "status")]
+
+
 SIGNATURES = {
     "kv_append": {
         "ncb_status_string": ([c_int], ctypes.c_char_p),
@@ -56,6 +89,8 @@ SIGNATURES = {
         "skinny_gemm": ([c_ptr] * 4 + [c_int] * 5 + [c_ptr], c_int),
         "skinny_gemm_supported": ([c_int] * 4, c_int),
         "skinny_gemm_mix": ([c_ptr] * 4 + [c_float, c_float, c_ptr] + [c_int] * 4 + [c_ptr], c_int),
+        "skinny_gemm_rs": ([c_ptr, c_ptr], c_int),
+        "embed_rs": ([c_ptr] * 6 + [c_ll, c_int, c_int, c_int, c_ptr], c_int),
         "embed_norm": ([c_ptr] * 3 + [c_int] * 3 + [c_ptr], c_int),
         "embed_norm_mix": ([c_ptr] * 4 + [c_float, c_float] + [c_int] * 3 + [c_ptr], c_int),
         "add_rms_norm": ([c_ptr] * 3 + [c_ll, c_int, c_ptr], c_int),
@@ -64,11 +99,21 @@ SIGNATURES = {
         "sample_choice": ([c_ptr] * 7 + [c_float, c_ptr, c_ptr, c_int, c_int, c_ptr, c_int, c_ptr], c_int),
         "greedy_choice": ([c_ptr] * 3 + [c_int] * 2 + [c_ptr, c_int, c_ptr], c_int),
     },
+    "gemm_f32": {"gemm_f32_rs": ([c_ptr, c_ptr], c_int)},
+    "latent_attn": {name: ([c_ptr, c_int, c_ptr], c_int) for name in ("latent_append", "latent_query", "latent_split",
+                                                                       "latent_out")},
+    "gla": {
+        "gla_chunk_tokens": ([c_int], c_int),
+        "gla_step": ([c_ptr, c_int, c_ptr], c_int),
+        "gla_chunked": ([c_ptr, c_int, c_ptr], c_int),
+    },
     "tile_gemm": {
+        "tile_gemm_rs": ([c_ptr, c_ptr], c_int),
         "tile_gemm": ([c_ptr] * 4 + [c_ll, c_int, c_int, c_int, c_ptr, c_ptr], c_int),
         "tile_gemm_form": ([c_ptr] * 4 + [c_ll, c_int, c_int, c_int, c_int, c_ptr, c_ptr], c_int),
     },
     "stream_gemm": {
+        "stream_gemm_rs": ([c_ptr, c_ptr], c_int),
         "stream_gemm_split": ([c_int, c_int, c_int], c_int),
         "stream_gemm": ([c_ptr] * 4 + [c_int] * 6 + [c_ptr, c_ll, c_ptr, c_ptr], c_int),
         "stream_gemm_mix": ([c_ptr] * 4 + [c_float, c_float, c_ptr] + [c_int] * 5 + [c_ptr, c_ll, c_ptr, c_ptr], c_int),
@@ -109,6 +154,14 @@ def build_library(name: str) -> Path:
             subprocess.run([*command(), str(built), str(KERNELS / f"{name}.cu")], check=True)
             built.replace(path)
     return path
+
+
+def build_libraries(names: "tuple[str, ...] | list[str]") -> None:
+    """Build several libraries at once, one nvcc process each."""
+    from concurrent.futures import ThreadPoolExecutor
+
+    with ThreadPoolExecutor(max(len(names), 1)) as pool:
+        list(pool.map(build_library, names))
 
 
 @functools.cache

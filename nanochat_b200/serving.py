@@ -24,7 +24,7 @@ from typing import Protocol
 import numpy as np
 import torch
 
-from .decoder import Decoder
+from .decoder import StepDecoder
 
 
 class Constraint(Protocol):
@@ -145,12 +145,10 @@ class NativeDecoder:
     GPU tests check bit for bit. end_token: the token that ends a continuation without being emitted (the
     reference's BOS, inference/decoder.py:305-307)."""
 
-    def __init__(self, decoder: Decoder, *, end_token: int):
+    def __init__(self, decoder: StepDecoder, *, end_token: int):
         self.decoder, self.end_token, self.batch = decoder, end_token, decoder.n_slots
         self.timings: dict[int, tuple[float, float, float]] = {}
         self.pending: list[tuple[int, list[int]]] = []  # started slots whose prompts await prefill
-        dev, V = decoder.device, decoder.cfg.vocab
-        assert V % 32 == 0, "the allowed-token masks need a vocabulary that is a multiple of 32"
         # the sampled step serves greedy rows too (temperature 0 takes the argmax)
         graph, side, tokens, pos, logits, trace, ctl = decoder._step_graph(self.batch, True, 0, masked=True)
         self.graph, self.side, self.dev_tokens, self.dev_pos, self.ctl = graph, side, tokens, pos, ctl
