@@ -618,6 +618,277 @@ def bench_decoder_d32(rank: int, world: int, device, new_tokens: int, profile: b
             "scaling": "weak (batch-sharded replicas)"}
 
 
+HYBRID_SIZES = {  # equal layers, width and parameters as the closest model of the same name
+    "d20": {"width": 1280, "layers": 20, "heads": 10, "gla_heads": 5, "ff": 3072, "batch": 8, "plain_ff": 5120, "kv_heads": 10},
+    "d32": {"width": 2048, "layers": 32, "heads": 16, "gla_heads": 8, "ff": 4096, "batch": 32, "plain_ff": 8192, "kv_heads": 4}}
+
+
+def hybrid_config(size: dict, max_len: int):
+    """A Pudisun model of real layer sizes: one gated-linear-attention layer, then three latent-attention layers, repeated."""
+    from nanochat_b200.hybrid import HybridConfig
+
+    latent = {"dim": 128, "heads": size["heads"], "kv_rank": 512, "rot_dim": 64, "vdim": 128, "scale": 192 ** -0.5,
+              "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0, "fast": 32.0, "original": 4096, "slow": 1.0}}}
+    gla = {"dim": 128, "heads": size["gla_heads"], "tau": 16.0, "vdim": 256}
+    layers = [{"type": "gla" if i % 4 == 0 else "latent_attention", "mixer": gla if i % 4 == 0 else latent,
+               "mlp": {"ff": size["ff"], "kind": "dense"}} for i in range(size["layers"])]
+    return HybridConfig.from_pudisun({"layers": layers, "width": size["width"], "vocab": 65536, "norm": {"eps": 1e-6},
+                                      "residual_mult": 0.2, "logit_scale": 0.1}, max_len)
+
+
+def bench_hybrid(device, new_tokens: int = 128, profile: str = "") -> dict:
+    """Prefill and decode throughput of Pudisun at two sizes beside this package's other model at equal width, depth and
+    parameter count (random weights, one GPU, device time between CUDA events): prefill of 8 x 511 rows, and decode of the
+    size's batch at contexts of 512 (d20) or uniform in [256, 8192] (d32; caches and states hold synthetic rows). `profile`
+    ("d20-prefill", "d20-decode", ...) brackets one pass or one step with cudaProfilerStart/Stop."""
+    from nanochat_b200.decoder import Decoder, DecoderConfig, DecoderWeights
+    from nanochat_b200.hybrid import HybridDecoder, HybridWeights
+
+    def elapsed(fn, repeats: int) -> float:
+        times = []
+        for _ in range(repeats):
+            start, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            torch.cuda.synchronize()
+            start.record()
+            fn()
+            end.record()
+            torch.cuda.synchronize()
+            times.append(start.elapsed_time(end))
+        return statistics.median(times)
+
+    def bracketed(name, fn):
+        if profile == name:
+            torch.cuda.synchronize()
+            torch.cuda.profiler.start()
+        fn()
+        if profile == name:
+            torch.cuda.synchronize()
+            torch.cuda.profiler.stop()
+
+    result = {}
+    for name, size in HYBRID_SIZES.items():
+        if profile and not profile.startswith(name):
+            continue
+        B = size["batch"]
+        gen = torch.Generator().manual_seed(400)
+        ctx = [511] * B if name == "d20" else torch.randint(256, 8193, (B,), generator=gen).tolist()
+        max_len = max(max(ctx), 511) + new_tokens + 8
+        prompts = torch.randint(0, 65536, (8, 512), generator=gen).tolist()
+        first = torch.randint(0, 65536, (B,), generator=gen).tolist()
+        hybrid = hybrid_config(size, max_len)
+        plain = DecoderConfig(n_layers=size["layers"], hidden=size["width"], n_heads=size["heads"], n_kv_heads=size["kv_heads"],
+                              intermediate=size["plain_ff"], vocab=65536, rope_theta=10000.0, max_len=max_len)
+
+        def pudisun():
+            return HybridDecoder(hybrid, HybridWeights.from_state_dict(HybridWeights.random_state(hybrid, 2, device), hybrid,
+                                                                       device=device), B, device)
+
+        def nanochat():
+            return Decoder(plain, DecoderWeights.random_init(plain, 2, device, on_device=True), B, device)
+
+        row = {"workload": f"{size['layers']} layers, width {size['width']}, vocab 65536; prefill 8 x 511 rows; decode batch {B}, "
+                           + ("context 512" if name == "d20" else "contexts uniform in [256, 8192]")}
+        for model, make in (("pudisun", pudisun), ("nanochat", nanochat)):
+            if profile and model == "nanochat":
+                continue
+            dec = make()
+            dec.prefill(prompts, list(range(8)))
+            bracketed(f"{name}-prefill", lambda: dec.prefill(prompts, list(range(8))))
+            prefill_ms = elapsed(lambda: dec.prefill(prompts, list(range(8))), REPEATS)
+            if name != "d20":  # synthetic cache rows for the long contexts
+                for cache in dec.caches:
+                    if hasattr(cache, "rows"):
+                        cache.rows.normal_()
+            dec.decode_from(first, ctx, 4)
+            if profile == f"{name}-decode":
+                dec.decode_from(first, ctx, 1)
+                bracketed(profile, lambda: dec.decode_from(first, ctx, 1))
+                dec.decode_from(first, ctx, 1)
+            if not profile:
+                dec.decode_from(first, ctx, new_tokens)  # captures the step of this length's chunk size
+            seconds = statistics.median([dec.decode_from(first, ctx, new_tokens)[1] for _ in range(REPEATS if not profile else 1)])
+            row[model] = {"prefill_ms": prefill_ms, "prefill_tokens_per_s": 8 * 511 / prefill_ms * 1e3,
+                          "decode_us_per_step": seconds / new_tokens * 1e6, "decode_tokens_per_s": B * new_tokens / seconds,
+                          "parameters_bytes": weight_bytes(dec), "cache_bytes_per_step": cache_bytes_read(dec, ctx, new_tokens)}
+            del dec
+            torch.cuda.empty_cache()
+        result[name] = row
+    if not profile:
+        result["kernels"] = bench_hybrid_kernels(device)
+    return result
+
+
+def weight_bytes(dec) -> int:
+    """Bytes of weights a decode step streams (the embedding counts once, as the head)."""
+    if hasattr(dec.w, "lm_head"):
+        return sum(t.numel() * 2 for l in dec.w.layers for t in (l.wqkv, l.wo, l.wup, l.wdown)) + dec.w.lm_head.numel() * 2
+    total = dec.w.embed.numel() * 2
+    for l in dec.w.layers:
+        total += 2 * sum(t.numel() for t in (l.mixer.w_in, l.mixer.w_out, l.w_up, l.w_down))
+        total += 2 * sum(getattr(l.mixer, n).numel() for n in ("w_uk_t", "w_uv") if hasattr(l.mixer, n))
+    return total
+
+
+def cache_bytes_read(dec, ctx, new_tokens: int) -> int:
+    """Cache and state bytes a decode step moves half way through the run."""
+    positions = sum(n + new_tokens // 2 for n in ctx)
+    total = 0
+    for cache in dec.caches:
+        if hasattr(cache, "state"):
+            total += 2 * len(ctx) * cache.state[0].numel() * 4
+        elif hasattr(cache, "rows"):
+            total += positions * cache.width * 2
+        else:
+            total += positions * cache.kv_heads * 264
+    return total
+
+
+def bench_hybrid_kernels(device) -> dict:
+    """The token mixers' kernels alone at the d20 and d32 sizes, against HBM bandwidth (decode) or the bf16 tensor peak
+    (prefill). Decode launches rotate over caches that together exceed L2; prefill inputs are larger than or re-read from L2
+    as in a pass."""
+    import ctypes
+
+    from nanochat_b200.mixers import GatedLinearAttention, LatentAttention, RowPlan, Rows
+    from nanochat_b200.native import Gla, Latent, cuda_library, stream
+
+    hbm, _ = peaks()
+    tensor = 1610.8
+    if (ROOT / "MEASURED_PEAKS.json").exists():
+        tensor = float(json.loads((ROOT / "MEASURED_PEAKS.json").read_text())["bf16_tflops"])
+    status = torch.zeros(1, dtype=torch.int32, device=device)
+
+    def per_call(fn, calls: int) -> float:
+        """Microseconds per call of `calls` calls captured in one graph (host launch costs left out), median of REPEATS."""
+        side = torch.cuda.Stream()
+        side.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(side):
+            for i in range(3):
+                fn(i)
+            side.synchronize()
+            graph = torch.cuda.CUDAGraph()
+            with torch.cuda.graph(graph, stream=side):
+                for i in range(calls):
+                    fn(i)
+        times = []
+        for _ in range(REPEATS + 1):
+            start, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            torch.cuda.synchronize()
+            start.record()
+            graph.replay()
+            end.record()
+            torch.cuda.synchronize()
+            times.append(start.elapsed_time(end) * 1e3 / calls)
+        return statistics.median(times[1:])
+
+    def spy(lib, fn, wanted):
+        """The argument structures `fn` passes to the entry points `wanted`, by name."""
+        seen, real = {}, cuda_library(lib)
+
+        class Recorder:
+            def __getattr__(self, name):
+                entry = getattr(real, name)
+                if name not in wanted:
+                    return entry
+
+                def call(args, *rest):
+                    kind = Latent if lib == "latent_attn" else Gla
+                    copy = kind()
+                    ctypes.memmove(ctypes.byref(copy), ctypes.byref(args._obj), ctypes.sizeof(kind))
+                    seen[name] = copy
+                    return entry(args, *rest)
+                return call
+
+        import nanochat_b200.mixers as module
+        original = module.cuda_library
+        module.cuda_library = lambda name: Recorder() if name == lib else original(name)
+        try:
+            fn()
+        finally:
+            module.cuda_library = original
+        return seen
+
+    out = {}
+    gen = torch.Generator(device=device).manual_seed(900)
+    for name, size in HYBRID_SIZES.items():
+        B, C, H = size["batch"], size["width"], size["heads"]
+        cgen = torch.Generator().manual_seed(400)
+        ctx = [576] * B if name == "d20" else torch.randint(256, 8193, (B,), generator=cgen).tolist()
+        cfg = hybrid_config(size, max(ctx) + 8)
+
+        def mixer_of(i, cls):
+            from nanochat_b200.hybrid import HybridConfig, HybridWeights
+            one = HybridConfig(C, 128, [cfg.layers[i].__class__(cfg.layers[i].kind, cfg.layers[i].mixer, 0, 0)], 1e-6)
+            state = HybridWeights.random_state(one, 3, device)
+            return cls(one.layers[0].mixer, {k[7:]: v for k, v in state.items() if k.startswith("l0.mix.")}, 1e-6, C, torch.bfloat16, device)
+
+        latent, gla = mixer_of(1, LatentAttention), mixer_of(0, GatedLinearAttention)
+        pos = torch.tensor([n - 1 for n in ctx], dtype=torch.int32, device=device)
+        slots = torch.arange(B, dtype=torch.int32, device=device)
+        # ---- decode
+        copies = max(2, int(400e6 // (sum(ctx) * 1152)) + 1) if name == "d20" else 2
+        caches = [latent.new_cache(B, max(ctx)) for _ in range(copies)]
+        for c in caches:
+            c.rows.normal_(generator=gen)
+        proj = torch.randn(B, latent.in_width, generator=gen, device=device).bfloat16()
+        mixed = torch.empty(B, latent.out_width, dtype=torch.bfloat16, device=device)
+        rows = Rows(B, pos, slots, max(ctx), status)
+        seen = spy("latent_attn", lambda: latent.run(proj, caches[0], rows, mixed), ("latent_query", "latent_split", "latent_out"))
+        lib = cuda_library("latent_attn")
+
+        def launch(entry, i):
+            a = seen[entry]
+            a.cache = caches[i % copies].rows.data_ptr()
+            assert getattr(lib, entry)(ctypes.byref(a), 0, stream()) == 0
+
+        nbytes = sum(ctx) * 1152 + B * H * 1152
+        us = per_call(lambda i: launch("latent_split", i), 40)
+        out[f"{name} latent_split"] = {"us": us, "bytes": nbytes, "gbs": nbytes / us / 1e3, "frac_hbm": nbytes / us / 1e3 / hbm,
+                                       "chunk_tiles": seen["latent_split"].chunk_tiles}
+        for entry, nbytes in (("latent_query", latent.w_uk_t.numel() * 2 + proj.numel() * 2 + B * H * 1152),
+                              ("latent_out", latent.w_uv.numel() * 2 + B * H * seen["latent_out"].max_chunks * 516 * 4 + mixed.numel() * 2)):
+            us = per_call(lambda i: launch(entry, i), 40)
+            out[f"{name} {entry}"] = {"us": us, "bytes": nbytes, "gbs": nbytes / us / 1e3, "frac_hbm": nbytes / us / 1e3 / hbm}
+        del caches
+        states = [gla.new_cache(B, 64) for _ in range(max(2, int(300e6 // (B * gla.heads * 128 * 256 * 4)) + 1))]
+        proj = torch.randn(B, gla.in_width, generator=gen, device=device).bfloat16()
+        mixed = torch.empty(B, gla.out_width, dtype=torch.bfloat16, device=device)
+        us = per_call(lambda i: gla.run(proj, states[i % len(states)], rows, mixed), 40)
+        nbytes = 2 * states[0].state.numel() * 4 + proj.numel() * 2 + mixed.numel() * 2
+        out[f"{name} gla_step"] = {"us": us, "bytes": nbytes, "gbs": nbytes / us / 1e3, "frac_hbm": nbytes / us / 1e3 / hbm}
+        del states
+        # ---- prefill: 8 prompts of 511 rows
+        import numpy as np
+        n, prompts = 511, 8
+        host = np.repeat(np.arange(prompts, dtype=np.int32), n), np.tile(np.arange(n, dtype=np.int32), prompts)
+        pos_p, slots_p = torch.from_numpy(host[1]).to(device), torch.from_numpy(host[0]).to(device)
+        rows = Rows(n * prompts, pos_p, slots_p, n, status, RowPlan(*host, device))
+        cache = latent.new_cache(prompts, n)
+        proj = torch.randn(n * prompts, latent.in_width, generator=gen, device=device).bfloat16()
+        mixed = torch.empty(n * prompts, latent.out_width, dtype=torch.bfloat16, device=device)
+        seen = spy("latent_attn", lambda: latent.run(proj, cache, rows, mixed), ("latent_append", "latent_gather", "latent_prefill"))
+        flops = prompts * n * (n + 1) // 2 * H * 2 * (192 + 128)
+        us = per_call(lambda i: lib.latent_prefill(ctypes.byref(seen["latent_prefill"]), stream()), 20)
+        out[f"{name} latent_prefill"] = {"us": us, "flops": flops, "tflops": flops / us / 1e6, "frac_tensor": flops / us / 1e6 / tensor}
+        us = per_call(lambda i: lib.latent_append(ctypes.byref(seen["latent_append"]), 0, stream()), 20)
+        nbytes = n * prompts * 2 * (2 * 576 + 2 * H * 64)
+        out[f"{name} latent_append"] = {"us": us, "bytes": nbytes, "gbs": nbytes / us / 1e3, "frac_hbm": nbytes / us / 1e3 / hbm}
+        us = per_call(lambda i: lib.latent_gather(ctypes.byref(seen["latent_gather"]), stream()), 20)
+        out[f"{name} latent_gather"] = {"us": us, "bytes": n * prompts * 2304, "gbs": n * prompts * 2304 / us / 1e3,
+                                        "frac_hbm": n * prompts * 2304 / us / 1e3 / hbm}
+        state = gla.new_cache(prompts, 64)
+        proj = torch.randn(n * prompts, gla.in_width, generator=gen, device=device).bfloat16()
+        mixed = torch.empty(n * prompts, gla.out_width, dtype=torch.bfloat16, device=device)
+        us = per_call(lambda i: gla.run(proj, state, rows, mixed), 20)
+        flops = n * prompts * gla.heads * (4 * 128 * 256 + 64 * (128 + 256))
+        nbytes = (proj.numel() + mixed.numel()) * 2 + 2 * state.state.numel() * 4
+        out[f"{name} gla_chunked"] = {"us": us, "flops": flops, "tflops": flops / us / 1e6, "bytes": nbytes, "gbs": nbytes / us / 1e3,
+                                      "frac_hbm": nbytes / us / 1e3 / hbm, "note": "four launches"}
+        assert int(status.item()) == 0
+        torch.cuda.empty_cache()
+    return out
+
+
 def pin_to_local_cores(local: int, world: int) -> str:
     """With several ranks on one host, give each rank its own slice of the cores this process may use, taken from the
     NUMA node its GPU hangs off when sysfs tells (else an even slice): the end-to-end loop is driven by the host (one
@@ -736,6 +1007,9 @@ def main() -> None:
     ap.add_argument("--longctx", type=int, default=1, help="also time the KV-length-sharded long-context case (0: skip)")
     ap.add_argument("--e2e-steps", type=int, default=200, help="steps of the end-to-end loop (profiling runs shrink it)")
     ap.add_argument("--e2e-parts", type=int, default=0, help="row groups of the end-to-end step that run as parallel graph branches (0: DecodeStep's choice)")
+    ap.add_argument("--hybrid", type=int, default=0, help="also time Pudisun's prefill, decode and kernels beside the closest model "
+                    "(N = 1); 2: print only that")
+    ap.add_argument("--hybrid-profile", default="", help="bracket one pass or step of that for ncu: d20-prefill, d20-decode, d32-...")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
 
@@ -757,6 +1031,12 @@ def main() -> None:
     device = torch.device("cuda", local)
     if world > 1:
         dist.init_process_group("nccl", device_id=device)
+
+    if args.hybrid == 2 and world == 1:
+        with ClockSampler(local) as clocks:
+            result = bench_hybrid(device, profile=args.hybrid_profile)
+        print(json.dumps({"hybrid": result, "clocks": clocks.summary()}))
+        return
 
     def barrier():
         if world > 1:
@@ -911,6 +1191,8 @@ def main() -> None:
     decoder_d32 = bench_decoder_d32(rank, world, device, 2 if d32_profiled else 128, d32_profiled) \
         if args.decoder_d32 else None
 
+    hybrid = bench_hybrid(device) if args.hybrid and world == 1 else None
+
     if rank == 0:
         value = head["total_bytes"] / (head["ms_step"] * 1e-3) / 1e9
         traffic = profiled_traffic() if args.workload == "target8k" and not args.chunk_pages else None
@@ -939,6 +1221,8 @@ def main() -> None:
             line["decoder"] = decoder
         if serving:
             line["serving"] = serving
+        if hybrid:
+            line["hybrid"] = hybrid
         if decoder_d32:
             line["decoder_d32"] = decoder_d32
         if world == 1 and args.cpu_seconds > 0:

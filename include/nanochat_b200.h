@@ -458,7 +458,14 @@ int gla_chunked(const ncb_gla *args, int f32, void *stream);
  *   latent_split   states of chunks of at most chunk_tiles tiles of NCB_LATENT_TILE positions: parts fp32
  *                  [rows][heads][max_chunks][rank + 4]; max_len bounds every position + 1
  *   latent_out     out [rows][ldo] = sigmoid(gate) * w_uv merged(states); w_uv [heads][vdim][rank]; sink fp32 [heads] or
- *                  NULL; gated 0: no gate */
+ *                  NULL; gated 0: no gate
+ * Prompts, bf16 (after latent_append with rotate_q):
+ *   latent_gather  the cached rows of n_contexts sequences (ctx_slot, row range ctx_first [n_contexts + 1]; max_len bounds
+ *                  their lengths) as ctx (latent, columns rank .. ctx_ld zeroed) and ctx_rot; a GEMM of ctx with the
+ *                  per-head rows [w_uk; w_uv] gives ctx_kv, per head [dim | vdim] at stride dim + vdim
+ *   latent_prefill out of row tiles: tile_rows (at most 64) rows from tile_row, the first at position tile_pos of the
+ *                  sequence whose context starts at row tile_ctx. List the tiles that reach furthest first. dim + rot at
+ *                  most 192, vdim at most 128 (latent_prefill_supported) */
 #define NCB_LATENT_TILE 32
 typedef struct {
     void *proj;
@@ -472,8 +479,15 @@ typedef struct {
     const float *norm, *cos, *sin, *sink;
     const int *pos, *slot_map; /* per row; slot_map NULL: row r is slot r */
     float *parts;
+    void *ctx, *ctx_rot, *ctx_kv; /* expanded form: [ctx][ctx_ld], [ctx][rot], [ctx][ctx_kv_ld] */
+    int ctx_ld, ctx_kv_ld, n_contexts, n_tiles;
+    const int *ctx_slot, *ctx_first; /* [n_contexts], [n_contexts + 1] */
+    const int *tile_row, *tile_rows, *tile_ctx, *tile_pos; /* [n_tiles] */
     int *status;
 } ncb_latent;
+int latent_gather(const ncb_latent *args, void *stream);
+int latent_prefill_supported(int dim, int rot, int vdim);
+int latent_prefill(const ncb_latent *args, void *stream);
 int latent_append(const ncb_latent *args, int f32, void *stream);
 int latent_query(const ncb_latent *args, int f32, void *stream);
 int latent_split(const ncb_latent *args, int f32, void *stream);

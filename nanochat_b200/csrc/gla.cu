@@ -8,11 +8,11 @@
  *   - k_gla_step: token by token. A block (or a cluster of blocks that share the norm's sum through distributed shared
  *     memory) owns a slice of vdim of one head and streams the state once per token: a decode step, bound by the state's
  *     bytes, and portions of a few tokens;
- *   - chunks of up to 64 tokens (prefill): k_gla_decay (running sums of log2 alpha inside a chunk), k_gla_chunk_state (each
- *     chunk's own contribution to the state, all chunks in parallel), k_gla_scan (the states at the chunks' starts, and
- *     the sequence's state at the end), k_gla_chunk_out (outputs of a chunk from its starting state and from itself).
- *     Products of decays are only ever formed as 2^(difference of running sums) with a difference <= 0, so no decay,
- *     however strong, over- or underflows into a wrong value.
+ *   - chunks of up to 64 tokens (prefill): k_gla_decay (alpha of every row), k_gla_chunk_state (each chunk's own
+ *     contribution to the state, all chunks in parallel), k_gla_scan (the states at the chunks' starts, and the sequence's
+ *     state at the end), k_gla_chunk_out (outputs of a chunk from its starting state and from itself). Decays between two
+ *     tokens are always products of the alphas between them, never quotients or differences of long sums, so no decay,
+ *     however strong, overflows or loses the small ones beside it.
  * T is the type of projections and outputs: bf16, or float for a model that runs in 32-bit.
  */
 #include "ncb_common.cuh"
@@ -133,39 +133,33 @@ template <typename T> __global__ void __launch_bounds__(STEP_THREADS) k_gla_step
 constexpr int CHUNK_THREADS = 256;
 constexpr int SUB = 16; /* tokens per sub-chunk of the intra-chunk scores */
 
-/* Grid (chunks, ceil(heads dim / 64)): running sums over a chunk's tokens of log2 alpha, fp32 [rows][heads dim]. */
+/* Grid (ceil(rows / DECAY_ROWS), ceil(heads dim / 256)): alpha fp32 [rows][heads dim]; a thread keeps its channel's low-rank
+ * weights across the rows. */
+constexpr int DECAY_ROWS = 16;
 template <typename T> __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_decay(const ncb_gla a) {
-    __shared__ float sum[4][64];
-    extern __shared__ float sm[]; /* a rows of the chunk: [count][rank] */
+    extern __shared__ float sm[]; /* the rows' low-rank inputs, [DECAY_ROWS][rank] */
     asm volatile("griddepcontrol.wait;" ::: "memory");
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-    const int first = a.chunk_first[blockIdx.x], n = a.chunk_count[blockIdx.x], HD = a.heads * a.dim;
+    const long long first = (long long)blockIdx.x * DECAY_ROWS;
+    const int n = (int)(a.rows - first < DECAY_ROWS ? a.rows - first : DECAY_ROWS), HD = a.heads * a.dim;
     for (int i = threadIdx.x; i < n * a.rank; i += CHUNK_THREADS)
         sm[i] = to_f(((const T *)a.proj)[(size_t)(first + i / a.rank) * a.ldp + a.off_a + i % a.rank]);
     __syncthreads();
-    const int ch = blockIdx.y * 64 + (threadIdx.x & 63), tg = threadIdx.x >> 6, per = a.chunk / 4;
-    const int t0 = tg * per, t1 = min(t0 + per, n);
-    const bool live = ch < HD;
-    const float *w = a.a2 + (size_t)(live ? ch : 0) * a.rank;
-    const float bias = live ? a.a2_bias[ch] : 0.f;
-    float run = 0.f, vals[16];
+    const int ch = blockIdx.y * CHUNK_THREADS + threadIdx.x;
+    if (ch >= HD) return;
+    const float *w = a.a2 + (size_t)ch * a.rank;
+    float z[DECAY_ROWS];
 #pragma unroll
-    for (int i = 0; i < 16; i++) {
-        vals[i] = 0.f;
-        if (i < per && t0 + i < t1) {
-            float z = bias;
-            for (int r = 0; r < a.rank; r++) z = fmaf(w[r], sm[(t0 + i) * a.rank + r], z);
-            run += log2_decay(z, a.inv_tau);
-            vals[i] = run;
-        }
+    for (int t = 0; t < DECAY_ROWS; t++) z[t] = a.a2_bias[ch];
+    for (int r = 0; r < a.rank; r++) {
+        const float wr = w[r];
+#pragma unroll
+        for (int t = 0; t < DECAY_ROWS; t++)
+            if (t < n) z[t] = fmaf(wr, sm[t * a.rank + r], z[t]);
     }
-    sum[tg][threadIdx.x & 63] = run;
-    __syncthreads();
-    float before = 0.f;
-    for (int j = 0; j < tg; j++) before += sum[j][threadIdx.x & 63];
 #pragma unroll
-    for (int i = 0; i < 16; i++)
-        if (live && i < per && t0 + i < t1) a.decay[(size_t)(first + t0 + i) * HD + ch] = before + vals[i];
+    for (int t = 0; t < DECAY_ROWS; t++)
+        if (t < n) a.decay[(size_t)(first + t) * HD + ch] = exp2f(log2_decay(z[t], a.inv_tau));
 }
 
 /* acc[4][4] += sum over k of A[k][i0 + i] B[k][j0 + j], both in shared memory with row strides sa and sb. */
@@ -181,7 +175,7 @@ __device__ __forceinline__ void tile_fma(float (&acc)[4][4], const float *A, int
     }
 }
 
-/* Grid (chunks, heads, ceil(vdim / 64)): the state a chunk adds, sum_t (k_t 2^(b_end - b_t)) v_t^T, and its decay. */
+/* Grid (chunks, heads, ceil(vdim / 64)): the state a chunk adds, sum_t (k_t alpha_(t+1) .. alpha_end) v_t^T, and its decay. */
 template <typename T> __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_chunk_state(const ncb_gla a) {
     extern __shared__ float sm[];
     asm volatile("griddepcontrol.wait;" ::: "memory");
@@ -190,15 +184,16 @@ template <typename T> __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_chu
     const int first = a.chunk_first[chunk], n = a.chunk_count[chunk], D = a.dim, V = a.vdim, HD = a.heads * D;
     const int sk = (D + 63) / 64 * 64;
     float *kt = sm, *vt = kt + a.chunk * sk; /* [n][sk], [n][64] */
-    for (int i = tid; i < n * sk; i += CHUNK_THREADS) {
-        const int t = i / sk, d = i % sk;
-        float v = 0.f;
-        if (d < D) {
-            const float *b = a.decay + (size_t)first * HD + h * D + d;
-            v = to_f(((const T *)a.proj)[(size_t)(first + t) * a.ldp + a.off_k + h * D + d]) *
-                exp2f(b[(size_t)(n - 1) * HD] - b[(size_t)t * HD]);
+    for (int d = tid; d < sk; d += CHUNK_THREADS) {
+        const float *al = a.decay + (size_t)first * HD + h * D + d;
+        const T *kp = (const T *)a.proj + (size_t)first * a.ldp + a.off_k + h * D + d;
+        float f = 1.f;
+#pragma unroll 8
+        for (int t = n - 1; t >= 0; t--) {
+            kt[t * sk + d] = d < D ? to_f(kp[(size_t)t * a.ldp]) * f : 0.f;
+            if (d < D) f *= al[(size_t)t * HD];
         }
-        kt[i] = v;
+        if (blockIdx.z == 0 && d < D) a.chunk_decay[(size_t)chunk * HD + h * D + d] = f;
     }
     for (int i = tid; i < n * 64; i += CHUNK_THREADS) {
         const int t = i >> 6, v = v0 + (i & 63);
@@ -217,9 +212,6 @@ template <typename T> __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_chu
                 *reinterpret_cast<float4 *>(out + (size_t)d * V + v0 + tx * 4) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
         }
     }
-    if (blockIdx.z == 0)
-        for (int d = tid; d < D; d += CHUNK_THREADS)
-            a.chunk_decay[(size_t)chunk * HD + h * D + d] = exp2f(a.decay[(size_t)(first + n - 1) * HD + h * D + d]);
 }
 
 /* Grid (heads dim vdim / 4 / 256, segments): states[c] <- the state before chunk c; the slot's state <- the last one. */
@@ -262,13 +254,14 @@ __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_scan(const ncb_gla a) {
 /* Floats of shared memory k_gla_chunk_out takes. */
 __host__ __device__ inline size_t out_floats(int chunk, int D) {
     const int sd = D + 4, sc = chunk + 4;
-    return (size_t)3 * chunk * sd + (size_t)chunk * sd + (size_t)SUB * sd /* q, k, b, scaled k, scaled q */
+    return (size_t)3 * chunk * sd + (size_t)SUB * sd + D /* q, k, alpha, scaled q, product so far */
            + (size_t)chunk * sc + (size_t)16 * sc + 16 * 64 + chunk;
 }
 
-/* Grid (chunks, heads): o_t = (q_t 2^b_t) S + sum_(s <= t) A[t][s] v_s with A[t][s] = sum_d q_td k_sd 2^(b_td - b_sd), then
- * norm and gate. Scores between different sub-chunks of 16 tokens go through the running sum r at the end of the
- * sub-chunk before t's: 2^(b_t - r) 2^(r - b_s), both factors at most 1; inside a sub-chunk each pair is formed directly. */
+/* Grid (chunks, heads): o_t = (q_t alpha_1 .. alpha_t) S + sum_(s <= t) A[t][s] v_s with
+ * A[t][s] = sum_d q_td k_sd alpha_(s+1)d .. alpha_td, then norm and gate. The chunk is walked in sub-chunks of 16 tokens: inside
+ * one, the products run along t for every s; against earlier sub-chunks the decay factors into what q has seen since its
+ * sub-chunk began and what k has seen up to there, and k's rows in shared memory are kept at that value as the walk goes on. */
 template <typename T> __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_chunk_out(const ncb_gla a) {
     extern __shared__ float sm[];
     asm volatile("griddepcontrol.wait;" ::: "memory");
@@ -276,8 +269,8 @@ template <typename T> __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_chu
     const int chunk = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
     const int first = a.chunk_first[chunk], n = a.chunk_count[chunk], D = a.dim, V = a.vdim, HD = a.heads * D, C = a.chunk;
     const int sd = D + 4, sc = C + 4;
-    float *q = sm, *k = q + C * sd, *b = k + C * sd, *ks = b + C * sd, *qs = ks + C * sd;
-    float *at = qs + SUB * sd;                 /* scores transposed: [s][t] */
+    float *q = sm, *k = q + C * sd, *al = k + C * sd, *qs = al + C * sd, *done = qs + SUB * sd;
+    float *at = done + D;                      /* scores transposed: [s][t] */
     float *lt = at + C * sc, *rt = lt + 16 * sc; /* staging of the output product: 16 k-values x (t | 64 columns of v) */
     float *ss = rt + 16 * 64;
     const T *proj = (const T *)a.proj;
@@ -286,44 +279,65 @@ template <typename T> __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_chu
         const T *p = proj + (size_t)(first + t) * a.ldp + h * D + d;
         q[t * sd + d] = t < n ? to_f(p[a.off_q]) * a.q_scale : 0.f;
         k[t * sd + d] = t < n ? to_f(p[a.off_k]) : 0.f;
-        b[t * sd + d] = t < n ? a.decay[(size_t)(first + t) * HD + h * D + d] : 0.f;
+        al[t * sd + d] = t < n ? a.decay[(size_t)(first + t) * HD + h * D + d] : 1.f;
     }
     for (int i = tid; i < C * sc; i += CHUNK_THREADS) at[i] = 0.f;
+    for (int d = tid; d < D; d += CHUNK_THREADS) done[d] = 1.f;
     __syncthreads();
     for (int i0 = 0; i0 < n; i0 += SUB) {
-        const float *ref = b + (i0 - 1) * sd; /* the running sum before this sub-chunk (i0 > 0) */
-        if (i0 > 0) {
-            for (int i = tid; i < i0 * D; i += CHUNK_THREADS) {
-                const int s = i / D, d = i % D;
-                ks[s * sd + d] = k[s * sd + d] * exp2f(ref[d] - b[s * sd + d]);
+        for (int d = tid; d < D; d += CHUNK_THREADS) { /* q with the decays since the sub-chunk's start */
+            float f = 1.f;
+#pragma unroll
+            for (int t = 0; t < SUB; t++) {
+                f *= al[(i0 + t) * sd + d];
+                qs[t * sd + d] = q[(i0 + t) * sd + d] * f;
             }
-            for (int i = tid; i < SUB * D; i += CHUNK_THREADS) {
-                const int t = i / D, d = i % D;
-                qs[t * sd + d] = i0 + t < n ? q[(i0 + t) * sd + d] * exp2f(b[(i0 + t) * sd + d] - ref[d]) : 0.f;
-            }
-            __syncthreads();
         }
-        for (int e = tid; e < SUB * (i0 + SUB); e += CHUNK_THREADS) {
+        __syncthreads();
+        for (int e = tid; e < SUB * i0; e += CHUNK_THREADS) { /* against earlier sub-chunks */
             const int t = e % SUB, s = e / SUB;
-            if (i0 + t >= n || s > i0 + t) continue;
+            const float4 *x = reinterpret_cast<const float4 *>(qs + t * sd), *y = reinterpret_cast<const float4 *>(k + s * sd);
             float v = 0.f;
-            if (s < i0) {
-                const float4 *x = reinterpret_cast<const float4 *>(qs + t * sd), *y = reinterpret_cast<const float4 *>(ks + s * sd);
-                for (int d = 0; d < D / 4; d++) {
-                    const float4 xv = x[d], yv = y[d];
-                    v = fmaf(xv.x, yv.x, v), v = fmaf(xv.y, yv.y, v), v = fmaf(xv.z, yv.z, v), v = fmaf(xv.w, yv.w, v);
-                }
-            } else {
-                const float *x = q + (i0 + t) * sd, *y = k + s * sd, *bt = b + (i0 + t) * sd, *bs = b + s * sd;
-                for (int d = 0; d < D; d++) v = fmaf(x[d] * y[d], exp2f(bt[d] - bs[d]), v);
+            for (int d = 0; d < D / 4; d++) {
+                const float4 xv = x[d], yv = y[d];
+                v = fmaf(xv.x, yv.x, v), v = fmaf(xv.y, yv.y, v), v = fmaf(xv.z, yv.z, v), v = fmaf(xv.w, yv.w, v);
             }
             at[s * sc + i0 + t] = v;
         }
+        { /* inside: thread (s, every 16th channel) runs along t */
+            const int s = tid >> 4, lane = tid & 15;
+            float acc[SUB];
+#pragma unroll
+            for (int t = 0; t < SUB; t++) acc[t] = 0.f;
+            for (int d = lane; d < D; d += 16) {
+                float f = k[(i0 + s) * sd + d];
+#pragma unroll
+                for (int t = 0; t < SUB; t++) {
+                    if (t > s) f *= al[(i0 + t) * sd + d];
+                    if (t >= s) acc[t] = fmaf(q[(i0 + t) * sd + d], f, acc[t]);
+                }
+            }
+#pragma unroll
+            for (int t = 0; t < SUB; t++) {
+                float v = acc[t];
+                for (int o = 8; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+                if (lane == t && t >= s) at[(i0 + s) * sc + i0 + t] = v;
+            }
+        }
         __syncthreads();
-    }
-    for (int i = tid; i < C * D; i += CHUNK_THREADS) { /* q <- q 2^b: what meets the starting state */
-        const int t = i / D, d = i % D;
-        q[t * sd + d] *= exp2f(b[t * sd + d]);
+        for (int d = tid; d < D; d += CHUNK_THREADS) { /* on to the next sub-chunk */
+            const float before = done[d];
+            float f = 1.f;
+#pragma unroll
+            for (int t = SUB - 1; t >= 0; t--) {
+                k[(i0 + t) * sd + d] *= f;
+                f *= al[(i0 + t) * sd + d];
+                q[(i0 + t) * sd + d] = qs[t * sd + d] * before; /* what meets the starting state */
+            }
+            for (int s = 0; s < i0; s++) k[s * sd + d] *= f;
+            done[d] = before * f;
+        }
+        __syncthreads();
     }
     if (tid < C) ss[tid] = 0.f;
     __syncthreads();
@@ -445,10 +459,10 @@ int gla_chunked(const ncb_gla *g, int f32, void *stream_ptr) {
         !g->chunk_count || !g->decay || !g->chunk_decay || !g->states || (g->out && !g->raw))
         return NCB_ERR_ARG;
     cudaStream_t stream = (cudaStream_t)stream_ptr;
-    const size_t decay_smem = (size_t)C * g->rank * 4, state_smem = ((size_t)C * ((g->dim + 63) / 64 * 64) + (size_t)C * 64) * 4,
+    const size_t decay_smem = (size_t)DECAY_ROWS * g->rank * 4, state_smem = ((size_t)C * ((g->dim + 63) / 64 * 64) + (size_t)C * 64) * 4,
                  out_smem = out_floats(C, g->dim) * 4;
     if (decay_smem > 200 * 1024 || out_smem > 226 * 1024) return NCB_ERR_UNSUPPORTED;
-    const dim3 decay_grid(g->n_chunks, (g->heads * g->dim + 63) / 64), state_grid(g->n_chunks, g->heads, (g->vdim + 63) / 64),
+    const dim3 decay_grid((unsigned)((g->rows + DECAY_ROWS - 1) / DECAY_ROWS), (g->heads * g->dim + CHUNK_THREADS - 1) / CHUNK_THREADS), state_grid(g->n_chunks, g->heads, (g->vdim + 63) / 64),
         out_grid(g->n_chunks, g->heads),
         scan_grid((unsigned)(((size_t)g->heads * g->dim * g->vdim / 4 + CHUNK_THREADS - 1) / CHUNK_THREADS), g->n_segments);
     rc = f32 ? launch(k_gla_decay<float>, decay_grid, CHUNK_THREADS, decay_smem, 1, stream, *g)

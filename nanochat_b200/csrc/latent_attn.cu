@@ -569,6 +569,199 @@ template <typename T> __global__ void __launch_bounds__(THREADS) k_latent_append
     }
 }
 
+/* Grid (ceil(longest context / 4), segments): the cached rows of a segment's whole context as matrices, latent part
+ * [ctx][ctx_ld] (columns past rank are zeroed: the GEMM over them wants a multiple of 64) and rotated part [ctx][rot]. */
+__global__ void __launch_bounds__(THREADS) k_latent_gather(const ncb_latent a) {
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    const int seg = blockIdx.y, p = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    const int slot = a.ctx_slot[seg], first = a.ctx_first[seg], len = a.ctx_first[seg + 1] - first;
+    if (p >= len) return;
+    const bool ok = slot >= 0 && slot < a.n_slots && p < a.capacity;
+    if (!ok && p == 0 && lane == 0) flag(a.status, NCB_DEV_BAD_POSITION);
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+    const uint4 *src = reinterpret_cast<const uint4 *>((const bf16 *)a.cache + ((size_t)(ok ? slot : 0) * a.capacity + (ok ? p : 0)) * (a.rank + a.rot));
+    uint4 *c = reinterpret_cast<uint4 *>((bf16 *)a.ctx + (size_t)(first + p) * a.ctx_ld), *k = reinterpret_cast<uint4 *>((bf16 *)a.ctx_rot + (size_t)(first + p) * a.rot);
+    for (int i = lane; i < a.ctx_ld / 8; i += 32) c[i] = ok && i < a.rank / 8 ? src[i] : zero;
+    for (int i = lane; i < a.rot / 8; i += 32) k[i] = ok ? src[a.rank / 8 + i] : zero;
+}
+
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void *src, bool on) { /* 16 bytes, zeros when off */
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
+}
+
+constexpr int PF_ROWS = 64, PF_KEYS = 64; /* query rows and keys per tile: four warps of 16 rows */
+
+/* Grid (heads, row tiles): PF_ROWS consecutive rows of one sequence against its expanded keys and values, one head. Keys
+ * and values of 64 positions per stage (cp.async, two stages); a warp owns 16 rows over the whole range: scores, fp32
+ * softmax and the second product (probabilities as two bf16 terms) in registers. QS: 16-wide steps of the score depth;
+ * VN: 16-wide column tiles of the values (both upper bounds). */
+template <int QS, int VN> __global__ void __launch_bounds__(THREADS, 2) k_latent_prefill(const ncb_latent a) {
+    extern __shared__ __align__(128) uint8_t raw[];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const int h = blockIdx.x, tile = blockIdx.y, depth = a.dim + a.rot, steps = depth / 16, cols = a.vdim / 16;
+    const int krow = depth * 2 + 16, vrow = a.vdim * 2 + 16, stage_bytes = PF_KEYS * (krow + vrow);
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    const int row0 = a.tile_row[tile], n_rows = min(a.tile_rows[tile], PF_ROWS), ctx0 = a.tile_ctx[tile], pos0 = a.tile_pos[tile];
+    const int keys = pos0 + n_rows, n_tiles = (keys + PF_KEYS - 1) / PF_KEYS; /* the last row sees positions < keys */
+    const uint32_t smem = smem_addr(raw);
+    const bf16 *kv = (const bf16 *)a.ctx_kv + (size_t)ctx0 * a.ctx_kv_ld + (size_t)h * (a.dim + a.vdim);
+    const bf16 *kr = (const bf16 *)a.ctx_rot + (size_t)ctx0 * a.rot;
+    auto fetch = [&](int i) {
+        const uint32_t ks = smem + (i & 1) * stage_bytes, vs = ks + PF_KEYS * krow;
+        const int p0 = i * PF_KEYS, nd = a.dim / 8, nr = a.rot / 8, nv = a.vdim / 8;
+        for (int j = tid; j < PF_KEYS * nd; j += THREADS) {
+            const int r = j / nd, c = j % nd;
+            const bool on = p0 + r < keys;
+            cp_async16(ks + r * krow + c * 16, kv + (size_t)(on ? p0 + r : 0) * a.ctx_kv_ld + c * 8, on);
+        }
+        for (int j = tid; j < PF_KEYS * nr; j += THREADS) {
+            const int r = j / nr, c = j % nr;
+            const bool on = p0 + r < keys;
+            cp_async16(ks + r * krow + (nd + c) * 16, kr + (size_t)(on ? p0 + r : 0) * a.rot + c * 8, on);
+        }
+        for (int j = tid; j < PF_KEYS * nv; j += THREADS) {
+            const int r = j / nv, c = j % nv;
+            const bool on = p0 + r < keys;
+            cp_async16(vs + r * vrow + c * 16, kv + (size_t)(on ? p0 + r : 0) * a.ctx_kv_ld + a.dim + c * 8, on);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    fetch(0);
+    uint32_t qf[QS][4];
+    const int lo_row = warp * 16 + g, hi_row = lo_row + 8;
+    const bool lo_on = lo_row < n_rows, hi_on = hi_row < n_rows;
+    {
+        const bf16 *q = (const bf16 *)a.proj + (size_t)row0 * a.ldp + a.off_q + (size_t)h * depth + 2 * t;
+        const bf16 *lo = q + (size_t)lo_row * a.ldp, *hi = q + (size_t)hi_row * a.ldp;
+#pragma unroll
+        for (int i = 0; i < QS; i++) {
+            const bool on = i < steps;
+            qf[i][0] = on && lo_on ? *reinterpret_cast<const uint32_t *>(lo + i * 16) : 0u;
+            qf[i][1] = on && hi_on ? *reinterpret_cast<const uint32_t *>(hi + i * 16) : 0u;
+            qf[i][2] = on && lo_on ? *reinterpret_cast<const uint32_t *>(lo + i * 16 + 8) : 0u;
+            qf[i][3] = on && hi_on ? *reinterpret_cast<const uint32_t *>(hi + i * 16 + 8) : 0u;
+        }
+    }
+    float o[VN][2][4];
+#pragma unroll
+    for (int i = 0; i < VN; i++)
+#pragma unroll
+        for (int j = 0; j < 8; j++) o[i][j >> 2][j & 3] = 0.f;
+    float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
+    const float scale = a.scale * LOG2E;
+    const int lo_pos = pos0 + lo_row, hi_pos = pos0 + hi_row, warp_last = pos0 + warp * 16 + 15;
+    for (int i = 0; i < n_tiles; i++) {
+        if (i + 1 < n_tiles) {
+            fetch(i + 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        const uint32_t ks = smem + (i & 1) * stage_bytes, vs = ks + PF_KEYS * krow;
+        const int p0 = i * PF_KEYS;
+        if (p0 <= warp_last) { /* some row of this warp sees some key of the tile */
+            float s[PF_KEYS / 8][4];
+#pragma unroll
+            for (int n = 0; n < PF_KEYS / 8; n++) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+            const uint32_t kbase = ks + ((lane >> 4) * 8 + (lane & 7)) * krow + ((lane >> 3) & 1) * 16;
+#pragma unroll
+            for (int k = 0; k < QS; k++)
+                if (k < steps) {
+#pragma unroll
+                    for (int n = 0; n < PF_KEYS / 16; n++) {
+                        uint32_t b[4];
+                        ldsm4(b, kbase + n * 16 * krow + k * 32);
+                        mma_bf16(s[2 * n], qf[k][0], qf[k][1], qf[k][2], qf[k][3], b[0], b[1]);
+                        mma_bf16(s[2 * n + 1], qf[k][0], qf[k][1], qf[k][2], qf[k][3], b[2], b[3]);
+                    }
+                }
+            const bool edge = p0 + PF_KEYS - 1 > pos0 + warp * 16; /* the causal border crosses this tile */
+            float mx_lo = m_lo, mx_hi = m_hi;
+#pragma unroll
+            for (int n = 0; n < PF_KEYS / 8; n++)
+#pragma unroll
+                for (int e = 0; e < 2; e++) {
+                    const int p = p0 + n * 8 + 2 * t + e;
+                    s[n][e] = edge && p > lo_pos ? -INFINITY : s[n][e] * scale;
+                    s[n][2 + e] = edge && p > hi_pos ? -INFINITY : s[n][2 + e] * scale;
+                    mx_lo = fmaxf(mx_lo, s[n][e]);
+                    mx_hi = fmaxf(mx_hi, s[n][2 + e]);
+                }
+            mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 1));
+            mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 2));
+            mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 1));
+            mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 2));
+            /* position 0 is visible to every row and in the first tile, so the maxima are finite from there on */
+            if (__any_sync(0xffffffffu, mx_lo != m_lo || mx_hi != m_hi)) {
+                const float al = ex2(m_lo - mx_lo), ah = ex2(m_hi - mx_hi);
+                l_lo *= al, l_hi *= ah;
+#pragma unroll
+                for (int c = 0; c < VN; c++)
+#pragma unroll
+                    for (int n = 0; n < 2; n++) o[c][n][0] *= al, o[c][n][1] *= al, o[c][n][2] *= ah, o[c][n][3] *= ah;
+                m_lo = mx_lo, m_hi = mx_hi;
+            }
+            const uint32_t vbase = vs + (lane & 15) * vrow + (lane >> 4) * 16;
+#pragma unroll
+            for (int j = 0; j < PF_KEYS / 16; j++) { /* 16 keys: two score tiles are one A operand */
+                uint32_t hi[4], lo[4];
+#pragma unroll
+                for (int e = 0; e < 4; e++) { /* e: rows g / g + 8, keys 2 t, + 1 / + 8, + 9 */
+                    const int n = 2 * j + (e >> 1);
+                    const float m = (e & 1) ? m_hi : m_lo;
+                    const float a0 = ex2(s[n][2 * (e & 1)] - m), a1 = ex2(s[n][2 * (e & 1) + 1] - m);
+                    if (e & 1) l_hi += a0 + a1;
+                    else l_lo += a0 + a1;
+                    split_bf16(a0, a1, hi[e], lo[e]);
+                }
+#pragma unroll
+                for (int c = 0; c < VN; c++)
+                    if (c < cols) {
+                        uint32_t b[4];
+                        ldsm4_t(b, vbase + j * 16 * vrow + c * 32);
+                        mma_bf16(o[c][0], hi[0], hi[1], hi[2], hi[3], b[0], b[1]);
+                        mma_bf16(o[c][1], hi[0], hi[1], hi[2], hi[3], b[2], b[3]);
+                        mma_bf16(o[c][0], lo[0], lo[1], lo[2], lo[3], b[0], b[1]);
+                        mma_bf16(o[c][1], lo[0], lo[1], lo[2], lo[3], b[2], b[3]);
+                    }
+            }
+        }
+        __syncthreads(); /* the stage may be overwritten */
+    }
+    l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1);
+    l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
+    l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
+    l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
+    float f_lo = 1.f, f_hi = 1.f;
+    if (a.sink) {
+        const float sink = a.sink[h] * LOG2E, ml = fmaxf(m_lo, sink), mh = fmaxf(m_hi, sink);
+        f_lo = exp2f(m_lo - ml), f_hi = exp2f(m_hi - mh);
+        l_lo = fmaf(l_lo, f_lo, exp2f(sink - ml)), l_hi = fmaf(l_hi, f_hi, exp2f(sink - mh));
+    }
+    f_lo /= l_lo, f_hi /= l_hi;
+#pragma unroll
+    for (int c = 0; c < VN; c++)
+        if (c < cols)
+#pragma unroll
+            for (int n = 0; n < 2; n++)
+#pragma unroll
+                for (int r = 0; r < 2; r++)
+                    if (r ? hi_on : lo_on) {
+                        const int row = row0 + (r ? hi_row : lo_row), at = h * a.vdim + c * 16 + n * 8 + 2 * t;
+                        const float f = r ? f_hi : f_lo;
+                        float g0 = 1.f, g1 = 1.f;
+                        if (a.gated) {
+                            const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>((const bf16 *)a.proj + (size_t)row * a.ldp + a.off_g + at));
+                            g0 = 1.f / (1.f + expf(-z.x)), g1 = 1.f / (1.f + expf(-z.y));
+                        }
+                        *reinterpret_cast<uint32_t *>((bf16 *)a.out + (size_t)row * a.ldo + at) =
+                            pack_bf16(o[c][n][2 * r] * f * g0, o[c][n][2 * r + 1] * f * g1);
+                    }
+}
+
 /* ---- host side ------------------------------------------------------------------------------------------------------ */
 
 template <typename... A>
@@ -669,6 +862,36 @@ int latent_out(const ncb_latent *g, int f32, void *stream) {
     if (smem > 200 * 1024) return NCB_ERR_UNSUPPORTED;
     const dim3 grid(g->heads, (unsigned)g->rows);
     return f32 ? launch(k_latent_out_any<float>, grid, smem, 1, s, *g) : launch(k_latent_out_any<bf16>, grid, smem, 1, s, *g);
+}
+
+int latent_gather(const ncb_latent *g, void *stream) {
+    if (!g) return NCB_ERR_ARG;
+    const int rc = check(*g);
+    if (rc != NCB_OK || g->n_contexts == 0) return rc;
+    if (!g->ctx || !g->ctx_rot || !g->ctx_slot || !g->ctx_first || g->n_contexts < 0 || g->n_contexts > 65535 || g->max_len <= 0 ||
+        g->ctx_ld < g->rank || g->ctx_ld % 8)
+        return NCB_ERR_ARG;
+    return launch(k_latent_gather, dim3((g->max_len + 3) / 4, g->n_contexts), 0, 1, (cudaStream_t)stream, *g);
+}
+
+/* 1 if latent_prefill takes these (padded) sizes. */
+int latent_prefill_supported(int dim, int rot, int vdim) {
+    return dim > 0 && rot > 0 && vdim > 0 && dim % 32 == 0 && rot % 16 == 0 && vdim % 16 == 0 && dim + rot <= 192 && vdim <= 128;
+}
+
+int latent_prefill(const ncb_latent *g, void *stream) {
+    if (!g) return NCB_ERR_ARG;
+    const int rc = check(*g);
+    if (rc != NCB_OK || g->n_tiles == 0) return rc;
+    if (!latent_prefill_supported(g->dim, g->rot, g->vdim)) return NCB_ERR_UNSUPPORTED;
+    if (!g->ctx_kv || !g->ctx_rot || !g->out || !g->tile_row || !g->tile_rows || !g->tile_ctx || !g->tile_pos || g->n_tiles < 0 ||
+        g->n_tiles > 65535 || g->ctx_kv_ld < g->heads * (g->dim + g->vdim) || g->ctx_kv_ld % 8 || g->ldo % 2)
+        return NCB_ERR_ARG;
+    const dim3 grid(g->heads, g->n_tiles);
+    const size_t smem = (size_t)2 * PF_KEYS * ((g->dim + g->rot) * 2 + 16 + g->vdim * 2 + 16);
+    cudaStream_t s = (cudaStream_t)stream;
+    return g->dim + g->rot <= 128 ? launch(k_latent_prefill<8, 8>, grid, smem, 1, s, *g)
+                                  : launch(k_latent_prefill<12, 8>, grid, smem, 1, s, *g);
 }
 
 } /* extern "C" */

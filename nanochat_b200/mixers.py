@@ -16,7 +16,7 @@ import torch
 from torch import Tensor
 
 from .kv_cache import LatentCache, StateCache
-from .native import Gla, Latent, check, cuda_library, stream
+from .native import GemmRs, Gla, Latent, check, cuda_library, stream
 from .rotary import half_tables
 
 LATENT_TILE = 32  # NCB_LATENT_TILE
@@ -86,6 +86,23 @@ class RowPlan:
 
     def segments(self) -> list[Tensor]:
         return self.upload("segments", [self.first, self.count])
+
+    def contexts(self) -> list[Tensor]:
+        """[segment's slot, first row of its context (n + 1)]: the contexts (all positions up to the segment's end) laid
+        out one after the other."""
+        return self.upload("contexts", [self.slots, np.concatenate([[0], np.cumsum(self.starts + self.count)])])
+
+    def row_tiles(self, size: int) -> tuple[list[Tensor], int]:
+        """([tile's first row, its rows, its context's first row, its first position], number of tiles) of at most `size`
+        rows of one segment, those that reach furthest into their sequences first."""
+        per = (self.count + size - 1) // size
+        within = np.arange(per.sum(), dtype=np.int32) - np.repeat(np.cumsum(per) - per, per)
+        first = np.repeat(self.first, per) + within * size
+        rows = np.minimum(size, np.repeat(self.first + self.count, per) - first)
+        context = np.repeat(np.cumsum(self.starts + self.count) - (self.starts + self.count), per)
+        pos = np.repeat(self.starts, per) + within * size
+        order = np.argsort(-pos.astype(np.int64), kind="stable")
+        return self.upload(("tiles", size), [v[order] for v in (first, rows, context, pos)]), len(first)
 
     def chunks(self, size: int) -> tuple[list[Tensor], int]:
         """([segment's first chunk (n + 1), chunk's first row, chunk's rows], number of chunks) for chunks of `size` rows."""
@@ -208,6 +225,11 @@ class LatentAttention:
         self.norm = pad_to(t["dkv.norm"].float(), self.rank)
         uk = pad_to(t["uk"].reshape(H, D, rank), H, self.dim, self.rank)
         uv = pad_to(t["uv"].reshape(H, V, rank), H, self.vdim, self.rank)
+        self.expanded = dtype == torch.bfloat16 and bool(
+            cuda_library("latent_attn").latent_prefill_supported(self.dim, self.rot, self.vdim))
+        if self.expanded:  # both expansions of a latent row as one GEMM: per head the key's rows, then the value's
+            both = torch.cat([uk, uv], 1).reshape(H * (self.dim + self.vdim), self.rank)
+            self.w_ukv = pad_to(both, up(both.shape[0], 128), up(self.rank, 64)).to(dtype)
         self.w_uk_t = uk.transpose(1, 2).contiguous().to(dtype)
         self.w_uv = uv.contiguous().to(dtype)
         self.sink = t["sink"].float().contiguous() if "sink" in t else None
@@ -235,6 +257,37 @@ class LatentAttention:
         wanted = max(1, (2 * SM_COUNT) // blocks)
         return max(2, (tiles + wanted - 1) // wanted, (tiles + 127) // 128)
 
+    ROW_TILE = 64  # rows per tile of latent_prefill
+
+    def expands(self, plan: RowPlan) -> bool:
+        """Whether a pass is cheaper with expanded keys and values: expanding every context once and attending in head
+        space, against attending in latent space (whose kernel reads the cache once per row and head tile)."""
+        if not self.expanded:
+            return False
+        count, length = plan.count.astype(np.float64), (plan.starts + plan.count).astype(np.float64)
+        pairs = float((count * (length - count / 2)).sum())
+        expanded = float(length.sum()) * self.rank * (self.dim + self.vdim) + pairs * (self.dim + self.rot + self.vdim)
+        return expanded < 2.0 * pairs * (2 * self.rank + self.rot)
+
+    def run_expanded(self, a: Latent, rows: Rows) -> None:
+        plan, lib, bf = rows.plan, cuda_library("latent_attn"), torch.bfloat16
+        n_ctx = int((plan.starts + plan.count).sum())
+        (slots, first), (tiles, a.n_tiles) = plan.contexts(), plan.row_tiles(self.ROW_TILE)
+        N, K = self.w_ukv.shape
+        a.rotate_q, a.max_len, a.n_contexts = 1, int((plan.starts + plan.count).max()), plan.n_segments
+        a.ctx_slot, a.ctx_first = slots.data_ptr(), first.data_ptr()
+        a.tile_row, a.tile_rows, a.tile_ctx, a.tile_pos = (t.data_ptr() for t in tiles)
+        a.ctx_ld, a.ctx_kv_ld = K, N
+        a.ctx = rows.buffer("latent_ctx", n_ctx * K, bf, self.device).data_ptr()
+        a.ctx_rot = rows.buffer("latent_ctx_rot", n_ctx * self.rot, bf, self.device).data_ptr()
+        a.ctx_kv = rows.buffer("latent_ctx_kv", n_ctx * N, bf, self.device).data_ptr()
+        check(lib.latent_append(pointer_to(a), 0, stream()), "latent_append")
+        check(lib.latent_gather(pointer_to(a), stream()), "latent_gather")
+        g = GemmRs(x=a.ctx, w=self.w_ukv.data_ptr(), y=a.ctx_kv, rows=n_ctx, ldy=N, N=N, K=K, n_store=N, epilogue=0, scale=1.0,
+                   status=a.status)
+        check(cuda_library("tile_gemm").tile_gemm_rs(pointer_to(g), stream()), "tile_gemm_rs")
+        check(lib.latent_prefill(pointer_to(a), stream()), "latent_prefill")
+
     def run(self, proj: Tensor, cache: LatentCache, rows: Rows, out: "Tensor | None") -> None:
         n, f32, lib = rows.n, int(self.dtype == torch.float32), cuda_library("latent_attn")
         cos, sin = self.tables
@@ -249,10 +302,14 @@ class LatentAttention:
             check(lib.latent_append(pointer_to(a), f32, stream()), "latent_append")
             return
         max_len = min(rows.max_len, cache.capacity)
+        a.out, a.ldo = out.data_ptr(), out.stride(0)
+        if rows.plan is not None and self.expands(rows.plan):
+            self.run_expanded(a, rows)
+            return
         tiles = (max_len + LATENT_TILE - 1) // LATENT_TILE
         a.max_len, a.chunk_tiles = max_len, rows.chunk_tiles or self.default_chunk(n, max_len)
         a.max_chunks = (tiles + a.chunk_tiles - 1) // a.chunk_tiles
-        a.out, a.ldo, a.w_uk_t, a.w_uv = out.data_ptr(), out.stride(0), self.w_uk_t.data_ptr(), self.w_uv.data_ptr()
+        a.w_uk_t, a.w_uv = self.w_uk_t.data_ptr(), self.w_uv.data_ptr()
         a.q_abs = rows.buffer("latent_q", n * self.heads * (self.rank + self.rot), self.dtype, self.device).data_ptr()
         a.parts = rows.buffer("latent_parts", n * self.heads * a.max_chunks * (self.rank + 4), torch.float32,
                               self.device).data_ptr()

@@ -43,7 +43,9 @@ class Latent(ctypes.Structure):
                                      "norm_count", "n_slots", "capacity", "table_len", "max_len", "chunk_tiles",
                                      "max_chunks")] + \
                [("scale", c_float), ("eps", c_float)] + \
-               [(n, c_ptr) for n in ("norm", "cos", "sin", "sink", "pos", "slot_map", "parts", "status")]
+               [(n, c_ptr) for n in ("norm", "cos", "sin", "sink", "pos", "slot_map", "parts", "ctx", "ctx_rot", "ctx_kv")] + \
+               [(n, c_int) for n in ("ctx_ld", "ctx_kv_ld", "n_contexts", "n_tiles")] + \
+               [(n, c_ptr) for n in ("ctx_slot", "ctx_first", "tile_row", "tile_rows", "tile_ctx", "tile_pos", "status")]
 
 
 class Gla(ctypes.Structure):
@@ -100,8 +102,15 @@ SIGNATURES = {
         "greedy_choice": ([c_ptr] * 3 + [c_int] * 2 + [c_ptr, c_int, c_ptr], c_int),
     },
     "gemm_f32": {"gemm_f32_rs": ([c_ptr, c_ptr], c_int)},
-    "latent_attn": {name: ([c_ptr, c_int, c_ptr], c_int) for name in ("latent_append", "latent_query", "latent_split",
-                                                                       "latent_out")},
+    "latent_attn": {
+        "latent_append": ([c_ptr, c_int, c_ptr], c_int),
+        "latent_query": ([c_ptr, c_int, c_ptr], c_int),
+        "latent_split": ([c_ptr, c_int, c_ptr], c_int),
+        "latent_out": ([c_ptr, c_int, c_ptr], c_int),
+        "latent_gather": ([c_ptr, c_ptr], c_int),
+        "latent_prefill_supported": ([c_int] * 3, c_int),
+        "latent_prefill": ([c_ptr, c_ptr], c_int),
+    },
     "gla": {
         "gla_chunk_tokens": ([c_int], c_int),
         "gla_step": ([c_ptr, c_int, c_ptr], c_int),
