@@ -832,7 +832,7 @@ def bench_hybrid_kernels(device) -> dict:
             c.rows.normal_(generator=gen)
         proj = torch.randn(B, latent.in_width, generator=gen, device=device).bfloat16()
         mixed = torch.empty(B, latent.out_width, dtype=torch.bfloat16, device=device)
-        rows = Rows(B, pos, slots, max(ctx), status)
+        rows = Rows(B, pos, slots, max(ctx), status, chunk_tiles=latent.chunk_for(ctx, max(ctx)))
         seen = spy("latent_attn", lambda: latent.run(proj, caches[0], rows, mixed), ("latent_query", "latent_split", "latent_out"))
         lib = cuda_library("latent_attn")
 

@@ -37,13 +37,12 @@ __device__ __forceinline__ float log2_decay(float z, float inv_tau) {
 __device__ __forceinline__ float silu(float z) { return z / (1.f + expf(-z)); }
 
 constexpr int STEP_THREADS = 256;
+constexpr int AHEAD_ROWS = 8; /* state rows per thread that are loaded ahead */
 
 /* Grid (slices, heads, segments), cluster (slices, 1, 1); segment z = rows first[z] .. + count[z] - 1 of one slot at
  * ascending positions (first NULL: row z alone). */
 template <typename T> __global__ void __launch_bounds__(STEP_THREADS) k_gla_step(const ncb_gla a) {
     extern __shared__ float sm[];
-    asm volatile("griddepcontrol.wait;" ::: "memory");
-    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     const int tid = threadIdx.x, h = blockIdx.y, slices = gridDim.x, rank = blockIdx.x;
     const int D = a.dim, V = a.vdim, VS = V / slices, v0 = rank * VS;
     const int groups = VS / 4, dgs = STEP_THREADS / groups;
@@ -53,6 +52,19 @@ template <typename T> __global__ void __launch_bounds__(STEP_THREADS) k_gla_step
     cg::cluster_group cluster = cg::this_cluster();
     const int pos0 = a.pos[first], slot = a.slot_map ? a.slot_map[first] : first;
     const bool bad = pos0 >= 0 && (slot < 0 || slot >= a.n_slots);
+    float *state = a.state + ((size_t)(bad ? 0 : slot) * a.heads + h) * D * V;
+    const int c = tid % groups, dg = tid / groups;
+    /* Positions, slots and this state were last written many launches ago (the launch before this one writes the projection
+     * alone), so the state's first elements start towards registers before the dependency wait. */
+    float4 ahead[AHEAD_ROWS];
+#pragma unroll
+    for (int i = 0; i < AHEAD_ROWS; i++) {
+        const int d = dg + i * dgs;
+        ahead[i] = pos0 > 0 && !bad && dg < dgs && d < D ? *reinterpret_cast<const float4 *>(state + (size_t)d * V + v0 + 4 * c)
+                                                         : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     if (bad && tid == 0) flag(a.status, NCB_DEV_BAD_POSITION);
     if (pos0 < 0 || bad) { /* an idle row: no state touched, a zero output (every block of the cluster takes this exit) */
         if (a.out)
@@ -60,8 +72,6 @@ template <typename T> __global__ void __launch_bounds__(STEP_THREADS) k_gla_step
                 ((T *)a.out)[(size_t)(first + i / VS) * a.ldo + h * V + v0 + i % VS] = from_f<T>(0.f);
         return;
     }
-    float *state = a.state + ((size_t)slot * a.heads + h) * D * V;
-    const int c = tid % groups, dg = tid / groups;
     for (int t = 0; t < count; t++) {
         const int row = first + t;
         const T *p = (const T *)a.proj + (size_t)row * a.ldp;
@@ -79,17 +89,25 @@ template <typename T> __global__ void __launch_bounds__(STEP_THREADS) k_gla_step
             const T *vp = p + a.off_v + h * V + v0 + 4 * c;
             const float vx = to_f(vp[0]), vy = to_f(vp[1]), vz = to_f(vp[2]), vw = to_f(vp[3]);
             float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 4
-            for (int d = dg; d < D; d += dgs) {
-                float4 *sp = reinterpret_cast<float4 *>(state + (size_t)d * V + v0 + 4 * c);
-                float4 s = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *sp;
+            auto update = [&](int d, float4 s) {
                 const float al = alpha[d], kd = k[d], qd = q[d];
                 s.x = fmaf(al, s.x, kd * vx), s.y = fmaf(al, s.y, kd * vy);
                 s.z = fmaf(al, s.z, kd * vz), s.w = fmaf(al, s.w, kd * vw);
-                *sp = s;
+                *reinterpret_cast<float4 *>(state + (size_t)d * V + v0 + 4 * c) = s;
                 acc.x = fmaf(qd, s.x, acc.x), acc.y = fmaf(qd, s.y, acc.y);
                 acc.z = fmaf(qd, s.z, acc.z), acc.w = fmaf(qd, s.w, acc.w);
+            };
+            auto stored = [&](int d) {
+                return fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4 *>(state + (size_t)d * V + v0 + 4 * c);
+            };
+            int d = dg;
+            if (t == 0) {
+#pragma unroll
+                for (int i = 0; i < AHEAD_ROWS; i++, d += dgs)
+                    if (d < D) update(d, ahead[i]);
             }
+#pragma unroll 4
+            for (; d < D; d += dgs) update(d, stored(d));
             *reinterpret_cast<float4 *>(part + dg * VS + 4 * c) = acc;
         }
         __syncthreads();
@@ -386,6 +404,384 @@ template <typename T> __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_chu
     }
 }
 
+/* ---- chunked form on the tensor cores (bf16 projections, dim <= 256) ------------------------------------------------------ */
+
+__device__ __forceinline__ void mma_bf16(float *d, const uint32_t *a, uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, "
+                 "{%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldsm4(uint32_t *r, uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t *r, uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ uint32_t bits(__nv_bfloat162 v) { return *reinterpret_cast<uint32_t *>(&v); }
+/* hi = bf16(v), lo = bf16(v - hi) of two values: 16 bits of mantissa. */
+__device__ __forceinline__ void split2(float x, float y, uint32_t &hi, uint32_t &lo) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+    const float2 f = __bfloat1622float2(h);
+    hi = bits(h);
+    lo = bits(__floats2bfloat162_rn(x - f.x, y - f.y));
+}
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void *src, bool on) { /* 16 bytes, zeros when off */
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
+}
+constexpr int VT = 256; /* columns of v a block handles at a time: eight warps of 32 */
+
+/* The chunk's v rows, columns v0 .. v0 + VT, as bf16 [C][VT + 8]; rows past n and columns past V are zero. */
+template <int C> __device__ __forceinline__ void stage_v(const ncb_gla &a, uint32_t dst, int first, int n, int h, int v0) {
+    const bf16 *v = (const bf16 *)a.proj + (size_t)first * a.ldp + a.off_v + h * a.vdim;
+    for (int i = threadIdx.x; i < C * (VT / 8); i += CHUNK_THREADS) {
+        const int t = i / (VT / 8), c = v0 + i % (VT / 8) * 8;
+        const bool on = t < n && c < a.vdim;
+        cp_async16(dst + (t * (VT + 8) + i % (VT / 8) * 8) * 2, v + (on ? (size_t)t * a.ldp + c : 0), on);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+}
+
+/* k_gla_chunk_state with the decayed k as three bf16 terms (24 bits, v is exact): U [dim][vdim] = sum over tokens, dim as M.
+ * Grid (chunks, heads, ceil(vdim / VT)). C = 64 for dim <= 128, 32 for dim <= 256: C dim / 256 <= 32 values per thread. */
+template <int C> __host__ __device__ inline size_t state_mma_bytes(int D) {
+    const size_t work = (size_t)C * D * 4 + (size_t)C * D * 2, terms = (size_t)3 * C * (D + 8) * 2;
+    return (size_t)C * (VT + 8) * 2 + (work > terms ? work : terms) + (size_t)2 * D * 4;
+}
+template <int C> __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_chunk_state_mma(const ncb_gla a) {
+    extern __shared__ __align__(16) uint8_t raw[];
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    const int chunk = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * VT, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int first = a.chunk_first[chunk], n = a.chunk_count[chunk], D = a.dim, V = a.vdim, HD = a.heads * D;
+    constexpr int HALF = C / 2;
+    bf16 *vs = reinterpret_cast<bf16 *>(raw);
+    uint8_t *rest = raw + C * (VT + 8) * 2;
+    float *al = reinterpret_cast<float *>(rest);           /* [C][D], then the terms of k over it */
+    bf16 *ks = reinterpret_cast<bf16 *>(al + C * D);       /* [C][D] */
+    bf16 *terms = reinterpret_cast<bf16 *>(rest);          /* [3][C][D + 8] */
+    const size_t work = (size_t)C * D * 6, three = (size_t)3 * C * (D + 8) * 2;
+    float *total = reinterpret_cast<float *>(rest + (work > three ? work : three)); /* [2][D]: the halves' products */
+    stage_v<C>(a, smem_addr(vs), first, n, h, v0);
+    for (int i = tid; i < C * (D / 4); i += CHUNK_THREADS) {
+        const int t = i / (D / 4), d = i % (D / 4) * 4;
+        cp_async16(smem_addr(al + t * D + d), a.decay + (size_t)(first + (t < n ? t : 0)) * HD + h * D + d, t < n);
+    }
+    for (int i = tid; i < C * (D / 8); i += CHUNK_THREADS) {
+        const int t = i / (D / 8), d = i % (D / 8) * 8;
+        cp_async16(smem_addr(ks + t * D + d), (const bf16 *)a.proj + (size_t)(first + (t < n ? t : 0)) * a.ldp + a.off_k + h * D + d, t < n);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    /* suffix products: item (d, half) walks its half of the tokens backwards */
+    float vals[32];
+#pragma unroll
+    for (int j = 0; j < 32 / HALF; j++) {
+        const int item = tid + j * CHUNK_THREADS, d = item % D, half = item / D;
+        if (item < 2 * D) {
+            float f = 1.f;
+#pragma unroll
+            for (int i = HALF - 1; i >= 0; i--) {
+                const int t = half * HALF + i;
+                vals[j * HALF + i] = to_f(ks[t * D + d]) * f;
+                if (t < n) f *= al[t * D + d];
+            }
+            total[half * D + d] = f;
+        }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int j = 0; j < 32 / HALF; j++) {
+        const int item = tid + j * CHUNK_THREADS, d = item % D, half = item / D;
+        if (item < 2 * D) {
+            const float after = half == 0 ? total[D + d] : 1.f;
+#pragma unroll
+            for (int i = 0; i < HALF; i++) {
+                const float x = vals[j * HALF + i] * after;
+                const bf16 hi = __float2bfloat16_rn(x), mid = __float2bfloat16_rn(x - to_f(hi)), lo = __float2bfloat16_rn(x - to_f(hi) - to_f(mid));
+                bf16 *p = terms + (half * HALF + i) * (D + 8) + d;
+                p[0] = hi, p[C * (D + 8)] = mid, p[2 * C * (D + 8)] = lo;
+            }
+            if (half == 0 && blockIdx.z == 0) a.chunk_decay[(size_t)chunk * HD + h * D + d] = total[d] * after;
+        }
+    }
+    __syncthreads();
+    float *out = a.states + ((size_t)chunk * a.heads + h) * D * V;
+    const int g = lane >> 2, t2 = (lane & 3) * 2, col0 = warp * 32;
+    if (v0 + col0 >= V) return;
+    const uint32_t vb = smem_addr(vs) + ((lane & 15) * (VT + 8) + col0 + (lane >> 4) * 8) * 2;
+    const uint32_t kb = smem_addr(terms) + (((lane >> 4) * 8 + (lane & 7)) * (D + 8) + ((lane >> 3) & 1) * 8) * 2;
+    for (int m0 = 0; m0 < D; m0 += 32) { /* two 16-row tiles of key channels at a time */
+        float acc[2][4][4];
+#pragma unroll
+        for (int i = 0; i < 32; i++) acc[i >> 4][(i >> 2) & 3][i & 3] = 0.f;
+        const int mts = D - m0 >= 32 ? 2 : 1;
+#pragma unroll
+        for (int k = 0; k < C / 16; k++) {
+            uint32_t b[2][4];
+            ldsm4_t(b[0], vb + k * 16 * (VT + 8) * 2);
+            ldsm4_t(b[1], vb + k * 16 * (VT + 8) * 2 + 32);
+#pragma unroll
+            for (int m = 0; m < 2; m++)
+                if (m < mts) {
+#pragma unroll
+                    for (int e = 0; e < 3; e++) {
+                        uint32_t x[4];
+                        ldsm4_t(x, kb + ((e * C + k * 16) * (D + 8) + m0 + m * 16) * 2);
+#pragma unroll
+                        for (int c = 0; c < 4; c++) mma_bf16(acc[m][c], x, b[c >> 1][(c & 1) * 2], b[c >> 1][(c & 1) * 2 + 1]);
+                    }
+                }
+        }
+#pragma unroll
+        for (int m = 0; m < 2; m++)
+#pragma unroll
+            for (int c = 0; c < 4; c++) {
+                const int v = v0 + col0 + c * 8 + t2, d = m0 + m * 16 + g;
+                if (m < mts && v < V) {
+                    *reinterpret_cast<float2 *>(out + (size_t)d * V + v) = make_float2(acc[m][c][0], acc[m][c][1]);
+                    *reinterpret_cast<float2 *>(out + (size_t)(d + 8) * V + v) = make_float2(acc[m][c][2], acc[m][c][3]);
+                }
+            }
+    }
+}
+
+/* k_gla_chunk_out with its output product on the tensor cores: what meets the starting state and the state itself as two bf16
+ * terms each, the intra-chunk scores as two terms against v. Grid (chunks, heads), C = 16 MT. */
+template <int MT> __host__ __device__ inline size_t out_mma_bytes(int D) {
+    constexpr int C = 16 * MT;
+    return ((size_t)3 * C * (D + 4) + (size_t)SUB * (D + 4) + D + 8 * C + C) * 4 /* q, k, alpha, scaled q, product, sums */
+           + (size_t)2 * C * (C + 8) * 2 + (size_t)2 * C * (D + 8) * 2 + (size_t)C * (VT + 8) * 2;
+}
+template <int MT> __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_chunk_out_mma(const ncb_gla a) {
+    extern __shared__ __align__(16) uint8_t raw[];
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    constexpr int C = 16 * MT, sc = C + 8;
+    const int chunk = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int first = a.chunk_first[chunk], n = a.chunk_count[chunk], D = a.dim, V = a.vdim, HD = a.heads * D;
+    const int sd = D + 4, sq = D + 8;
+    bf16 *vs = reinterpret_cast<bf16 *>(raw);                     /* [C][VT + 8] */
+    bf16 *at = vs + C * (VT + 8);                                 /* [2][C][sc]: scores' terms, [t][s] */
+    bf16 *qt = at + 2 * C * sc;                                   /* [2][C][sq]: terms of q with the decays since the chunk's start */
+    float *q = reinterpret_cast<float *>(qt + 2 * C * sq), *k = q + C * sd, *al = k + C * sd, *qs = al + C * sd, *done = qs + SUB * sd;
+    float *sums = done + D, *rstd = sums + 8 * C;
+    const bf16 *proj = (const bf16 *)a.proj;
+    stage_v<C>(a, smem_addr(vs), first, n, h, 0);
+    for (int i = tid; i < C * (D / 4); i += CHUNK_THREADS) {
+        const int t = i / (D / 4), d = i % (D / 4) * 4;
+        cp_async16(smem_addr(al + t * sd + d), a.decay + (size_t)(first + (t < n ? t : 0)) * HD + h * D + d, t < n);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    for (int i = tid; i < C * (D / 8); i += CHUNK_THREADS) {
+        const int t = i / (D / 8), d = i % (D / 8) * 8;
+        const bf16 *p = proj + (size_t)(first + (t < n ? t : 0)) * a.ldp + h * D + d;
+        const uint4 z = make_uint4(0u, 0u, 0u, 0u);
+        const uint4 qv = t < n ? *reinterpret_cast<const uint4 *>(p + a.off_q) : z, kv = t < n ? *reinterpret_cast<const uint4 *>(p + a.off_k) : z;
+        const __nv_bfloat162 *qp = reinterpret_cast<const __nv_bfloat162 *>(&qv), *kp = reinterpret_cast<const __nv_bfloat162 *>(&kv);
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const float2 x = __bfloat1622float2(qp[j]), y = __bfloat1622float2(kp[j]);
+            *reinterpret_cast<float2 *>(q + t * sd + d + 2 * j) = make_float2(x.x * a.q_scale, x.y * a.q_scale);
+            *reinterpret_cast<float2 *>(k + t * sd + d + 2 * j) = y;
+        }
+    }
+    for (int i = tid; i < C * sc; i += CHUNK_THREADS) reinterpret_cast<uint32_t *>(at)[i] = 0u; /* both terms */
+    for (int d = tid; d < D; d += CHUNK_THREADS) done[d] = 1.f;
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    auto put_score = [&](int t, int s, float v) {
+        const bf16 hi = __float2bfloat16_rn(v);
+        at[t * sc + s] = hi;
+        at[(C + t) * sc + s] = __float2bfloat16_rn(v - to_f(hi));
+    };
+#pragma unroll 1
+    for (int i0 = 0; i0 < n; i0 += SUB) { /* the walk of k_gla_chunk_out; alpha, q and k of tokens past n are zero */
+        for (int d = tid; d < D; d += CHUNK_THREADS) {
+            float f = 1.f;
+#pragma unroll
+            for (int t = 0; t < SUB; t++) {
+                f *= al[(i0 + t) * sd + d];
+                qs[t * sd + d] = q[(i0 + t) * sd + d] * f;
+            }
+        }
+        __syncthreads();
+        for (int e = tid; e < SUB * i0; e += CHUNK_THREADS) {
+            const int t = e % SUB, s = e / SUB;
+            const float4 *x = reinterpret_cast<const float4 *>(qs + t * sd), *y = reinterpret_cast<const float4 *>(k + s * sd);
+            float v0 = 0.f, v1 = 0.f;
+#pragma unroll 4
+            for (int d = 0; d < D / 4; d++) {
+                const float4 xv = x[d], yv = y[d];
+                v0 = fmaf(xv.x, yv.x, v0), v1 = fmaf(xv.y, yv.y, v1), v0 = fmaf(xv.z, yv.z, v0), v1 = fmaf(xv.w, yv.w, v1);
+            }
+            put_score(i0 + t, s, v0 + v1);
+        }
+        {
+            const int s = tid >> 4, l16 = tid & 15;
+            float acc[SUB];
+#pragma unroll
+            for (int t = 0; t < SUB; t++) acc[t] = 0.f;
+            for (int d = l16; d < D; d += 16) {
+                float f = k[(i0 + s) * sd + d];
+#pragma unroll
+                for (int t = 0; t < SUB; t++) {
+                    if (t > s) f *= al[(i0 + t) * sd + d];
+                    if (t >= s) acc[t] = fmaf(q[(i0 + t) * sd + d], f, acc[t]);
+                }
+            }
+#pragma unroll
+            for (int t = 0; t < SUB; t++) {
+                float v = acc[t];
+                for (int o = 8; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+                if (l16 == t && t >= s) put_score(i0 + t, i0 + s, v);
+            }
+        }
+        __syncthreads();
+        for (int d = tid; d < D; d += CHUNK_THREADS) {
+            const float before = done[d];
+            float f = 1.f;
+#pragma unroll
+            for (int t = SUB - 1; t >= 0; t--) {
+                k[(i0 + t) * sd + d] *= f;
+                f *= al[(i0 + t) * sd + d];
+                const float x = qs[t * sd + d] * before;
+                const bf16 hi = __float2bfloat16_rn(x);
+                qt[(i0 + t) * sq + d] = hi;
+                qt[(C + i0 + t) * sq + d] = __float2bfloat16_rn(x - to_f(hi));
+            }
+            for (int s = 0; s < i0; s++) k[s * sd + d] *= f;
+            done[d] = before * f;
+        }
+        __syncthreads();
+    }
+    const float *state = a.states + ((size_t)chunk * a.heads + h) * D * V;
+    const int g = lane >> 2, t2 = (lane & 3) * 2, col0 = warp * 32;
+    const uint32_t qb = smem_addr(qt) + ((lane & 15) * sq + (lane >> 4) * 8) * 2, ab = smem_addr(at) + ((lane & 15) * sc + (lane >> 4) * 8) * 2;
+    const uint32_t vb = smem_addr(vs) + ((lane & 15) * (VT + 8) + col0 + (lane >> 4) * 8) * 2;
+    const bool direct = V <= VT; /* the whole row of a token is in this block's registers */
+    for (int i = tid; i < 8 * C; i += CHUNK_THREADS) sums[i] = 0.f;
+    for (int v0 = 0; v0 < V; v0 += VT) {
+        if (v0 > 0) {
+            __syncthreads();
+            stage_v<C>(a, smem_addr(vs), first, n, h, v0);
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+            __syncthreads();
+        }
+        float acc[MT][4][4];
+#pragma unroll
+        for (int i = 0; i < MT * 16; i++) acc[i >> 4][(i >> 2) & 3][i & 3] = 0.f;
+        const int cols = min(32, V - v0 - col0); /* <= 0: this warp has none */
+        float next[4][4];
+        auto load = [&](int k0) {
+#pragma unroll
+            for (int c = 0; c < 4; c++) {
+                const float *p = state + (size_t)(k0 + t2) * V + v0 + col0 + c * 8 + g;
+                const bool on = c * 8 < cols;
+                next[c][0] = on ? p[0] : 0.f, next[c][1] = on ? p[V] : 0.f;
+                next[c][2] = on ? p[(size_t)8 * V] : 0.f, next[c][3] = on ? p[(size_t)9 * V] : 0.f;
+            }
+        };
+        load(0);
+        for (int k0 = 0; k0 < D; k0 += 16) {
+            uint32_t hi[4][2], lo[4][2];
+#pragma unroll
+            for (int c = 0; c < 4; c++) split2(next[c][0], next[c][1], hi[c][0], lo[c][0]), split2(next[c][2], next[c][3], hi[c][1], lo[c][1]);
+            if (k0 + 16 < D) load(k0 + 16);
+#pragma unroll
+            for (int m = 0; m < MT; m++) {
+                uint32_t xh[4], xl[4];
+                ldsm4(xh, qb + (m * 16 * sq + k0) * 2);
+                ldsm4(xl, qb + ((C + m * 16) * sq + k0) * 2);
+#pragma unroll
+                for (int c = 0; c < 4; c++) {
+                    mma_bf16(acc[m][c], xh, hi[c][0], hi[c][1]);
+                    mma_bf16(acc[m][c], xh, lo[c][0], lo[c][1]);
+                    mma_bf16(acc[m][c], xl, hi[c][0], hi[c][1]);
+                }
+            }
+        }
+#pragma unroll
+        for (int kk = 0; kk < MT; kk++) { /* 16 tokens of the chunk itself; rows before them see none of it */
+            uint32_t b[2][4];
+            ldsm4_t(b[0], vb + kk * 16 * (VT + 8) * 2);
+            ldsm4_t(b[1], vb + kk * 16 * (VT + 8) * 2 + 32);
+#pragma unroll
+            for (int m = kk; m < MT; m++) {
+                uint32_t xh[4], xl[4];
+                ldsm4(xh, ab + (m * 16 * sc + kk * 16) * 2);
+                ldsm4(xl, ab + ((C + m * 16) * sc + kk * 16) * 2);
+#pragma unroll
+                for (int c = 0; c < 4; c++) {
+                    mma_bf16(acc[m][c], xh, b[c >> 1][(c & 1) * 2], b[c >> 1][(c & 1) * 2 + 1]);
+                    mma_bf16(acc[m][c], xl, b[c >> 1][(c & 1) * 2], b[c >> 1][(c & 1) * 2 + 1]);
+                }
+            }
+        }
+        __syncthreads(); /* the sums are cleared */
+#pragma unroll
+        for (int m = 0; m < MT; m++)
+#pragma unroll
+            for (int r = 0; r < 2; r++) {
+                float s = 0.f;
+#pragma unroll
+                for (int c = 0; c < 4; c++) s += acc[m][c][2 * r] * acc[m][c][2 * r] + acc[m][c][2 * r + 1] * acc[m][c][2 * r + 1];
+                s += __shfl_xor_sync(0xffffffffu, s, 1);
+                s += __shfl_xor_sync(0xffffffffu, s, 2);
+                if ((lane & 3) == 0) sums[warp * C + m * 16 + r * 8 + g] += s;
+            }
+        if (direct) {
+            __syncthreads();
+            if (tid < C) {
+                float s = 0.f;
+                for (int w = 0; w < 8; w++) s += sums[w * C + tid];
+                rstd[tid] = 1.f / sqrtf(s / (float)a.norm_count + a.eps);
+            }
+            __syncthreads();
+        }
+#pragma unroll
+        for (int m = 0; m < MT; m++)
+#pragma unroll
+            for (int r = 0; r < 2; r++) {
+                const int t = m * 16 + r * 8 + g;
+                if (t >= n) continue;
+                const bf16 *gp = proj + (size_t)(first + t) * a.ldp + a.off_g + h * V;
+#pragma unroll
+                for (int c = 0; c < 4; c++) {
+                    const int v = v0 + col0 + c * 8 + t2;
+                    if (c * 8 >= cols) continue;
+                    if (direct) {
+                        const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(gp + v));
+                        const float2 w = *reinterpret_cast<const float2 *>(a.norm + v);
+                        *reinterpret_cast<__nv_bfloat162 *>((bf16 *)a.out + (size_t)(first + t) * a.ldo + h * V + v) =
+                            __floats2bfloat162_rn(acc[m][c][2 * r] * rstd[t] * w.x * silu(z.x), acc[m][c][2 * r + 1] * rstd[t] * w.y * silu(z.y));
+                    } else {
+                        *reinterpret_cast<float2 *>(a.raw + ((size_t)(first + t) * a.heads + h) * V + v) =
+                            make_float2(acc[m][c][2 * r], acc[m][c][2 * r + 1]);
+                    }
+                }
+            }
+    }
+    if (direct) return;
+    __syncthreads();
+    if (tid < C) {
+        float s = 0.f;
+        for (int w = 0; w < 8; w++) s += sums[w * C + tid];
+        rstd[tid] = 1.f / sqrtf(s / (float)a.norm_count + a.eps);
+    }
+    __syncthreads(); /* this block's raw outputs are visible to all of its threads */
+    for (int i = tid; i < n * V; i += CHUNK_THREADS) {
+        const int t = i / V, v = i % V;
+        const float gate = silu(to_f(proj[(size_t)(first + t) * a.ldp + a.off_g + h * V + v]));
+        ((bf16 *)a.out)[(size_t)(first + t) * a.ldo + h * V + v] =
+            __float2bfloat16_rn(a.raw[((size_t)(first + t) * a.heads + h) * V + v] * rstd[t] * a.norm[v] * gate);
+    }
+}
+
 /* ---- host side ------------------------------------------------------------------------------------------------------ */
 
 template <typename... A>
@@ -468,6 +864,19 @@ int gla_chunked(const ncb_gla *g, int f32, void *stream_ptr) {
     rc = f32 ? launch(k_gla_decay<float>, decay_grid, CHUNK_THREADS, decay_smem, 1, stream, *g)
              : launch(k_gla_decay<bf16>, decay_grid, CHUNK_THREADS, decay_smem, 1, stream, *g);
     if (rc != NCB_OK) return rc;
+    /* 16-byte copies of rows: every offset of the projection a multiple of 8 */
+    const bool mma = !f32 && g->dim <= 256 && !(g->ldp % 8 | g->off_q % 8 | g->off_k % 8 | g->off_v % 8 | g->off_g % 8 | g->ldo % 2) &&
+                     !((uintptr_t)g->proj % 16 | (uintptr_t)g->decay % 16);
+    if (mma) {
+        const dim3 grid(g->n_chunks, g->heads, (g->vdim + VT - 1) / VT);
+        rc = C == 64 ? launch(k_gla_chunk_state_mma<64>, grid, CHUNK_THREADS, state_mma_bytes<64>(g->dim), 1, stream, *g)
+                     : launch(k_gla_chunk_state_mma<32>, grid, CHUNK_THREADS, state_mma_bytes<32>(g->dim), 1, stream, *g);
+        if (rc != NCB_OK) return rc;
+        rc = launch(k_gla_scan, scan_grid, CHUNK_THREADS, 0, 1, stream, *g);
+        if (rc != NCB_OK || !g->out) return rc;
+        return C == 64 ? launch(k_gla_chunk_out_mma<4>, out_grid, CHUNK_THREADS, out_mma_bytes<4>(g->dim), 1, stream, *g)
+                       : launch(k_gla_chunk_out_mma<2>, out_grid, CHUNK_THREADS, out_mma_bytes<2>(g->dim), 1, stream, *g);
+    }
     rc = f32 ? launch(k_gla_chunk_state<float>, state_grid, CHUNK_THREADS, state_smem, 1, stream, *g)
              : launch(k_gla_chunk_state<bf16>, state_grid, CHUNK_THREADS, state_smem, 1, stream, *g);
     if (rc != NCB_OK) return rc;

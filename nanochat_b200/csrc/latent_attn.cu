@@ -4,14 +4,14 @@
  * so the cache holds only c (RMS-normed, `rank` values) and the rotated key part k_rot (`rot` values) shared by the heads.
  * Softmax optionally with a sink (exp(sink_h) in the denominator), output optionally gated by sigmoid(gate).
  *
- * Cache: T [n_slots][capacity][rank + rot], T = bf16 (float for a model that runs in 32-bit): a row per position, so a
- * block streams consecutive positions with one bulk copy per row and both contractions read the same bytes.
+ * Cache: T [n_slots][capacity][rank + rot], T = bf16 (float for a model that runs in 32-bit): a row per position, so all
+ * slots are one matrix that TMA reads in boxes, and both contractions read the same bytes.
  *
  * Absorbed form (decode, short portions of prompts): q is taken into latent space, q_abs = [W_uk,h^T q_plain | q_rot],
  * and every head attends the latent rows themselves, as the query heads of ONE key/value head:
  *   - k_latent_query: norm + rotate + append of the new row, rotation of q, and the per-head product with W_uk^T;
- *   - k_latent_split: split over positions. mma.sync m16n8k16 with 16 heads as M; a 32-position tile is fetched by 32 bulk
- *     copies into padded rows (conflict-free ldmatrix). Two warps halve the score contraction's depth so that q stays in
+ *   - k_latent_split: split over positions. mma.sync m16n8k16 with 16 heads as M; a 32-position tile comes as TMA boxes of 32
+ *     rows x 64 columns (128-byte swizzle, conflict-free ldmatrix). Two warps halve the score contraction's depth so that q stays in
  *     registers, two halve the positions; for the second contraction the four warps own a quarter of the latent's columns
  *     each. Scores and probabilities are fp32; a probability enters the second product as two bf16 terms (hi + lo), so its
  *     weight keeps 16 bits. Per (row, head, chunk) an un-normalised state (m in log2 units, l, o);
@@ -20,7 +20,7 @@
  * [W_uk; W_uv] is an ordinary GEMM) and k_latent_prefill: a tile of a prompt's rows against the expanded keys and values.
  * k_latent_split_any and k_latent_out_any are the same steps in plain fp32 arithmetic for any sizes and for T = float.
  */
-#include "ncb_common.cuh"
+#include "umma.cuh"
 
 #include <cooperative_groups.h>
 
@@ -55,6 +55,9 @@ __device__ __forceinline__ void ldsm4_t(uint32_t *r, uint32_t addr) {
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
 __device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void *src, bool on) { /* 16 bytes, zeros when off */
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
+}
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const uint32_t *>(&v);
@@ -127,42 +130,52 @@ template <typename T> __device__ __forceinline__ void rotate_pair(const ncb_late
 /* ---- absorbed form: query ------------------------------------------------------------------------------------------- */
 
 /* Grid (rank / 64 rounded up, + 1, heads, ceil(rows / 16)). Block x < last: 64 latent columns of q_abs for one head and 16
- * rows; block x == last: the rotated part of that head's q and, for head 0, the rows' appends. */
+ * rows, its weights on their way to shared memory before the dependency wait; block x == last: the rotated part of that
+ * head's q, and the appends of the rows dealt to that head. */
 template <typename T> __global__ void __launch_bounds__(THREADS) k_latent_query(const ncb_latent a) {
+    extern __shared__ __align__(128) uint8_t raw[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, r0 = blockIdx.z * 16;
-    const int W = a.rank + a.rot, stride_q = a.dim + a.rot;
+    const int W = a.rank + a.rot, stride_q = a.dim + a.rot, f0 = blockIdx.x * 64, ws = a.dim + 8;
+    const bool rotate = blockIdx.x == gridDim.x - 1;
+    if (sizeof(T) == 2 && !rotate) {
+        const int n = min(64, a.rank - f0), per = a.dim / 8;
+        const bf16 *src = (const bf16 *)a.w_uk_t + ((size_t)h * a.rank + f0) * a.dim;
+        for (int i = tid; i < n * per; i += THREADS) cp_async16(smem_addr(raw) + (i / per * ws + i % per * 8) * 2, src + (size_t)i * 8, true);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    }
     asm volatile("griddepcontrol.wait;" ::: "memory");
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     const int rows = (int)(a.rows - r0 < 16 ? a.rows - r0 : 16);
     const T *q = (const T *)a.proj + a.off_q + (size_t)h * stride_q;
     T *out = (T *)a.q_abs;
-    if (blockIdx.x == gridDim.x - 1) {
+    if (rotate) {
+        for (int r = h + warp * a.heads; r < rows; r += a.heads * (THREADS / 32)) append_row<T>(a, r0 + r, lane);
         const int half = a.rot / 2;
         for (int i = tid; i < rows * half; i += THREADS) {
             const int row = r0 + i / half, pos = a.pos[row];
             if (pos >= 0 && pos < a.table_len)
                 rotate_pair(a, q + (size_t)row * a.ldp + a.dim, out + ((size_t)row * a.heads + h) * W + a.rank, pos, i % half);
         }
-        if (h == 0)
-            for (int r = warp; r < rows; r += THREADS / 32) append_row<T>(a, r0 + r, lane);
         return;
     }
-    const T *w = (const T *)a.w_uk_t + (size_t)h * a.rank * a.dim; /* [rank][dim] of this head */
-    const int f0 = blockIdx.x * 64;
     if constexpr (sizeof(T) == 2) {
         /* 16 rows x 16 columns per warp, depth dim: the same permutation of the k slots for both operands, 32 k-values per
-         * 16-byte load, so neither operand needs staging */
+         * 16-byte load */
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
         const int g = lane >> 2, t = lane & 3, c0 = f0 + warp * 16;
         if (c0 >= a.rank) return;
+        const bf16 *ws0 = reinterpret_cast<const bf16 *>(raw) + warp * 16 * ws;
         float acc[2][2][4] = {};
         const T *xl = q + (size_t)(r0 + g) * a.ldp + 8 * t, *xh = xl + (size_t)8 * a.ldp;
         const bool lo_on = g < rows, hi_on = g + 8 < rows;
+#pragma unroll 4
         for (int k = 0; k < a.dim; k += 32) {
             const uint4 z = make_uint4(0u, 0u, 0u, 0u);
             const uint4 lo = lo_on ? *reinterpret_cast<const uint4 *>(xl + k) : z, hi = hi_on ? *reinterpret_cast<const uint4 *>(xh + k) : z;
 #pragma unroll
             for (int j = 0; j < 2; j++) {
-                const uint4 b = *reinterpret_cast<const uint4 *>(w + (size_t)(c0 + j * 8 + g) * a.dim + k + 8 * t);
+                const uint4 b = *reinterpret_cast<const uint4 *>(ws0 + (j * 8 + g) * ws + k + 8 * t);
                 mma_bf16(acc[j][0], lo.x, hi.x, lo.y, hi.y, b.x, b.y);
                 mma_bf16(acc[j][1], lo.z, hi.z, lo.w, hi.w, b.z, b.w);
             }
@@ -175,6 +188,7 @@ template <typename T> __global__ void __launch_bounds__(THREADS) k_latent_query(
                     *reinterpret_cast<uint32_t *>(out + ((size_t)(r0 + g + 8 * r) * a.heads + h) * W + c0 + j * 8 + 2 * t) =
                         pack_bf16(acc[j][0][2 * r] + acc[j][1][2 * r], acc[j][0][2 * r + 1] + acc[j][1][2 * r + 1]);
     } else {
+        const T *w = (const T *)a.w_uk_t + (size_t)h * a.rank * a.dim; /* [rank][dim] of this head */
         const int cols = a.rank - f0 < 64 ? a.rank - f0 : 64;
         for (int i = tid; i < rows * cols; i += THREADS) {
             const int row = r0 + i / cols, c = f0 + i % cols;
@@ -188,37 +202,29 @@ template <typename T> __global__ void __launch_bounds__(THREADS) k_latent_query(
 
 /* ---- absorbed form: split over positions ---------------------------------------------------------------------------- */
 
-__device__ __forceinline__ void bar_init(uint32_t bar) { asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"(bar) : "memory"); }
-__device__ __forceinline__ bool bar_wait(uint32_t bar, uint32_t parity) { /* bounded: about two seconds of the SM clock */
-    const long long start = clock64();
-    for (;;) {
-        uint32_t done;
-        asm volatile("{\n\t.reg .pred p;\n\t"
-                     "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
-                     "selp.u32 %0, 1, 0, p;\n\t}"
-                     : "=r"(done) : "r"(bar), "r"(parity) : "memory");
-        if (done) return true;
-        if (clock64() - start > 4000000000ll) return false;
-    }
-}
+constexpr int BOX_BYTES = TILE * 128; /* 32 rows of 64 bf16 columns */
 
 template <int STAGES> struct SplitSmem {
-    __host__ __device__ static int row_bytes(int W) { return W * 2 + 16; } /* an odd number of 16-byte units: no conflicts */
-    __host__ __device__ static int bytes(int W) { return STAGES * TILE * row_bytes(W) + 2 * HEADS_M * (TILE + 4) * 4 + 64; }
+    __host__ __device__ static int boxes(int W) { return (W + 63) / 64; }
+    __host__ __device__ static int bytes(int W) { return 1024 + STAGES * boxes(W) * BOX_BYTES + 2 * HEADS_M * (TILE + 4) * 4 + 64; }
 };
 
 /* Grid (max chunks, ceil(heads / 16), rows). MK: 16-wide k-steps per half of the score contraction; MN: 16-wide column
- * tiles of the latent per warp. */
-template <int MK, int MN, int STAGES> __global__ void __launch_bounds__(THREADS, 2) k_latent_split(const ncb_latent a) {
+ * tiles of the latent per warp. map: all slots' rows as one matrix [n_slots capacity][rank + rot], boxes of 32 x 64. */
+template <int MK, int MN, int STAGES>
+__global__ void __launch_bounds__(THREADS, 2) k_latent_split(const __grid_constant__ CUtensorMap map, const ncb_latent a) {
     extern __shared__ __align__(128) uint8_t raw[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-    const int W = a.rank + a.rot, row_bytes = SplitSmem<STAGES>::row_bytes(W), stage_bytes = TILE * row_bytes;
-    float *scores = reinterpret_cast<float *>(raw + STAGES * stage_bytes); /* [2][16][TILE + 4]: the two depth halves */
-    const uint32_t ring = smem_addr(raw), bars = ring + STAGES * stage_bytes + 2 * HEADS_M * (TILE + 4) * 4;
+    const int W = a.rank + a.rot, boxes = SplitSmem<STAGES>::boxes(W), stage_bytes = boxes * BOX_BYTES;
+    const uint32_t ring = (smem_addr(raw) + 1023u) & ~1023u; /* swizzled boxes sit on 1024-byte boundaries */
+    uint8_t *ring_ptr = raw + (ring - smem_addr(raw));
+    float *scores = reinterpret_cast<float *>(ring_ptr + STAGES * stage_bytes); /* [2][16][TILE + 4]: the two depth halves */
+    const uint32_t bars = ring + STAGES * stage_bytes + 2 * HEADS_M * (TILE + 4) * 4;
     if (tid == 0) {
-        for (int s = 0; s < STAGES; s++) bar_init(bars + 8 * s);
+        for (int s = 0; s < STAGES; s++) mbar_init(bars + 8 * s, 1);
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+        asm volatile("prefetch.tensormap [%0];" ::"l"(&map) : "memory");
     }
     asm volatile("griddepcontrol.wait;" ::: "memory");
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
@@ -228,20 +234,16 @@ template <int MK, int MN, int STAGES> __global__ void __launch_bounds__(THREADS,
     const int t0 = blockIdx.x * cut.per, t1 = min(t0 + cut.per, cut.tiles);
     if (blockIdx.x >= cut.n_chunks || t0 >= t1) return;
     __syncthreads();
-    const bf16 *cache = (const bf16 *)a.cache + (size_t)slot * a.capacity * W;
-    auto fetch = [&](int i) { /* warp 0: a tile's rows, one bulk copy per lane */
-        const int tile = t0 + i, s = i % STAGES, n = min(TILE, cut.len - tile * TILE);
-        if (lane == 0)
-            asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bars + 8 * s), "r"(n * W * 2) : "memory");
-        __syncwarp();
-        if (lane < n)
-            asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
-                             ring + s * stage_bytes + lane * row_bytes),
-                         "l"(cache + (size_t)(tile * TILE + lane) * W), "r"(W * 2), "r"(bars + 8 * s)
-                         : "memory");
+    const uint64_t policy = policy_evict_first();
+    auto fetch = [&](int i) { /* one thread: a tile's boxes */
+        const int s = i % STAGES, r = slot * a.capacity + (t0 + i) * TILE;
+        mbar_expect_tx(bars + 8 * s, stage_bytes);
+        for (int b = 0; b < boxes; b++) tma_load(ring + s * stage_bytes + b * BOX_BYTES, &map, b * 64, r, bars + 8 * s, policy);
     };
+    /* the address of 16-byte chunk c of row r in a stage */
+    auto chunk_at = [](uint32_t stage, int r, int c) { return stage + (c >> 3) * BOX_BYTES + r * 128 + (((c & 7) ^ (r & 7)) << 4); };
     const int n_tiles = t1 - t0;
-    if (warp == 0)
+    if (tid == 0)
         for (int i = 0; i < min(STAGES, n_tiles); i++) fetch(i);
 
     /* this warp's half of the score depth, as A operand fragments */
@@ -274,21 +276,23 @@ template <int MK, int MN, int STAGES> __global__ void __launch_bounds__(THREADS,
     for (int i = 0; i < n_tiles; i++) {
         const int s = i % STAGES, p0 = (t0 + i) * TILE;
         const uint32_t stage = ring + s * stage_bytes;
-        if (!bar_wait(bars + 8 * s, (i / STAGES) & 1)) ok = false;
+        if (!mbar_wait(bars + 8 * s, (i / STAGES) & 1)) ok = false;
+        __syncwarp();
         const int live = min(TILE, cut.len - p0);
-        if (live < TILE) { /* the sequence's last tile: rows that were not copied must not hold stale NaNs */
-            for (int j = tid; j < (TILE - live) * (row_bytes / 16); j += THREADS)
-                *reinterpret_cast<uint4 *>(raw + s * stage_bytes + live * row_bytes + j * 16) = make_uint4(0u, 0u, 0u, 0u);
+        if (live < TILE) { /* the sequence's last tile: whatever lies past its end must not reach the second product */
+            for (int j = tid; j < (TILE - live) * boxes * 8; j += THREADS)
+                *reinterpret_cast<uint4 *>(ring_ptr + s * stage_bytes + (j >> 3) / (TILE - live) * BOX_BYTES + (live + (j >> 3) % (TILE - live)) * 128 +
+                                           (j & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
             __syncthreads();
         }
         { /* scores of 16 positions over half of the depth */
             float acc[2][2][4] = {};
-            const uint32_t base = stage + (ph * 16 + (lane >> 4) * 8 + (lane & 7)) * row_bytes + (ks0 * 16 + ((lane >> 3) & 1) * 8) * 2;
+            const int r = ph * 16 + (lane >> 4) * 8 + (lane & 7), c = 2 * ks0 + ((lane >> 3) & 1);
 #pragma unroll
             for (int ks = 0; ks < MK; ks++)
                 if (ks < nks) {
                     uint32_t b[4];
-                    ldsm4(b, base + ks * 32);
+                    ldsm4(b, chunk_at(stage, r, c + 2 * ks));
                     mma_bf16(acc[ks & 1][0], qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3], b[0], b[1]);
                     mma_bf16(acc[ks & 1][1], qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3], b[2], b[3]);
                 }
@@ -340,14 +344,13 @@ template <int MK, int MN, int STAGES> __global__ void __launch_bounds__(THREADS,
                 else l_lo += a0 + a1;
                 split_bf16(a0, a1, hi[j][e], lo[j][e]);
             }
-        const uint32_t vbase = stage + (lane & 15) * row_bytes + (ct0 * 16 + (lane >> 4) * 8) * 2;
 #pragma unroll
         for (int c = 0; c < MN; c++)
             if (c < nct) {
 #pragma unroll
                 for (int j = 0; j < 2; j++) {
                     uint32_t b[4];
-                    ldsm4_t(b, vbase + j * 16 * row_bytes + c * 32);
+                    ldsm4_t(b, chunk_at(stage, j * 16 + (lane & 15), 2 * (ct0 + c) + (lane >> 4)));
                     mma_bf16(o[c][0], hi[j][0], hi[j][1], hi[j][2], hi[j][3], b[0], b[1]);
                     mma_bf16(o[c][1], hi[j][0], hi[j][1], hi[j][2], hi[j][3], b[2], b[3]);
                     mma_bf16(o[c][0], lo[j][0], lo[j][1], lo[j][2], lo[j][3], b[0], b[1]);
@@ -355,7 +358,7 @@ template <int MK, int MN, int STAGES> __global__ void __launch_bounds__(THREADS,
                 }
             }
         __syncthreads(); /* the stage and the scores may be overwritten */
-        if (warp == 0 && i + STAGES < n_tiles) fetch(i + STAGES);
+        if (tid == 0 && i + STAGES < n_tiles) fetch(i + STAGES);
     }
     if (!ok && lane == 0) flag(a.status, NCB_DEV_WAIT_TIMEOUT);
     l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1);
@@ -486,9 +489,12 @@ template <typename T> __global__ void __launch_bounds__(THREADS) k_latent_out_an
     }
 }
 
+constexpr int OUT_THREADS = 256;
+
 /* Grid (slices, heads, ceil(rows / 16)), cluster (slices, 1, 1): a block merges rank / slices latent columns of 16 rows,
- * multiplies them by its columns of W_uv for all of the head's values, and the cluster adds the partial products up. */
-__global__ void __launch_bounds__(THREADS) k_latent_out(const ncb_latent a) {
+ * multiplies them by its columns of W_uv (on their way to shared memory before the dependency wait) for all of the head's
+ * values, and the cluster adds the partial products up. */
+__global__ void __launch_bounds__(OUT_THREADS) k_latent_out(const ncb_latent a) {
     extern __shared__ __align__(128) uint8_t raw[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     const int slices = gridDim.x, rank_block = blockIdx.x, h = blockIdx.y, r0 = blockIdx.z * 16;
@@ -496,38 +502,65 @@ __global__ void __launch_bounds__(THREADS) k_latent_out(const ncb_latent a) {
     float *w = reinterpret_cast<float *>(raw);                          /* [16][max_chunks] */
     float *sum = w + 16 * a.max_chunks;                                 /* [16][vdim + 4] partial products */
     bf16 *x = reinterpret_cast<bf16 *>(sum + 16 * (V + 4));             /* [16][cols + 8] merged latent */
+    bf16 *u = x + 16 * xs;                                              /* [vdim][cols + 8] */
     __shared__ int n_chunks[16];
+    {
+        const int per = cols / 8;
+        const bf16 *src = (const bf16 *)a.w_uv + (size_t)h * V * a.rank + c0;
+        for (int i = tid; i < V * per; i += OUT_THREADS) cp_async16(smem_addr(u + i / per * xs + i % per * 8), src + (size_t)(i / per) * a.rank + i % per * 8, true);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    }
     asm volatile("griddepcontrol.wait;" ::: "memory");
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     const int rows = (int)(a.rows - r0 < 16 ? a.rows - r0 : 16);
-    for (int r = warp; r < 16; r += THREADS / 32) {
+    const size_t state = (size_t)(a.rank + STATE_PAD);
+    { /* the factor of every chunk's state, 16 threads per row: 2^(m - M) / L with the sink in M and L */
+        const int r = tid >> 4, j = tid & 15;
         int n = 0, slot;
-        if (r < rows) {
-            n = cut_of(length_of(a, r0 + r, slot), a.chunk_tiles).n_chunks;
-            merge_weights(a, r0 + r, h, n, w + r * a.max_chunks, lane);
+        if (r < rows) n = cut_of(length_of(a, r0 + r, slot), a.chunk_tiles).n_chunks;
+        const float *p = a.parts + ((size_t)(r0 + r) * a.heads + h) * a.max_chunks * state;
+        const float sink = a.sink ? a.sink[h] * LOG2E : -INFINITY;
+        float M = sink, L = 0.f;
+        for (int c = j; c < n; c += 16) M = fmaxf(M, p[c * state]);
+        for (int o = 8; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
+        for (int c = j; c < n; c += 16) {
+            const float2 ml = *reinterpret_cast<const float2 *>(p + c * state);
+            const float e = exp2f(ml.x - M);
+            w[r * a.max_chunks + c] = e;
+            L = fmaf(e, ml.y, L);
         }
-        if (lane == 0) n_chunks[r] = n;
+        for (int o = 8; o > 0; o >>= 1) L += __shfl_xor_sync(0xffffffffu, L, o);
+        if (a.sink) L += exp2f(sink - M);
+        const float inv = n > 0 ? 1.f / L : 0.f;
+        for (int c = j; c < n; c += 16) w[r * a.max_chunks + c] *= inv;
+        if (j == 0) n_chunks[r] = n;
     }
     __syncthreads();
-    const size_t state = (size_t)(a.rank + STATE_PAD);
-    for (int i = tid; i < 16 * (cols / 4); i += THREADS) {
+    for (int i = tid; i < 16 * (cols / 4); i += OUT_THREADS) {
         const int r = i / (cols / 4), c4 = i % (cols / 4) * 4;
         float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
         const int n = n_chunks[r];
         const float *p = a.parts + ((size_t)(r0 + r) * a.heads + h) * a.max_chunks * state + STATE_PAD + c0 + c4;
-#pragma unroll 4
-        for (int c = 0; c < n; c++) {
-            const float4 s = *reinterpret_cast<const float4 *>(p + c * state);
-            const float f = w[r * a.max_chunks + c];
-            v.x = fmaf(f, s.x, v.x), v.y = fmaf(f, s.y, v.y), v.z = fmaf(f, s.z, v.z), v.w = fmaf(f, s.w, v.w);
+        const float *f = w + r * a.max_chunks;
+        constexpr int AHEAD = 8; /* states whose loads are in flight together */
+        for (int c = 0; c < n; c += AHEAD) {
+            float4 s[AHEAD];
+#pragma unroll
+            for (int j = 0; j < AHEAD; j++)
+                s[j] = c + j < n ? *reinterpret_cast<const float4 *>(p + (c + j) * state) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int j = 0; j < AHEAD; j++) {
+                const float e = c + j < n ? f[c + j] : 0.f;
+                v.x = fmaf(e, s[j].x, v.x), v.y = fmaf(e, s[j].y, v.y), v.z = fmaf(e, s[j].z, v.z), v.w = fmaf(e, s[j].w, v.w);
+            }
         }
         *reinterpret_cast<uint2 *>(x + r * xs + c4) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
     }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
-    const bf16 *u = (const bf16 *)a.w_uv + (size_t)h * V * a.rank + c0 + 8 * t;
-    for (int n0 = warp * 8; n0 < V; n0 += 32) { /* 8 output values at a time */
+    for (int n0 = warp * 8; n0 < V; n0 += OUT_THREADS / 4) { /* 8 output values at a time */
         float acc[2][4] = {};
-        const bf16 *wr = u + (size_t)(n0 + g) * a.rank, *xl = x + g * xs + 8 * t, *xh = xl + 8 * xs;
+        const bf16 *wr = u + (n0 + g) * xs + 8 * t, *xl = x + g * xs + 8 * t, *xh = xl + 8 * xs;
 #pragma unroll 4
         for (int k = 0; k < cols; k += 32) {
             const uint4 lo = *reinterpret_cast<const uint4 *>(xl + k), hi = *reinterpret_cast<const uint4 *>(xh + k);
@@ -542,11 +575,12 @@ __global__ void __launch_bounds__(THREADS) k_latent_out(const ncb_latent a) {
     cg::cluster_group cluster = cg::this_cluster();
     if (slices > 1) cluster.sync();
     else __syncthreads();
-    for (int i = rank_block * THREADS + tid; i < rows * V; i += slices * THREADS) {
+    for (int i = rank_block * OUT_THREADS + tid; i < rows * V; i += slices * OUT_THREADS) {
         const int r = i / V, j = i % V;
+        const float gate = gate_of<bf16>(a, r0 + r, h * V + j);
         float v = 0.f;
         for (int s = 0; s < slices; s++) v += slices > 1 ? cluster.map_shared_rank(sum, s)[r * (V + 4) + j] : sum[r * (V + 4) + j];
-        ((bf16 *)a.out)[(size_t)(r0 + r) * a.ldo + h * V + j] = __float2bfloat16_rn(v * gate_of<bf16>(a, r0 + r, h * V + j));
+        ((bf16 *)a.out)[(size_t)(r0 + r) * a.ldo + h * V + j] = __float2bfloat16_rn(v * gate);
     }
     if (slices > 1) cluster.sync(); /* nobody leaves while a peer still reads its shared memory */
 }
@@ -584,10 +618,6 @@ __global__ void __launch_bounds__(THREADS) k_latent_gather(const ncb_latent a) {
     uint4 *c = reinterpret_cast<uint4 *>((bf16 *)a.ctx + (size_t)(first + p) * a.ctx_ld), *k = reinterpret_cast<uint4 *>((bf16 *)a.ctx_rot + (size_t)(first + p) * a.rot);
     for (int i = lane; i < a.ctx_ld / 8; i += 32) c[i] = ok && i < a.rank / 8 ? src[i] : zero;
     for (int i = lane; i < a.rot / 8; i += 32) k[i] = ok ? src[a.rank / 8 + i] : zero;
-}
-
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void *src, bool on) { /* 16 bytes, zeros when off */
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
 }
 
 constexpr int PF_ROWS = 64, PF_KEYS = 64; /* query rows and keys per tile: four warps of 16 rows */
@@ -765,12 +795,12 @@ template <int QS, int VN> __global__ void __launch_bounds__(THREADS, 2) k_latent
 /* ---- host side ------------------------------------------------------------------------------------------------------ */
 
 template <typename... A>
-int launch(void (*kernel)(A...), dim3 grid, size_t smem, int cluster, cudaStream_t stream, A... args) {
+int launch(void (*kernel)(A...), dim3 grid, size_t smem, int threads, int cluster, cudaStream_t stream, A... args) {
     if (smem > 48 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
         return NCB_ERR_LAUNCH;
     cudaLaunchConfig_t config = {};
     config.gridDim = grid;
-    config.blockDim = dim3(THREADS);
+    config.blockDim = dim3(threads);
     config.dynamicSmemBytes = smem;
     config.stream = stream;
     cudaLaunchAttribute attribute[2];
@@ -798,8 +828,10 @@ int check(const ncb_latent &g) {
 }
 
 template <int MK, int MN, int STAGES> int launch_split(const ncb_latent &g, cudaStream_t s) {
+    CUtensorMap map;
+    if (!tensor_map(g.cache, g.n_slots * g.capacity, g.rank + g.rot, TILE, &map)) return NCB_ERR_LAUNCH;
     return launch(k_latent_split<MK, MN, STAGES>, dim3(g.max_chunks, (g.heads + HEADS_M - 1) / HEADS_M, (unsigned)g.rows),
-                  (size_t)SplitSmem<STAGES>::bytes(g.rank + g.rot), 1, s, g);
+                  (size_t)SplitSmem<STAGES>::bytes(g.rank + g.rot), THREADS, 1, s, map, g);
 }
 
 } /* namespace */
@@ -811,8 +843,8 @@ int latent_append(const ncb_latent *g, int f32, void *stream) {
     const int rc = check(*g);
     if (rc != NCB_OK || g->rows == 0) return rc;
     const dim3 grid((unsigned)((g->rows + 3) / 4));
-    return f32 ? launch(k_latent_append<float>, grid, 0, 1, (cudaStream_t)stream, *g)
-               : launch(k_latent_append<bf16>, grid, 0, 1, (cudaStream_t)stream, *g);
+    return f32 ? launch(k_latent_append<float>, grid, 0, THREADS, 1, (cudaStream_t)stream, *g)
+               : launch(k_latent_append<bf16>, grid, 0, THREADS, 1, (cudaStream_t)stream, *g);
 }
 
 int latent_query(const ncb_latent *g, int f32, void *stream) {
@@ -821,8 +853,10 @@ int latent_query(const ncb_latent *g, int f32, void *stream) {
     if (rc != NCB_OK || g->rows == 0) return rc;
     if (!g->q_abs || !g->w_uk_t || (g->rows + 15) / 16 > 65535) return NCB_ERR_ARG;
     const dim3 grid((g->rank + 63) / 64 + 1, g->heads, (unsigned)((g->rows + 15) / 16));
-    return f32 ? launch(k_latent_query<float>, grid, 0, 1, (cudaStream_t)stream, *g)
-               : launch(k_latent_query<bf16>, grid, 0, 1, (cudaStream_t)stream, *g);
+    const size_t smem = f32 ? 0 : (size_t)64 * (g->dim + 8) * 2;
+    if (smem > 200 * 1024) return NCB_ERR_UNSUPPORTED;
+    return f32 ? launch(k_latent_query<float>, grid, smem, THREADS, 1, (cudaStream_t)stream, *g)
+               : launch(k_latent_query<bf16>, grid, smem, THREADS, 1, (cudaStream_t)stream, *g);
 }
 
 int latent_split(const ncb_latent *g, int f32, void *stream) {
@@ -833,7 +867,7 @@ int latent_split(const ncb_latent *g, int f32, void *stream) {
     if ((long long)g->max_chunks * g->chunk_tiles < (g->max_len + TILE - 1) / TILE || g->max_len <= 0) return NCB_ERR_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     const int half = ((g->rank + g->rot) / 16 + 1) / 2, per_warp = (g->rank / 16 + 3) / 4;
-    if (!f32) {
+    if (!f32 && g->capacity % TILE == 0 && (long long)g->n_slots * g->capacity < 0x7fffffffLL) {
         if (half <= 3 && per_warp <= 1) return launch_split<3, 1, 4>(*g, s);
         if (half <= 6 && per_warp <= 2) return launch_split<6, 2, 4>(*g, s);
         if (half <= 10 && per_warp <= 4) return launch_split<10, 4, 3>(*g, s);
@@ -842,7 +876,7 @@ int latent_split(const ncb_latent *g, int f32, void *stream) {
     const size_t smem = ((size_t)2 * g->rank + g->rot + ANY_TILE + 8) * sizeof(float);
     if (smem > 200 * 1024) return NCB_ERR_UNSUPPORTED;
     const dim3 grid(g->max_chunks, g->heads, (unsigned)g->rows);
-    return f32 ? launch(k_latent_split_any<float>, grid, smem, 1, s, *g) : launch(k_latent_split_any<bf16>, grid, smem, 1, s, *g);
+    return f32 ? launch(k_latent_split_any<float>, grid, smem, THREADS, 1, s, *g) : launch(k_latent_split_any<bf16>, grid, smem, THREADS, 1, s, *g);
 }
 
 int latent_out(const ncb_latent *g, int f32, void *stream) {
@@ -854,14 +888,14 @@ int latent_out(const ncb_latent *g, int f32, void *stream) {
     if (!f32) {
         int slices = 4;
         while (slices > 1 && g->rank % (slices * 32)) slices /= 2;
-        const size_t smem = (size_t)16 * g->max_chunks * 4 + (size_t)16 * (g->vdim + 4) * 4 + (size_t)16 * (g->rank / slices + 8) * 2;
+        const size_t smem = (size_t)16 * g->max_chunks * 4 + (size_t)16 * (g->vdim + 4) * 4 + (size_t)(16 + g->vdim) * (g->rank / slices + 8) * 2;
         if (smem <= 200 * 1024)
-            return launch(k_latent_out, dim3(slices, g->heads, (unsigned)((g->rows + 15) / 16)), smem, slices, s, *g);
+            return launch(k_latent_out, dim3(slices, g->heads, (unsigned)((g->rows + 15) / 16)), smem, OUT_THREADS, slices, s, *g);
     }
     const size_t smem = ((size_t)g->max_chunks + g->rank) * sizeof(float);
     if (smem > 200 * 1024) return NCB_ERR_UNSUPPORTED;
     const dim3 grid(g->heads, (unsigned)g->rows);
-    return f32 ? launch(k_latent_out_any<float>, grid, smem, 1, s, *g) : launch(k_latent_out_any<bf16>, grid, smem, 1, s, *g);
+    return f32 ? launch(k_latent_out_any<float>, grid, smem, THREADS, 1, s, *g) : launch(k_latent_out_any<bf16>, grid, smem, THREADS, 1, s, *g);
 }
 
 int latent_gather(const ncb_latent *g, void *stream) {
@@ -871,7 +905,7 @@ int latent_gather(const ncb_latent *g, void *stream) {
     if (!g->ctx || !g->ctx_rot || !g->ctx_slot || !g->ctx_first || g->n_contexts < 0 || g->n_contexts > 65535 || g->max_len <= 0 ||
         g->ctx_ld < g->rank || g->ctx_ld % 8)
         return NCB_ERR_ARG;
-    return launch(k_latent_gather, dim3((g->max_len + 3) / 4, g->n_contexts), 0, 1, (cudaStream_t)stream, *g);
+    return launch(k_latent_gather, dim3((g->max_len + 3) / 4, g->n_contexts), 0, THREADS, 1, (cudaStream_t)stream, *g);
 }
 
 /* 1 if latent_prefill takes these (padded) sizes. */
@@ -890,8 +924,8 @@ int latent_prefill(const ncb_latent *g, void *stream) {
     const dim3 grid(g->heads, g->n_tiles);
     const size_t smem = (size_t)2 * PF_KEYS * ((g->dim + g->rot) * 2 + 16 + g->vdim * 2 + 16);
     cudaStream_t s = (cudaStream_t)stream;
-    return g->dim + g->rot <= 128 ? launch(k_latent_prefill<8, 8>, grid, smem, 1, s, *g)
-                                  : launch(k_latent_prefill<12, 8>, grid, smem, 1, s, *g);
+    return g->dim + g->rot <= 128 ? launch(k_latent_prefill<8, 8>, grid, smem, THREADS, 1, s, *g)
+                                  : launch(k_latent_prefill<12, 8>, grid, smem, THREADS, 1, s, *g);
 }
 
 } /* extern "C" */

@@ -299,6 +299,5 @@ class HybridDecoder(StepDecoder):
         latent = next((l.mixer for l in self.w.layers if isinstance(l.mixer, LatentAttention)), None)
         if latent is None:
             return 0
-        longest = min(max(positions) + 1 + steps // 2, self.capacity)
-        tiles = (self.capacity + 31) // 32
-        return max(latent.default_chunk(len(positions), longest), (tiles + 127) // 128)
+        lens = [min(p + 1 + steps // 2, self.capacity) for p in positions]
+        return latent.chunk_for(lens, self.capacity)

@@ -238,6 +238,7 @@ class LatentAttention:
         self.w_out = pad_to(o, columns, self.out_width).to(dtype)
         self.in_width = self.w_in.shape[0]
         self.tables: "tuple[Tensor, Tensor] | None" = None
+        self._chunks: dict[tuple[int, int], int] = {}
 
     def new_cache(self, n_slots: int, max_len: int) -> LatentCache:
         cache = LatentCache(n_slots, self.rank + self.rot, max_len, self.dtype, device=self.device)
@@ -250,12 +251,25 @@ class LatentAttention:
     def cache_bytes(sizes: dict, max_len: int, itemsize: int) -> int:
         return up(max_len, 64) * (up(int(sizes["kv_rank"]), 32) + up(int(sizes["rot_dim"]), 16)) * itemsize
 
+    def chunk_for(self, lens: "list[int]", most: int) -> int:
+        """Tiles per chunk of the split kernel for rows of these lengths: the size with the least modelled time, waves of the
+        blocks that fit the GPU (two per SM) times a block's tiles plus a fixed cost. At most 128 chunks for `most` positions
+        (a bound of every length)."""
+        tiles = np.maximum((np.asarray(lens, dtype=np.int64) + LATENT_TILE - 1) // LATENT_TILE, 1)
+        top, least = int(tiles.max()), max(2, ((most + LATENT_TILE - 1) // LATENT_TILE + 127) // 128)
+        best, cost = least, float("inf")
+        for c in range(least, max(top, least) + 1):
+            blocks = int(((tiles + c - 1) // c).sum()) * ((self.heads + 15) // 16)
+            now = -(-blocks // (2 * SM_COUNT)) * (min(c, top) + 2.0)
+            if now < cost:
+                best, cost = c, now
+        return best
+
     def default_chunk(self, rows: int, max_len: int) -> int:
-        """Tiles per chunk of the split kernel for `rows` rows of at most max_len positions: about two blocks per SM, at
-        least two tiles (a chunk's state has to be merged again) and at most 128 chunks."""
-        tiles, blocks = (max_len + LATENT_TILE - 1) // LATENT_TILE, rows * ((self.heads + 15) // 16)
-        wanted = max(1, (2 * SM_COUNT) // blocks)
-        return max(2, (tiles + wanted - 1) // wanted, (tiles + 127) // 128)
+        """chunk_for rows that all have max_len positions, remembered (it only depends on these)."""
+        if (rows, max_len) not in self._chunks:
+            self._chunks[rows, max_len] = self.chunk_for([max_len] * rows, max_len)
+        return self._chunks[rows, max_len]
 
     ROW_TILE = 64  # rows per tile of latent_prefill
 
