@@ -48,6 +48,7 @@ inline int check_rs(const ncb_gemm_rs &g) {
     if (g.rows == 0) return NCB_OK;
     if (!g.x || !g.w) return NCB_ERR_ARG;
     if (g.ss && (g.ss_parts <= 0 || g.norm_count <= 0)) return NCB_ERR_ARG;
+    if ((uintptr_t)g.ss % 16) return NCB_ERR_ALIGN;
     if (g.epilogue == 6) {
         if (!g.h || !g.gain || !g.x_next || !g.ss_next) return NCB_ERR_ARG;
         if (((uintptr_t)g.h | (uintptr_t)g.gain | (uintptr_t)g.x_next) % 16) return NCB_ERR_ALIGN;

@@ -432,12 +432,12 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t &hi, uint32_t 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void *src, bool on) { /* 16 bytes, zeros when off */
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
 }
-constexpr int VT = 256; /* columns of v a block handles at a time: eight warps of 32 */
+constexpr int VT = 256; /* columns of v a block handles at a time */
 
 /* The chunk's v rows, columns v0 .. v0 + VT, as bf16 [C][VT + 8]; rows past n and columns past V are zero. */
-template <int C> __device__ __forceinline__ void stage_v(const ncb_gla &a, uint32_t dst, int first, int n, int h, int v0) {
+template <int C, int THREADS = CHUNK_THREADS> __device__ __forceinline__ void stage_v(const ncb_gla &a, uint32_t dst, int first, int n, int h, int v0) {
     const bf16 *v = (const bf16 *)a.proj + (size_t)first * a.ldp + a.off_v + h * a.vdim;
-    for (int i = threadIdx.x; i < C * (VT / 8); i += CHUNK_THREADS) {
+    for (int i = threadIdx.x; i < C * (VT / 8); i += THREADS) {
         const int t = i / (VT / 8), c = v0 + i % (VT / 8) * 8;
         const bool on = t < n && c < a.vdim;
         cp_async16(dst + (t * (VT + 8) + i % (VT / 8) * 8) * 2, v + (on ? (size_t)t * a.ldp + c : 0), on);
@@ -550,186 +550,249 @@ template <int C> __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_chunk_st
     }
 }
 
-/* k_gla_chunk_out with its output product on the tensor cores: what meets the starting state and the state itself as two bf16
- * terms each, the intra-chunk scores as two terms against v. Grid (chunks, heads), C = 16 MT. */
+/* k_gla_chunk_out on the tensor cores, sub-chunks side by side. Per sub-chunk i of 16 tokens: q with the decays since its start
+ * (qs), k with the decays to its end (kd), its whole product G_i; all kept as two bf16 terms. Then
+ *   scores inside a sub-chunk: a warp per (sub-chunk, four s), products running along t in fp32, lanes over key channels;
+ *   scores against sub-chunk j < i: a warp per pair, (qs_i G_(j+1) .. G_(i-1)) . kd_j, three MMAs per step (two-term operands);
+ *   output: (qs_i G_0 .. G_(i-1)) S with S as two terms, plus scores (two terms) times v; a warp per 16 columns.
+ * Grid (chunks, heads), C = 16 MT, 512 threads. */
+constexpr int OUT_THREADS = 512, OUT_WARPS = OUT_THREADS / 32;
 template <int MT> __host__ __device__ inline size_t out_mma_bytes(int D) {
     constexpr int C = 16 * MT;
-    return ((size_t)3 * C * (D + 4) + (size_t)SUB * (D + 4) + D + 8 * C + C) * 4 /* q, k, alpha, scaled q, product, sums */
-           + (size_t)2 * C * (C + 8) * 2 + (size_t)2 * C * (D + 8) * 2 + (size_t)C * (VT + 8) * 2;
+    return (size_t)C * (VT + 8) * 2 + (size_t)2 * C * (C + 8) * 2 + (size_t)4 * C * (D + 8) * 2 /* v, scores, qs, kd */
+           + (size_t)2 * C * D * 2 + ((size_t)C * D + MT * D + OUT_WARPS * C + C) * 4;          /* q, k, alpha, G, sums, rstd */
 }
-template <int MT> __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_chunk_out_mma(const ncb_gla a) {
+/* v[0 .. 63] summed over the warp by halving: lane l ends up with the sums of values 2 l and 2 l + 1 in v[0], v[1]. */
+__device__ __forceinline__ void reduce64(float (&v)[64], int lane) {
+#pragma unroll
+    for (int step = 0; step < 5; step++) {
+        const int n = 32 >> step, off = 16 >> step;
+        const bool upper = lane & off;
+#pragma unroll
+        for (int i = 0; i < n; i++) {
+            const float mine = upper ? v[i + n] : v[i], theirs = upper ? v[i] : v[i + n];
+            v[i] = mine + __shfl_xor_sync(0xffffffffu, theirs, off);
+        }
+    }
+}
+/* The two-term pair (hi, lo) times f0, f1 as a new two-term pair. */
+__device__ __forceinline__ void rescale2(uint32_t &hi, uint32_t &lo, float f0, float f1) {
+    const float2 h = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&hi)), l = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&lo));
+    split2((h.x + l.x) * f0, (h.y + l.y) * f1, hi, lo);
+}
+template <int MT> __global__ void __launch_bounds__(OUT_THREADS, 1) k_gla_chunk_out_mma(const ncb_gla a) {
     extern __shared__ __align__(16) uint8_t raw[];
     asm volatile("griddepcontrol.wait;" ::: "memory");
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     constexpr int C = 16 * MT, sc = C + 8;
     const int chunk = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int first = a.chunk_first[chunk], n = a.chunk_count[chunk], D = a.dim, V = a.vdim, HD = a.heads * D;
-    const int sd = D + 4, sq = D + 8;
+    const int first = a.chunk_first[chunk], n = a.chunk_count[chunk], D = a.dim, V = a.vdim, HD = a.heads * D, sq = D + 8;
     bf16 *vs = reinterpret_cast<bf16 *>(raw);                     /* [C][VT + 8] */
     bf16 *at = vs + C * (VT + 8);                                 /* [2][C][sc]: scores' terms, [t][s] */
-    bf16 *qt = at + 2 * C * sc;                                   /* [2][C][sq]: terms of q with the decays since the chunk's start */
-    float *q = reinterpret_cast<float *>(qt + 2 * C * sq), *k = q + C * sd, *al = k + C * sd, *qs = al + C * sd, *done = qs + SUB * sd;
-    float *sums = done + D, *rstd = sums + 8 * C;
+    bf16 *qs = at + 2 * C * sc, *kd = qs + 2 * C * sq;            /* [2][C][sq] each */
+    bf16 *q = kd + 2 * C * sq, *k = q + C * D;                    /* [C][D], as projected */
+    float *al = reinterpret_cast<float *>(k + C * D), *G = al + C * D, *sums = G + MT * D, *rstd = sums + OUT_WARPS * C;
     const bf16 *proj = (const bf16 *)a.proj;
-    stage_v<C>(a, smem_addr(vs), first, n, h, 0);
-    for (int i = tid; i < C * (D / 4); i += CHUNK_THREADS) {
+    for (int i = tid; i < C * (D / 4); i += OUT_THREADS) {
         const int t = i / (D / 4), d = i % (D / 4) * 4;
-        cp_async16(smem_addr(al + t * sd + d), a.decay + (size_t)(first + (t < n ? t : 0)) * HD + h * D + d, t < n);
+        cp_async16(smem_addr(al + t * D + d), a.decay + (size_t)(first + (t < n ? t : 0)) * HD + h * D + d, t < n);
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    for (int i = tid; i < C * (D / 8); i += CHUNK_THREADS) {
+    for (int i = tid; i < C * (D / 8); i += OUT_THREADS) {
         const int t = i / (D / 8), d = i % (D / 8) * 8;
         const bf16 *p = proj + (size_t)(first + (t < n ? t : 0)) * a.ldp + h * D + d;
-        const uint4 z = make_uint4(0u, 0u, 0u, 0u);
-        const uint4 qv = t < n ? *reinterpret_cast<const uint4 *>(p + a.off_q) : z, kv = t < n ? *reinterpret_cast<const uint4 *>(p + a.off_k) : z;
-        const __nv_bfloat162 *qp = reinterpret_cast<const __nv_bfloat162 *>(&qv), *kp = reinterpret_cast<const __nv_bfloat162 *>(&kv);
+        cp_async16(smem_addr(q + t * D + d), p + a.off_q, t < n);
+        cp_async16(smem_addr(k + t * D + d), p + a.off_k, t < n);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    stage_v<C, OUT_THREADS>(a, smem_addr(vs), first, n, h, 0);
+    for (int i = tid; i < C * sc; i += OUT_THREADS) reinterpret_cast<uint32_t *>(at)[i] = 0u; /* both terms */
+    for (int i = tid; i < OUT_WARPS * C; i += OUT_THREADS) sums[i] = 0.f;
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    __syncthreads();
+    for (int i = tid; i < MT * D; i += OUT_THREADS) { /* alpha, q and k of tokens past n are zero */
+        const int sub = i / D, d = i - sub * D;
+        float f = 1.f, v[SUB];
 #pragma unroll
-        for (int j = 0; j < 4; j++) {
-            const float2 x = __bfloat1622float2(qp[j]), y = __bfloat1622float2(kp[j]);
-            *reinterpret_cast<float2 *>(q + t * sd + d + 2 * j) = make_float2(x.x * a.q_scale, x.y * a.q_scale);
-            *reinterpret_cast<float2 *>(k + t * sd + d + 2 * j) = y;
+        for (int t = 0; t < SUB; t++) {
+            v[t] = al[(sub * SUB + t) * D + d];
+            f *= v[t];
+            const int r = sub * SUB + t;
+            const float x = to_f(q[r * D + d]) * a.q_scale * f;
+            const bf16 hi = __float2bfloat16_rn(x);
+            qs[r * sq + d] = hi;
+            qs[(C + r) * sq + d] = __float2bfloat16_rn(x - to_f(hi));
+        }
+        G[i] = f;
+        f = 1.f;
+#pragma unroll
+        for (int t = SUB - 1; t >= 0; t--) {
+            const int r = sub * SUB + t;
+            const float x = to_f(k[r * D + d]) * f;
+            const bf16 hi = __float2bfloat16_rn(x);
+            kd[r * sq + d] = hi;
+            kd[(C + r) * sq + d] = __float2bfloat16_rn(x - to_f(hi));
+            f *= v[t];
         }
     }
-    for (int i = tid; i < C * sc; i += CHUNK_THREADS) reinterpret_cast<uint32_t *>(at)[i] = 0u; /* both terms */
-    for (int d = tid; d < D; d += CHUNK_THREADS) done[d] = 1.f;
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
+    const int g = lane >> 2, t2 = (lane & 3) * 2;
     auto put_score = [&](int t, int s, float v) {
         const bf16 hi = __float2bfloat16_rn(v);
         at[t * sc + s] = hi;
         at[(C + t) * sc + s] = __float2bfloat16_rn(v - to_f(hi));
     };
-#pragma unroll 1
-    for (int i0 = 0; i0 < n; i0 += SUB) { /* the walk of k_gla_chunk_out; alpha, q and k of tokens past n are zero */
-        for (int d = tid; d < D; d += CHUNK_THREADS) {
-            float f = 1.f;
+    for (int task = warp; task < MT * (MT - 1) / 2; task += OUT_WARPS) { /* pairs (i, j), j < i */
+        int i = 1, j = task;
+        while (j >= i) j -= i, i++;
+        if (i * SUB >= n) continue;
+        float acc[2][4] = {};
+        const uint32_t xa = smem_addr(qs) + ((i * SUB + (lane & 15)) * sq + (lane >> 4) * 8) * 2;
+        const uint32_t ya = smem_addr(kd) + ((j * SUB + (lane >> 4) * 8 + (lane & 7)) * sq + ((lane >> 3) & 1) * 8) * 2;
+        for (int d0 = 0; d0 < D; d0 += 16) {
+            uint32_t xh[4], xl[4], yh[4], yl[4];
+            ldsm4(xh, xa + d0 * 2);
+            ldsm4(xl, xa + (C * sq + d0) * 2);
+            ldsm4(yh, ya + d0 * 2);
+            ldsm4(yl, ya + (C * sq + d0) * 2);
+            if (i - j > 1) {
+                float f[4] = {1.f, 1.f, 1.f, 1.f}; /* columns t2, t2 + 1, t2 + 8, t2 + 9 */
+                for (int m = j + 1; m < i; m++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) f[e] *= G[m * D + d0 + t2 + (e & 1) + (e >> 1) * 8];
+                rescale2(xh[0], xl[0], f[0], f[1]), rescale2(xh[1], xl[1], f[0], f[1]);
+                rescale2(xh[2], xl[2], f[2], f[3]), rescale2(xh[3], xl[3], f[2], f[3]);
+            }
+#pragma unroll
+            for (int c = 0; c < 2; c++) {
+                mma_bf16(acc[c], xh, yh[2 * c], yh[2 * c + 1]);
+                mma_bf16(acc[c], xh, yl[2 * c], yl[2 * c + 1]);
+                mma_bf16(acc[c], xl, yh[2 * c], yh[2 * c + 1]);
+            }
+        }
+#pragma unroll
+        for (int c = 0; c < 2; c++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) put_score(i * SUB + g + (e >> 1) * 8, j * SUB + c * 8 + t2 + (e & 1), acc[c][e]);
+    }
+    for (int task = OUT_WARPS - 1 - warp; task < MT * 4; task += OUT_WARPS) { /* (sub-chunk, four s) */
+        const int i0 = task / 4 * SUB, s0 = task % 4 * 4;
+        if (i0 >= n) continue;
+        float acc[64]; /* [s][t] */
+#pragma unroll
+        for (int e = 0; e < 64; e++) acc[e] = 0.f;
+        for (int d = lane; d < D; d += 32) {
+            float f[4];
+#pragma unroll
+            for (int e = 0; e < 4; e++) f[e] = to_f(k[(i0 + s0 + e) * D + d]) * a.q_scale;
 #pragma unroll
             for (int t = 0; t < SUB; t++) {
-                f *= al[(i0 + t) * sd + d];
-                qs[t * sd + d] = q[(i0 + t) * sd + d] * f;
-            }
-        }
-        __syncthreads();
-        for (int e = tid; e < SUB * i0; e += CHUNK_THREADS) {
-            const int t = e % SUB, s = e / SUB;
-            const float4 *x = reinterpret_cast<const float4 *>(qs + t * sd), *y = reinterpret_cast<const float4 *>(k + s * sd);
-            float v0 = 0.f, v1 = 0.f;
-#pragma unroll 4
-            for (int d = 0; d < D / 4; d++) {
-                const float4 xv = x[d], yv = y[d];
-                v0 = fmaf(xv.x, yv.x, v0), v1 = fmaf(xv.y, yv.y, v1), v0 = fmaf(xv.z, yv.z, v0), v1 = fmaf(xv.w, yv.w, v1);
-            }
-            put_score(i0 + t, s, v0 + v1);
-        }
-        {
-            const int s = tid >> 4, l16 = tid & 15;
-            float acc[SUB];
+                if (t < s0) continue;
+                const float x = to_f(q[(i0 + t) * D + d]), al_t = al[(i0 + t) * D + d];
 #pragma unroll
-            for (int t = 0; t < SUB; t++) acc[t] = 0.f;
-            for (int d = l16; d < D; d += 16) {
-                float f = k[(i0 + s) * sd + d];
-#pragma unroll
-                for (int t = 0; t < SUB; t++) {
-                    if (t > s) f *= al[(i0 + t) * sd + d];
-                    if (t >= s) acc[t] = fmaf(q[(i0 + t) * sd + d], f, acc[t]);
+                for (int e = 0; e < 4; e++) {
+                    if (t > s0 + e) f[e] *= al_t;
+                    if (t >= s0 + e) acc[e * 16 + t] = fmaf(x, f[e], acc[e * 16 + t]);
                 }
             }
-#pragma unroll
-            for (int t = 0; t < SUB; t++) {
-                float v = acc[t];
-                for (int o = 8; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-                if (l16 == t && t >= s) put_score(i0 + t, i0 + s, v);
-            }
         }
-        __syncthreads();
-        for (int d = tid; d < D; d += CHUNK_THREADS) {
-            const float before = done[d];
-            float f = 1.f;
+        reduce64(acc, lane);
+        const int at0 = 2 * lane;
 #pragma unroll
-            for (int t = SUB - 1; t >= 0; t--) {
-                k[(i0 + t) * sd + d] *= f;
-                f *= al[(i0 + t) * sd + d];
-                const float x = qs[t * sd + d] * before;
-                const bf16 hi = __float2bfloat16_rn(x);
-                qt[(i0 + t) * sq + d] = hi;
-                qt[(C + i0 + t) * sq + d] = __float2bfloat16_rn(x - to_f(hi));
-            }
-            for (int s = 0; s < i0; s++) k[s * sd + d] *= f;
-            done[d] = before * f;
+        for (int e = 0; e < 2; e++) {
+            const int s = s0 + (at0 + e) / 16, t = (at0 + e) % 16;
+            if (t >= s) put_score(i0 + t, i0 + s, acc[e]);
         }
-        __syncthreads();
     }
+    __syncthreads();
+    for (int i = tid; i < (MT - 1) * D / 2; i += OUT_THREADS) { /* qs <- qs G_0 .. G_(sub - 1), channels d, d + 1 */
+        const int sub = 1 + i / (D / 2), d = i % (D / 2) * 2;
+        float f0 = 1.f, f1 = 1.f;
+        for (int m = 0; m < sub; m++) f0 *= G[m * D + d], f1 *= G[m * D + d + 1];
+#pragma unroll 4
+        for (int t = 0; t < SUB; t++) {
+            uint32_t *hi = reinterpret_cast<uint32_t *>(qs + (sub * SUB + t) * sq + d), *lo = reinterpret_cast<uint32_t *>(qs + (C + sub * SUB + t) * sq + d);
+            uint32_t x = *hi, y = *lo;
+            rescale2(x, y, f0, f1);
+            *hi = x, *lo = y;
+        }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
     const float *state = a.states + ((size_t)chunk * a.heads + h) * D * V;
-    const int g = lane >> 2, t2 = (lane & 3) * 2, col0 = warp * 32;
-    const uint32_t qb = smem_addr(qt) + ((lane & 15) * sq + (lane >> 4) * 8) * 2, ab = smem_addr(at) + ((lane & 15) * sc + (lane >> 4) * 8) * 2;
+    const int col0 = warp * 16;
+    const uint32_t qb = smem_addr(qs) + ((lane & 15) * sq + (lane >> 4) * 8) * 2, ab = smem_addr(at) + ((lane & 15) * sc + (lane >> 4) * 8) * 2;
     const uint32_t vb = smem_addr(vs) + ((lane & 15) * (VT + 8) + col0 + (lane >> 4) * 8) * 2;
     const bool direct = V <= VT; /* the whole row of a token is in this block's registers */
-    for (int i = tid; i < 8 * C; i += CHUNK_THREADS) sums[i] = 0.f;
     for (int v0 = 0; v0 < V; v0 += VT) {
         if (v0 > 0) {
             __syncthreads();
-            stage_v<C>(a, smem_addr(vs), first, n, h, v0);
+            stage_v<C, OUT_THREADS>(a, smem_addr(vs), first, n, h, v0);
             asm volatile("cp.async.wait_group 0;" ::: "memory");
             __syncthreads();
         }
-        float acc[MT][4][4];
+        float acc[MT][2][4];
 #pragma unroll
-        for (int i = 0; i < MT * 16; i++) acc[i >> 4][(i >> 2) & 3][i & 3] = 0.f;
-        const int cols = min(32, V - v0 - col0); /* <= 0: this warp has none */
-        float next[4][4];
-        auto load = [&](int k0) {
+        for (int i = 0; i < MT * 8; i++) acc[i >> 3][(i >> 2) & 1][i & 3] = 0.f;
+        const bool live = v0 + col0 < V; /* vdim is a multiple of 16: both column tiles or none */
+        constexpr int DEPTH = 3;         /* k-steps of the state in flight */
+        float next[DEPTH][2][4];
+        auto load = [&](int k0, int slot) {
 #pragma unroll
-            for (int c = 0; c < 4; c++) {
+            for (int c = 0; c < 2; c++) {
                 const float *p = state + (size_t)(k0 + t2) * V + v0 + col0 + c * 8 + g;
-                const bool on = c * 8 < cols;
-                next[c][0] = on ? p[0] : 0.f, next[c][1] = on ? p[V] : 0.f;
-                next[c][2] = on ? p[(size_t)8 * V] : 0.f, next[c][3] = on ? p[(size_t)9 * V] : 0.f;
+                const bool on = live && k0 < D;
+                next[slot][c][0] = on ? p[0] : 0.f, next[slot][c][1] = on ? p[V] : 0.f;
+                next[slot][c][2] = on ? p[(size_t)8 * V] : 0.f, next[slot][c][3] = on ? p[(size_t)9 * V] : 0.f;
             }
         };
-        load(0);
-        for (int k0 = 0; k0 < D; k0 += 16) {
-            uint32_t hi[4][2], lo[4][2];
 #pragma unroll
-            for (int c = 0; c < 4; c++) split2(next[c][0], next[c][1], hi[c][0], lo[c][0]), split2(next[c][2], next[c][3], hi[c][1], lo[c][1]);
-            if (k0 + 16 < D) load(k0 + 16);
+        for (int j = 0; j < DEPTH; j++) load(16 * j, j);
+        for (int kb = 0; kb < D; kb += 16 * DEPTH) {
 #pragma unroll
-            for (int m = 0; m < MT; m++) {
-                uint32_t xh[4], xl[4];
-                ldsm4(xh, qb + (m * 16 * sq + k0) * 2);
-                ldsm4(xl, qb + ((C + m * 16) * sq + k0) * 2);
+            for (int j = 0; j < DEPTH; j++) {
+                const int k0 = kb + 16 * j;
+                if (k0 >= D) break;
+                uint32_t hi[2][2], lo[2][2];
 #pragma unroll
-                for (int c = 0; c < 4; c++) {
-                    mma_bf16(acc[m][c], xh, hi[c][0], hi[c][1]);
-                    mma_bf16(acc[m][c], xh, lo[c][0], lo[c][1]);
-                    mma_bf16(acc[m][c], xl, hi[c][0], hi[c][1]);
+                for (int c = 0; c < 2; c++) split2(next[j][c][0], next[j][c][1], hi[c][0], lo[c][0]), split2(next[j][c][2], next[j][c][3], hi[c][1], lo[c][1]);
+                load(k0 + 16 * DEPTH, j);
+#pragma unroll
+                for (int m = 0; m < MT; m++) {
+                    uint32_t xh[4], xl[4];
+                    ldsm4(xh, qb + (m * 16 * sq + k0) * 2);
+                    ldsm4(xl, qb + ((C + m * 16) * sq + k0) * 2);
+#pragma unroll
+                    for (int c = 0; c < 2; c++) {
+                        mma_bf16(acc[m][c], xh, hi[c][0], hi[c][1]);
+                        mma_bf16(acc[m][c], xh, lo[c][0], lo[c][1]);
+                        mma_bf16(acc[m][c], xl, hi[c][0], hi[c][1]);
+                    }
                 }
             }
         }
 #pragma unroll
         for (int kk = 0; kk < MT; kk++) { /* 16 tokens of the chunk itself; rows before them see none of it */
-            uint32_t b[2][4];
-            ldsm4_t(b[0], vb + kk * 16 * (VT + 8) * 2);
-            ldsm4_t(b[1], vb + kk * 16 * (VT + 8) * 2 + 32);
+            uint32_t b[4];
+            ldsm4_t(b, vb + kk * 16 * (VT + 8) * 2);
 #pragma unroll
             for (int m = kk; m < MT; m++) {
                 uint32_t xh[4], xl[4];
                 ldsm4(xh, ab + (m * 16 * sc + kk * 16) * 2);
                 ldsm4(xl, ab + ((C + m * 16) * sc + kk * 16) * 2);
 #pragma unroll
-                for (int c = 0; c < 4; c++) {
-                    mma_bf16(acc[m][c], xh, b[c >> 1][(c & 1) * 2], b[c >> 1][(c & 1) * 2 + 1]);
-                    mma_bf16(acc[m][c], xl, b[c >> 1][(c & 1) * 2], b[c >> 1][(c & 1) * 2 + 1]);
+                for (int c = 0; c < 2; c++) {
+                    mma_bf16(acc[m][c], xh, b[2 * c], b[2 * c + 1]);
+                    mma_bf16(acc[m][c], xl, b[2 * c], b[2 * c + 1]);
                 }
             }
         }
-        __syncthreads(); /* the sums are cleared */
 #pragma unroll
         for (int m = 0; m < MT; m++)
 #pragma unroll
             for (int r = 0; r < 2; r++) {
                 float s = 0.f;
 #pragma unroll
-                for (int c = 0; c < 4; c++) s += acc[m][c][2 * r] * acc[m][c][2 * r] + acc[m][c][2 * r + 1] * acc[m][c][2 * r + 1];
+                for (int c = 0; c < 2; c++) s += acc[m][c][2 * r] * acc[m][c][2 * r] + acc[m][c][2 * r + 1] * acc[m][c][2 * r + 1];
                 s += __shfl_xor_sync(0xffffffffu, s, 1);
                 s += __shfl_xor_sync(0xffffffffu, s, 2);
                 if ((lane & 3) == 0) sums[warp * C + m * 16 + r * 8 + g] += s;
@@ -738,11 +801,12 @@ template <int MT> __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_chunk_o
             __syncthreads();
             if (tid < C) {
                 float s = 0.f;
-                for (int w = 0; w < 8; w++) s += sums[w * C + tid];
+                for (int w = 0; w < OUT_WARPS; w++) s += sums[w * C + tid];
                 rstd[tid] = 1.f / sqrtf(s / (float)a.norm_count + a.eps);
             }
             __syncthreads();
         }
+        if (!live) continue;
 #pragma unroll
         for (int m = 0; m < MT; m++)
 #pragma unroll
@@ -751,9 +815,8 @@ template <int MT> __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_chunk_o
                 if (t >= n) continue;
                 const bf16 *gp = proj + (size_t)(first + t) * a.ldp + a.off_g + h * V;
 #pragma unroll
-                for (int c = 0; c < 4; c++) {
+                for (int c = 0; c < 2; c++) {
                     const int v = v0 + col0 + c * 8 + t2;
-                    if (c * 8 >= cols) continue;
                     if (direct) {
                         const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(gp + v));
                         const float2 w = *reinterpret_cast<const float2 *>(a.norm + v);
@@ -770,11 +833,11 @@ template <int MT> __global__ void __launch_bounds__(CHUNK_THREADS) k_gla_chunk_o
     __syncthreads();
     if (tid < C) {
         float s = 0.f;
-        for (int w = 0; w < 8; w++) s += sums[w * C + tid];
+        for (int w = 0; w < OUT_WARPS; w++) s += sums[w * C + tid];
         rstd[tid] = 1.f / sqrtf(s / (float)a.norm_count + a.eps);
     }
     __syncthreads(); /* this block's raw outputs are visible to all of its threads */
-    for (int i = tid; i < n * V; i += CHUNK_THREADS) {
+    for (int i = tid; i < n * V; i += OUT_THREADS) {
         const int t = i / V, v = i % V;
         const float gate = silu(to_f(proj[(size_t)(first + t) * a.ldp + a.off_g + h * V + v]));
         ((bf16 *)a.out)[(size_t)(first + t) * a.ldo + h * V + v] =
@@ -874,8 +937,8 @@ int gla_chunked(const ncb_gla *g, int f32, void *stream_ptr) {
         if (rc != NCB_OK) return rc;
         rc = launch(k_gla_scan, scan_grid, CHUNK_THREADS, 0, 1, stream, *g);
         if (rc != NCB_OK || !g->out) return rc;
-        return C == 64 ? launch(k_gla_chunk_out_mma<4>, out_grid, CHUNK_THREADS, out_mma_bytes<4>(g->dim), 1, stream, *g)
-                       : launch(k_gla_chunk_out_mma<2>, out_grid, CHUNK_THREADS, out_mma_bytes<2>(g->dim), 1, stream, *g);
+        return C == 64 ? launch(k_gla_chunk_out_mma<4>, out_grid, OUT_THREADS, out_mma_bytes<4>(g->dim), 1, stream, *g)
+                       : launch(k_gla_chunk_out_mma<2>, out_grid, OUT_THREADS, out_mma_bytes<2>(g->dim), 1, stream, *g);
     }
     rc = f32 ? launch(k_gla_chunk_state<float>, state_grid, CHUNK_THREADS, state_smem, 1, stream, *g)
              : launch(k_gla_chunk_state<bf16>, state_grid, CHUNK_THREADS, state_smem, 1, stream, *g);

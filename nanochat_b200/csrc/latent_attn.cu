@@ -94,6 +94,22 @@ __device__ __forceinline__ int length_of(const ncb_latent &a, int row, int &slot
     return pos + 1;
 }
 
+/* Two neighbouring values as one load and store. */
+template <typename T> __device__ __forceinline__ float2 load2(const T *p);
+template <> __device__ __forceinline__ float2 load2<float>(const float *p) { return *reinterpret_cast<const float2 *>(p); }
+template <> __device__ __forceinline__ float2 load2<bf16>(const bf16 *p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(p)); }
+__device__ __forceinline__ void store2(float *p, float x, float y) { *reinterpret_cast<float2 *>(p) = make_float2(x, y); }
+__device__ __forceinline__ void store2(bf16 *p, float x, float y) { *reinterpret_cast<__nv_bfloat162 *>(p) = __floats2bfloat162_rn(x, y); }
+
+/* Rotation of pairs i, i + 1 (i even) of one head's or key's rotated part, from `q` to `out` (may be the same). */
+template <typename T> __device__ __forceinline__ void rotate_pairs(const ncb_latent &a, const T *q, T *out, int pos, int i) {
+    const int half = a.rot / 2;
+    const float2 c = *reinterpret_cast<const float2 *>(a.cos + (size_t)pos * half + i), t = *reinterpret_cast<const float2 *>(a.sin + (size_t)pos * half + i);
+    const float2 u = load2<T>(q + i), v = load2<T>(q + half + i);
+    store2(out + i, u.x * c.x - v.x * t.x, u.y * c.y - v.y * t.y);
+    store2(out + half + i, v.x * c.x + u.x * t.x, v.y * c.y + u.y * t.y);
+}
+
 /* One warp: norm of the latent, rotation of the key part, one cache row. */
 template <typename T> __device__ __forceinline__ void append_row(const ncb_latent &a, int row, int lane) {
     int slot;
@@ -102,29 +118,19 @@ template <typename T> __device__ __forceinline__ void append_row(const ncb_laten
     const T *kv = (const T *)a.proj + (size_t)row * a.ldp + a.off_kv;
     T *out = (T *)a.cache + ((size_t)slot * a.capacity + (len - 1)) * (a.rank + a.rot);
     float s = 0.f;
-    for (int i = lane; i < a.rank; i += 32) {
-        const float v = to_f(kv[i]);
-        s = fmaf(v, v, s);
+#pragma unroll 8
+    for (int i = lane * 2; i < a.rank; i += 64) {
+        const float2 v = load2<T>(kv + i);
+        s = fmaf(v.x, v.x, fmaf(v.y, v.y, s));
     }
     for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
     const float rstd = 1.f / sqrtf(s / (float)a.norm_count + a.eps);
-    for (int i = lane; i < a.rank; i += 32) out[i] = from_f<T>(to_f(kv[i]) * rstd * a.norm[i]);
-    const int half = a.rot / 2;
-    const float *cs = a.cos + (size_t)(len - 1) * half, *sn = a.sin + (size_t)(len - 1) * half;
-    for (int i = lane; i < half; i += 32) {
-        const float u = to_f(kv[a.rank + i]), v = to_f(kv[a.rank + half + i]), c = cs[i], t = sn[i];
-        out[a.rank + i] = from_f<T>(u * c - v * t);
-        out[a.rank + half + i] = from_f<T>(v * c + u * t);
+#pragma unroll 8
+    for (int i = lane * 2; i < a.rank; i += 64) {
+        const float2 v = load2<T>(kv + i), w = *reinterpret_cast<const float2 *>(a.norm + i);
+        store2(out + i, v.x * rstd * w.x, v.y * rstd * w.y);
     }
-}
-
-/* Rotation of one head's q_rot for one row, from `q` to `out` (may be the same); one pair per call index. */
-template <typename T> __device__ __forceinline__ void rotate_pair(const ncb_latent &a, const T *q, T *out, int pos, int i) {
-    const int half = a.rot / 2;
-    const float c = a.cos[(size_t)pos * half + i], t = a.sin[(size_t)pos * half + i];
-    const float u = to_f(q[i]), v = to_f(q[half + i]);
-    out[i] = from_f<T>(u * c - v * t);
-    out[half + i] = from_f<T>(v * c + u * t);
+    for (int i = lane * 2; i < a.rot / 2; i += 64) rotate_pairs(a, kv + a.rank, out + a.rank, len - 1, i);
 }
 
 /* ---- absorbed form: query ------------------------------------------------------------------------------------------- */
@@ -150,11 +156,11 @@ template <typename T> __global__ void __launch_bounds__(THREADS) k_latent_query(
     T *out = (T *)a.q_abs;
     if (rotate) {
         for (int r = h + warp * a.heads; r < rows; r += a.heads * (THREADS / 32)) append_row<T>(a, r0 + r, lane);
-        const int half = a.rot / 2;
-        for (int i = tid; i < rows * half; i += THREADS) {
-            const int row = r0 + i / half, pos = a.pos[row];
+        const int pairs = a.rot / 4;
+        for (int i = tid; i < rows * pairs; i += THREADS) {
+            const int row = r0 + i / pairs, pos = a.pos[row];
             if (pos >= 0 && pos < a.table_len)
-                rotate_pair(a, q + (size_t)row * a.ldp + a.dim, out + ((size_t)row * a.heads + h) * W + a.rank, pos, i % half);
+                rotate_pairs(a, q + (size_t)row * a.ldp + a.dim, out + ((size_t)row * a.heads + h) * W + a.rank, pos, i % pairs * 2);
         }
         return;
     }
@@ -594,12 +600,13 @@ template <typename T> __global__ void __launch_bounds__(THREADS) k_latent_append
     const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (row >= a.rows) return;
     append_row<T>(a, row, lane);
-    const int pos = a.pos[row], half = a.rot / 2;
+    const int pos = a.pos[row], pairs = a.rot / 4;
     if (!a.rotate_q || pos < 0 || pos >= a.table_len) return;
     T *q = (T *)a.proj + (size_t)row * a.ldp + a.off_q + a.dim;
-    for (int i = lane; i < a.heads * half; i += 32) {
-        T *p = q + (size_t)(i / half) * (a.dim + a.rot);
-        rotate_pair(a, p, p, pos, i % half);
+#pragma unroll 4
+    for (int i = lane; i < a.heads * pairs; i += 32) {
+        T *p = q + (size_t)(i / pairs) * (a.dim + a.rot);
+        rotate_pairs(a, p, p, pos, i % pairs * 2);
     }
 }
 
@@ -625,12 +632,13 @@ constexpr int PF_ROWS = 64, PF_KEYS = 64; /* query rows and keys per tile: four 
 /* Grid (heads, row tiles): PF_ROWS consecutive rows of one sequence against its expanded keys and values, one head. Keys
  * and values of 64 positions per stage (cp.async, two stages); a warp owns 16 rows over the whole range: scores, fp32
  * softmax and the second product (probabilities as two bf16 terms) in registers. QS: 16-wide steps of the score depth;
- * VN: 16-wide column tiles of the values (both upper bounds). */
-template <int QS, int VN> __global__ void __launch_bounds__(THREADS, 2) k_latent_prefill(const ncb_latent a) {
+ * VN: 16-wide column tiles of the values (both upper bounds, or with EXACT the sizes). */
+template <int QS, int VN, bool EXACT> __global__ void __launch_bounds__(THREADS, 2) k_latent_prefill(const ncb_latent a) {
     extern __shared__ __align__(128) uint8_t raw[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-    const int h = blockIdx.x, tile = blockIdx.y, depth = a.dim + a.rot, steps = depth / 16, cols = a.vdim / 16;
-    const int krow = depth * 2 + 16, vrow = a.vdim * 2 + 16, stage_bytes = PF_KEYS * (krow + vrow);
+    const int h = blockIdx.x, tile = blockIdx.y, depth = EXACT ? QS * 16 : a.dim + a.rot, vdim = EXACT ? VN * 16 : a.vdim;
+    const int steps = depth / 16, cols = vdim / 16;
+    const int krow = depth * 2 + 16, vrow = vdim * 2 + 16, stage_bytes = PF_KEYS * (krow + vrow);
     asm volatile("griddepcontrol.wait;" ::: "memory");
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     const int row0 = a.tile_row[tile], n_rows = min(a.tile_rows[tile], PF_ROWS), ctx0 = a.tile_ctx[tile], pos0 = a.tile_pos[tile];
@@ -640,21 +648,16 @@ template <int QS, int VN> __global__ void __launch_bounds__(THREADS, 2) k_latent
     const bf16 *kr = (const bf16 *)a.ctx_rot + (size_t)ctx0 * a.rot;
     auto fetch = [&](int i) {
         const uint32_t ks = smem + (i & 1) * stage_bytes, vs = ks + PF_KEYS * krow;
-        const int p0 = i * PF_KEYS, nd = a.dim / 8, nr = a.rot / 8, nv = a.vdim / 8;
-        for (int j = tid; j < PF_KEYS * nd; j += THREADS) {
-            const int r = j / nd, c = j % nd;
+        const int p0 = i * PF_KEYS, nd = a.dim / 8, nr = a.rot / 8, nv = a.vdim / 8, c0 = tid & 7;
+#pragma unroll
+        for (int j = 0; j < PF_KEYS / 16; j++) { /* eight threads per row, 16 rows at a time */
+            const int r = (tid >> 3) + 16 * j;
             const bool on = p0 + r < keys;
-            cp_async16(ks + r * krow + c * 16, kv + (size_t)(on ? p0 + r : 0) * a.ctx_kv_ld + c * 8, on);
-        }
-        for (int j = tid; j < PF_KEYS * nr; j += THREADS) {
-            const int r = j / nr, c = j % nr;
-            const bool on = p0 + r < keys;
-            cp_async16(ks + r * krow + (nd + c) * 16, kr + (size_t)(on ? p0 + r : 0) * a.rot + c * 8, on);
-        }
-        for (int j = tid; j < PF_KEYS * nv; j += THREADS) {
-            const int r = j / nv, c = j % nv;
-            const bool on = p0 + r < keys;
-            cp_async16(vs + r * vrow + c * 16, kv + (size_t)(on ? p0 + r : 0) * a.ctx_kv_ld + a.dim + c * 8, on);
+            const bf16 *src = kv + (size_t)(on ? p0 + r : 0) * a.ctx_kv_ld, *rot = kr + (size_t)(on ? p0 + r : 0) * a.rot;
+            const uint32_t kd = ks + r * krow, vd = vs + r * vrow;
+            for (int c = c0; c < nd; c += 8) cp_async16(kd + c * 16, src + c * 8, on);
+            for (int c = c0; c < nr; c += 8) cp_async16(kd + (nd + c) * 16, rot + c * 8, on);
+            for (int c = c0; c < nv; c += 8) cp_async16(vd + c * 16, src + a.dim + c * 8, on);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -924,8 +927,9 @@ int latent_prefill(const ncb_latent *g, void *stream) {
     const dim3 grid(g->heads, g->n_tiles);
     const size_t smem = (size_t)2 * PF_KEYS * ((g->dim + g->rot) * 2 + 16 + g->vdim * 2 + 16);
     cudaStream_t s = (cudaStream_t)stream;
-    return g->dim + g->rot <= 128 ? launch(k_latent_prefill<8, 8>, grid, smem, THREADS, 1, s, *g)
-                                  : launch(k_latent_prefill<12, 8>, grid, smem, THREADS, 1, s, *g);
+    if (g->dim + g->rot == 192 && g->vdim == 128) return launch(k_latent_prefill<12, 8, true>, grid, smem, THREADS, 1, s, *g);
+    return g->dim + g->rot <= 128 ? launch(k_latent_prefill<8, 8, false>, grid, smem, THREADS, 1, s, *g)
+                                  : launch(k_latent_prefill<12, 8, false>, grid, smem, THREADS, 1, s, *g);
 }
 
 } /* extern "C" */

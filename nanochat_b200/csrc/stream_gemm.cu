@@ -199,8 +199,18 @@ __global__ void __launch_bounds__(THREADS) k_stream_gemm(const __grid_constant__
     if (warp >= 2 && !a.norm_input) { /* row scales from the stream's partial sums; every block needs every row's */
         for (int r = tid - 64; r < a.rows; r += 64) {
             float v = 0.f;
-            if (a.rs.ss)
-                for (int i = 0; i < a.rs.ss_parts; i++) v += a.rs.ss[(size_t)r * a.rs.ss_parts + i];
+            if (a.rs.ss) {
+                const float *p = a.rs.ss + (size_t)r * a.rs.ss_parts;
+                if ((a.rs.ss_parts & 3) == 0) { /* the usual counts: four at a time, independent loads */
+#pragma unroll 8
+                    for (int i = 0; i < a.rs.ss_parts; i += 4) {
+                        const float4 s = *reinterpret_cast<const float4 *>(p + i);
+                        v += (s.x + s.y) + (s.z + s.w);
+                    }
+                } else {
+                    for (int i = 0; i < a.rs.ss_parts; i++) v += p[i];
+                }
+            }
             sumsq[r] = row_scale(a.rs, v);
         }
     }

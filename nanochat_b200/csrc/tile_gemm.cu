@@ -31,6 +31,8 @@ constexpr int BM = 128;          /* rows per tile = MMA M */
 constexpr int THREADS = 192;     /* producer warp, MMA warp, four epilogue warps */
 constexpr int A_BYTES = BM * KBLK * 2;
 
+constexpr int TURN_FLOATS = 32 * 33; /* per epilogue warp: see stream_columns */
+
 enum { EPI_STORE = 0, EPI_RESID = 1, EPI_RELU2 = 2, EPI_F32 = 3, EPI_GEGLU = 5, EPI_STREAM = 6 };
 
 template <int BN> struct Tile {
@@ -38,7 +40,8 @@ template <int BN> struct Tile {
     static constexpr int STAGE_BYTES = A_BYTES + B_BYTES;          /* 48 KB (BN 256) or 32 KB (BN 128) */
     static constexpr int STAGES = BN == 256 ? 4 : 6;               /* 192 KB of ring either way */
     static constexpr int RING_BYTES = STAGES * STAGE_BYTES;
-    static constexpr int SMEM_BYTES = 1024 + RING_BYTES + 256;     /* 1024: the ring is aligned by hand; 256: barriers */
+    /* 1024: the ring is aligned by hand; 256: barriers; then the stream update's staging */
+    static constexpr int smem_bytes(int epi) { return 1024 + RING_BYTES + 256 + (epi == EPI_STREAM ? 4 * TURN_FLOATS * 4 : 0); }
     static constexpr int TMEM_COLS = 2 * BN;                       /* two accumulators */
 };
 
@@ -93,30 +96,6 @@ template <int EPI> static __device__ __forceinline__ void store_columns(const Ti
             o[j] = __floats2bfloat162_rn(gelu_tanh(v[4 * j]) * v[4 * j + 1], gelu_tanh(v[4 * j + 2]) * v[4 * j + 3]);
         uint4 *dst = reinterpret_cast<uint4 *>(reinterpret_cast<bf16 *>(a.y) + (size_t)row * a.ldy + (n >> 1));
         dst[0] = packed[0], dst[1] = packed[1];
-    } else if (EPI == EPI_STREAM) {
-        float4 *h = reinterpret_cast<float4 *>(a.rs.h + at);
-        const float4 *gain = reinterpret_cast<const float4 *>(a.rs.gain + n);
-        uint4 packed[4];
-        __nv_bfloat162 *o = reinterpret_cast<__nv_bfloat162 *>(packed);
-        float4 hv[8];
-#pragma unroll
-        for (int j = 0; j < 8; j++) hv[j] = h[j];
-        float q = 0.f;
-#pragma unroll
-        for (int j = 0; j < 8; j++) {
-            float4 x = hv[j];
-            x.x += a.rs.mult * v[4 * j], x.y += a.rs.mult * v[4 * j + 1];
-            x.z += a.rs.mult * v[4 * j + 2], x.w += a.rs.mult * v[4 * j + 3];
-            q += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
-            h[j] = x;
-            const float4 g = gain[j];
-            o[2 * j] = __floats2bfloat162_rn(x.x * g.x, x.y * g.y);
-            o[2 * j + 1] = __floats2bfloat162_rn(x.z * g.z, x.w * g.w);
-        }
-        uint4 *dst = reinterpret_cast<uint4 *>(reinterpret_cast<bf16 *>(a.rs.x_next) + at);
-#pragma unroll
-        for (int j = 0; j < 4; j++) dst[j] = packed[j];
-        a.rs.ss_next[(size_t)row * (a.N >> 5) + (n >> 5)] = q;
     } else if ((EPI == EPI_STORE || EPI == EPI_F32) && (n + 32 > a.n_store || (a.ldy & 7))) {
 #pragma unroll
         for (int j = 0; j < 32; j++) /* the last stored columns, or rows without vector alignment */
@@ -152,6 +131,47 @@ template <int EPI> static __device__ __forceinline__ void store_columns(const Ti
 #pragma unroll
         for (int j = 0; j < 4; j++) dst[j] = packed[j];
     }
+}
+
+/* The stream update of 32 rows (first row m) x 32 columns (from n) by one warp. A thread's products belong to one row; the
+ * stream wants whole 128-byte lines, so they turn around in shared memory (`turn`, 32 x 33 floats of this warp) and are
+ * worked on as four rows x 32 columns per instruction. */
+static __device__ __forceinline__ void stream_columns(const TileArgs &a, int m, int n, const float *v, float factor, float *turn,
+                                                      int lane) {
+    const int r4 = lane >> 3, c4 = (lane & 7) * 4;
+    float4 h[8];
+#pragma unroll
+    for (int i = 0; i < 8; i++) {
+        const int row = m + 4 * i + r4;
+        h[i] = row < a.rows ? *reinterpret_cast<const float4 *>(a.rs.h + (size_t)row * a.N + n + c4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    const float4 gain = *reinterpret_cast<const float4 *>(a.rs.gain + n + c4);
+    factor *= a.rs.mult;
+#pragma unroll
+    for (int j = 0; j < 32; j++) turn[lane * 33 + j] = v[j] * factor;
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < 8; i++) {
+        const int row = m + 4 * i + r4;
+        const float *p = turn + (4 * i + r4) * 33 + c4;
+        float4 x = h[i];
+        x.x += p[0], x.y += p[1], x.z += p[2], x.w += p[3];
+        float q = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+        q += __shfl_xor_sync(0xffffffffu, q, 1);
+        q += __shfl_xor_sync(0xffffffffu, q, 2);
+        q += __shfl_xor_sync(0xffffffffu, q, 4);
+        if (row < a.rows) {
+            const size_t at = (size_t)row * a.N + n + c4;
+            *reinterpret_cast<float4 *>(a.rs.h + at) = x;
+            uint2 out;
+            __nv_bfloat162 *o = reinterpret_cast<__nv_bfloat162 *>(&out);
+            o[0] = __floats2bfloat162_rn(x.x * gain.x, x.y * gain.y);
+            o[1] = __floats2bfloat162_rn(x.z * gain.z, x.w * gain.w);
+            *reinterpret_cast<uint2 *>(reinterpret_cast<bf16 *>(a.rs.x_next) + at) = out;
+            if ((lane & 7) == 0) a.rs.ss_next[(size_t)row * (a.N >> 5) + (n >> 5)] = q;
+        }
+    }
+    __syncwarp(); /* the staging is free again */
 }
 
 template <int BN, int EPI>
@@ -264,6 +284,7 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm(const __grid_constant_
         }
     } else { /* epilogue warps 2..5: tensor-memory lanes 32 (warp % 4) .. + 31 */
         const int quarter = warp & 3;
+        float *turn = reinterpret_cast<float *>(tail + 256) + quarter * TURN_FLOATS; /* EPI_STREAM only */
         uint32_t it = 0;
         for (int u = blockIdx.x; u < units; u += gridDim.x, it++) {
             const uint32_t buf = it & 1;
@@ -282,6 +303,10 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm(const __grid_constant_
             for (int c = 0; c < un.width / 32; c++) {
                 float v[32];
                 tmem_load32(tmem + ((uint32_t)(quarter * 32) << 16) + buf * BN + c * 32, v);
+                if (EPI == EPI_STREAM) {
+                    stream_columns(a, m0 + quarter * 32, n0 + c * 32, v, factor, turn, lane);
+                    continue;
+                }
                 if (!live) continue;
                 store_columns<EPI>(a, row, n0 + c * 32, v, factor);
             }
@@ -318,14 +343,15 @@ constexpr bool PAIR_BY_DEFAULT = true;
  * neighbouring accumulator columns. <256, 1> is the standard tile; <160, 2> (320 wide, one accumulator) exists for
  * widths like 1280, where 256-wide tiles leave a last round that is nearly empty (80 tiles for 74 pairs) and 320-wide
  * tiles fit one round (64). Of an MMA's NMMA W rows each block stages NMMA / 2. */
-template <int NMMA, int NSUB> struct Pair {
+template <int NMMA, int NSUB, int EPI> struct Pair {
     static constexpr int WIDTH = NMMA * NSUB;
+    static constexpr int TURN_BYTES = EPI == EPI_STREAM ? 4 * TURN_FLOATS * 4 : 0; /* the stream update's staging */
     static constexpr int SUB_BYTES = (NMMA / 2) * KBLK * 2;        /* this block's W rows of one MMA */
     static constexpr int B_BYTES = NSUB * SUB_BYTES;
     static constexpr int STAGE_BYTES = A_BYTES + B_BYTES;          /* 32 KB (256 wide) or 36 KB (320 wide) */
-    static constexpr int STAGES = 6;
+    static constexpr int STAGES = WIDTH > 256 && EPI == EPI_STREAM ? 5 : 6;
     static constexpr int RING_BYTES = STAGES * STAGE_BYTES;
-    static constexpr int SMEM_BYTES = 1024 + RING_BYTES + 256;
+    static constexpr int SMEM_BYTES = 1024 + RING_BYTES + 256 + TURN_BYTES;
     static constexpr int ACCS = 2 * WIDTH <= 512 ? 2 : 1;          /* accumulators in tensor memory */
     static constexpr int TMEM_COLS = 512;
     static_assert(SUB_BYTES % 1024 == 0 && NMMA % 32 == 0 && NMMA <= 256 && WIDTH <= 512, "swizzle atoms, MMA shape");
@@ -382,7 +408,7 @@ template <int NMMA, int NSUB, int EPI>
 __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm_pair(const __grid_constant__ CUtensorMap map_x,
                                                                const __grid_constant__ CUtensorMap map_w,
                                                                const __grid_constant__ CUtensorMap map_w_half, const TileArgs a) {
-    using P = Pair<NMMA, NSUB>;
+    using P = Pair<NMMA, NSUB, EPI>;
     constexpr int STAGES = P::STAGES, WIDTH = P::WIDTH, ACCS = P::ACCS;
     extern __shared__ uint8_t raw[];
     const uint32_t raw_addr = smem_u32(raw);
@@ -507,6 +533,7 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm_pair(const __grid_cons
         }
     } else { /* epilogue warps 2..5 of both blocks: this block's tensor-memory lanes 32 (warp % 4) .. + 31 */
         const int quarter = warp & 3;
+        float *turn = reinterpret_cast<float *>(tail + 256) + quarter * TURN_FLOATS; /* EPI_STREAM only */
         uint32_t it = 0;
         for (int u = pair; u < units; u += n_pairs, it++) {
             const uint32_t buf = acc_of(it);
@@ -525,6 +552,10 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm_pair(const __grid_cons
             for (int c = 0; c < un.width / 32; c++) {
                 float v[32];
                 tmem_load32(tmem + ((uint32_t)(quarter * 32) << 16) + buf * WIDTH + c * 32, v);
+                if (EPI == EPI_STREAM) {
+                    stream_columns(a, m0 + quarter * 32, n0 + c * 32, v, factor, turn, lane);
+                    continue;
+                }
                 if (!live) continue;
                 store_columns<EPI>(a, row, n0 + c * 32, v, factor);
             }
@@ -560,7 +591,7 @@ int launch(const CUtensorMap &map_x, const CUtensorMap &map_w, const CUtensorMap
         int device = 0;
         cudaGetDevice(&device);
         if (prepared_device != device) {
-            if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, Tile<BN>::SMEM_BYTES) != cudaSuccess)
+            if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, Tile<BN>::smem_bytes(EPI)) != cudaSuccess)
                 return NCB_ERR_LAUNCH;
             prepared_device = device;
         }
@@ -572,7 +603,7 @@ int launch(const CUtensorMap &map_x, const CUtensorMap &map_w, const CUtensorMap
     cudaLaunchConfig_t config = {};
     config.gridDim = dim3(tiles < sms ? tiles : sms);
     config.blockDim = dim3(THREADS);
-    config.dynamicSmemBytes = Tile<BN>::SMEM_BYTES;
+    config.dynamicSmemBytes = Tile<BN>::smem_bytes(EPI);
     config.stream = stream;
     cudaLaunchAttribute attribute[1];
     attribute[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
@@ -624,10 +655,10 @@ int resident_pairs() {
     std::lock_guard<std::mutex> guard(lock);
     if (!have[device]) {
         auto kernel = k_tile_gemm_pair<160, 2, EPI_STORE>; /* the larger ring of the two */
-        if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, Pair<160, 2>::SMEM_BYTES) != cudaSuccess)
+        if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, Pair<160, 2, EPI_STORE>::SMEM_BYTES) != cudaSuccess)
             known[device] = 0;
         else
-            known[device] = resident_pairs_of(kernel, Pair<160, 2>::SMEM_BYTES);
+            known[device] = resident_pairs_of(kernel, Pair<160, 2, EPI_STORE>::SMEM_BYTES);
         have[device] = true;
     }
     return known[device];
@@ -637,7 +668,7 @@ int resident_pairs() {
 template <int NMMA, int NSUB, int EPI>
 int launch_pair(const CUtensorMap &map_x, const CUtensorMap &map_w, const CUtensorMap &map_w_half, TileArgs a, int pairs,
                 cudaStream_t stream) {
-    using P = Pair<NMMA, NSUB>;
+    using P = Pair<NMMA, NSUB, EPI>;
     auto kernel = k_tile_gemm_pair<NMMA, NSUB, EPI>;
     static std::mutex lock;
     static int prepared_device = -1;

@@ -49,6 +49,8 @@ def stack_fields(fields: list[Tensor], width: int, columns: int) -> tuple[Tensor
     for f in fields:
         offsets.append(at)
         at += up(f.shape[0], 8)
+    if at >= 1024:  # the widest tiles of tile_gemm take multiples of 256
+        width = up(width, 256)
     out = torch.zeros((up(at, width), columns), dtype=fields[0].dtype, device=fields[0].device)
     for f, o in zip(fields, offsets):
         out[o:o + f.shape[0], :f.shape[1]] = f
