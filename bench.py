@@ -665,6 +665,8 @@ def bench_hybrid(device, new_tokens: int = 128, profile: str = "") -> dict:
             torch.cuda.synchronize()
             torch.cuda.profiler.stop()
 
+    if profile == "kernels":
+        return {"kernels": bench_hybrid_kernels(device, profiled=True)}
     result = {}
     for name, size in HYBRID_SIZES.items():
         if profile and not profile.startswith(name):
@@ -743,10 +745,10 @@ def cache_bytes_read(dec, ctx, new_tokens: int) -> int:
     return total
 
 
-def bench_hybrid_kernels(device) -> dict:
+def bench_hybrid_kernels(device, profiled: bool = False) -> dict:
     """The token mixers' kernels alone at the d20 and d32 sizes, against HBM bandwidth (decode) or the bf16 tensor peak
     (prefill). Decode launches rotate over caches that together exceed L2; prefill inputs are larger than or re-read from L2
-    as in a pass."""
+    as in a pass. profiled: launch each d32 kernel once between cudaProfilerStart and Stop and time nothing."""
     import ctypes
 
     from nanochat_b200.mixers import GatedLinearAttention, LatentAttention, RowPlan, Rows
@@ -760,6 +762,14 @@ def bench_hybrid_kernels(device) -> dict:
 
     def per_call(fn, calls: int) -> float:
         """Microseconds per call of `calls` calls captured in one graph (host launch costs left out), median of REPEATS."""
+        if profiled:
+            fn(0)
+            torch.cuda.synchronize()
+            torch.cuda.profiler.start()
+            fn(1)
+            torch.cuda.synchronize()
+            torch.cuda.profiler.stop()
+            return 1.0
         side = torch.cuda.Stream()
         side.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(side):
@@ -811,6 +821,8 @@ def bench_hybrid_kernels(device) -> dict:
     out = {}
     gen = torch.Generator(device=device).manual_seed(900)
     for name, size in HYBRID_SIZES.items():
+        if profiled and name != "d32":
+            continue
         B, C, H = size["batch"], size["width"], size["heads"]
         cgen = torch.Generator().manual_seed(400)
         ctx = [576] * B if name == "d20" else torch.randint(256, 8193, (B,), generator=cgen).tolist()
@@ -1009,7 +1021,8 @@ def main() -> None:
     ap.add_argument("--e2e-parts", type=int, default=0, help="row groups of the end-to-end step that run as parallel graph branches (0: DecodeStep's choice)")
     ap.add_argument("--hybrid", type=int, default=0, help="also time Pudisun's prefill, decode and kernels beside the closest model "
                     "(N = 1); 2: print only that")
-    ap.add_argument("--hybrid-profile", default="", help="bracket one pass or step of that for ncu: d20-prefill, d20-decode, d32-...")
+    ap.add_argument("--hybrid-profile", default="", help="bracket one pass or step of that for ncu: d20-prefill, d20-decode, d32-..., or one "
+                    "launch of each d32 kernel: kernels")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
 
