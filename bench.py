@@ -896,6 +896,50 @@ def bench_hybrid_kernels(device, profiled: bool = False) -> dict:
         nbytes = (proj.numel() + mixed.numel()) * 2 + 2 * state.state.numel() * 4
         out[f"{name} gla_chunked"] = {"us": us, "flops": flops, "tflops": flops / us / 1e6, "bytes": nbytes, "gbs": nbytes / us / 1e3,
                                       "frac_hbm": nbytes / us / 1e3 / hbm, "note": "four launches"}
+        # ---- the closest model's kernels at the same sizes, and its GEMM epilogue beside the stream update
+        import nanochat_b200 as ncb
+        from nanochat_b200 import attention as ops
+        from nanochat_b200.native import GemmRs, pointer
+
+        del cache, state, proj, mixed
+        Hkv = size["kv_heads"]
+        kv = [ncb.Fp8KVCache(B, Hkv, max(ctx), device=device) for _ in range(copies)]
+        for c in kv:  # random finite bytes below the e4m3 NaN, small scales
+            c.pages.random_(0, 100, generator=gen)
+            c.pages.view(B, Hkv, -1, 16896)[..., 16384:].view(torch.float32).fill_(0.01)
+        q = torch.randn(B, H, D, generator=gen, device=device).bfloat16()
+        lens_t = torch.tensor(ctx, dtype=torch.int32, device=device)
+        chunk = ops.plan_chunk_pages(ctx, Hkv, max(ctx))
+        work = torch.empty(max(ops.workspace_bytes(B, H, Hkv, max(ctx), chunk), 16), dtype=torch.uint8, device=device)
+        att = torch.empty_like(q)
+        nbytes = sum(ctx) * Hkv * 264 + B * H * 512
+        us = per_call(lambda i: ops.decode_attention(q, kv[i % copies], lens_t, max(ctx), chunk_pages=chunk, workspace=work, out=att,
+                                                     status=status), 40)
+        out[f"{name} nanochat decode_attn + merge"] = {"us": us, "bytes": nbytes, "gbs": nbytes / us / 1e3, "frac_hbm": nbytes / us / 1e3 / hbm}
+        pkv = ncb.Fp8KVCache(prompts, Hkv, n, device=device)
+        pkv.pages.copy_(torch.zeros_like(pkv.pages))
+        q = torch.randn(n * prompts, H, D, generator=gen, device=device).bfloat16()
+        plan = ops.PrefillPlan(*host, H, pkv, device)
+        att = torch.empty_like(q)
+        flops = prompts * n * (n + 1) // 2 * H * 4 * D
+        us = per_call(lambda i: ops.prefill_attention(q, pkv, plan, out=att, status=status), 20)
+        out[f"{name} nanochat prefill_attn"] = {"us": us, "flops": flops, "tflops": flops / us / 1e6, "frac_tensor": flops / us / 1e6 / tensor}
+        del kv, pkv, q, att
+        rows_n = n * prompts
+        h = torch.randn(rows_n, C, generator=gen, device=device)
+        gain = torch.ones(C, device=device)
+        y, ss = torch.empty(rows_n, C, dtype=torch.bfloat16, device=device), torch.empty(rows_n, C // 32, device=device)
+        for what, K in (("o", latent.out_width), ("down", size["ff"])):
+            x = torch.randn(rows_n, K, generator=gen, device=device).bfloat16()
+            w = (torch.randn(C, K, generator=gen, device=device) * 0.02).bfloat16()
+            a = GemmRs(x=x.data_ptr(), w=w.data_ptr(), rows=rows_n, N=C, K=K, n_store=C, epilogue=6, scale=1.0, mult=0.2, h=h.data_ptr(),
+                       gain=gain.data_ptr(), x_next=y.data_ptr(), ss_next=ss.data_ptr(), status=status.data_ptr())
+            flops = 2 * rows_n * C * K
+            for form, call in (("stream update", lambda i: cuda_library("tile_gemm").tile_gemm_rs(ctypes.byref(a), stream())),
+                               ("bf16 residual", lambda i: cuda_library("tile_gemm").tile_gemm(
+                                   pointer(x), pointer(w), pointer(y), pointer(y), rows_n, C, K, 1, pointer(status), stream()))):
+                us = per_call(call, 20)
+                out[f"{name} tile_gemm {what}, {form}"] = {"us": us, "flops": flops, "tflops": flops / us / 1e6, "frac_tensor": flops / us / 1e6 / tensor}
         assert int(status.item()) == 0
         torch.cuda.empty_cache()
     return out
