@@ -1,6 +1,6 @@
 """Token mixers of models whose layers differ in kind: weights prepared for the kernels, the cache or state each needs, and
 the launches between the input projection and the output projection. A mixer is built from its sizes and a dict of
-checkpoint tensors, so any model whose layers use it can share it; models/hybrid decoders only see
+checkpoint tensors, so any model whose layers use it can share it. A decoder only sees
 
     w_in, w_out                    fused input projection [in_width, C], output projection [C, out_width]
     new_cache(n_slots, max_len)    one layer's cache

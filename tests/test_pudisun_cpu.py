@@ -1,4 +1,4 @@
-"""Pudisun without a GPU: the checker's own mechanisms against independent statements of them (and against planted mistakes,
+"""Pudisun without a GPU: the oracle's own mechanisms against independent statements of them (and against planted mistakes,
 so that the tolerances of the GPU tests are known to catch them), the checkpoint reader, configuration, registry, row plans."""
 
 import json
@@ -23,7 +23,7 @@ ROOT = Path(__file__).resolve().parent.parent
 BF16_TOLERANCE = 0.05  # of the GPU tests, on relative_error of a bf16 run
 
 
-# ---- the checker ------------------------------------------------------------------------------------------------------
+# ---- the oracle -------------------------------------------------------------------------------------------------------
 
 def test_gla_recurrence_equals_its_unrolled_sum():
     """o_t = sum over s <= t of (q_t . prod of decays . k_s) v_s, written without a state."""
@@ -85,7 +85,7 @@ def test_activations():
 @pytest.mark.parametrize("mistake", ["no sink", "sink scaled", "late key", "first key lost", "rotation off by one", "no yarn factor",
                                      "state lost", "decay late", "own weights for a shared layer", "plain residual"])
 def test_a_planted_mistake_exceeds_the_gpu_tests_tolerance(mistake, monkeypatch):
-    """Each mistake changes the checker's logits by more than what the GPU comparisons allow (in bf16, the looser ones)."""
+    """Each mistake changes the oracle's logits by more than what the GPU comparisons allow (in bf16, the looser ones)."""
     cfg = json.loads(json.dumps(cases.CONFIGS["ragged"]))
     state, toks = cases.random_state(cfg, 5), cases.tokens(cfg, 40, 6)
     want = oracle.forward(toks, cfg, state)
@@ -132,7 +132,7 @@ def test_a_planted_mistake_exceeds_the_gpu_tests_tolerance(mistake, monkeypatch)
 
 # ---- tables, files, configuration ---------------------------------------------------------------------------------------
 
-def test_rotary_tables_follow_the_checkers_frequencies():
+def test_rotary_tables_follow_the_oracles_frequencies():
     for rot in ({"dims": 24, "base": 10000.0, "scaling": cases.YARN}, {"dims": 2, "base": 500.0},
                 {"dims": 64, "base": 20.0, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}):
         want, factor = oracle.rotary_frequencies(rot)

@@ -1,4 +1,4 @@
-"""Pudisun on the GPU against the plain checker (oracle/pudisun.py): each mechanism alone, whole prompts, portions, decoding,
+"""Pudisun on the GPU against the plain oracle (oracle/pudisun.py): each mechanism alone, whole prompts, portions, decoding,
 batches, slots used again, generation through the scheduler, the command line and the trace runner."""
 
 import json
@@ -36,7 +36,7 @@ _oracle: dict = {}
 
 
 def case(name: str, n: int, seed: int = 1):
-    """(configuration, weights, tokens, the checker's logits), computed once per test run."""
+    """(configuration, weights, tokens, the oracle's logits), computed once per test run."""
     if (name, n, seed) not in _oracle:
         cfg = cases.CONFIGS[name]
         state, toks = cases.random_state(cfg, seed), cases.tokens(cfg, n, seed + 50)
@@ -116,7 +116,7 @@ def test_latent_attention_alone(dtype, sizes, mode):
 @pytest.mark.parametrize("mode", ["absorbed", "expanded", "decoded"])
 def test_a_key_that_stands_out_is_found_wherever_it_lies(dtype, mode):
     """One earlier row's key is made to dominate a later row's score (same input, large scale), at tile, page and chunk
-    borders, first and last positions; the outputs are those of the checker."""
+    borders, first and last positions; the outputs are those of the oracle."""
     if mode == "expanded" and dtype == F32:
         pytest.skip("no expanded form in 32-bit")
     entry = cases.latent(heads=2, dim=32, rot_dim=16, vdim=32, kv_rank=64, scale=1.5, scaling=None)
@@ -260,7 +260,7 @@ def test_long_prompts_far_keys_and_passes_of_a_prompt(dtype):
 @DTYPES
 def test_batches_of_unequal_requests_match_each_request_alone(dtype):
     """Prompts of different lengths in one pass (also cut by the pass's size), then decode steps over all slots in another
-    order than the slots', against the checker; an idle slot's cache and state stay as they are."""
+    order than the slots', against the oracle; an idle slot's cache and state stay as they are."""
     name = "ragged"
     lens = (5, 71, 1, 130, 64)
     seqs = [case(name, n + 9, seed=s) for s, n in enumerate(lens)]
@@ -297,9 +297,9 @@ def greedy(cfg, state, prompt, n) -> list[int]:
     return out[len(prompt):]
 
 
-def test_greedy_generation_through_the_scheduler_matches_the_checker():
+def test_greedy_generation_through_the_scheduler_matches_the_oracle():
     """Seven requests through three slots (slots are freed and used again while others run), and generate(); 32-bit, where the
-    choice is the checker's."""
+    choice is the oracle's."""
     cfg = cases.CONFIGS["ragged"]
     state = cases.random_state(cfg, 31)
     prompts = [cases.tokens(cfg, n, 60 + n) for n in (1, 30, 7, 66, 2, 64, 12)]
