@@ -67,7 +67,12 @@ const char *ncb_status_string(int status);
  *   epilogue 5: features 2 j and 2 j + 1 are a gate and its value: y[row][j] = gelu_tanh(gate) * value (N / 2 columns).
  *   epilogue 6: h [rows][N] += mult * product; x_next [rows][N] = h * gain[N]; ss_next [rows][parts] with a count of partial
  *               sums per row that depends on the entry point (see their declarations).
+ *   epilogue 7: several streams in place of one, h [rows][streams][N]: all of them at once from the old ones,
+ *               h_t <- sum_s mix[s * NCB_MAX_STREAMS + t] h_s + out[t] * product; what the next norm reads is
+ *               u = sum_t in[t] h_t: x_next = u * gain, ss_next of u. (in: the next branch's.)
+ *   epilogue 8: as 5 with silu(gate) * value.
  */
+#define NCB_MAX_STREAMS 8
 typedef struct {
     const void *x;      /* [rows][K] */
     const void *w;      /* [N][K] */
@@ -85,6 +90,8 @@ typedef struct {
     const void *next_w; /* stream_gemm_rs: see stream_gemm */
     long long next_bytes;
     int *status;
+    int streams;        /* epilogue 7: how many, at most NCB_MAX_STREAMS */
+    float in[NCB_MAX_STREAMS], out[NCB_MAX_STREAMS], mix[NCB_MAX_STREAMS * NCB_MAX_STREAMS];
 } ncb_gemm_rs;
 
 /* ---- library kv_append -------------------------------------------------------------------------------------- */
@@ -493,6 +500,80 @@ int latent_query(const ncb_latent *args, int f32, void *stream);
 int latent_split(const ncb_latent *args, int f32, void *stream);
 int latent_out(const ncb_latent *args, int f32, void *stream);
 
+/* ---- library short_conv ------------------------------------------------------------------------------------------------
+ * A short causal convolution over time on the first `width` channels of projected rows (csrc/short_conv.cuh): proj T
+ * [rows][ldp], w fp32 [taps][width], ring T [n_slots][taps][width] (the projected value of position p at p % taps; what lies
+ * before position 0 is never read). Rows of a sequence are consecutive and at ascending positions; a negative position is idle.
+ * The mixers that take an ncb_conv read it; short_conv_tail stores the sequences' last rows into the ring afterwards. */
+typedef struct {
+    const void *proj;
+    void *ring;
+    const float *w;
+    long long rows, ldp;
+    int taps, width, n_slots;
+    const int *pos, *slot_map; /* per row; slot_map NULL: row r is slot r */
+} ncb_conv;
+int short_conv_tail(const ncb_conv *args, int f32, int *status, void *stream);
+
+/* ---- library gqa_attn --------------------------------------------------------------------------------------------------
+ * Softmax attention of grouped query heads with a short convolution on q, k and v, rotation of the first `rot` dimensions of
+ * a head (pairs i, i + rot / 2), an RMS norm of q and k over norm_count values after it, and a sigmoid gate per head
+ * (csrc/gqa_attn.cu). T: bf16, or fp32 when the entry point's f32 is not 0. Projected rows hold q [heads dim], k [kv_heads
+ * dim], v [kv_heads vdim] (inside the convolution's channels; k and v only with own_kv) and the gate [heads] at the given
+ * offsets. dim and vdim multiples of 16 (zero-padded values stay zero). cos, sin fp32 [table_len][rot / 2]. kv T
+ * [n_slots][kv_heads][capacity][dim + vdim]. A row with a negative position is idle: a zero output row.
+ *   gqa_rows     q T [rows][heads dim]; with own_kv k, v appended to kv; keep: also the ring (every row a slot of its own);
+ *                q NULL: only the appends
+ *   gqa_split    states of chunks of at most chunk_tiles tiles of NCB_GQA_TILE positions: parts fp32
+ *                [rows][heads][max_chunks][vdim + 4]; max_len bounds every position + 1
+ *   gqa_merge    out [rows][ldo] = sigmoid(gate) * merged states
+ *   gqa_prefill  out of row tiles, bf16: tile_rows (at most 64) rows from tile_row, the first at position tile_pos. List the
+ *                tiles that reach furthest first. For gqa_prefill_supported(dim, vdim) */
+#define NCB_GQA_TILE 16
+typedef struct {
+    ncb_conv conv;
+    void *q, *kv, *out;
+    long long ldo;
+    int off_q, off_k, off_v, off_g, own_kv, keep;
+    int heads, kv_heads, dim, vdim, norm_count, rot;
+    int capacity, table_len, max_len, chunk_tiles, max_chunks, n_tiles;
+    float scale, eps;
+    const float *cos, *sin;
+    float *parts;
+    const int *tile_row, *tile_rows, *tile_pos; /* [n_tiles] */
+    int *status;
+} ncb_gqa;
+int gqa_rows(const ncb_gqa *args, int f32, void *stream);
+int gqa_split(const ncb_gqa *args, int f32, void *stream);
+int gqa_merge(const ncb_gqa *args, int f32, void *stream);
+int gqa_prefill_supported(int dim, int vdim);
+int gqa_prefill(const ncb_gqa *args, void *stream);
+
+/* ---- library delta_rule ------------------------------------------------------------------------------------------------
+ * Gated delta rule with a decay per key channel (csrc/delta_rule.cu has the recurrence). T as above. Projected rows hold q, k
+ * [kv_heads dim] and v [heads vdim] (the convolution's channels), beta [heads] and the low-rank inputs of the decay [rank_a]
+ * and of the output gate [rank_g] at the given offsets; dim and vdim multiples of 16 (zero-padded channels stay zero),
+ * norm_count the vdim that counts in the output norm. a2 T [heads][rank_a][dim], g2 T [heads][rank_g][vdim]; a_exp fp32
+ * [heads] = exp(A_log). state fp32 [n_slots][heads][dim][vdim]. Rows of a segment are consecutive, of one slot and at
+ * ascending positions; a row at position 0 starts from a zero state; a segment whose first position is negative is idle.
+ * out NULL: only the state is advanced.
+ *   delta_step   token by token; seg_first NULL: every row is a segment; keep: also the ring (every row a slot of its own) */
+typedef struct {
+    ncb_conv conv;
+    void *out;
+    long long ldo;
+    int off_q, off_k, off_v, off_b, off_a, off_g, keep;
+    int heads, kv_heads, dim, vdim, rank_a, rank_g, norm_count;
+    float q_scale, eps;
+    const void *a2, *g2;
+    const float *dt_bias, *a_exp, *norm; /* [heads dim], [heads], [vdim] */
+    float *state;
+    const int *seg_first, *seg_count;
+    int n_segments;
+    int *status;
+} ncb_delta;
+int delta_step(const ncb_delta *args, int f32, void *stream);
+
 /* ---- GEMMs around an fp32 residual stream (ncb_gemm_rs above) ------------------------------------------------
  * Shapes as for the plain entry points: skinny_gemm_rs at most 16 rows, K as skinny_gemm without norm, N a multiple of 8,
  * N / 8 partial sums; stream_gemm_rs at most 256 rows, N a multiple of 128, K of 64, N / 128 partial sums; tile_gemm_rs
@@ -506,6 +587,10 @@ int gemm_f32_rs(const ncb_gemm_rs *args, void *stream);
  * embed, x: bf16, or fp32 with f32 != 0; C columns are read, all of them written. A token outside [0, vocab) reads row 0. */
 int embed_rs(const void *embed, const void *tokens, void *h, const void *gain, void *x, void *ss, long long rows, int C,
              int vocab, int f32, void *stream);
+/* The same for `streams` equal streams, h fp32 [rows][streams][C] = scale * embed[tokens] each; the first norm reads
+ * in_sum times one of them (in_sum: the sum of the first branch's weights of the streams). */
+int embed_streams(const void *embed, const void *tokens, void *h, const void *gain, void *x, void *ss, long long rows, int C,
+                  int vocab, int f32, int streams, float scale, float in_sum, void *stream);
 
 #ifdef __cplusplus
 }

@@ -31,7 +31,7 @@ constexpr int GEMM_THREADS = GEMM_WARPS * 32;
 constexpr int TILE_N = 8;         /* output features per block */
 constexpr int MAX_ROWS = 16;
 
-enum { EPI_STORE = 0, EPI_RESID = 1, EPI_RELU2 = 2, EPI_F32 = 3, EPI_MIX = 4, EPI_GEGLU = 5, EPI_STREAM = 6 };
+enum { EPI_STORE = 0, EPI_RESID = 1, EPI_RELU2 = 2, EPI_F32 = 3, EPI_MIX = 4, EPI_GEGLU = 5, EPI_STREAM = 6, EPI_STREAMS = 7, EPI_SWIGLU = 8 };
 
 struct GemmArgs {
     const bf16 *x;     /* [rows][K] */
@@ -209,14 +209,14 @@ __global__ void __launch_bounds__(GEMM_THREADS, ITERS > 8 ? 2 : 1) k_skinny_gemm
             for (int w = 0; w < GEMM_WARPS; w++) v += part[w][row][col];
             if (!NORM) v *= rstd[row];
             const size_t at = (size_t)row * a.N + (size_t)tile * TILE_N + col;
-            if (EPI == EPI_GEGLU) {
+            if (EPI == EPI_GEGLU || EPI == EPI_SWIGLU) {
                 const float up = __shfl_xor_sync(0xffffffffu, v, 1);
                 if (row < a.rows && (col & 1) == 0)
-                    reinterpret_cast<bf16 *>(a.y)[row * a.ldy + tile * (TILE_N / 2) + col / 2] = __float2bfloat16_rn(gelu_tanh(v) * up);
-            } else if (EPI == EPI_STREAM) {
+                    reinterpret_cast<bf16 *>(a.y)[row * a.ldy + tile * (TILE_N / 2) + col / 2] = __float2bfloat16_rn(gate_of<EPI == EPI_SWIGLU>(v) * up);
+            } else if (EPI == EPI_STREAM || EPI == EPI_STREAMS) {
                 float hv = 0.f;
                 if (row < a.rows) {
-                    hv = stream_add(a.rs, at, v);
+                    hv = EPI == EPI_STREAM ? stream_add(a.rs, at, v) : streams_add(a.rs, row, tile * TILE_N + col, a.N, v);
                     reinterpret_cast<bf16 *>(a.rs.x_next)[at] = __float2bfloat16_rn(hv * a.rs.gain[tile * TILE_N + col]);
                 }
                 float q = hv * hv;
@@ -273,11 +273,12 @@ __global__ void __launch_bounds__(128) k_embed_norm(const bf16 *embed, const lon
     }
 }
 
-/* The first rows of an fp32 residual stream: h = embed[token], x = h * gain for the first norm, one sum of squares. */
+/* The first rows of an fp32 residual stream (or of `streams` equal ones): h = scale embed[token], x = in_sum h gain for the
+ * first norm, one sum of squares. */
 constexpr int EMBED_THREADS = 128;
 template <typename T>
 __global__ void __launch_bounds__(EMBED_THREADS) k_embed_rs(const T *embed, const long long *tokens, float *h, const float *gain,
-                                                            T *x, float *ss, int C, int vocab) {
+                                                            T *x, float *ss, int C, int vocab, int streams, float scale, float in_sum) {
     __shared__ float warp_sums[EMBED_THREADS / 32];
     asm volatile("griddepcontrol.wait;" ::: "memory");
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
@@ -287,10 +288,10 @@ __global__ void __launch_bounds__(EMBED_THREADS) k_embed_rs(const T *embed, cons
     const size_t base = (size_t)blockIdx.x * C;
     float s = 0.f;
     for (int i = threadIdx.x; i < C; i += EMBED_THREADS) {
-        const float v = (float)e[i];
-        h[base + i] = v;
-        x[base + i] = (T)(v * gain[i]);
-        s += v * v;
+        const float v = scale * (float)e[i], u = in_sum * v;
+        for (int j = 0; j < streams; j++) h[(base * streams) + (size_t)j * C + i] = v;
+        x[base + i] = (T)(u * gain[i]);
+        s += u * u;
     }
     for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
     if ((threadIdx.x & 31) == 0) warp_sums[threadIdx.x >> 5] = s;
@@ -592,6 +593,8 @@ template <int ITERS, bool HI, bool NORM> static int launch_gemm_epi(const GemmAr
     }
     if constexpr (!NORM) { /* the residual-stream forms scale by row instead of norming their input */
         if (epilogue == EPI_GEGLU) { auto k = k_skinny_gemm<ITERS, HI, EPI_GEGLU, false>; return launch_pdl(k, dim3(grid_for(k, tiles, ITERS <= 8)), block, stream, a); }
+        if (epilogue == EPI_SWIGLU) { auto k = k_skinny_gemm<ITERS, HI, EPI_SWIGLU, false>; return launch_pdl(k, dim3(grid_for(k, tiles, ITERS <= 8)), block, stream, a); }
+        if (epilogue == EPI_STREAMS) { auto k = k_skinny_gemm<ITERS, HI, EPI_STREAMS, false>; return launch_pdl(k, dim3(grid_for(k, tiles, ITERS <= 8)), block, stream, a); }
         if (epilogue == EPI_STREAM) { auto k = k_skinny_gemm<ITERS, HI, EPI_STREAM, false>; return launch_pdl(k, dim3(grid_for(k, tiles, ITERS <= 8)), block, stream, a); }
     }
     return NCB_ERR_ARG;
@@ -621,7 +624,7 @@ static int launch_skinny(const GemmArgs &a, int epilogue, cudaStream_t s) {
     if (rows < 0 || rows > MAX_ROWS || N <= 0 || K <= 0 || N % TILE_N || K % (GEMM_WARPS * 32)) return NCB_ERR_ARG;
     if (!skinny_depth_ok(K)) return NCB_ERR_UNSUPPORTED;
     if (rows == 0) return NCB_OK;
-    if (!a.x || !a.w || (!a.y && epilogue != EPI_STREAM) || ((epilogue == EPI_RESID || epilogue == EPI_MIX) && !a.resid) ||
+    if (!a.x || !a.w || (!a.y && epilogue != EPI_STREAM && epilogue != EPI_STREAMS) || ((epilogue == EPI_RESID || epilogue == EPI_MIX) && !a.resid) ||
         (epilogue == EPI_MIX && !a.x0))
         return NCB_ERR_ARG;
     if (((uintptr_t)a.x | (uintptr_t)a.w) % 16 || (uintptr_t)a.y % 4) return NCB_ERR_ALIGN;
@@ -685,17 +688,22 @@ int skinny_gemm_rs(const ncb_gemm_rs *g, void *stream) {
     return launch_skinny(a, g->epilogue, (cudaStream_t)stream);
 }
 
-int embed_rs(const void *embed, const void *tokens, void *h, const void *gain, void *x, void *ss, long long rows, int C,
-             int vocab, int f32, void *stream) {
-    if (rows < 0 || rows > 0x7fffffffLL || C <= 0 || vocab <= 0) return NCB_ERR_ARG;
+int embed_streams(const void *embed, const void *tokens, void *h, const void *gain, void *x, void *ss, long long rows, int C,
+                  int vocab, int f32, int streams, float scale, float in_sum, void *stream) {
+    if (rows < 0 || rows > 0x7fffffffLL || C <= 0 || vocab <= 0 || streams < 1 || streams > NCB_MAX_STREAMS) return NCB_ERR_ARG;
     if (rows == 0) return NCB_OK;
     if (!embed || !tokens || !h || !gain || !x || !ss) return NCB_ERR_ARG;
     const dim3 grid((unsigned)rows), block(EMBED_THREADS);
     if (f32)
         return launch_pdl(k_embed_rs<float>, grid, block, (cudaStream_t)stream, (const float *)embed, (const long long *)tokens,
-                          (float *)h, (const float *)gain, (float *)x, (float *)ss, C, vocab);
+                          (float *)h, (const float *)gain, (float *)x, (float *)ss, C, vocab, streams, scale, in_sum);
     return launch_pdl(k_embed_rs<bf16>, grid, block, (cudaStream_t)stream, (const bf16 *)embed, (const long long *)tokens,
-                      (float *)h, (const float *)gain, (bf16 *)x, (float *)ss, C, vocab);
+                      (float *)h, (const float *)gain, (bf16 *)x, (float *)ss, C, vocab, streams, scale, in_sum);
+}
+
+int embed_rs(const void *embed, const void *tokens, void *h, const void *gain, void *x, void *ss, long long rows, int C,
+             int vocab, int f32, void *stream) {
+    return embed_streams(embed, tokens, h, gain, x, ss, rows, C, vocab, f32, 1, 1.f, 1.f, stream);
 }
 
 static int launch_embed(const void *embed, const void *tokens, void *h, void *x0, float l1, float l2, int mix, int rows,

@@ -9,7 +9,7 @@
 namespace {
 
 constexpr int TM = 64, TN = 64, TK = 16, THREADS = 256;
-enum { EPI_STORE = 0, EPI_F32 = 3, EPI_GEGLU = 5, EPI_STREAM = 6 };
+enum { EPI_STORE = 0, EPI_F32 = 3, EPI_GEGLU = 5, EPI_STREAM = 6, EPI_STREAMS = 7, EPI_SWIGLU = 8 };
 
 struct Args {
     const float *x, *w;
@@ -65,18 +65,23 @@ __global__ void __launch_bounds__(THREADS) k_gemm_f32(const Args a) {
         float v[4];
 #pragma unroll
         for (int j = 0; j < 4; j++) v[j] = acc[i][j] * factor[r];
-        if (a.epilogue == EPI_GEGLU) {
+        if (a.epilogue == EPI_SWIGLU) {
+            if (live) {
+                a.y[row * a.ldy + (n >> 1)] = silu(v[0]) * v[1];
+                a.y[row * a.ldy + (n >> 1) + 1] = silu(v[2]) * v[3];
+            }
+        } else if (a.epilogue == EPI_GEGLU) {
             if (live) {
                 a.y[row * a.ldy + (n >> 1)] = gelu_tanh(v[0]) * v[1];
                 a.y[row * a.ldy + (n >> 1) + 1] = gelu_tanh(v[2]) * v[3];
             }
-        } else if (a.epilogue == EPI_STREAM) {
+        } else if (a.epilogue == EPI_STREAM || a.epilogue == EPI_STREAMS) {
             float q = 0.f;
             if (live)
 #pragma unroll
                 for (int j = 0; j < 4; j++) {
                     const size_t at = (size_t)row * a.N + n + j;
-                    const float h = stream_add(a.rs, at, v[j]);
+                    const float h = a.epilogue == EPI_STREAM ? stream_add(a.rs, at, v[j]) : streams_add(a.rs, row, n + j, a.N, v[j]);
                     reinterpret_cast<float *>(a.rs.x_next)[at] = h * a.rs.gain[n + j];
                     q += h * h;
                 }

@@ -37,7 +37,7 @@ constexpr int RING_KB_SMALL = 100;               /* ring of the <= 128-row shape
 constexpr int THREADS = 128;
 constexpr int MAX_SPLIT = 8;                     /* portable cluster size */
 
-enum { EPI_STORE = 0, EPI_RESID = 1, EPI_RELU2 = 2, EPI_F32 = 3, EPI_MIX = 4, EPI_GEGLU = 5, EPI_STREAM = 6 };
+enum { EPI_STORE = 0, EPI_RESID = 1, EPI_RELU2 = 2, EPI_F32 = 3, EPI_MIX = 4, EPI_GEGLU = 5, EPI_STREAM = 6, EPI_STREAMS = 7, EPI_SWIGLU = 8 };
 
 template <int NP> struct Shape {
     /* A stage holds KSUB consecutive boxes of W and the matching boxes of x. Wider stages (2 or 4 boxes, i.e. 256
@@ -292,15 +292,15 @@ __global__ void __launch_bounds__(THREADS) k_stream_gemm(const __grid_constant__
 #pragma unroll
             for (int j = 0; j < 32; j++) {
                 const int r = c * 32 + j;
-                if (EPI == EPI_GEGLU) { /* gate and value are neighbouring features, so neighbouring lanes */
+                if (EPI == EPI_GEGLU || EPI == EPI_SWIGLU) { /* gate and value are neighbouring features, so neighbouring lanes */
                     const float up = __shfl_down_sync(0xffffffffu, v[j], 1);
                     if (r < a.rows && (tid & 1) == 0)
-                        reinterpret_cast<bf16 *>(a.y)[r * a.ldy + (col >> 1)] = __float2bfloat16_rn(gelu_tanh(v[j]) * up);
-                } else if (EPI == EPI_STREAM) {
+                        reinterpret_cast<bf16 *>(a.y)[r * a.ldy + (col >> 1)] = __float2bfloat16_rn(gate_of<EPI == EPI_SWIGLU>(v[j]) * up);
+                } else if (EPI == EPI_STREAM || EPI == EPI_STREAMS) {
                     const size_t at = (size_t)r * a.N + col;
                     float h = 0.f;
                     if (r < a.rows) {
-                        h = stream_add(a.rs, at, v[j]);
+                        h = EPI == EPI_STREAM ? stream_add(a.rs, at, v[j]) : streams_add(a.rs, r, (int)col, a.N, v[j]);
                         reinterpret_cast<bf16 *>(a.rs.x_next)[at] = __float2bfloat16_rn(h * a.rs.gain[col]);
                     }
                     h *= h;
@@ -315,7 +315,7 @@ __global__ void __launch_bounds__(THREADS) k_stream_gemm(const __grid_constant__
                 }
             }
         }
-        if (EPI == EPI_STREAM) {
+        if (EPI == EPI_STREAM || EPI == EPI_STREAMS) {
             __syncthreads();
             for (int r = tid; r < a.rows; r += THREADS)
                 a.rs.ss_next[(size_t)r * gridDim.y + tile] = (park[r] + park[NP + r]) + (park[2 * NP + r] + park[3 * NP + r]);
@@ -355,6 +355,7 @@ __global__ void __launch_bounds__(THREADS) k_stream_gemm(const __grid_constant__
         float ps[RB][MAX_SPLIT];
         uint2 res[RB], mix[RB];
         float4 hold[EPI == EPI_STREAM ? RB : 1];
+        Streams<2, float4> pair[EPI == EPI_STREAMS ? RB : 1]; /* more than two streams are loaded where they are used */
 #pragma unroll
         for (int i = 0; i < RB; i++) {
             const int r = r0 + i * 4 * S;
@@ -367,6 +368,7 @@ __global__ void __launch_bounds__(THREADS) k_stream_gemm(const __grid_constant__
             res[i] = HAS_RESID && ok ? *reinterpret_cast<const uint2 *>(a.resid + (size_t)r * a.N + col4) : make_uint2(0u, 0u);
             if (EPI == EPI_STREAM)
                 hold[i] = ok ? *reinterpret_cast<const float4 *>(a.rs.h + (size_t)r * a.N + col4) : make_float4(0.f, 0.f, 0.f, 0.f);
+            if (EPI == EPI_STREAMS && a.rs.streams <= 2) pair[i].load(a.rs, (size_t)r * a.rs.streams * a.N + col4, a.N, ok);
             mix[i] = EPI == EPI_MIX && ok ? *reinterpret_cast<const uint2 *>(a.x0 + (size_t)r * a.N + col4) : make_uint2(0u, 0u);
         }
 #pragma unroll
@@ -386,15 +388,29 @@ __global__ void __launch_bounds__(THREADS) k_stream_gemm(const __grid_constant__
                 const float f = sumsq[r];
                 v.x *= f, v.y *= f, v.z *= f, v.w *= f;
             }
-            if (EPI == EPI_STREAM) { /* a warp holds the whole row of this tile (r is the same for its lanes) */
-                float4 h = hold[i];
-                h.x += a.rs.mult * v.x, h.y += a.rs.mult * v.y, h.z += a.rs.mult * v.z, h.w += a.rs.mult * v.w;
+            if (EPI == EPI_STREAM || EPI == EPI_STREAMS) { /* a warp holds the whole row of this tile (r is the same for its lanes) */
+                float4 h;
+                if (EPI == EPI_STREAM) {
+                    h = hold[i];
+                    h.x += a.rs.mult * v.x, h.y += a.rs.mult * v.y, h.z += a.rs.mult * v.z, h.w += a.rs.mult * v.w;
+                } else {
+                    const size_t at = (size_t)r * a.rs.streams * a.N + col4;
+                    with_streams(a.rs.streams, [&](auto S) {
+                        if constexpr (decltype(S)::value == 2) {
+                            h = pair[i].update(a.rs, at, a.N, v, r < a.rows);
+                        } else {
+                            Streams<decltype(S)::value, float4> x;
+                            x.load(a.rs, at, a.N, r < a.rows);
+                            h = x.update(a.rs, at, a.N, v, r < a.rows);
+                        }
+                    });
+                }
                 float q = h.x * h.x + h.y * h.y + h.z * h.z + h.w * h.w;
                 for (int o = 16; o > 0; o >>= 1) q += __shfl_xor_sync(0xffffffffu, q, o);
                 if (r < a.rows) {
                     const size_t at = (size_t)r * a.N + col4;
                     const float4 g = *reinterpret_cast<const float4 *>(a.rs.gain + col4);
-                    *reinterpret_cast<float4 *>(a.rs.h + at) = h;
+                    if (EPI == EPI_STREAM) *reinterpret_cast<float4 *>(a.rs.h + at) = h;
                     uint2 out;
                     __nv_bfloat162 *oo = reinterpret_cast<__nv_bfloat162 *>(&out);
                     oo[0] = __floats2bfloat162_rn(h.x * g.x, h.y * g.y);
@@ -406,9 +422,9 @@ __global__ void __launch_bounds__(THREADS) k_stream_gemm(const __grid_constant__
             }
             if (r >= a.rows) continue;
             const size_t at = (size_t)r * a.N + col4;
-            if (EPI == EPI_GEGLU) {
+            if (EPI == EPI_GEGLU || EPI == EPI_SWIGLU) {
                 *reinterpret_cast<__nv_bfloat162 *>(reinterpret_cast<bf16 *>(a.y) + (size_t)r * a.ldy + (col4 >> 1)) =
-                    __floats2bfloat162_rn(gelu_tanh(v.x) * v.y, gelu_tanh(v.z) * v.w);
+                    __floats2bfloat162_rn(gate_of<EPI == EPI_SWIGLU>(v.x) * v.y, gate_of<EPI == EPI_SWIGLU>(v.z) * v.w);
             } else if ((EPI == EPI_STORE || EPI == EPI_F32) && ((int)col4 + 4 > a.n_store || (a.ldy & 3))) {
                 const float e[4] = {v.x, v.y, v.z, v.w}; /* the last stored columns, or rows without vector alignment */
 #pragma unroll
@@ -494,6 +510,8 @@ int launch_epi(const CUtensorMap &map_w, const CUtensorMap &map_x, const GemmArg
     case EPI_MIX: return launch<NP, EPI_MIX>(map_w, map_x, a, split, stream);
     case EPI_GEGLU: return launch<NP, EPI_GEGLU>(map_w, map_x, a, split, stream);
     case EPI_STREAM: return launch<NP, EPI_STREAM>(map_w, map_x, a, split, stream);
+    case EPI_STREAMS: return launch<NP, EPI_STREAMS>(map_w, map_x, a, split, stream);
+    case EPI_SWIGLU: return launch<NP, EPI_SWIGLU>(map_w, map_x, a, split, stream);
     default: return NCB_ERR_ARG;
     }
 }
@@ -515,10 +533,10 @@ static int run_stream_gemm(const void *x, const void *w, const void *resid, void
                            int epilogue, int split, const void *next_w, long long next_bytes, int *status, void *stream,
                            const void *x0, float l1, float l2, long long ldy, int n_store, const StreamIO &rs) {
     if (rows < 0 || rows > 256 || N <= 0 || K <= 0 || N % TILE_F || K % KBLK) return NCB_ERR_ARG;
-    if (epilogue < EPI_STORE || epilogue > EPI_STREAM || split < 0 || split > MAX_SPLIT || split > K / KBLK) return NCB_ERR_ARG;
+    if (epilogue < EPI_STORE || epilogue > EPI_SWIGLU || split < 0 || split > MAX_SPLIT || split > K / KBLK) return NCB_ERR_ARG;
     if (rows == 0) return NCB_OK;
     const bool has_resid = epilogue == EPI_RESID || epilogue == EPI_MIX;
-    if (!x || !w || (!y && epilogue != EPI_STREAM) || (has_resid && !resid) || (epilogue == EPI_MIX && !x0)) return NCB_ERR_ARG;
+    if (!x || !w || (!y && epilogue != EPI_STREAM && epilogue != EPI_STREAMS) || (has_resid && !resid) || (epilogue == EPI_MIX && !x0)) return NCB_ERR_ARG;
     if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)y | (uintptr_t)resid | (uintptr_t)x0) % 16) return NCB_ERR_ALIGN;
     if (next_w && ((uintptr_t)next_w % 16 || next_bytes % 16 || next_bytes < 0)) return NCB_ERR_ALIGN;
     if (split == 0) split = auto_split(rows, N / TILE_F, K / KBLK);

@@ -33,7 +33,9 @@ constexpr int A_BYTES = BM * KBLK * 2;
 
 constexpr int TURN_FLOATS = 32 * 33; /* per epilogue warp: see stream_columns */
 
-enum { EPI_STORE = 0, EPI_RESID = 1, EPI_RELU2 = 2, EPI_F32 = 3, EPI_GEGLU = 5, EPI_STREAM = 6 };
+enum { EPI_STORE = 0, EPI_RESID = 1, EPI_RELU2 = 2, EPI_F32 = 3, EPI_GEGLU = 5, EPI_STREAM = 6, EPI_STREAMS = 7, EPI_SWIGLU = 8 };
+
+constexpr bool writes_stream(int epi) { return epi == EPI_STREAM || epi == EPI_STREAMS; }
 
 template <int BN> struct Tile {
     static constexpr int B_BYTES = BN * KBLK * 2;
@@ -41,7 +43,7 @@ template <int BN> struct Tile {
     static constexpr int STAGES = BN == 256 ? 4 : 6;               /* 192 KB of ring either way */
     static constexpr int RING_BYTES = STAGES * STAGE_BYTES;
     /* 1024: the ring is aligned by hand; 256: barriers; then the stream update's staging */
-    static constexpr int smem_bytes(int epi) { return 1024 + RING_BYTES + 256 + (epi == EPI_STREAM ? 4 * TURN_FLOATS * 4 : 0); }
+    static constexpr int smem_bytes(int epi) { return 1024 + RING_BYTES + 256 + (writes_stream(epi) ? 4 * TURN_FLOATS * 4 : 0); }
     static constexpr int TMEM_COLS = 2 * BN;                       /* two accumulators */
 };
 
@@ -88,12 +90,12 @@ template <int EPI> static __device__ __forceinline__ void store_columns(const Ti
     const size_t at = (size_t)row * (EPI == EPI_STORE || EPI == EPI_F32 ? a.ldy : (long long)a.N) + n;
 #pragma unroll
     for (int j = 0; j < 32; j++) v[j] *= factor;
-    if (EPI == EPI_GEGLU) {
+    if (EPI == EPI_GEGLU || EPI == EPI_SWIGLU) {
         uint4 packed[2];
         __nv_bfloat162 *o = reinterpret_cast<__nv_bfloat162 *>(packed);
 #pragma unroll
         for (int j = 0; j < 8; j++)
-            o[j] = __floats2bfloat162_rn(gelu_tanh(v[4 * j]) * v[4 * j + 1], gelu_tanh(v[4 * j + 2]) * v[4 * j + 3]);
+            o[j] = __floats2bfloat162_rn(gate_of<EPI == EPI_SWIGLU>(v[4 * j]) * v[4 * j + 1], gate_of<EPI == EPI_SWIGLU>(v[4 * j + 2]) * v[4 * j + 3]);
         uint4 *dst = reinterpret_cast<uint4 *>(reinterpret_cast<bf16 *>(a.y) + (size_t)row * a.ldy + (n >> 1));
         dst[0] = packed[0], dst[1] = packed[1];
     } else if ((EPI == EPI_STORE || EPI == EPI_F32) && (n + 32 > a.n_store || (a.ldy & 7))) {
@@ -171,6 +173,48 @@ static __device__ __forceinline__ void stream_columns(const TileArgs &a, int m, 
             if ((lane & 7) == 0) a.rs.ss_next[(size_t)row * (a.N >> 5) + (n >> 5)] = q;
         }
     }
+    __syncwarp(); /* the staging is free again */
+}
+
+/* stream_columns for at most S streams: 16 values of the streams per thread are in flight at a time. */
+template <int S> static __device__ __forceinline__ void columns_of_streams(const TileArgs &a, int m, int n, const float *turn, int lane) {
+    constexpr int G = 16 / S > 8 ? 8 : 16 / S;
+    const int r4 = lane >> 3, c4 = (lane & 7) * 4;
+    const float4 gain = *reinterpret_cast<const float4 *>(a.rs.gain + n + c4);
+#pragma unroll
+    for (int i0 = 0; i0 < 8; i0 += G) {
+        Streams<S, float4> h[G];
+#pragma unroll
+        for (int i = 0; i < G; i++) {
+            const int row = m + 4 * (i0 + i) + r4;
+            h[i].load(a.rs, (size_t)row * a.rs.streams * a.N + n + c4, a.N, row < a.rows);
+        }
+#pragma unroll
+        for (int i = 0; i < G; i++) {
+            const int row = m + 4 * (i0 + i) + r4;
+            const float *p = turn + (4 * (i0 + i) + r4) * 33 + c4;
+            const float4 x = h[i].update(a.rs, (size_t)row * a.rs.streams * a.N + n + c4, a.N, make_float4(p[0], p[1], p[2], p[3]), row < a.rows);
+            float q = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+            q += __shfl_xor_sync(0xffffffffu, q, 1);
+            q += __shfl_xor_sync(0xffffffffu, q, 2);
+            q += __shfl_xor_sync(0xffffffffu, q, 4);
+            if (row < a.rows) {
+                uint2 out;
+                __nv_bfloat162 *o = reinterpret_cast<__nv_bfloat162 *>(&out);
+                o[0] = __floats2bfloat162_rn(x.x * gain.x, x.y * gain.y);
+                o[1] = __floats2bfloat162_rn(x.z * gain.z, x.w * gain.w);
+                *reinterpret_cast<uint2 *>(reinterpret_cast<bf16 *>(a.rs.x_next) + (size_t)row * a.N + n + c4) = out;
+                if ((lane & 7) == 0) a.rs.ss_next[(size_t)row * (a.N >> 5) + (n >> 5)] = q;
+            }
+        }
+    }
+}
+static __device__ __forceinline__ void streams_columns(const TileArgs &a, int m, int n, const float *v, float factor, float *turn,
+                                                       int lane) {
+#pragma unroll
+    for (int j = 0; j < 32; j++) turn[lane * 33 + j] = v[j] * factor;
+    __syncwarp();
+    with_streams(a.rs.streams, [&](auto S) { columns_of_streams<decltype(S)::value>(a, m, n, turn, lane); });
     __syncwarp(); /* the staging is free again */
 }
 
@@ -307,6 +351,10 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm(const __grid_constant_
                     stream_columns(a, m0 + quarter * 32, n0 + c * 32, v, factor, turn, lane);
                     continue;
                 }
+                if (EPI == EPI_STREAMS) {
+                    streams_columns(a, m0 + quarter * 32, n0 + c * 32, v, factor, turn, lane);
+                    continue;
+                }
                 if (!live) continue;
                 store_columns<EPI>(a, row, n0 + c * 32, v, factor);
             }
@@ -345,11 +393,11 @@ constexpr bool PAIR_BY_DEFAULT = true;
  * tiles fit one round (64). Of an MMA's NMMA W rows each block stages NMMA / 2. */
 template <int NMMA, int NSUB, int EPI> struct Pair {
     static constexpr int WIDTH = NMMA * NSUB;
-    static constexpr int TURN_BYTES = EPI == EPI_STREAM ? 4 * TURN_FLOATS * 4 : 0; /* the stream update's staging */
+    static constexpr int TURN_BYTES = writes_stream(EPI) ? 4 * TURN_FLOATS * 4 : 0; /* the stream update's staging */
     static constexpr int SUB_BYTES = (NMMA / 2) * KBLK * 2;        /* this block's W rows of one MMA */
     static constexpr int B_BYTES = NSUB * SUB_BYTES;
     static constexpr int STAGE_BYTES = A_BYTES + B_BYTES;          /* 32 KB (256 wide) or 36 KB (320 wide) */
-    static constexpr int STAGES = WIDTH > 256 && EPI == EPI_STREAM ? 5 : 6;
+    static constexpr int STAGES = WIDTH > 256 && writes_stream(EPI) ? 5 : 6;
     static constexpr int RING_BYTES = STAGES * STAGE_BYTES;
     static constexpr int SMEM_BYTES = 1024 + RING_BYTES + 256 + TURN_BYTES;
     static constexpr int ACCS = 2 * WIDTH <= 512 ? 2 : 1;          /* accumulators in tensor memory */
@@ -556,6 +604,10 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm_pair(const __grid_cons
                     stream_columns(a, m0 + quarter * 32, n0 + c * 32, v, factor, turn, lane);
                     continue;
                 }
+                if (EPI == EPI_STREAMS) {
+                    streams_columns(a, m0 + quarter * 32, n0 + c * 32, v, factor, turn, lane);
+                    continue;
+                }
                 if (!live) continue;
                 store_columns<EPI>(a, row, n0 + c * 32, v, factor);
             }
@@ -623,6 +675,8 @@ int launch_epi(const CUtensorMap &map_x, const CUtensorMap &map_w, const CUtenso
     case EPI_F32: return launch<BN, EPI_F32>(map_x, map_w, map_w_half, a, stream);
     case EPI_GEGLU: return launch<BN, EPI_GEGLU>(map_x, map_w, map_w_half, a, stream);
     case EPI_STREAM: return launch<BN, EPI_STREAM>(map_x, map_w, map_w_half, a, stream);
+    case EPI_STREAMS: return launch<BN, EPI_STREAMS>(map_x, map_w, map_w_half, a, stream);
+    case EPI_SWIGLU: return launch<BN, EPI_SWIGLU>(map_x, map_w, map_w_half, a, stream);
     default: return NCB_ERR_ARG;
     }
 }
@@ -712,6 +766,8 @@ int launch_pair_epi(const CUtensorMap &map_x, const CUtensorMap &map_w, const CU
     case EPI_F32: return launch_pair<NMMA, NSUB, EPI_F32>(map_x, map_w, map_w_half, a, pairs, stream);
     case EPI_GEGLU: return launch_pair<NMMA, NSUB, EPI_GEGLU>(map_x, map_w, map_w_half, a, pairs, stream);
     case EPI_STREAM: return launch_pair<NMMA, NSUB, EPI_STREAM>(map_x, map_w, map_w_half, a, pairs, stream);
+    case EPI_STREAMS: return launch_pair<NMMA, NSUB, EPI_STREAMS>(map_x, map_w, map_w_half, a, pairs, stream);
+    case EPI_SWIGLU: return launch_pair<NMMA, NSUB, EPI_SWIGLU>(map_x, map_w, map_w_half, a, pairs, stream);
     default: return NCB_ERR_ARG;
     }
 }
@@ -784,7 +840,7 @@ int tile_gemm_rs(const ncb_gemm_rs *g, void *stream) {
     if (!g || g->rows > 0x7fffff00LL || g->N % 128 || g->K % KBLK) return NCB_ERR_ARG;
     const int rc = check_rs(*g);
     if (rc != NCB_OK || g->rows == 0) return rc;
-    if (g->epilogue == EPI_GEGLU && g->ldy % 8) return NCB_ERR_ALIGN;
+    if ((g->epilogue == EPI_GEGLU || g->epilogue == EPI_SWIGLU) && g->ldy % 8) return NCB_ERR_ALIGN;
     const TileArgs a = {nullptr, g->y, (int)g->rows, g->N, g->K, g->status, 0, g->ldy, g->n_store, stream_io(*g)};
     return run_tile_gemm(g->x, g->w, a, g->epilogue, 0, (cudaStream_t)stream);
 }

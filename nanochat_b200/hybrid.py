@@ -1,5 +1,7 @@
 """Decoder for models whose layers differ in kind: each layer a mixer (mixers.MIXERS) and optionally a gated feed-forward,
-pre-norm, around a residual stream kept in fp32. Layers may share another layer's weights with a cache of their own.
+pre-norm, around a residual stream kept in fp32. Layers may share another layer's weights with a cache of their own, or read
+another layer's keys and values. In place of the one stream there may be several with hyper-connections: a branch reads a
+weighted sum of them, and its result and the old streams make the new ones (HyperConnection).
 
 One layer is
     input projection (norm as a row scale) -> mixer's launches -> output projection, stream update ->
@@ -17,11 +19,11 @@ from torch import Tensor
 
 from .decoder import StepDecoder
 from .kv_cache import cache_pages
-from .mixers import MIXERS, LatentAttention, RowPlan, Rows, pad_to, up
-from .native import GemmRs, check, cuda_library, pointer, stream
+from .mixers import MIXERS, RowPlan, Rows, pad_to, up
+from .native import MAX_STREAMS, GemmRs, check, cuda_library, pointer, stream
 from .prompt_store import PromptStore
 
-STORE, STORE_F32, GEGLU, STREAM = 0, 3, 5, 6
+STORE, STORE_F32, GEGLU, STREAM, STREAMS, SWIGLU = 0, 3, 5, 6, 7, 8
 
 
 @dataclass(frozen=True)
@@ -43,6 +45,11 @@ class HybridConfig:
     logit_scale: float = 1.0
     max_len: int = 1024
     itemsize: int = 2  # bytes of a cached value
+    streams: int = 0   # streams with hyper-connections; 0: one plain residual stream
+    embed_scale: float = 1.0
+    tied_head: bool = True      # the head is the embedding; else the checkpoint's "head"
+    norm_base: float = 0.0      # norms multiply by norm_base + weight
+    unit: int = GEGLU           # the feed-forward's gated unit: GEGLU or SWIGLU
 
     @staticmethod
     def from_pudisun(config: dict, max_len: int) -> "HybridConfig":
@@ -61,6 +68,27 @@ class HybridConfig:
                             eps=float(config["norm"]["eps"]), residual_mult=float(config["residual_mult"]),
                             logit_scale=float(config["logit_scale"]), max_len=max_len)
 
+    @staticmethod
+    def from_rekudra(config: dict, max_len: int) -> "HybridConfig":
+        """From the config.json of a Rekudra model."""
+        entries, layers = config["layers"], []
+        for i, entry in enumerate(entries):
+            kind, mixer, mlp = entry["type"], entry["mixer"], entry.get("mlp")
+            if kind not in MIXERS:
+                raise ValueError(f"layer {i}: no mixer '{kind}' (known: {', '.join(sorted(MIXERS))})")
+            if mlp is not None and mlp["kind"] != "dense":
+                raise ValueError(f"layer {i}: no feed-forward '{mlp['kind']}'")
+            of = mixer.get("kv_from")
+            if of is not None and not (0 <= of < i and entries[of]["type"] == kind and entries[of]["mixer"].get("kv_from") is None):
+                raise ValueError(f"layer {i}: keys and values of layer {of}, which has none of its own")
+            layers.append(LayerSpec(kind, mixer, 0 if mlp is None else int(mlp["ff"]), i))
+        streams = int(config["streams"])
+        if not 1 <= streams <= MAX_STREAMS:
+            raise ValueError(f"{streams} streams: the kernels take up to {MAX_STREAMS}")
+        return HybridConfig(width=int(config["width"]), vocab=int(config["vocab"]), layers=layers, eps=float(config["norm"]["eps"]),
+                            max_len=max_len, streams=streams, embed_scale=float(config["embedding"]["scale"]), tied_head=False,
+                            norm_base=1.0, unit=SWIGLU)
+
     def slot_bytes(self) -> int:
         """Device bytes one more slot costs: its rows and states in every layer's cache and its rows of a decode step."""
         cache = sum(MIXERS[s.kind].cache_bytes(s.mixer, self.max_len, self.itemsize) for s in self.layers)
@@ -70,18 +98,39 @@ class HybridConfig:
 
 
 @dataclass
+class HyperConnection:
+    """How one branch reads and writes the streams, as the arrays a GEMM's epilogue takes: u = sum_s read[s] x_s,
+    x_t <- sum_s mix[s, t] x_s + write[t] y."""
+    read: ctypes.Array
+    write: ctypes.Array
+    mix: ctypes.Array
+    read_sum: float
+
+    @staticmethod
+    def of(read: Tensor, write: Tensor, mix: Tensor) -> "HyperConnection":
+        full = torch.zeros((MAX_STREAMS, MAX_STREAMS))
+        full[:mix.shape[0], :mix.shape[1]] = mix.float()
+        row, square = ctypes.c_float * MAX_STREAMS, ctypes.c_float * (MAX_STREAMS * MAX_STREAMS)
+        return HyperConnection(row(*read.float().tolist()), row(*write.float().tolist()), square(*full.flatten().tolist()),
+                               float(read.float().sum()))
+
+
+@dataclass
 class LayerWeights:
     gain1: Tensor  # fp32 [C]
     mixer: object
     gain2: "Tensor | None" = None
     w_up: "Tensor | None" = None    # [2 F, C]: gate and up rows alternating
     w_down: "Tensor | None" = None  # [C, F]
+    hc1: "HyperConnection | None" = None
+    hc2: "HyperConnection | None" = None
 
 
 @dataclass
 class HybridWeights:
     """C = width and every other GEMM size padded with zeros to what the kernels tile."""
-    embed: Tensor        # [vocab up to 128, C]; also the head
+    embed: Tensor        # [vocab up to 128, C]
+    head: Tensor         # the same shape, maybe the same tensor
     final_gain: Tensor   # fp32 [C]
     layers: list[LayerWeights]
     dtype: torch.dtype
@@ -90,11 +139,19 @@ class HybridWeights:
     def from_state_dict(state: dict, cfg: HybridConfig, dtype: torch.dtype = torch.bfloat16,
                         device: "torch.device | str" = "cuda") -> "HybridWeights":
         """From a checkpoint's tensors by name: embed, final.norm, and per layer l<i>.norm1 / norm2, l<i>.mix.*, l<i>.mlp.gate
-        / up / down. A layer that uses another one's weights has no tensors of its own and shares the prepared ones."""
+        / up / down; with several streams l<i>.hc1 / hc2.in / out / mix; the head where it is not the embedding. A layer that uses another one's weights has no tensors of its own and shares the prepared ones."""
         C = up(cfg.width, 128)
 
         def gain(name: str) -> Tensor:
-            return pad_to(state[name].to(device).float(), C)
+            return pad_to(cfg.norm_base + state[name].to(device).float(), C)
+
+        def connection(name: str) -> "HyperConnection | None":
+            if not cfg.streams:
+                return None
+            read, write, mix = (state[name + part].cpu() for part in (".in", ".out", ".mix"))
+            if read.shape != (cfg.streams,) or write.shape != (cfg.streams,) or mix.shape != (cfg.streams, cfg.streams):
+                raise ValueError(f"{name}: not of {cfg.streams} streams")
+            return HyperConnection.of(read, write, mix)
 
         layers: list[LayerWeights] = [None] * len(cfg.layers)
         for i, spec in enumerate(cfg.layers):
@@ -102,19 +159,22 @@ class HybridWeights:
                 continue
             p = f"l{i}."
             mix = {name[len(p) + 4:]: t for name, t in state.items() if name.startswith(p + "mix.")}
-            layer = LayerWeights(gain(p + "norm1"), MIXERS[spec.kind](spec.mixer, mix, cfg.eps, C, dtype, device))
+            layer = LayerWeights(gain(p + "norm1"), MIXERS[spec.kind](spec.mixer, mix, cfg.eps, C, dtype, device),
+                                 hc1=connection(p + "hc1"))
             if spec.ff:
                 F = up(spec.ff, 128)
                 w = torch.zeros((F, 2, C), dtype=dtype, device=device)
                 for j, name in enumerate(("gate", "up")):
                     w[:spec.ff, j, :cfg.width] = state[p + "mlp." + name].to(device=device, dtype=dtype)
+                layer.hc2 = connection(p + "hc2")
                 layer.gain2, layer.w_up = gain(p + "norm2"), w.view(2 * F, C)
                 layer.w_down = pad_to(state[p + "mlp.down"].to(device=device, dtype=dtype), C, F)
             layers[i] = layer
         for i, spec in enumerate(cfg.layers):
             layers[i] = layers[spec.weights_of]
-        embed = pad_to(state["embed"].to(device=device, dtype=dtype), up(cfg.vocab, 128), C)
-        return HybridWeights(embed, gain("final.norm"), layers, dtype)
+        embed, head = (pad_to(state[name].to(device=device, dtype=dtype), up(cfg.vocab, 128), C) if name else None
+                       for name in ("embed", None if cfg.tied_head else "head"))
+        return HybridWeights(embed, embed if head is None else head, gain("final.norm"), layers, dtype)
 
     @staticmethod
     def random_state(cfg: HybridConfig, seed: int, device: "torch.device | str" = "cpu", std: float = 0.02) -> dict:
@@ -153,10 +213,11 @@ class HybridWeights:
 
 
 class Stream:
-    """The fp32 residual stream of some rows and what the next norm reads: h, x = h * gain, partial sums of squares."""
+    """The fp32 residual stream of some rows (or several streams) and what the next norm reads: h, x = h * gain (of several: of
+    their weighted sum), partial sums of squares."""
 
-    def __init__(self, rows: int, columns: int, dtype: torch.dtype, device):
-        self.h = torch.empty((rows, columns), dtype=torch.float32, device=device)
+    def __init__(self, rows: int, columns: int, dtype: torch.dtype, device, streams: int = 1):
+        self.h = torch.empty((rows, streams, columns) if streams > 1 else (rows, columns), dtype=torch.float32, device=device)
         self.x = torch.empty((rows, columns), dtype=dtype, device=device)
         self.ss = torch.empty((rows, columns // 8), dtype=torch.float32, device=device)
         self.parts = 1
@@ -169,9 +230,13 @@ class HybridDecoder(StepDecoder):
                  prompt_store: int = 0, softcap: float = 0.0):
         self._start(cfg, weights, n_slots, device, softcap)
         self.dtype, self.f32 = weights.dtype, weights.dtype == torch.float32
-        self.caches = [layer.mixer.new_cache(n_slots, cfg.max_len) for layer in weights.layers]
+        self.caches = []
+        for layer in weights.layers:
+            of = layer.mixer.kv_from
+            self.caches.append(layer.mixer.new_cache(n_slots, cfg.max_len, None if of is None else self.caches[of]))
         self.capacity = cache_pages(cfg.max_len) * 64
-        self.store = PromptStore(self.caches, prompt_store) if prompt_store > 0 else None
+        self.sum_of_streams = HyperConnection.of(*(torch.ones(cfg.streams),) * 2, torch.zeros(cfg.streams, cfg.streams))
+        self.store = PromptStore([part for cache in self.caches for part in cache.parts], prompt_store) if prompt_store > 0 else None
         self.columns = up(cfg.width, 128)
         self.in_width = max(layer.mixer.in_width for layer in weights.layers)
         self.out_width = max(layer.mixer.out_width for layer in weights.layers)
@@ -195,9 +260,10 @@ class HybridDecoder(StepDecoder):
 
     def gemm(self, rows: int, x: Tensor, w: Tensor, epilogue: int, st: Stream, out: "Tensor | None" = None,
              gain: "Tensor | None" = None, n_store: int = 0, scale: float = 1.0, normed: bool = False,
-             then: "Tensor | None" = None) -> None:
+             then: "Tensor | None" = None, hc: "tuple | None" = None) -> None:
         """epilogue(x . w^T): see ncb_gemm_rs. normed: x is the stream's and its norm is applied; gain: the next norm's
-        (epilogue STREAM); then: the weights the next GEMM reads (prefetched into L2 by stream_gemm)."""
+        (epilogues STREAM, STREAMS); then: the weights the next GEMM reads (prefetched into L2 by stream_gemm); hc: this branch's
+        and the next one's hyper-connections (STREAMS)."""
         N, K = w.shape
         kind = self.gemm_kernel(rows, N, K)
         lib, entry, part = self.ENTRY[kind]
@@ -205,7 +271,9 @@ class HybridDecoder(StepDecoder):
                    eps=self.cfg.eps, norm_count=self.cfg.width, mult=self.cfg.residual_mult, status=self.status.data_ptr())
         if normed:
             a.ss, a.ss_parts = st.ss.data_ptr(), st.parts
-        if epilogue == STREAM:
+        if epilogue == STREAMS:
+            a.streams, a.out, a.mix, a.in_ = self.cfg.streams, hc[0].write, hc[0].mix, hc[1].read
+        if epilogue in (STREAM, STREAMS):
             a.h, a.gain, a.x_next, a.ss_next = st.h.data_ptr(), gain.data_ptr(), st.x.data_ptr(), st.ss.data_ptr()
             st.parts = N // part
         else:
@@ -218,7 +286,7 @@ class HybridDecoder(StepDecoder):
 
     def buffers(self, rows: int) -> dict:
         dev, d = self.device, self.dtype
-        buf = {"stream": Stream(rows, self.columns, d, dev),
+        buf = {"stream": Stream(rows, self.columns, d, dev, max(self.cfg.streams, 1)),
                "proj": torch.empty((rows, self.in_width), dtype=d, device=dev),
                # columns past a mixer's heads are padding that the output projection multiplies by zero weights
                "mixed": torch.zeros((rows, self.out_width), dtype=d, device=dev)}
@@ -230,9 +298,12 @@ class HybridDecoder(StepDecoder):
         """The stream after the last layer, with x = h * final gain; fill_only: stop when the last layer's cache is filled."""
         cfg, w, st, n = self.cfg, self.w, buf["stream"], rows.n
         layers = w.layers
-        check(cuda_library("decode_step").embed_rs(pointer(w.embed), pointer(tokens), pointer(st.h), pointer(layers[0].gain1),
-                                                   pointer(st.x), pointer(st.ss), n, self.columns, cfg.vocab, int(self.f32),
-                                                   stream()), "embed_rs")
+        many = cfg.streams > 0
+        write = STREAMS if many else STREAM
+        check(cuda_library("decode_step").embed_streams(pointer(w.embed), pointer(tokens), pointer(st.h), pointer(layers[0].gain1),
+                                                        pointer(st.x), pointer(st.ss), n, self.columns, cfg.vocab, int(self.f32),
+                                                        max(cfg.streams, 1), cfg.embed_scale,
+                                                        layers[0].hc1.read_sum if many else 1.0, stream()), "embed_streams")
         st.parts = 1
         for i, layer in enumerate(layers):
             mixer, last = layer.mixer, i + 1 == len(layers)
@@ -245,16 +316,19 @@ class HybridDecoder(StepDecoder):
                 return st
             mixer.run(proj, self.caches[i], rows, mixed)
             dense = layer.w_up is not None
-            following = layer.w_up if dense else w.embed if last else layers[i + 1].mixer.w_in
-            self.gemm(n, mixed, mixer.w_out, STREAM, st, gain=layer.gain2 if dense else after, then=following)
+            following = layer.w_up if dense else w.head if last else layers[i + 1].mixer.w_in
+            read = self.sum_of_streams if last else layers[i + 1].hc1
+            self.gemm(n, mixed, mixer.w_out, write, st, gain=layer.gain2 if dense else after, then=following,
+                      hc=(layer.hc1, layer.hc2 if dense else read))
             if dense:
                 u = buf["u"].view(-1)[:n * layer.w_down.shape[1]].view(n, layer.w_down.shape[1])
-                self.gemm(n, st.x, layer.w_up, GEGLU, st, out=u, normed=True, then=layer.w_down)
-                self.gemm(n, u, layer.w_down, STREAM, st, gain=after, then=None if last else layers[i + 1].mixer.w_in)
+                self.gemm(n, st.x, layer.w_up, cfg.unit, st, out=u, normed=True, then=layer.w_down)
+                self.gemm(n, u, layer.w_down, write, st, gain=after, then=None if last else layers[i + 1].mixer.w_in,
+                          hc=(layer.hc2, read))
         return st
 
     def head(self, st: Stream, rows: int, out: Tensor) -> None:
-        self.gemm(rows, st.x, self.w.embed, STORE_F32, st, out=out, n_store=self.cfg.vocab, scale=self.cfg.logit_scale,
+        self.gemm(rows, st.x, self.w.head, STORE_F32, st, out=out, n_store=self.cfg.vocab, scale=self.cfg.logit_scale,
                   normed=True)
 
     # ---- what StepDecoder drives ----------------------------------------------------------------------------------------
@@ -295,9 +369,10 @@ class HybridDecoder(StepDecoder):
         self.head(self.run_layers(tokens, rows, buf), n, buf["logits"])
 
     def planned_chunk(self, positions: list[int], steps: int) -> int:
-        """Tiles per chunk of the latent layers' split kernel for lengths half way through the run."""
-        latent = next((l.mixer for l in self.w.layers if isinstance(l.mixer, LatentAttention)), None)
-        if latent is None:
+        """Tiles per chunk of the attention layers' split kernel (the first such layer's choice) for lengths half way through
+        the run."""
+        attention = next((l.mixer for l in self.w.layers if hasattr(l.mixer, "chunk_for")), None)
+        if attention is None:
             return 0
         lens = [min(p + 1 + steps // 2, self.capacity) for p in positions]
-        return latent.chunk_for(lens, self.capacity)
+        return attention.chunk_for(lens, self.capacity)

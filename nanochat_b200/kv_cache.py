@@ -101,7 +101,15 @@ class Fp8KVCache:
         return k, floats[:, fbase + PAGE_KS // 4], v, floats[:, fbase + PAGE_VS // 4]
 
 
-class LatentCache:
+class SingleCache:
+    """A layer's cache that is one buffer."""
+
+    @property
+    def parts(self) -> list:
+        return [self]
+
+
+class LatentCache(SingleCache):
     """One latent-attention layer's cache: a row of `width` values (normed latent, then the rotated key part) per position,
     T [n_slots, capacity, width]. `pages` is the same memory in the unit the prompt store copies: 64 positions of a slot."""
 
@@ -124,7 +132,51 @@ class LatentCache:
         return cache_pages(positions)
 
 
-class StateCache:
+class HeadCache:
+    """One attention layer's keys and values in the model's number format: a row [key | value] per position and key/value head,
+    T [n_slots, kv_heads, capacity, dim + vdim]. `pages`: the same memory in units of 64 positions."""
+
+    def __init__(self, n_slots: int, kv_heads: int, width: int, max_len: int, dtype: torch.dtype, device: "torch.device | str" = "cuda"):
+        self.n_slots, self.kv_heads, self.width = n_slots, kv_heads, width
+        self.pages_per_slot = cache_pages(max_len)
+        self.capacity = self.pages_per_slot * PAGE_TOKENS
+        self.rows = torch.zeros((n_slots, kv_heads, self.capacity, width), dtype=dtype, device=device)
+        self.pages = self.rows.view(torch.uint8).view(n_slots, kv_heads, self.pages_per_slot, -1)
+
+    @property
+    def device(self) -> torch.device:
+        return self.rows.device
+
+    def nbytes(self) -> int:
+        return self.pages.numel()
+
+    @staticmethod
+    def pages_for(positions: int) -> int:
+        return cache_pages(positions)
+
+
+class RingCache:
+    """A short convolution's state: the last projected rows of every slot, position p's at p % taps, T [n_slots, taps, width].
+    Positions before 0 count as zeros wherever they are read, so a slot that is used again needs no clearing."""
+
+    def __init__(self, n_slots: int, taps: int, width: int, dtype: torch.dtype, device: "torch.device | str" = "cuda"):
+        self.n_slots, self.taps, self.width = n_slots, taps, width
+        self.rows = torch.zeros((n_slots, taps, width), dtype=dtype, device=device)
+        self.pages = self.rows.view(torch.uint8).view(n_slots, 1, 1, -1)
+
+    @property
+    def device(self) -> torch.device:
+        return self.rows.device
+
+    def nbytes(self) -> int:
+        return self.pages.numel()
+
+    @staticmethod
+    def pages_for(positions: int) -> int:
+        return 1 if positions > 0 else 0
+
+
+class StateCache(SingleCache):
     """One recurrent layer's state: fp32 [n_slots, heads, dim, vdim], carried from token to token. A row at position 0
     starts from zero whatever its slot holds, so a slot that is used again needs no clearing. As `pages`, a slot is a
     single page: the state after the last position that was run."""

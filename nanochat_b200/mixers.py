@@ -3,23 +3,27 @@ the launches between the input projection and the output projection. A mixer is 
 checkpoint tensors, so any model whose layers use it can share it. A decoder only sees
 
     w_in, w_out                    fused input projection [in_width, C], output projection [C, out_width]
-    new_cache(n_slots, max_len)    one layer's cache
+    new_cache(n_slots, max_len)    one layer's cache; its `parts` are what a prompt store copies
+    kv_from                        the layer whose keys and values this one reads (None: its own); that layer's cache is then
+                                   new_cache's third argument
     run(proj, cache, rows, out)    proj [rows, in_width] -> out [rows, out_width]; out None: only fill the cache
 
 Sizes the kernels want as multiples (of 16, 32 or 128) are reached by zero-padding weights here: padded values are zero
 everywhere they appear, so they change nothing, and no kernel has ragged edges."""
 
+import functools
 from dataclasses import dataclass, field
 
 import numpy as np
 import torch
 from torch import Tensor
 
-from .kv_cache import LatentCache, StateCache
-from .native import GemmRs, Gla, Latent, check, cuda_library, stream
+from .kv_cache import HeadCache, LatentCache, RingCache, StateCache
+from .native import Conv, Delta, GemmRs, Gla, Gqa, Latent, check, cuda_library, pointer, stream
 from .rotary import half_tables
 
 LATENT_TILE = 32  # NCB_LATENT_TILE
+GQA_TILE = 16     # NCB_GQA_TILE
 SM_COUNT = 148
 
 
@@ -136,10 +140,215 @@ class Rows:
         return t
 
 
+def padded_heads(w: Tensor, heads: int, size: int, padded: int) -> Tensor:
+    """[heads size, n] -> [heads padded, n]: zero rows at the end of every head."""
+    return pad_to(w.reshape(heads, size, -1), heads, padded, w.shape[-1]).reshape(heads * padded, -1)
+
+
+class ShortConv:
+    """The short causal convolution on the first channels of a mixer's projection: fields [(channels x taps weights or None where
+    there are none, the field's offset)]; channels outside the fields are zero."""
+
+    def __init__(self, fields: list, width: int, dtype: torch.dtype, device):
+        self.width, self.dtype, self.device = width, dtype, torch.device(device)
+        self.taps = max((w.shape[1] for w, _ in fields), default=1)
+        self.w = torch.zeros((self.taps, width), dtype=torch.float32, device=device)
+        for w, at in fields:
+            if w.shape[1] != self.taps:
+                raise ValueError(f"convolutions of {w.shape[1]} and {self.taps} taps in one layer")
+            self.w[:, at:at + w.shape[0]] = w.float().T
+
+    def new_ring(self, n_slots: int) -> RingCache:
+        return RingCache(n_slots, self.taps, self.width, self.dtype, self.device)
+
+    def args(self, proj: Tensor, ring: RingCache, rows: "Rows") -> Conv:
+        return Conv(proj=proj.data_ptr(), ring=ring.rows.data_ptr(), w=self.w.data_ptr(), rows=rows.n, ldp=proj.stride(0),
+                    taps=self.taps, width=self.width, n_slots=ring.n_slots, pos=rows.pos.data_ptr(),
+                    slot_map=rows.slot_map.data_ptr())
+
+    def keep_tail(self, conv: Conv, rows: "Rows") -> None:
+        """After a pass of several rows per slot; a decode step's kernels keep their rows themselves."""
+        if rows.plan is not None:
+            check(cuda_library("short_conv").short_conv_tail(pointer_to(conv), int(self.dtype == torch.float32),
+                                                             pointer(rows.status), stream()), "short_conv_tail")
+
+
+@dataclass
+class AttentionCache:
+    kv: HeadCache
+    ring: RingCache
+    own: bool
+
+    @property
+    def parts(self) -> list:
+        return [self.kv, self.ring] if self.own else [self.ring]
+
+
+@dataclass
+class RecurrentCache:
+    state: StateCache
+    ring: RingCache
+
+    @property
+    def parts(self) -> list:
+        return [self.state, self.ring]
+
+
+class GroupedAttention:
+    """Softmax attention of grouped query heads: short convolutions, rotation, norm of queries and keys, a gate per head
+    (csrc/gqa_attn.cu). sizes: heads, kv_heads, dim, vdim, scale, rot (dims, base, scaling; may be absent), kv_from. tensors: q,
+    q.conv, g, o and, unless another layer's are read, k, k.conv, v, v.conv."""
+
+    def __init__(self, sizes: dict, tensors: dict, eps: float, columns: int, dtype: torch.dtype, device):
+        H, G, D, V = (int(sizes[n]) for n in ("heads", "kv_heads", "dim", "vdim"))
+        if H % G:
+            raise ValueError(f"{H} query heads over {G} key/value heads")
+        self.heads, self.kv_heads, self.true_dim, self.rot_spec = H, G, D, sizes.get("rot")
+        self.rot = int(self.rot_spec["dims"]) if self.rot_spec else 0
+        if self.rot % 2 or self.rot > D:
+            raise ValueError(f"rotation of {self.rot} of {D} dimensions")
+        self.dim, self.vdim, self.kv_from = up(D, 16), up(V, 16), sizes.get("kv_from")
+        self.scale, self.eps, self.dtype, self.device = float(sizes["scale"]), float(eps), dtype, torch.device(device)
+        t = {k: v.to(device) for k, v in tensors.items()}
+        heads = [("q", H, D, self.dim)] + ([("k", G, D, self.dim), ("v", G, V, self.vdim)] if self.kv_from is None else [])
+        fields = [padded_heads(t[n], h, d, p).to(dtype) for n, h, d, p in heads] + [t["g"].to(dtype)]
+        self.w_in, offsets = stack_fields(fields, 128, columns)
+        self.off_q, self.off_g = offsets[0], offsets[-1]
+        self.off_k, self.off_v = offsets[1:3] if self.kv_from is None else (0, 0)
+        self.conv = ShortConv([(padded_heads(t[n + ".conv"], h, d, p), at) for (n, h, d, p), at in zip(heads, offsets)], self.off_g,
+                              dtype, device)
+        o = pad_to(t["o"].reshape(-1, H, V), columns, H, self.vdim).reshape(columns, H * self.vdim)
+        self.out_width = up(H * self.vdim, 128)
+        self.w_out = pad_to(o, columns, self.out_width).to(dtype)
+        self.in_width = self.w_in.shape[0]
+        self.tables: "tuple[Tensor, Tensor] | None" = None
+        self._chunks: dict[tuple[int, int], int] = {}
+
+    def new_cache(self, n_slots: int, max_len: int, of: "AttentionCache | None" = None) -> AttentionCache:
+        if (of is None) != (self.kv_from is None):
+            raise ValueError("a layer reads its own keys and values or another layer's")
+        kv = HeadCache(n_slots, self.kv_heads, self.dim + self.vdim, max_len, self.dtype, self.device) if of is None else of.kv
+        if kv.width != self.dim + self.vdim or kv.kv_heads != self.kv_heads:
+            raise ValueError("layers that share keys and values differ in their heads")
+        if self.rot and (self.tables is None or self.tables[0].shape[0] < kv.capacity):
+            self.tables = shared_tables(kv.capacity, self.rot, float(self.rot_spec["base"]),
+                                        tuple(sorted((self.rot_spec.get("scaling") or {}).items())), self.device)
+        return AttentionCache(kv, self.conv.new_ring(n_slots), of is None)
+
+    @staticmethod
+    def cache_bytes(sizes: dict, max_len: int, itemsize: int) -> int:
+        H, G, dim, vdim = int(sizes["heads"]), int(sizes["kv_heads"]), up(int(sizes["dim"]), 16), up(int(sizes["vdim"]), 16)
+        own = sizes.get("kv_from") is None
+        ring = int(sizes.get("conv", 1)) * (H * dim + (G * (dim + vdim) if own else 0))
+        return (ring + (up(max_len, 64) * G * (dim + vdim) if own else 0)) * itemsize
+
+    def chunk_for(self, lens: "list[int]", most: int) -> int:
+        """Tiles per chunk of the split kernel for rows of these lengths, at most 128 chunks for `most` positions: enough blocks
+        to fill the GPU twice over, chunks long enough to be worth a state."""
+        tiles = np.maximum((np.asarray(lens, dtype=np.int64) + GQA_TILE - 1) // GQA_TILE, 1)
+        top, least = int(tiles.max()), max(8, ((most + GQA_TILE - 1) // GQA_TILE + 127) // 128)
+        per_chunk = self.kv_heads * ((self.heads // self.kv_heads + 15) // 16)
+        best, cost = least, float("inf")
+        c = least
+        while c < 2 * max(top, least):
+            blocks = int(((tiles + c - 1) // c).sum()) * per_chunk
+            now = -(-blocks // (2 * SM_COUNT)) * (min(c, top) + 8.0)
+            if now < cost:
+                best, cost = c, now
+            c += max(1, c // 8)
+        return best
+
+    def default_chunk(self, rows: int, max_len: int) -> int:
+        if (rows, max_len) not in self._chunks:
+            self._chunks[rows, max_len] = self.chunk_for([max_len] * rows, max_len)
+        return self._chunks[rows, max_len]
+
+    def run(self, proj: Tensor, cache: AttentionCache, rows: Rows, out: "Tensor | None") -> None:
+        n, f32, lib, kv = rows.n, int(self.dtype == torch.float32), cuda_library("gqa_attn"), cache.kv
+        a = Gqa(conv=self.conv.args(proj, cache.ring, rows), kv=kv.rows.data_ptr(), off_q=self.off_q, off_k=self.off_k, off_v=self.off_v,
+                off_g=self.off_g, own_kv=int(cache.own), keep=int(rows.plan is None and self.conv.taps > 1), heads=self.heads,
+                kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim, norm_count=self.true_dim, rot=self.rot, capacity=kv.capacity,
+                table_len=kv.capacity, scale=self.scale, eps=self.eps, status=rows.status.data_ptr())
+        if self.rot:
+            a.cos, a.sin = (t.data_ptr() for t in self.tables)
+        if out is not None:
+            a.q = rows.buffer("gqa_q", n * self.heads * self.dim, self.dtype, self.device).data_ptr()
+        check(lib.gqa_rows(pointer_to(a), f32, stream()), "gqa_rows")
+        if out is not None:
+            a.out, a.ldo = out.data_ptr(), out.stride(0)
+            max_len = min(rows.max_len, kv.capacity)
+            tiles = (max_len + GQA_TILE - 1) // GQA_TILE
+            a.max_len, a.chunk_tiles = max_len, rows.chunk_tiles or self.default_chunk(n, max_len)
+            a.max_chunks = (tiles + a.chunk_tiles - 1) // a.chunk_tiles
+            a.parts = rows.buffer("gqa_parts", n * self.heads * a.max_chunks * (self.vdim + 4), torch.float32, self.device).data_ptr()
+            check(lib.gqa_split(pointer_to(a), f32, stream()), "gqa_split")
+            check(lib.gqa_merge(pointer_to(a), f32, stream()), "gqa_merge")
+        self.conv.keep_tail(a.conv, rows)
+
+
+class ChannelDelta:
+    """Gated delta rule with a decay per key channel, short convolutions, per-head output norm and a low-rank sigmoid gate
+    (csrc/delta_rule.cu). sizes: heads, kv_heads, dim, vdim. tensors: q, k, v and their .conv, b, A_log, a1, a2, dt_bias, g1, g2,
+    norm, o."""
+
+    kv_from = None
+
+    def __init__(self, sizes: dict, tensors: dict, eps: float, columns: int, dtype: torch.dtype, device):
+        H, G, D, V = (int(sizes[n]) for n in ("heads", "kv_heads", "dim", "vdim"))
+        if H % G:
+            raise ValueError(f"{H} value heads over {G} query/key heads")
+        self.heads, self.kv_heads, self.true_vdim = H, G, V
+        self.dim, self.vdim, self.q_scale = up(D, 16), up(V, 16), float(D) ** -0.5
+        self.eps, self.dtype, self.device = float(eps), dtype, torch.device(device)
+        t = {k: v.to(device) for k, v in tensors.items()}
+        heads = [("q", G, D, self.dim), ("k", G, D, self.dim), ("v", H, V, self.vdim)]
+        fields = [padded_heads(t[n], h, d, p).to(dtype) for n, h, d, p in heads] + [t[n].to(dtype) for n in ("b", "a1", "g1")]
+        self.w_in, self.offsets = stack_fields(fields, 128, columns)
+        self.conv = ShortConv([(padded_heads(t[n + ".conv"], h, d, p), at) for (n, h, d, p), at in zip(heads, self.offsets)],
+                              self.offsets[3], dtype, device)
+        self.rank_a, self.rank_g = t["a1"].shape[0], t["g1"].shape[0]
+
+        def second(w: Tensor, n: int, padded: int) -> Tensor:  # [heads n, rank] -> [heads, rank, padded]
+            return pad_to(w.reshape(H, n, -1), H, padded, w.shape[1]).transpose(1, 2).contiguous().to(dtype)
+
+        self.a2, self.g2 = second(t["a2"], D, self.dim), second(t["g2"], V, self.vdim)
+        self.dt_bias = pad_to(t["dt_bias"].float().reshape(H, D), H, self.dim).contiguous()
+        self.a_exp = t["A_log"].float().exp()
+        self.norm = pad_to(t["norm"].float(), self.vdim)
+        o = pad_to(t["o"].reshape(-1, H, V), columns, H, self.vdim).reshape(columns, H * self.vdim)
+        self.out_width = up(H * self.vdim, 128)
+        self.w_out = pad_to(o, columns, self.out_width).to(dtype)
+        self.in_width = self.w_in.shape[0]
+
+    def new_cache(self, n_slots: int, max_len: int, of: None = None) -> RecurrentCache:
+        return RecurrentCache(StateCache(n_slots, self.heads, self.dim, self.vdim, device=self.device), self.conv.new_ring(n_slots))
+
+    @staticmethod
+    def cache_bytes(sizes: dict, max_len: int, itemsize: int) -> int:
+        H, G, dim, vdim = int(sizes["heads"]), int(sizes["kv_heads"]), up(int(sizes["dim"]), 16), up(int(sizes["vdim"]), 16)
+        return H * dim * vdim * 4 + int(sizes.get("conv", 1)) * (2 * G * dim + H * vdim) * itemsize
+
+    def run(self, proj: Tensor, cache: RecurrentCache, rows: Rows, out: "Tensor | None") -> None:
+        f32, lib, plan = int(self.dtype == torch.float32), cuda_library("delta_rule"), rows.plan
+        a = Delta(conv=self.conv.args(proj, cache.ring, rows), out=None if out is None else out.data_ptr(),
+                  ldo=0 if out is None else out.stride(0), keep=int(plan is None and self.conv.taps > 1), heads=self.heads,
+                  kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim, rank_a=self.rank_a, rank_g=self.rank_g,
+                  norm_count=self.true_vdim, q_scale=self.q_scale, eps=self.eps, a2=self.a2.data_ptr(), g2=self.g2.data_ptr(),
+                  dt_bias=self.dt_bias.data_ptr(), a_exp=self.a_exp.data_ptr(), norm=self.norm.data_ptr(),
+                  state=cache.state.state.data_ptr(), status=rows.status.data_ptr())
+        a.off_q, a.off_k, a.off_v, a.off_b, a.off_a, a.off_g = self.offsets
+        if plan is not None:
+            first, count = plan.segments()
+            a.seg_first, a.seg_count, a.n_segments = first.data_ptr(), count.data_ptr(), plan.n_segments
+        check(lib.delta_step(pointer_to(a), f32, stream()), "delta_step")
+        self.conv.keep_tail(a.conv, rows)
+
+
 class GatedLinearAttention:
     """Linear attention with a decay per key channel, per-head output norm and silu gate (csrc/gla.cu).
     sizes: heads, dim, vdim, tau. tensors: q, k, v, g, o, a1, a2, a2.b, norm."""
 
+    kv_from = None
     CHUNKED_FROM = 24  # shorter segments run token by token
 
     def __init__(self, sizes: dict, tensors: dict, eps: float, columns: int, dtype: torch.dtype, device):
@@ -166,7 +375,7 @@ class GatedLinearAttention:
         self.in_width = self.w_in.shape[0]
         self.chunk = cuda_library("gla").gla_chunk_tokens(self.dim)
 
-    def new_cache(self, n_slots: int, max_len: int) -> StateCache:
+    def new_cache(self, n_slots: int, max_len: int, of: None = None) -> StateCache:
         return StateCache(n_slots, self.heads, self.dim, self.vdim, device=self.device)
 
     @staticmethod
@@ -205,6 +414,8 @@ class LatentAttention:
     sizes: heads, dim, rot_dim, vdim, kv_rank, scale, rot (dims, base, scaling). tensors: q, dkv, dkv.norm, uk, uv, o and
     optionally g (output gate) and sink."""
 
+    kv_from = None
+
     def __init__(self, sizes: dict, tensors: dict, eps: float, columns: int, dtype: torch.dtype, device):
         H, D, R = int(sizes["heads"]), int(sizes["dim"]), int(sizes["rot_dim"])
         V, rank, rot = int(sizes["vdim"]), int(sizes["kv_rank"]), sizes["rot"]
@@ -242,7 +453,7 @@ class LatentAttention:
         self.tables: "tuple[Tensor, Tensor] | None" = None
         self._chunks: dict[tuple[int, int], int] = {}
 
-    def new_cache(self, n_slots: int, max_len: int) -> LatentCache:
+    def new_cache(self, n_slots: int, max_len: int, of: None = None) -> LatentCache:
         cache = LatentCache(n_slots, self.rank + self.rot, max_len, self.dtype, device=self.device)
         if self.tables is None or self.tables[0].shape[0] < cache.capacity:
             self.tables = half_tables(cache.capacity, int(self.rot_spec["dims"]), float(self.rot_spec["base"]),
@@ -334,10 +545,17 @@ class LatentAttention:
         check(lib.latent_out(pointer_to(a), f32, stream()), "latent_out")
 
 
+@functools.lru_cache(maxsize=4)
+def shared_tables(positions: int, dims: int, base: float, scaling: tuple, device) -> tuple[Tensor, Tensor]:
+    """half_tables, one pair for all layers of a kind."""
+    return half_tables(positions, dims, base, dict(scaling) or None, dims, device)
+
+
 def pointer_to(struct):
     import ctypes
 
     return ctypes.byref(struct)
 
 
-MIXERS = {"latent_attention": LatentAttention, "gla": GatedLinearAttention}
+MIXERS = {"latent_attention": LatentAttention, "gla": GatedLinearAttention, "attention": GroupedAttention,
+          "channel_delta": ChannelDelta}

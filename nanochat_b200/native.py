@@ -22,8 +22,10 @@ KERNELS = PACKAGE / "csrc"
 INCLUDE = PACKAGE.parent / "include"
 NATIVE = PACKAGE / "_native"
 HEAD_DIM = 128
-LIBRARIES = ("kv_append", "decode_attn", "decode_step", "stream_gemm", "tile_gemm", "gemm_f32", "latent_attn", "gla")
+LIBRARIES = ("kv_append", "decode_attn", "decode_step", "stream_gemm", "tile_gemm", "gemm_f32", "latent_attn", "gla",
+             "short_conv", "gqa_attn", "delta_rule")
 
+MAX_STREAMS = 8  # NCB_MAX_STREAMS
 c_ptr, c_int, c_ll, c_float = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong, ctypes.c_float
 
 
@@ -32,7 +34,8 @@ class GemmRs(ctypes.Structure):
     _fields_ = [("x", c_ptr), ("w", c_ptr), ("y", c_ptr), ("rows", c_ll), ("ldy", c_ll), ("N", c_int), ("K", c_int),
                 ("n_store", c_int), ("epilogue", c_int), ("ss", c_ptr), ("ss_parts", c_int), ("norm_count", c_int),
                 ("eps", c_float), ("scale", c_float), ("h", c_ptr), ("gain", c_ptr), ("x_next", c_ptr), ("ss_next", c_ptr),
-                ("mult", c_float), ("next_w", c_ptr), ("next_bytes", c_ll), ("status", c_ptr)]
+                ("mult", c_float), ("next_w", c_ptr), ("next_bytes", c_ll), ("status", c_ptr), ("streams", c_int),
+                ("in_", c_float * MAX_STREAMS), ("out", c_float * MAX_STREAMS), ("mix", c_float * (MAX_STREAMS * MAX_STREAMS))]
 
 
 class Latent(ctypes.Structure):
@@ -58,6 +61,32 @@ class Gla(ctypes.Structure):
                                      "seg_chunk", "chunk_first", "chunk_count")] + \
                [(n, c_int) for n in ("n_segments", "n_chunks", "chunk")] + \
                [(n, c_ptr) for n in ("decay", "chunk_decay", "states", "raw", "status")]
+
+
+class Conv(ctypes.Structure):
+    """ncb_conv of include/nanochat_b200.h, field for field."""
+    _fields_ = [("proj", c_ptr), ("ring", c_ptr), ("w", c_ptr), ("rows", c_ll), ("ldp", c_ll), ("taps", c_int), ("width", c_int),
+                ("n_slots", c_int), ("pos", c_ptr), ("slot_map", c_ptr)]
+
+
+class Gqa(ctypes.Structure):
+    """ncb_gqa of include/nanochat_b200.h, field for field."""
+    _fields_ = [("conv", Conv), ("q", c_ptr), ("kv", c_ptr), ("out", c_ptr), ("ldo", c_ll)] + \
+               [(n, c_int) for n in ("off_q", "off_k", "off_v", "off_g", "own_kv", "keep", "heads", "kv_heads", "dim", "vdim",
+                                     "norm_count", "rot", "capacity", "table_len", "max_len", "chunk_tiles", "max_chunks",
+                                     "n_tiles")] + \
+               [("scale", c_float), ("eps", c_float)] + \
+               [(n, c_ptr) for n in ("cos", "sin", "parts", "tile_row", "tile_rows", "tile_pos", "status")]
+
+
+class Delta(ctypes.Structure):
+    """ncb_delta of include/nanochat_b200.h, field for field."""
+    _fields_ = [("conv", Conv), ("out", c_ptr), ("ldo", c_ll)] + \
+               [(n, c_int) for n in ("off_q", "off_k", "off_v", "off_b", "off_a", "off_g", "keep", "heads", "kv_heads", "dim", "vdim",
+                                     "rank_a", "rank_g", "norm_count")] + \
+               [("q_scale", c_float), ("eps", c_float)] + \
+               [(n, c_ptr) for n in ("a2", "g2", "dt_bias", "a_exp", "norm", "state", "seg_first", "seg_count")] + \
+               [("n_segments", c_int), ("status", c_ptr)]
 
 
 SIGNATURES = {
@@ -93,6 +122,7 @@ SIGNATURES = {
         "skinny_gemm_mix": ([c_ptr] * 4 + [c_float, c_float, c_ptr] + [c_int] * 4 + [c_ptr], c_int),
         "skinny_gemm_rs": ([c_ptr, c_ptr], c_int),
         "embed_rs": ([c_ptr] * 6 + [c_ll, c_int, c_int, c_int, c_ptr], c_int),
+        "embed_streams": ([c_ptr] * 6 + [c_ll, c_int, c_int, c_int, c_int, c_float, c_float, c_ptr], c_int),
         "embed_norm": ([c_ptr] * 3 + [c_int] * 3 + [c_ptr], c_int),
         "embed_norm_mix": ([c_ptr] * 4 + [c_float, c_float] + [c_int] * 3 + [c_ptr], c_int),
         "add_rms_norm": ([c_ptr] * 3 + [c_ll, c_int, c_ptr], c_int),
@@ -115,6 +145,15 @@ SIGNATURES = {
         "gla_chunk_tokens": ([c_int], c_int),
         "gla_step": ([c_ptr, c_int, c_ptr], c_int),
         "gla_chunked": ([c_ptr, c_int, c_ptr], c_int),
+    },
+    "short_conv": {"short_conv_tail": ([c_ptr, c_int, c_ptr, c_ptr], c_int)},
+    "gqa_attn": {
+        "gqa_rows": ([c_ptr, c_int, c_ptr], c_int),
+        "gqa_split": ([c_ptr, c_int, c_ptr], c_int),
+        "gqa_merge": ([c_ptr, c_int, c_ptr], c_int),
+    },
+    "delta_rule": {
+        "delta_step": ([c_ptr, c_int, c_ptr], c_int),
     },
     "tile_gemm": {
         "tile_gemm_rs": ([c_ptr, c_ptr], c_int),

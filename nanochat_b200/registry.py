@@ -46,6 +46,14 @@ def build_pudisun(config: dict, tensors: dict, n_slots: int, max_len: int, dtype
     return HybridDecoder(cfg, HybridWeights.from_state_dict(tensors, cfg, dtype, device), n_slots, device, **options)
 
 
+@register("Rekudra", libraries={torch.bfloat16: ("decode_step", "stream_gemm", "tile_gemm", "short_conv", "gqa_attn", "delta_rule"),
+                                torch.float32: ("decode_step", "gemm_f32", "short_conv", "gqa_attn", "delta_rule")})
+def build_rekudra(config: dict, tensors: dict, n_slots: int, max_len: int, dtype: torch.dtype, device, **options):
+    cfg = HybridConfig.from_rekudra(config, max_len)
+    cfg.itemsize = dtype.itemsize
+    return HybridDecoder(cfg, HybridWeights.from_state_dict(tensors, cfg, dtype, device), n_slots, device, **options)
+
+
 @register("NanochatForCausalLM", "nanochat",
           libraries={torch.bfloat16: ("kv_append", "decode_attn", "decode_step", "stream_gemm", "tile_gemm")})
 def build_nanochat(config: dict, tensors: dict, n_slots: int, max_len: int, dtype: torch.dtype, device, **options):

@@ -1,4 +1,5 @@
-"""Rotary tables for pairs (i, i + dims / 2), with optional YaRN interpolation of the frequencies."""
+"""Rotary tables for pairs (i, i + dims / 2), with optional interpolation of the frequencies: YaRN (scaling with fast and slow)
+or by bands of wavelengths (scaling with low and high)."""
 
 import math
 
@@ -25,10 +26,30 @@ def yarn_frequencies(dims: int, base: float, scaling: "dict | None") -> tuple[Te
     return freqs / factor * ramp + freqs * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
 
 
+def banded_frequencies(dims: int, base: float, scaling: dict) -> Tensor:
+    """Angle per position of each of the dims / 2 pairs, fp64. scaling: factor, original, low, high. A pair that turns more than
+    `high` times over the original context keeps its frequency, one that turns less than `low` times is divided by the factor,
+    and those between mix the two in proportion to their turns."""
+    freqs, _ = yarn_frequencies(dims, base, None)
+    turns = freqs * (float(scaling["original"]) / (2.0 * math.pi))
+    low, high = float(scaling["low"]), float(scaling["high"])
+    slowed = freqs / float(scaling["factor"])
+    share = ((turns - low) / (high - low)) if high > low else torch.zeros_like(turns)
+    mixed = torch.where(turns < low, slowed, slowed * (1.0 - share) + freqs * share)
+    return torch.where(turns > high, freqs, mixed)
+
+
+def frequencies(dims: int, base: float, scaling: "dict | None") -> tuple[Tensor, float]:
+    """(angle per position of each pair, factor of cos and sin) for either kind of scaling, or none."""
+    if scaling and "low" in scaling:
+        return banded_frequencies(dims, base, scaling), 1.0
+    return yarn_frequencies(dims, base, scaling)
+
+
 def half_tables(positions: int, dims: int, base: float, scaling: "dict | None", padded: int,
                 device: "torch.device | str") -> tuple[Tensor, Tensor]:
     """cos, sin fp32 (positions, padded / 2), evaluated in fp64 and rounded once; pairs past dims / 2 do not turn."""
-    freqs, factor = yarn_frequencies(dims, base, scaling)
+    freqs, factor = frequencies(dims, base, scaling)
     angle = torch.zeros((positions, padded // 2), dtype=torch.float64)
     angle[:, :dims // 2] = torch.arange(positions, dtype=torch.float64)[:, None] * freqs
     return (angle.cos() * factor).float().to(device), (angle.sin() * factor).float().to(device)
