@@ -524,7 +524,8 @@ int short_conv_tail(const ncb_conv *args, int f32, int *status, void *stream);
  * [n_slots][kv_heads][capacity][dim + vdim]. A row with a negative position is idle: a zero output row.
  *   gqa_rows     q T [rows][heads dim]; with own_kv k, v appended to kv; keep: also the ring (every row a slot of its own);
  *                q NULL: only the appends
- *   gqa_split    states of chunks of at most chunk_tiles tiles of NCB_GQA_TILE positions: parts fp32
+ *   gqa_split    (in bf16 with q NULL, for a decode step of sizes gqa_split_fused(dim, vdim): also everything gqa_rows does)
+ *                states of chunks of at most chunk_tiles tiles of NCB_GQA_TILE positions: parts fp32
  *                [rows][heads][max_chunks][vdim + 4]; max_len bounds every position + 1
  *   gqa_merge    out [rows][ldo] = sigmoid(gate) * merged states
  *   gqa_prefill  out of row tiles, bf16: tile_rows (at most 64) rows from tile_row, the first at position tile_pos. List the
@@ -544,6 +545,7 @@ typedef struct {
     int *status;
 } ncb_gqa;
 int gqa_rows(const ncb_gqa *args, int f32, void *stream);
+int gqa_split_fused(int dim, int vdim);
 int gqa_split(const ncb_gqa *args, int f32, void *stream);
 int gqa_merge(const ncb_gqa *args, int f32, void *stream);
 int gqa_prefill_supported(int dim, int vdim);

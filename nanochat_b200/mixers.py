@@ -223,6 +223,12 @@ class GroupedAttention:
         self.in_width = self.w_in.shape[0]
         self.tables: "tuple[Tensor, Tensor] | None" = None
         self._chunks: dict[tuple[int, int], int] = {}
+        lib, bf = cuda_library("gqa_attn"), dtype == torch.bfloat16
+        self.fused = bf and bool(lib.gqa_split_fused(self.dim, self.vdim))
+        self.tiled = bf and bool(lib.gqa_prefill_supported(self.dim, self.vdim))
+
+    ROW_TILE = 64     # rows per tile of gqa_prefill
+    TILED_FROM = 8    # shorter segments run as rows on their own
 
     def new_cache(self, n_slots: int, max_len: int, of: "AttentionCache | None" = None) -> AttentionCache:
         if (of is None) != (self.kv_from is None):
@@ -271,11 +277,18 @@ class GroupedAttention:
                 table_len=kv.capacity, scale=self.scale, eps=self.eps, status=rows.status.data_ptr())
         if self.rot:
             a.cos, a.sin = (t.data_ptr() for t in self.tables)
-        if out is not None:
-            a.q = rows.buffer("gqa_q", n * self.heads * self.dim, self.dtype, self.device).data_ptr()
-        check(lib.gqa_rows(pointer_to(a), f32, stream()), "gqa_rows")
+        fused = self.fused and rows.plan is None and out is not None
+        if not fused:
+            if out is not None:
+                a.q = rows.buffer("gqa_q", n * self.heads * self.dim, self.dtype, self.device).data_ptr()
+            check(lib.gqa_rows(pointer_to(a), f32, stream()), "gqa_rows")
         if out is not None:
             a.out, a.ldo = out.data_ptr(), out.stride(0)
+        if out is not None and self.tiled and rows.plan is not None and rows.plan.longest >= self.TILED_FROM:
+            tiles, a.n_tiles = rows.plan.row_tiles(self.ROW_TILE)
+            a.tile_row, a.tile_rows, a.tile_pos = (tiles[i].data_ptr() for i in (0, 1, 3))
+            check(lib.gqa_prefill(pointer_to(a), stream()), "gqa_prefill")
+        elif out is not None:
             max_len = min(rows.max_len, kv.capacity)
             tiles = (max_len + GQA_TILE - 1) // GQA_TILE
             a.max_len, a.chunk_tiles = max_len, rows.chunk_tiles or self.default_chunk(n, max_len)

@@ -151,6 +151,9 @@ SIGNATURES = {
         "gqa_rows": ([c_ptr, c_int, c_ptr], c_int),
         "gqa_split": ([c_ptr, c_int, c_ptr], c_int),
         "gqa_merge": ([c_ptr, c_int, c_ptr], c_int),
+        "gqa_split_fused": ([c_int] * 2, c_int),
+        "gqa_prefill_supported": ([c_int] * 2, c_int),
+        "gqa_prefill": ([c_ptr, c_ptr], c_int),
     },
     "delta_rule": {
         "delta_step": ([c_ptr, c_int, c_ptr], c_int),
