@@ -559,7 +559,12 @@ int gqa_prefill(const ncb_gqa *args, void *stream);
  * [heads] = exp(A_log). state fp32 [n_slots][heads][dim][vdim]. Rows of a segment are consecutive, of one slot and at
  * ascending positions; a row at position 0 starts from a zero state; a segment whose first position is negative is idle.
  * out NULL: only the state is advanced.
- *   delta_step   token by token; seg_first NULL: every row is a segment; keep: also the ring (every row a slot of its own) */
+ *   delta_step    token by token; seg_first NULL: every row is a segment; keep: also the ring (every row a slot of its own)
+ *   delta_chunked bf16, rank_a and rank_g multiples of 16: segments cut into chunks of at most delta_chunk_tokens(dim) rows
+ *                 (= chunk; 0: not taken): chunk_first / chunk_count [n_chunks], seg_chunk [n_segments + 1] (a segment's first
+ *                 chunk). a2_rows bf16 [heads][dim][rank_a], g2_rows [heads][vdim][rank_g]. Scratch per (chunk, head): w_terms,
+ *                 kd_terms, q_terms bf16 [2][chunk][dim], b_terms [2][chunk][chunk], s_terms [2][vdim][dim], u_terms
+ *                 [2][vdim][chunk], u0 fp32 [vdim][chunk], chunk_decay [dim]; raw fp32 [rows][heads][vdim]. Three launches. */
 typedef struct {
     ncb_conv conv;
     void *out;
@@ -572,8 +577,15 @@ typedef struct {
     float *state;
     const int *seg_first, *seg_count;
     int n_segments;
+    const void *a2_rows, *g2_rows;
+    const int *seg_chunk, *chunk_first, *chunk_count;
+    int n_chunks, chunk;
+    void *w_terms, *kd_terms, *q_terms, *b_terms, *s_terms, *u_terms;
+    float *u0, *chunk_decay, *raw;
     int *status;
 } ncb_delta;
+int delta_chunk_tokens(int dim);
+int delta_chunked(const ncb_delta *args, void *stream);
 int delta_step(const ncb_delta *args, int f32, void *stream);
 
 /* ---- GEMMs around an fp32 residual stream (ncb_gemm_rs above) ------------------------------------------------

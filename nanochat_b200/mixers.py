@@ -305,6 +305,7 @@ class ChannelDelta:
     norm, o."""
 
     kv_from = None
+    CHUNKED_FROM = 24  # shorter segments run token by token
 
     def __init__(self, sizes: dict, tensors: dict, eps: float, columns: int, dtype: torch.dtype, device):
         H, G, D, V = (int(sizes[n]) for n in ("heads", "kv_heads", "dim", "vdim"))
@@ -315,16 +316,16 @@ class ChannelDelta:
         self.eps, self.dtype, self.device = float(eps), dtype, torch.device(device)
         t = {k: v.to(device) for k, v in tensors.items()}
         heads = [("q", G, D, self.dim), ("k", G, D, self.dim), ("v", H, V, self.vdim)]
-        fields = [padded_heads(t[n], h, d, p).to(dtype) for n, h, d, p in heads] + [t[n].to(dtype) for n in ("b", "a1", "g1")]
+        fields = [padded_heads(t[n], h, d, p).to(dtype) for n, h, d, p in heads] + [t["b"].to(dtype)] + \
+            [pad_to(t[n], up(t[n].shape[0], 16), t[n].shape[1]).to(dtype) for n in ("a1", "g1")]
         self.w_in, self.offsets = stack_fields(fields, 128, columns)
         self.conv = ShortConv([(padded_heads(t[n + ".conv"], h, d, p), at) for (n, h, d, p), at in zip(heads, self.offsets)],
                               self.offsets[3], dtype, device)
-        self.rank_a, self.rank_g = t["a1"].shape[0], t["g1"].shape[0]
-
-        def second(w: Tensor, n: int, padded: int) -> Tensor:  # [heads n, rank] -> [heads, rank, padded]
-            return pad_to(w.reshape(H, n, -1), H, padded, w.shape[1]).transpose(1, 2).contiguous().to(dtype)
-
-        self.a2, self.g2 = second(t["a2"], D, self.dim), second(t["g2"], V, self.vdim)
+        self.rank_a, self.rank_g = (up(t[n].shape[0], 16) for n in ("a1", "g1"))
+        self.a2_rows = pad_to(t["a2"].reshape(H, D, -1), H, self.dim, self.rank_a).to(dtype)
+        self.g2_rows = pad_to(t["g2"].reshape(H, V, -1), H, self.vdim, self.rank_g).to(dtype)
+        self.a2, self.g2 = (w.transpose(1, 2).contiguous() for w in (self.a2_rows, self.g2_rows))
+        self.chunk = cuda_library("delta_rule").delta_chunk_tokens(self.dim) if dtype == torch.bfloat16 else 0
         self.dt_bias = pad_to(t["dt_bias"].float().reshape(H, D), H, self.dim).contiguous()
         self.a_exp = t["A_log"].float().exp()
         self.norm = pad_to(t["norm"].float(), self.vdim)
@@ -353,8 +354,23 @@ class ChannelDelta:
         if plan is not None:
             first, count = plan.segments()
             a.seg_first, a.seg_count, a.n_segments = first.data_ptr(), count.data_ptr(), plan.n_segments
-        check(lib.delta_step(pointer_to(a), f32, stream()), "delta_step")
+        if plan is None or self.chunk == 0 or plan.longest < self.CHUNKED_FROM:
+            check(lib.delta_step(pointer_to(a), f32, stream()), "delta_step")
+        else:
+            self.run_chunked(a, rows)
         self.conv.keep_tail(a.conv, rows)
+
+    def run_chunked(self, a: Delta, rows: Rows) -> None:
+        (seg_chunk, chunk_first, chunk_count), n = rows.plan.chunks(self.chunk)
+        a.seg_chunk, a.chunk_first, a.chunk_count = seg_chunk.data_ptr(), chunk_first.data_ptr(), chunk_count.data_ptr()
+        a.n_chunks, a.chunk, a.a2_rows, a.g2_rows = n, self.chunk, self.a2_rows.data_ptr(), self.g2_rows.data_ptr()
+        C, D, V, each, bf, f = self.chunk, self.dim, self.vdim, n * self.heads, torch.bfloat16, torch.float32
+        for name, size, kind in (("w_terms", 2 * C * D, bf), ("kd_terms", 2 * C * D, bf), ("q_terms", 2 * C * D, bf), ("b_terms", 2 * C * C, bf),
+                                 ("s_terms", 2 * V * D, bf), ("u_terms", 2 * V * C, bf), ("u0", V * C, f), ("chunk_decay", D, f)):
+            setattr(a, name, rows.buffer("delta_" + name, each * size, kind, self.device).data_ptr())
+        # values beyond one tile of the output kernel pass through memory for the norm
+        a.raw = rows.buffer("delta_raw", rows.n * self.heads * V if V > 128 else 4, f, self.device).data_ptr()
+        check(cuda_library("delta_rule").delta_chunked(pointer_to(a), stream()), "delta_chunked")
 
 
 class GatedLinearAttention:

@@ -121,7 +121,7 @@ def test_a_key_that_stands_out_is_found_wherever_it_lies(dtype, mode):
     """One earlier row's key is made to dominate a later row's score: the query's projection is the key's with its columns
     rolled, and the later row's inputs (over all taps) are the earlier row's, rolled as well, so that the two meet and the later
     row's own key does not. At tile, page and chunk borders, first and last positions."""
-    entry = cases.attention(heads=4, kv_heads=2, dim=32, vdim=32, conv=2, rot_dims=16, scale=3.0, base=1e6, scaling=None)
+    entry = cases.attention(heads=4, kv_heads=2, dim=32, vdim=32, conv=2, rot_dims=16, scale=1.2, base=1e6, scaling=None)
     C, n = 64, 200
     state = cases.random_state(cases.config([entry], width=C), 17)
     for name, size in (("", C), (".conv", 2)):
