@@ -619,8 +619,8 @@ def bench_decoder_d32(rank: int, world: int, device, new_tokens: int, profile: b
 
 
 HYBRID_SIZES = {  # equal layers, width and parameters as the closest model of the same name
-    "d20": {"width": 1280, "layers": 20, "heads": 10, "gla_heads": 5, "ff": 3072, "batch": 8, "plain_ff": 5120, "kv_heads": 10},
-    "d32": {"width": 2048, "layers": 32, "heads": 16, "gla_heads": 8, "ff": 4096, "batch": 32, "plain_ff": 8192, "kv_heads": 4}}
+    "d20": {"width": 1280, "layers": 20, "heads": 10, "gla_heads": 5, "ff": 3072, "batch": 8, "plain_ff": 5120, "kv_heads": 10, "silu_ff": 3072},
+    "d32": {"width": 2048, "layers": 32, "heads": 16, "gla_heads": 8, "ff": 4096, "batch": 32, "plain_ff": 8192, "kv_heads": 4, "silu_ff": 5376}}
 
 
 def hybrid_config(size: dict, max_len: int):
@@ -636,8 +636,27 @@ def hybrid_config(size: dict, max_len: int):
                                       "residual_mult": 0.2, "logit_scale": 0.1}, max_len)
 
 
-def bench_hybrid(device, new_tokens: int = 128, profile: str = "") -> dict:
-    """Prefill and decode throughput of Pudisun at two sizes beside this package's other model at equal width, depth and
+def rekudra_config(size: dict, max_len: int):
+    """A Rekudra model of real layer sizes: delta-rule and attention layers in turn, each with a feed-forward, two streams; every
+    second attention layer reads the keys and values of the one before."""
+    from nanochat_b200.hybrid import HybridConfig
+
+    rot = {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "high": 4.0, "low": 1.0, "original": 8192}}
+    heads = {"conv": 4, "dim": 128, "heads": size["heads"], "kv_heads": size["kv_heads"], "vdim": 128}
+    layers = []
+    for i in range(size["layers"]):
+        mixer = dict(heads)
+        if i % 2:
+            mixer.update(rot=rot, scale=128 ** -0.5)
+            if i % 4 == 3:
+                mixer["kv_from"] = i - 2
+        layers.append({"type": "attention" if i % 2 else "channel_delta", "mixer": mixer, "mlp": {"ff": size["silu_ff"], "kind": "dense"}})
+    return HybridConfig.from_rekudra({"layers": layers, "width": size["width"], "vocab": 65536, "norm": {"eps": 1e-6}, "streams": 2,
+                                      "embedding": {"scale": 1.0}}, max_len)
+
+
+def bench_hybrid(device, new_tokens: int = 128, profile: str = "", model_name: str = "pudisun") -> dict:
+    """Prefill and decode throughput of Pudisun or Rekudra at two sizes beside this package's other model at equal width, depth and
     parameter count (random weights, one GPU, device time between CUDA events): prefill of 8 x 511 rows, and decode of the
     size's batch at contexts of 512 (d20) or uniform in [256, 8192] (d32; caches and states hold synthetic rows). `profile`
     ("d20-prefill", "d20-decode", ...) brackets one pass or one step with cudaProfilerStart/Stop."""
@@ -665,8 +684,9 @@ def bench_hybrid(device, new_tokens: int = 128, profile: str = "") -> dict:
             torch.cuda.synchronize()
             torch.cuda.profiler.stop()
 
+    kernels = bench_rekudra_kernels if model_name == "rekudra" else bench_hybrid_kernels
     if profile == "kernels":
-        return {"kernels": bench_hybrid_kernels(device, profiled=True)}
+        return {"kernels": kernels(device, profiled=True)}
     result = {}
     for name, size in HYBRID_SIZES.items():
         if profile and not profile.startswith(name):
@@ -677,11 +697,11 @@ def bench_hybrid(device, new_tokens: int = 128, profile: str = "") -> dict:
         max_len = max(max(ctx), 511) + new_tokens + 8
         prompts = torch.randint(0, 65536, (8, 512), generator=gen).tolist()
         first = torch.randint(0, 65536, (B,), generator=gen).tolist()
-        hybrid = hybrid_config(size, max_len)
+        hybrid = (rekudra_config if model_name == "rekudra" else hybrid_config)(size, max_len)
         plain = DecoderConfig(n_layers=size["layers"], hidden=size["width"], n_heads=size["heads"], n_kv_heads=size["kv_heads"],
                               intermediate=size["plain_ff"], vocab=65536, rope_theta=10000.0, max_len=max_len)
 
-        def pudisun():
+        def mixed():
             return HybridDecoder(hybrid, HybridWeights.from_state_dict(HybridWeights.random_state(hybrid, 2, device), hybrid,
                                                                        device=device), B, device)
 
@@ -690,7 +710,7 @@ def bench_hybrid(device, new_tokens: int = 128, profile: str = "") -> dict:
 
         row = {"workload": f"{size['layers']} layers, width {size['width']}, vocab 65536; prefill 8 x 511 rows; decode batch {B}, "
                            + ("context 512" if name == "d20" else "contexts uniform in [256, 8192]")}
-        for model, make in (("pudisun", pudisun), ("nanochat", nanochat)):
+        for model, make in ((model_name, mixed), ("nanochat", nanochat)):
             if profile and model == "nanochat":
                 continue
             dec = make()
@@ -699,8 +719,9 @@ def bench_hybrid(device, new_tokens: int = 128, profile: str = "") -> dict:
             prefill_ms = elapsed(lambda: dec.prefill(prompts, list(range(8))), REPEATS)
             if name != "d20":  # synthetic cache rows for the long contexts
                 for cache in dec.caches:
-                    if hasattr(cache, "rows"):
-                        cache.rows.normal_()
+                    for one in getattr(cache, "parts", [cache]):
+                        if hasattr(one, "rows"):
+                            one.rows.normal_()
             dec.decode_from(first, ctx, 4)
             if profile == f"{name}-decode":
                 dec.decode_from(first, ctx, 1)
@@ -716,7 +737,7 @@ def bench_hybrid(device, new_tokens: int = 128, profile: str = "") -> dict:
             torch.cuda.empty_cache()
         result[name] = row
     if not profile:
-        result["kernels"] = bench_hybrid_kernels(device)
+        result["kernels"] = kernels(device)
     return result
 
 
@@ -727,7 +748,8 @@ def weight_bytes(dec) -> int:
     total = dec.w.embed.numel() * 2
     for l in dec.w.layers:
         total += 2 * sum(t.numel() for t in (l.mixer.w_in, l.mixer.w_out, l.w_up, l.w_down))
-        total += 2 * sum(getattr(l.mixer, n).numel() for n in ("w_uk_t", "w_uv") if hasattr(l.mixer, n))
+        low_rank = ("w_uk_t", "w_uv", *(("a2", "g2") if hasattr(l.mixer, "g2") else ()))
+        total += 2 * sum(getattr(l.mixer, n).numel() for n in low_rank if hasattr(l.mixer, n))
     return total
 
 
@@ -736,13 +758,79 @@ def cache_bytes_read(dec, ctx, new_tokens: int) -> int:
     positions = sum(n + new_tokens // 2 for n in ctx)
     total = 0
     for cache in dec.caches:
-        if hasattr(cache, "state"):
-            total += 2 * len(ctx) * cache.state[0].numel() * 4
+        if hasattr(cache, "kv"):
+            total += positions * cache.kv.kv_heads * cache.kv.width * 2
+        elif hasattr(cache, "state"):
+            state = getattr(cache.state, "state", cache.state)
+            total += 2 * len(ctx) * state[0].numel() * 4
         elif hasattr(cache, "rows"):
             total += positions * cache.width * 2
         else:
             total += positions * cache.kv_heads * 264
     return total
+
+
+def graph_time(fn, calls: int, profiled: bool = False) -> float:
+    """Microseconds per call of `calls` calls fn(i) captured in one graph (host launch costs left out), median of REPEATS.
+    profiled: one call between cudaProfilerStart and Stop instead."""
+    if profiled:
+        fn(0)
+        torch.cuda.synchronize()
+        torch.cuda.profiler.start()
+        fn(1)
+        torch.cuda.synchronize()
+        torch.cuda.profiler.stop()
+        return 1.0
+    side = torch.cuda.Stream()
+    side.wait_stream(torch.cuda.current_stream())
+    with torch.cuda.stream(side):
+        for i in range(3):
+            fn(i)
+        side.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph, stream=side):
+            for i in range(calls):
+                fn(i)
+    times = []
+    for _ in range(REPEATS + 1):
+        start, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        start.record()
+        graph.replay()
+        end.record()
+        torch.cuda.synchronize()
+        times.append(start.elapsed_time(end) * 1e3 / calls)
+    return statistics.median(times[1:])
+
+
+def spy(lib: str, fn, wanted) -> dict:
+    """The argument structures that `fn` passes to the entry points `wanted` of a mixers' library, by name."""
+    import ctypes
+
+    import nanochat_b200.mixers as module
+
+    original = module.cuda_library
+    seen, real = {}, original(lib)
+
+    class Recorder:
+        def __getattr__(self, name):
+            entry = getattr(real, name)
+            if name not in wanted:
+                return entry
+
+            def call(args, *rest):
+                copy = type(args._obj)()
+                ctypes.memmove(ctypes.byref(copy), ctypes.byref(args._obj), ctypes.sizeof(copy))
+                seen[name] = copy
+                return entry(args, *rest)
+            return call
+
+    module.cuda_library = lambda name: Recorder() if name == lib else original(name)
+    try:
+        fn()
+    finally:
+        module.cuda_library = original
+    return seen
 
 
 def bench_hybrid_kernels(device, profiled: bool = False) -> dict:
@@ -752,7 +840,7 @@ def bench_hybrid_kernels(device, profiled: bool = False) -> dict:
     import ctypes
 
     from nanochat_b200.mixers import GatedLinearAttention, LatentAttention, RowPlan, Rows
-    from nanochat_b200.native import Gla, Latent, cuda_library, stream
+    from nanochat_b200.native import cuda_library, stream
 
     hbm, _ = peaks()
     tensor = 1610.8
@@ -761,62 +849,7 @@ def bench_hybrid_kernels(device, profiled: bool = False) -> dict:
     status = torch.zeros(1, dtype=torch.int32, device=device)
 
     def per_call(fn, calls: int) -> float:
-        """Microseconds per call of `calls` calls captured in one graph (host launch costs left out), median of REPEATS."""
-        if profiled:
-            fn(0)
-            torch.cuda.synchronize()
-            torch.cuda.profiler.start()
-            fn(1)
-            torch.cuda.synchronize()
-            torch.cuda.profiler.stop()
-            return 1.0
-        side = torch.cuda.Stream()
-        side.wait_stream(torch.cuda.current_stream())
-        with torch.cuda.stream(side):
-            for i in range(3):
-                fn(i)
-            side.synchronize()
-            graph = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(graph, stream=side):
-                for i in range(calls):
-                    fn(i)
-        times = []
-        for _ in range(REPEATS + 1):
-            start, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            torch.cuda.synchronize()
-            start.record()
-            graph.replay()
-            end.record()
-            torch.cuda.synchronize()
-            times.append(start.elapsed_time(end) * 1e3 / calls)
-        return statistics.median(times[1:])
-
-    def spy(lib, fn, wanted):
-        """The argument structures `fn` passes to the entry points `wanted`, by name."""
-        seen, real = {}, cuda_library(lib)
-
-        class Recorder:
-            def __getattr__(self, name):
-                entry = getattr(real, name)
-                if name not in wanted:
-                    return entry
-
-                def call(args, *rest):
-                    kind = Latent if lib == "latent_attn" else Gla
-                    copy = kind()
-                    ctypes.memmove(ctypes.byref(copy), ctypes.byref(args._obj), ctypes.sizeof(kind))
-                    seen[name] = copy
-                    return entry(args, *rest)
-                return call
-
-        import nanochat_b200.mixers as module
-        original = module.cuda_library
-        module.cuda_library = lambda name: Recorder() if name == lib else original(name)
-        try:
-            fn()
-        finally:
-            module.cuda_library = original
-        return seen
+        return graph_time(fn, calls, profiled)
 
     out = {}
     gen = torch.Generator(device=device).manual_seed(900)
@@ -945,6 +978,158 @@ def bench_hybrid_kernels(device, profiled: bool = False) -> dict:
     return out
 
 
+def bench_rekudra_kernels(device, profiled: bool = False) -> dict:
+    """Rekudra's kernels alone at the d20 and d32 sizes, as bench_hybrid_kernels, and the closest model's beside them."""
+    import ctypes
+
+    import numpy as np
+
+    import nanochat_b200 as ncb
+    from nanochat_b200 import attention as ops
+    from nanochat_b200.hybrid import HybridConfig, HybridWeights, HyperConnection
+    from nanochat_b200.mixers import RowPlan, Rows
+    from nanochat_b200.native import GemmRs, cuda_library, pointer, stream
+
+    hbm, _ = peaks()
+    tensor = 1610.8
+    if (ROOT / "MEASURED_PEAKS.json").exists():
+        tensor = float(json.loads((ROOT / "MEASURED_PEAKS.json").read_text())["bf16_tflops"])
+    status = torch.zeros(1, dtype=torch.int32, device=device)
+    out = {}
+
+    def per_call(fn, calls):
+        return graph_time(fn, calls, profiled)
+
+    def moved(name, us, nbytes):
+        out[name] = {"us": us, "bytes": nbytes, "gbs": nbytes / us / 1e3, "frac_hbm": nbytes / us / 1e3 / hbm}
+
+    def multiplied(name, us, flops):
+        out[name] = {"us": us, "flops": flops, "tflops": flops / us / 1e6, "frac_tensor": flops / us / 1e6 / tensor}
+
+    gen = torch.Generator(device=device).manual_seed(900)
+    for name, size in HYBRID_SIZES.items():
+        if profiled and name != "d32":
+            continue
+        B, C, H, G = size["batch"], size["width"], size["heads"], size["kv_heads"]
+        cgen = torch.Generator().manual_seed(400)
+        ctx = [576] * B if name == "d20" else torch.randint(256, 8193, (B,), generator=cgen).tolist()
+        cfg = rekudra_config(size, max(ctx) + 8)
+        one = HybridConfig(C, 128, cfg.layers[:2], 1e-6, streams=2, tied_head=False, norm_base=1.0)
+        layers = HybridWeights.from_state_dict(HybridWeights.random_state(one, 3, device), one, device=device).layers
+        delta, attn = layers[0].mixer, layers[1].mixer
+        pos = torch.tensor([n - 1 for n in ctx], dtype=torch.int32, device=device)
+        slots = torch.arange(B, dtype=torch.int32, device=device)
+        # ---- decode
+        row_bytes = G * 256 * 2
+        copies = max(2, int(400e6 // (sum(ctx) * row_bytes)) + 1)
+        caches = [attn.new_cache(B, max(ctx)) for _ in range(copies)]
+        for c in caches:
+            c.kv.rows.normal_(generator=gen)
+        proj = torch.randn(B, attn.in_width, generator=gen, device=device).bfloat16()
+        mixed = torch.empty(B, attn.out_width, dtype=torch.bfloat16, device=device)
+        rows = Rows(B, pos, slots, max(ctx), status, chunk_tiles=attn.chunk_for(ctx, max(ctx)))
+        seen = spy("gqa_attn", lambda: attn.run(proj, caches[0], rows, mixed), ("gqa_split", "gqa_merge"))
+        lib = cuda_library("gqa_attn")
+
+        def launch(entry, i):
+            a = seen[entry]
+            a.kv = caches[i % copies].kv.rows.data_ptr()
+            assert getattr(lib, entry)(ctypes.byref(a), 0, stream()) == 0
+
+        nbytes = sum(ctx) * row_bytes + proj.numel() * 2
+        moved(f"{name} gqa_split", per_call(lambda i: launch("gqa_split", i), 40), nbytes)
+        out[f"{name} gqa_split"]["chunk_tiles"] = seen["gqa_split"].chunk_tiles
+        moved(f"{name} gqa_merge", per_call(lambda i: launch("gqa_merge", i), 40),
+              B * H * seen["gqa_merge"].max_chunks * 132 * 4 + mixed.numel() * 2)
+        if not profiled:
+            moved(f"{name} gqa_split + merge", per_call(lambda i: (launch("gqa_split", i), launch("gqa_merge", i)), 40), nbytes)
+        del caches
+        states = [delta.new_cache(B, 64) for _ in range(max(2, int(300e6 // (B * H * 128 * 128 * 4)) + 1))]
+        proj = torch.randn(B, delta.in_width, generator=gen, device=device).bfloat16()
+        mixed = torch.empty(B, delta.out_width, dtype=torch.bfloat16, device=device)
+        moved(f"{name} delta_step", per_call(lambda i: delta.run(proj, states[i % len(states)], rows, mixed), 40),
+              2 * states[0].state.state.numel() * 4 + (proj.numel() + mixed.numel() + delta.a2.numel() + delta.g2.numel()) * 2)
+        del states
+        # ---- prefill: 8 prompts of 511 rows, and one of 4,088
+        for label, prompts, n in (("", 8, 511), (" one prompt", 1, 4088)):
+            if profiled and label:
+                continue
+            host = np.repeat(np.arange(prompts, dtype=np.int32), n), np.tile(np.arange(n, dtype=np.int32), prompts)
+            pos_p, slots_p = torch.from_numpy(host[1]).to(device), torch.from_numpy(host[0]).to(device)
+            rows = Rows(n * prompts, pos_p, slots_p, n, status, RowPlan(*host, device))
+            cache = attn.new_cache(prompts, n)
+            proj = torch.randn(n * prompts, attn.in_width, generator=gen, device=device).bfloat16()
+            mixed = torch.empty(n * prompts, attn.out_width, dtype=torch.bfloat16, device=device)
+            seen = spy("gqa_attn", lambda: attn.run(proj, cache, rows, mixed), ("gqa_rows", "gqa_prefill"))
+            us = per_call(lambda i: lib.gqa_prefill(ctypes.byref(seen["gqa_prefill"]), stream()), 20)
+            multiplied(f"{name} gqa_prefill{label}", us, prompts * n * (n + 1) // 2 * H * 2 * 256)
+            us = per_call(lambda i: lib.gqa_rows(ctypes.byref(seen["gqa_rows"]), 0, stream()), 20)
+            moved(f"{name} gqa_rows{label}", us, 2 * 2 * n * prompts * (H * 128 + G * 256))
+            state = delta.new_cache(prompts, 64)
+            proj = torch.randn(n * prompts, delta.in_width, generator=gen, device=device).bfloat16()
+            mixed = torch.empty(n * prompts, delta.out_width, dtype=torch.bfloat16, device=device)
+            us = per_call(lambda i: delta.run(proj, state, rows, mixed), 20)
+            moved(f"{name} delta_chunked{label}", us, (proj.numel() + mixed.numel()) * 2 + 2 * state.state.state.numel() * 4)
+            out[f"{name} delta_chunked{label}"]["note"] = "three launches and the rings'"
+        # ---- the streams' update beside the closest model's residual, and its attention kernels
+        rows_n = n * prompts
+        hc = HyperConnection.of(torch.ones(2), torch.ones(2), torch.full((2, 2), 0.5))
+        h = torch.randn(rows_n, 2, C, generator=gen, device=device)
+        gain, x_next = torch.ones(C, device=device), torch.empty(rows_n, C, dtype=torch.bfloat16, device=device)
+        ss = torch.empty(rows_n, C // 8, device=device)
+        for what, K, N, epilogue in (("o", attn.out_width, C, 7), ("down", size["silu_ff"], C, 7), ("gate / up", C, 2 * size["silu_ff"], 8)):
+            x = torch.randn(rows_n, K, generator=gen, device=device).bfloat16()
+            w = (torch.randn(N, K, generator=gen, device=device) * 0.02).bfloat16()
+            y = torch.empty(rows_n, N, dtype=torch.bfloat16, device=device)
+            a = GemmRs(x=x.data_ptr(), w=w.data_ptr(), y=y.data_ptr(), ldy=N // 2 if epilogue == 8 else N, rows=rows_n, N=N, K=K, n_store=N,
+                       epilogue=epilogue, scale=1.0, h=h.data_ptr(), gain=gain.data_ptr(), x_next=x_next.data_ptr(), ss_next=ss.data_ptr(),
+                       status=status.data_ptr(), streams=2, in_=hc.read, out=hc.write, mix=hc.mix)
+            us = per_call(lambda i: cuda_library("tile_gemm").tile_gemm_rs(ctypes.byref(a), stream()), 20)
+            multiplied(f"{name} tile_gemm {what}, " + ("two streams" if epilogue == 7 else "silu gate"), us, 2 * rows_n * N * K)
+            if profiled:
+                continue
+            us = per_call(lambda i: cuda_library("tile_gemm").tile_gemm(pointer(x), pointer(w), pointer(y) if epilogue == 7 else None, pointer(y),
+                                                                        rows_n, N, K, 1 if epilogue == 7 else 2, pointer(status), stream()), 20)
+            multiplied(f"{name} tile_gemm {what}, " + ("bf16 residual" if epilogue == 7 else "relu^2"), us, 2 * rows_n * N * K)
+            a.rows = B
+            entry = ("decode_step", "skinny_gemm") if B <= 16 else ("stream_gemm", "stream_gemm")
+            us = per_call(lambda i: getattr(cuda_library(entry[0]), entry[1] + "_rs")(ctypes.byref(a), stream()), 40)
+            moved(f"{name} {entry[1]} {what}, " + ("two streams" if epilogue == 7 else "silu gate"), us, N * K * 2)
+            if B <= 16:
+                call = lambda i: cuda_library("decode_step").skinny_gemm(  # noqa: E731
+                    pointer(x), pointer(w), pointer(y) if epilogue == 7 else None, pointer(y), B, N, K, 0, 1 if epilogue == 7 else 2, stream())
+            else:
+                call = lambda i: cuda_library("stream_gemm").stream_gemm(  # noqa: E731
+                    pointer(x), pointer(w), pointer(y) if epilogue == 7 else None, pointer(y), B, N, K, 0, 1 if epilogue == 7 else 2, 0, None, 0,
+                    pointer(status), stream())
+            moved(f"{name} {entry[1]} {what}, " + ("bf16 residual" if epilogue == 7 else "relu^2"), per_call(call, 40), N * K * 2)
+        if not profiled:
+            kv = [ncb.Fp8KVCache(B, G, max(ctx), device=device) for _ in range(copies)]
+            for c in kv:  # random finite bytes below the e4m3 NaN, small scales
+                c.pages.random_(0, 100, generator=gen)
+                c.pages.view(B, G, -1, 16896)[..., 16384:].view(torch.float32).fill_(0.01)
+            q = torch.randn(B, H, D, generator=gen, device=device).bfloat16()
+            lens_t = torch.tensor(ctx, dtype=torch.int32, device=device)
+            chunk = ops.plan_chunk_pages(ctx, G, max(ctx))
+            work = torch.empty(max(ops.workspace_bytes(B, H, G, max(ctx), chunk), 16), dtype=torch.uint8, device=device)
+            att = torch.empty_like(q)
+            us = per_call(lambda i: ops.decode_attention(q, kv[i % copies], lens_t, max(ctx), chunk_pages=chunk, workspace=work, out=att,
+                                                         status=status), 40)
+            moved(f"{name} nanochat decode_attn + merge", us, sum(ctx) * G * 264 + B * H * 512)
+            for label, prompts, n in (("", 8, 511), (" one prompt", 1, 4088)):
+                host = np.repeat(np.arange(prompts, dtype=np.int32), n), np.tile(np.arange(n, dtype=np.int32), prompts)
+                pkv = ncb.Fp8KVCache(prompts, G, n, device=device)
+                pkv.pages.zero_()
+                q = torch.randn(n * prompts, H, D, generator=gen, device=device).bfloat16()
+                plan, att = ops.PrefillPlan(*host, H, pkv, device), torch.empty_like(q)
+                us = per_call(lambda i: ops.prefill_attention(q, pkv, plan, out=att, status=status), 20)
+                multiplied(f"{name} nanochat prefill_attn{label}", us, prompts * n * (n + 1) // 2 * H * 4 * D)
+            del kv
+        assert int(status.item()) == 0
+        torch.cuda.empty_cache()
+    return out
+
+
 def pin_to_local_cores(local: int, world: int) -> str:
     """With several ranks on one host, give each rank its own slice of the cores this process may use, taken from the
     NUMA node its GPU hangs off when sysfs tells (else an even slice): the end-to-end loop is driven by the host (one
@@ -1063,8 +1248,9 @@ def main() -> None:
     ap.add_argument("--longctx", type=int, default=1, help="also time the KV-length-sharded long-context case (0: skip)")
     ap.add_argument("--e2e-steps", type=int, default=200, help="steps of the end-to-end loop (profiling runs shrink it)")
     ap.add_argument("--e2e-parts", type=int, default=0, help="row groups of the end-to-end step that run as parallel graph branches (0: DecodeStep's choice)")
-    ap.add_argument("--hybrid", type=int, default=0, help="also time Pudisun's prefill, decode and kernels beside the closest model "
+    ap.add_argument("--hybrid", type=int, default=0, help="also time a mixed-layer model's prefill, decode and kernels beside the closest model "
                     "(N = 1); 2: print only that")
+    ap.add_argument("--hybrid-model", default="pudisun", choices=["pudisun", "rekudra"], help="the model that --hybrid times")
     ap.add_argument("--hybrid-profile", default="", help="bracket one pass or step of that for ncu: d20-prefill, d20-decode, d32-..., or one "
                     "launch of each d32 kernel: kernels")
     args = ap.parse_args()
@@ -1091,7 +1277,7 @@ def main() -> None:
 
     if args.hybrid == 2 and world == 1:
         with ClockSampler(local) as clocks:
-            result = bench_hybrid(device, profile=args.hybrid_profile)
+            result = bench_hybrid(device, profile=args.hybrid_profile, model_name=args.hybrid_model)
         print(json.dumps({"hybrid": result, "clocks": clocks.summary()}))
         return
 
@@ -1248,7 +1434,7 @@ def main() -> None:
     decoder_d32 = bench_decoder_d32(rank, world, device, 2 if d32_profiled else 128, d32_profiled) \
         if args.decoder_d32 else None
 
-    hybrid = bench_hybrid(device) if args.hybrid and world == 1 else None
+    hybrid = bench_hybrid(device, model_name=args.hybrid_model) if args.hybrid and world == 1 else None
 
     if rank == 0:
         value = head["total_bytes"] / (head["ms_step"] * 1e-3) / 1e9

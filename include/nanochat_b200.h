@@ -560,11 +560,11 @@ int gqa_prefill(const ncb_gqa *args, void *stream);
  * ascending positions; a row at position 0 starts from a zero state; a segment whose first position is negative is idle.
  * out NULL: only the state is advanced.
  *   delta_step    token by token; seg_first NULL: every row is a segment; keep: also the ring (every row a slot of its own)
- *   delta_chunked bf16, rank_a and rank_g multiples of 16: segments cut into chunks of at most delta_chunk_tokens(dim) rows
- *                 (= chunk; 0: not taken): chunk_first / chunk_count [n_chunks], seg_chunk [n_segments + 1] (a segment's first
- *                 chunk). a2_rows bf16 [heads][dim][rank_a], g2_rows [heads][vdim][rank_g]. Scratch per (chunk, head): w_terms,
- *                 kd_terms, q_terms bf16 [2][chunk][dim], b_terms [2][chunk][chunk], s_terms [2][vdim][dim], u_terms
- *                 [2][vdim][chunk], u0 fp32 [vdim][chunk], chunk_decay [dim]; raw fp32 [rows][heads][vdim]. Three launches. */
+ *   delta_chunked bf16, rank_a and rank_g multiples of 16: segments cut into chunks of at most delta_chunk_tokens() rows
+ *                 (= chunk; 0: not taken): chunk_first / chunk_count [n_chunks], chunk_within [n_chunks] (rows of the segment
+ *                 before the chunk), seg_chunk [n_segments + 1] (a segment's first chunk). a2_rows bf16 [heads][dim][rank_a], g2_rows [heads][vdim][rank_g]. Scratch per (chunk, head): w_terms,
+ *                 kd_terms, q_terms bf16 [2][chunk][dim + 8], b_terms [2][chunk][chunk + 8], s_terms [2][vdim][dim + 8], u_terms
+ *                 [2][vdim][chunk + 8], u0 fp32 [vdim][chunk + 4], chunk_decay [dim]; raw fp32 [rows][heads][vdim]. Three launches. */
 typedef struct {
     ncb_conv conv;
     void *out;
@@ -578,13 +578,13 @@ typedef struct {
     const int *seg_first, *seg_count;
     int n_segments;
     const void *a2_rows, *g2_rows;
-    const int *seg_chunk, *chunk_first, *chunk_count;
+    const int *seg_chunk, *chunk_first, *chunk_count, *chunk_within;
     int n_chunks, chunk;
     void *w_terms, *kd_terms, *q_terms, *b_terms, *s_terms, *u_terms;
     float *u0, *chunk_decay, *raw;
     int *status;
 } ncb_delta;
-int delta_chunk_tokens(int dim);
+int delta_chunk_tokens(int dim, int vdim, int taps, int rank_a, int rank_g);
 int delta_chunked(const ncb_delta *args, void *stream);
 int delta_step(const ncb_delta *args, int f32, void *stream);
 

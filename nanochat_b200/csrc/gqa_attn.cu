@@ -76,33 +76,72 @@ template <typename T> __device__ __forceinline__ void head_row(const ncb_gqa &a,
     for (int i = 2 * lane; i < a.dim; i += 64) store2(out + i, x[i] * r, x[i + 1] * r);
 }
 
-/* Grid (units / 4 rounded up, rows), a warp per unit of a row: the query heads, then with own_kv the key and the value heads.
- * q NULL: the query heads only keep their ring. */
+constexpr int RUN = 8; /* consecutive rows a warp of k_gqa_rows works on */
+
+/* Grid (units / 4 rounded up, rows / RUN rounded up), a warp per unit and run of rows: the query heads, then with own_kv the key
+ * and the value heads. q NULL: the query heads only keep their ring. */
 template <typename T> __global__ void __launch_bounds__(THREADS) k_gqa_rows(const ncb_gqa a) {
-    extern __shared__ float sm[];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, unit = blockIdx.x * (THREADS / 32) + warp, row = blockIdx.y;
-    const int H = a.heads, G = a.own_kv ? a.kv_heads : 0;
+    extern __shared__ float sm[]; /* [warps][RUN][dim], then the rows' places */
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, unit = blockIdx.x * (THREADS / 32) + warp;
+    const int H = a.heads, G = a.own_kv ? a.kv_heads : 0, row0 = blockIdx.y * RUN, n = (int)min((long long)RUN, a.conv.rows - row0);
+    Place *place = reinterpret_cast<Place *>(sm + (THREADS / 32) * RUN * a.dim) + warp * RUN;
     asm volatile("griddepcontrol.wait;" ::: "memory");
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     if (unit >= H + 2 * G) return;
-    int slot;
-    const int len = length_of(a, row, slot);
-    if (len == 0) return;
-    const Place at = place_of(a.conv, row);
-    float *x = sm + warp * a.dim;
-    if (unit < H) {
-        if (a.q) head_row<T>(a, row, at, a.off_q + unit * a.dim, x, (T *)a.q + ((size_t)row * H + unit) * a.dim, lane);
-        else if (a.keep)
-            for (int i = 2 * lane; i < a.dim; i += 64) keep2<T>(a.conv, row, at, a.off_q + unit * a.dim + i);
-    } else if (unit < H + G) {
-        head_row<T>(a, row, at, a.off_k + (unit - H) * a.dim, x, cache_row<T>(a, slot, unit - H, len - 1), lane);
-    } else {
-        const int g = unit - H - G, ch0 = a.off_v + g * a.vdim;
-        T *out = cache_row<T>(a, slot, g, len - 1) + a.dim;
-        for (int i = 2 * lane; i < a.vdim; i += 64) {
-            const float2 v = conv2<T>(a.conv, row, at, ch0 + i);
-            store2(out + i, v.x, v.y);
-            if (a.keep) keep2<T>(a.conv, row, at, ch0 + i);
+    if (lane < n) {
+        int slot;
+        const int len = length_of(a, row0 + lane, slot);
+        place[lane] = len ? place_of(a.conv, row0 + lane) : Place{-1, 0, 0};
+    }
+    __syncwarp();
+    const bool query = unit < H, key = !query && unit < H + G;
+    const int kvh = query ? 0 : key ? unit - H : unit - H - G, size = query || key ? a.dim : a.vdim;
+    const int ch0 = query ? a.off_q + unit * a.dim : key ? a.off_k + kvh * a.dim : a.off_v + kvh * a.vdim;
+    if (a.keep)
+        for (int r = 0; r < n; r++)
+            if (place[r].pos >= 0)
+                for (int i = 2 * lane; i < size; i += 64) keep2<T>(a.conv, row0 + r, place[r], ch0 + i);
+    if (query && !a.q) return;
+    float *x = sm + warp * RUN * a.dim;
+    for (int i = 2 * lane; i < size; i += 64) {
+        conv_run<T, RUN>(a.conv, row0, n, place, ch0 + i, [&](int r, float2 y) {
+            if (query || key) *reinterpret_cast<float2 *>(x + r * a.dim + i) = y;
+            else if (r < n && place[r].pos >= 0) store2(cache_row<T>(a, place[r].slot, kvh, place[r].pos) + a.dim + i, y.x, y.y);
+        });
+    }
+    if (!query && !key) return;
+    __syncwarp();
+    const int half = a.rot / 2;
+    for (int i = lane; i < half; i += 32) { /* in place: a pair belongs to one lane */
+        float c[RUN], s[RUN];
+#pragma unroll
+        for (int r = 0; r < RUN; r++) {
+            const size_t at = (size_t)(r < n && place[r].pos >= 0 ? place[r].pos : 0) * half + i;
+            c[r] = a.cos[at], s[r] = a.sin[at];
+        }
+#pragma unroll
+        for (int r = 0; r < RUN; r++) {
+            float *p = x + r * a.dim + i;
+            const float u = p[0], v = p[half];
+            p[0] = u * c[r] - v * s[r];
+            p[half] = v * c[r] + u * s[r];
+        }
+    }
+    __syncwarp();
+#pragma unroll
+    for (int r = 0; r < RUN; r++) {
+        float sum = 0.f;
+        for (int i = 2 * lane; i < a.dim; i += 64) {
+            const float2 v = *reinterpret_cast<const float2 *>(x + r * a.dim + i);
+            sum = fmaf(v.x, v.x, fmaf(v.y, v.y, sum));
+        }
+        for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+        if (r >= n || place[r].pos < 0) continue;
+        const float f = 1.f / sqrtf(sum / (float)a.norm_count + a.eps);
+        T *out = query ? (T *)a.q + ((size_t)(row0 + r) * H + unit) * a.dim : cache_row<T>(a, place[r].slot, kvh, place[r].pos);
+        for (int i = 2 * lane; i < a.dim; i += 64) {
+            const float2 v = *reinterpret_cast<const float2 *>(x + r * a.dim + i);
+            store2(out + i, v.x * f, v.y * f);
         }
     }
 }
@@ -180,11 +219,6 @@ __device__ __forceinline__ void ldsm4_t(uint32_t *r, uint32_t addr) {
 }
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void *src, bool on) { /* 16 bytes, zeros when off */
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
-}
-/* A contiguous run of global memory into shared memory; 16-byte aligned, a multiple of 16 bytes. */
-__device__ __forceinline__ void bulk_load(uint32_t dst, const void *src, uint32_t bytes, uint32_t bar) {
-    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-                 ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
 }
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
@@ -636,11 +670,10 @@ int gqa_rows(const ncb_gqa *g, int f32, void *stream) {
     if (!g) return NCB_ERR_ARG;
     const int rc = check(*g);
     if (rc != NCB_OK || g->conv.rows == 0) return rc;
-    if (g->conv.rows > 65535) return NCB_ERR_ARG;
-    const size_t smem = (size_t)(THREADS / 32) * g->dim * 4;
+    const size_t smem = (size_t)(THREADS / 32) * RUN * (g->dim * 4 + sizeof(Place));
     if (smem > 200 * 1024) return NCB_ERR_UNSUPPORTED;
     const int units = g->heads + (g->own_kv ? 2 * g->kv_heads : 0);
-    const dim3 grid((units + THREADS / 32 - 1) / (THREADS / 32), (unsigned)g->conv.rows);
+    const dim3 grid((units + THREADS / 32 - 1) / (THREADS / 32), (unsigned)((g->conv.rows + RUN - 1) / RUN));
     return f32 ? launch(k_gqa_rows<float>, grid, THREADS, smem, 1, (cudaStream_t)stream, *g)
                : launch(k_gqa_rows<bf16>, grid, THREADS, smem, 1, (cudaStream_t)stream, *g);
 }

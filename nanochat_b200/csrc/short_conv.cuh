@@ -35,19 +35,62 @@ __device__ __forceinline__ Place place_of(const ncb_conv &c, int row) {
     }
     return p;
 }
+constexpr int CONV_BATCH = 4; /* taps whose loads are in flight together */
+
 /* Channels ch, ch + 1 (ch even) of row `row` after the convolution. */
 template <typename T> __device__ __forceinline__ float2 conv2(const ncb_conv &c, int row, const Place &at, int ch) {
     const T *u = (const T *)c.proj + (size_t)row * c.ldp + ch;
     const T *ring = (const T *)c.ring + (size_t)at.slot * c.taps * c.width + ch;
+    const int here = at.pos % c.taps;
     float2 y = make_float2(0.f, 0.f);
-    for (int j = 0; j < c.taps; j++) {
-        const int back = c.taps - 1 - j;
-        if (at.pos - back < 0) continue;
-        const float2 w = *reinterpret_cast<const float2 *>(c.w + (size_t)j * c.width + ch);
-        const float2 x = load2<T>(back <= at.before ? u - (size_t)back * c.ldp : ring + (size_t)((at.pos - back) % c.taps) * c.width);
-        y.x = fmaf(w.x, x.x, y.x), y.y = fmaf(w.y, x.y, y.y);
+    for (int back0 = 0; back0 < c.taps; back0 += CONV_BATCH) {
+        float2 w[CONV_BATCH], x[CONV_BATCH];
+#pragma unroll
+        for (int i = 0; i < CONV_BATCH; i++) {
+            const int back = back0 + i;
+            w[i] = x[i] = make_float2(0.f, 0.f);
+            if (back < c.taps && back <= at.pos) {
+                w[i] = *reinterpret_cast<const float2 *>(c.w + (size_t)(c.taps - 1 - back) * c.width + ch);
+                x[i] = load2<T>(back <= at.before ? u - (ptrdiff_t)back * c.ldp : ring + (size_t)(here - back + (here < back ? c.taps : 0)) * c.width);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < CONV_BATCH; i++) y.x = fmaf(w[i].x, x[i].x, y.x), y.y = fmaf(w[i].y, x[i].y, y.y);
     }
     return y;
+}
+/* The same of the n (at most N) rows from row0, whose places are place[0 .. n), given to put(row - row0, y): each projected
+ * value is loaded once where the taps before a row are rows of the pass. put() is also called, with anything, for rows past n. */
+template <typename T, int N, typename F> __device__ __forceinline__ void conv_run(const ncb_conv &c, int row0, int n, const Place *place, int ch, F put) {
+    constexpr int OLD = CONV_BATCH - 1;
+    if (n <= 0) {
+#pragma unroll 1
+        for (int i = 0; i < N; i++) put(i, make_float2(0.f, 0.f));
+        return;
+    }
+    const T *u = (const T *)c.proj + (ptrdiff_t)row0 * c.ldp + ch;
+    float2 x[N + OLD], w[CONV_BATCH]; /* w[back]: zero past the taps */
+#pragma unroll
+    for (int i = 0; i < N + OLD; i++) { /* (loads of rows that are not needed go to one that is) */
+        const int r = i - OLD;
+        x[i] = load2<T>(u + (ptrdiff_t)(r < n && row0 + r >= 0 ? r : 0) * c.ldp);
+    }
+#pragma unroll
+    for (int back = 0; back < CONV_BATCH; back++) {
+        w[back] = *reinterpret_cast<const float2 *>(c.w + (size_t)max(c.taps - 1 - back, 0) * c.width + ch);
+        if (back >= c.taps) w[back] = make_float2(0.f, 0.f);
+    }
+#pragma unroll
+    for (int i = 0; i < N; i++) {
+        float2 y = make_float2(0.f, 0.f);
+#pragma unroll
+        for (int back = 0; back < CONV_BATCH; back++) y.x = fmaf(w[back].x, x[i + OLD - back].x, y.x), y.y = fmaf(w[back].y, x[i + OLD - back].y, y.y);
+        put(i, y);
+    }
+    const bool all = c.taps > CONV_BATCH;
+#pragma unroll 1
+    for (int i = 0; i < min(n, N); i++) /* the sequences' first rows in the pass */
+        if (all || place[i].before < c.taps - 1) put(i, place[i].pos < 0 ? make_float2(0.f, 0.f) : conv2<T>(c, row0 + i, place[i], ch));
 }
 /* Keeps channels ch, ch + 1 of the row in the ring. A row on its own may do so at once: it reads the other taps' places. */
 template <typename T> __device__ __forceinline__ void keep2(const ncb_conv &c, int row, const Place &at, int ch) {

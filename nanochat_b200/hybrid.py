@@ -178,27 +178,51 @@ class HybridWeights:
 
     @staticmethod
     def random_state(cfg: HybridConfig, seed: int, device: "torch.device | str" = "cpu", std: float = 0.02) -> dict:
-        """Random checkpoint tensors of this configuration (bf16): matrices ~ N(0, std), norms around 1, sinks and decay
-        biases ~ N(0, 1). For benchmarks and tests."""
+        """Random checkpoint tensors of this configuration (bf16): matrices ~ N(0, std), norms multiply by about 1, sinks and
+        decay biases ~ N(0, 1), convolutions pass mostly the current token on, streams mix gently. For benchmarks and tests."""
         gen = torch.Generator(device=device).manual_seed(seed)
 
         def w(*shape, scale=std, base=0.0):
             return (torch.randn(*shape, generator=gen, device=device) * scale + base).bfloat16()
 
         C = cfg.width
-        state = {"embed": w(cfg.vocab, C), "final.norm": w(C, scale=0.1, base=1.0)}
+        around = 1.0 - cfg.norm_base
+        state = {"embed": w(cfg.vocab, C), "final.norm": w(C, scale=0.1, base=around)}
+        if not cfg.tied_head:
+            state["head"] = w(cfg.vocab, C)
         for i, spec in enumerate(cfg.layers):
             if spec.weights_of != i:
                 continue
             m, p = spec.mixer, f"l{i}."
             H, D, V = m["heads"], m["dim"], m["vdim"]
-            state[p + "norm1"] = w(C, scale=0.1, base=1.0)
+            state[p + "norm1"] = w(C, scale=0.1, base=around)
+            if cfg.streams:
+                for q in (1, 2) if spec.ff else (1,):
+                    state.update({p + f"hc{q}.in": w(cfg.streams, scale=0.1, base=1.0 / cfg.streams), p + f"hc{q}.out": w(cfg.streams, scale=0.1, base=1.0),
+                                  p + f"hc{q}.mix": (w(cfg.streams, cfg.streams, scale=0.05) + torch.eye(cfg.streams, device=device)).bfloat16()})
             if spec.kind == "gla":
                 rank = m.get("decay_rank", 16)
                 shapes = {"q": (H * D, C), "k": (H * D, C), "v": (H * V, C), "g": (H * V, C), "o": (C, H * V),
                           "a1": (rank, C), "a2": (H * D, rank)}
                 state[p + "mix.a2.b"] = w(H * D, scale=1.0, base=2.0)
                 state[p + "mix.norm"] = w(V, scale=0.1, base=1.0)
+            elif spec.kind in ("attention", "channel_delta"):
+                G, delta = m["kv_heads"], spec.kind == "channel_delta"
+                rows = {"q": (G if delta else H) * D, "k": G * D, "v": (H if delta else G) * V}
+                if m.get("kv_from") is not None:
+                    rows = {"q": rows["q"]}
+                shapes = {**{n: (count, C) for n, count in rows.items()}, "o": (C, H * V)}
+                for n, count in rows.items():
+                    taps = w(count, m["conv"], scale=0.2)
+                    taps[:, -1] += 1.0
+                    state[p + f"mix.{n}.conv"] = taps
+                if delta:
+                    rank = m.get("low_rank", 128)
+                    shapes.update({"b": (H, C), "a1": (rank, C), "a2": (H * D, rank), "g1": (rank, C), "g2": (H * V, rank)})
+                    state.update({p + "mix.A_log": w(H, scale=0.5), p + "mix.dt_bias": w(H * D, scale=1.0, base=-4.0),
+                                  p + "mix.norm": w(V, scale=0.1, base=1.0)})
+                else:
+                    shapes["g"] = (H, C)
             else:
                 R, rank = m["rot_dim"], m["kv_rank"]
                 shapes = {"q": (H * (D + R), C), "dkv": (rank + R, C), "uk": (H * D, rank), "uv": (H * V, rank),
@@ -207,7 +231,7 @@ class HybridWeights:
                 state[p + "mix.sink"] = w(H, scale=1.0)
             state.update({p + "mix." + n: w(*s) for n, s in shapes.items()})
             if spec.ff:
-                state[p + "norm2"] = w(C, scale=0.1, base=1.0)
+                state[p + "norm2"] = w(C, scale=0.1, base=around)
                 state.update({p + "mlp.gate": w(spec.ff, C), p + "mlp.up": w(spec.ff, C), p + "mlp.down": w(C, spec.ff)})
         return state
 

@@ -111,13 +111,14 @@ class RowPlan:
         return self.upload(("tiles", size), [v[order] for v in (first, rows, context, pos)]), len(first)
 
     def chunks(self, size: int) -> tuple[list[Tensor], int]:
-        """([segment's first chunk (n + 1), chunk's first row, chunk's rows], number of chunks) for chunks of `size` rows."""
+        """([segment's first chunk (n + 1), chunk's first row, chunk's rows, the segment's rows before it], number of chunks) for
+        chunks of `size` rows."""
         per = (self.count + size - 1) // size
         base = np.concatenate([[0], np.cumsum(per)]).astype(np.int32)
         within = np.arange(base[-1], dtype=np.int32) - np.repeat(base[:-1], per)
         rows = np.repeat(self.first, per) + within * size
         count = np.minimum(size, np.repeat(self.first + self.count, per) - rows)
-        return self.upload(("chunks", size), [base, rows, count]), int(base[-1])
+        return self.upload(("chunks", size), [base, rows, count, within * size]), int(base[-1])
 
 
 @dataclass
@@ -325,7 +326,7 @@ class ChannelDelta:
         self.a2_rows = pad_to(t["a2"].reshape(H, D, -1), H, self.dim, self.rank_a).to(dtype)
         self.g2_rows = pad_to(t["g2"].reshape(H, V, -1), H, self.vdim, self.rank_g).to(dtype)
         self.a2, self.g2 = (w.transpose(1, 2).contiguous() for w in (self.a2_rows, self.g2_rows))
-        self.chunk = cuda_library("delta_rule").delta_chunk_tokens(self.dim) if dtype == torch.bfloat16 else 0
+        self.chunk = cuda_library("delta_rule").delta_chunk_tokens(self.dim, self.vdim, self.conv.taps, self.rank_a, self.rank_g) if dtype == torch.bfloat16 else 0
         self.dt_bias = pad_to(t["dt_bias"].float().reshape(H, D), H, self.dim).contiguous()
         self.a_exp = t["A_log"].float().exp()
         self.norm = pad_to(t["norm"].float(), self.vdim)
@@ -361,12 +362,13 @@ class ChannelDelta:
         self.conv.keep_tail(a.conv, rows)
 
     def run_chunked(self, a: Delta, rows: Rows) -> None:
-        (seg_chunk, chunk_first, chunk_count), n = rows.plan.chunks(self.chunk)
-        a.seg_chunk, a.chunk_first, a.chunk_count = seg_chunk.data_ptr(), chunk_first.data_ptr(), chunk_count.data_ptr()
+        arrays, n = rows.plan.chunks(self.chunk)
+        a.seg_chunk, a.chunk_first, a.chunk_count, a.chunk_within = (t.data_ptr() for t in arrays)
         a.n_chunks, a.chunk, a.a2_rows, a.g2_rows = n, self.chunk, self.a2_rows.data_ptr(), self.g2_rows.data_ptr()
         C, D, V, each, bf, f = self.chunk, self.dim, self.vdim, n * self.heads, torch.bfloat16, torch.float32
-        for name, size, kind in (("w_terms", 2 * C * D, bf), ("kd_terms", 2 * C * D, bf), ("q_terms", 2 * C * D, bf), ("b_terms", 2 * C * C, bf),
-                                 ("s_terms", 2 * V * D, bf), ("u_terms", 2 * V * C, bf), ("u0", V * C, f), ("chunk_decay", D, f)):
+        for name, size, kind in (("w_terms", 2 * C * (D + 8), bf), ("kd_terms", 2 * C * (D + 8), bf), ("q_terms", 2 * C * (D + 8), bf),
+                                 ("b_terms", 2 * C * (C + 8), bf), ("s_terms", 2 * V * (D + 8), bf), ("u_terms", 2 * V * (C + 8), bf),
+                                 ("u0", V * (C + 4), f), ("chunk_decay", D, f)):
             setattr(a, name, rows.buffer("delta_" + name, each * size, kind, self.device).data_ptr())
         # values beyond one tile of the output kernel pass through memory for the norm
         a.raw = rows.buffer("delta_raw", rows.n * self.heads * V if V > 128 else 4, f, self.device).data_ptr()
@@ -427,7 +429,7 @@ class GatedLinearAttention:
         if plan is None or self.chunk == 0 or plan.longest < self.CHUNKED_FROM:
             check(lib.gla_step(pointer_to(a), f32, stream()), "gla_step")
             return
-        (seg_chunk, chunk_first, chunk_count), n_chunks = plan.chunks(self.chunk)
+        (seg_chunk, chunk_first, chunk_count, _), n_chunks = plan.chunks(self.chunk)
         HD, HV, f = self.heads * self.dim, self.heads * self.vdim, torch.float32
         a.seg_chunk, a.chunk_first, a.chunk_count = seg_chunk.data_ptr(), chunk_first.data_ptr(), chunk_count.data_ptr()
         a.n_chunks, a.chunk = n_chunks, self.chunk

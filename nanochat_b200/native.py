@@ -87,7 +87,7 @@ class Delta(ctypes.Structure):
                [("q_scale", c_float), ("eps", c_float)] + \
                [(n, c_ptr) for n in ("a2", "g2", "dt_bias", "a_exp", "norm", "state", "seg_first", "seg_count")] + \
                [("n_segments", c_int)] + \
-               [(n, c_ptr) for n in ("a2_rows", "g2_rows", "seg_chunk", "chunk_first", "chunk_count")] + \
+               [(n, c_ptr) for n in ("a2_rows", "g2_rows", "seg_chunk", "chunk_first", "chunk_count", "chunk_within")] + \
                [("n_chunks", c_int), ("chunk", c_int)] + \
                [(n, c_ptr) for n in ("w_terms", "kd_terms", "q_terms", "b_terms", "s_terms", "u_terms", "u0", "chunk_decay", "raw", "status")]
 
@@ -160,7 +160,7 @@ SIGNATURES = {
     },
     "delta_rule": {
         "delta_step": ([c_ptr, c_int, c_ptr], c_int),
-        "delta_chunk_tokens": ([c_int], c_int),
+        "delta_chunk_tokens": ([c_int] * 5, c_int),
         "delta_chunked": ([c_ptr, c_ptr], c_int),
     },
     "tile_gemm": {

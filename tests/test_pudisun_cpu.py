@@ -204,7 +204,7 @@ def test_row_plans():
     plan = RowPlan(slots, positions, "cpu")
     assert plan.n_segments == 3 and plan.longest == 4
     assert plan.first.tolist() == [0, 3, 5] and plan.count.tolist() == [3, 2, 4]
-    (seg_chunk, first, count), n = plan.chunks(2)
+    (seg_chunk, first, count, within), n = plan.chunks(2)
     assert n == 5 and seg_chunk.tolist() == [0, 2, 3, 5] and first.tolist() == [0, 2, 3, 5, 7] and count.tolist() == [2, 1, 2, 2, 2]
     ctx_slot, ctx_first = plan.contexts()
     assert ctx_slot.tolist() == [4, 1, 7] and ctx_first.tolist() == [0, 3, 14, 23]
