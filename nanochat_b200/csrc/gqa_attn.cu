@@ -76,73 +76,106 @@ template <typename T> __device__ __forceinline__ void head_row(const ncb_gqa &a,
     for (int i = 2 * lane; i < a.dim; i += 64) store2(out + i, x[i] * r, x[i + 1] * r);
 }
 
-constexpr int RUN = 8; /* consecutive rows a warp of k_gqa_rows works on */
+constexpr int RUN = 16; /* consecutive rows a warp of k_gqa_rows works on */
 
-/* Grid (units / 4 rounded up, rows / RUN rounded up), a warp per unit and run of rows: the query heads, then with own_kv the key
- * and the value heads. q NULL: the query heads only keep their ring. */
+/* Shared memory per warp of k_gqa_rows: the projected rows with the taps before them, the convolution's weights (CONV_BATCH of
+ * them, zero past the taps), a head's row, the rows' places. */
+__host__ __device__ inline size_t rows_smem(int size, int itemsize) {
+    return (size_t)(RUN + CONV_BATCH - 1) * size * itemsize + (size_t)CONV_BATCH * size * 4 + (size_t)size * 4 + RUN * sizeof(Place) + 8;
+}
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void *src, bool on) { /* 16 bytes, zeros when off */
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
+}
+
+/* Grid (units / warps rounded up, rows / RUN rounded up), a warp per unit and run of rows: the query heads, then with own_kv the
+ * key and the value heads. q NULL: the query heads only keep their ring. A loop over the rows with a short body: the kernel has
+ * many warps, and what is unrolled far has to be fetched by each of them. */
 template <typename T> __global__ void __launch_bounds__(THREADS) k_gqa_rows(const ncb_gqa a) {
-    extern __shared__ float sm[]; /* [warps][RUN][dim], then the rows' places */
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, unit = blockIdx.x * (THREADS / 32) + warp;
+    extern __shared__ __align__(128) uint8_t raw[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, unit = blockIdx.x * (blockDim.x >> 5) + warp;
     const int H = a.heads, G = a.own_kv ? a.kv_heads : 0, row0 = blockIdx.y * RUN, n = (int)min((long long)RUN, a.conv.rows - row0);
-    Place *place = reinterpret_cast<Place *>(sm + (THREADS / 32) * RUN * a.dim) + warp * RUN;
+    constexpr int OLD = CONV_BATCH - 1, PER = 16 / sizeof(T);
+    const int largest = max(a.dim, a.vdim);
+    uint8_t *mine = raw + warp * ((rows_smem(largest, sizeof(T)) + 15) / 16 * 16);
+    T *tile = reinterpret_cast<T *>(mine);                                  /* [OLD + RUN][size] */
+    float *w = reinterpret_cast<float *>(tile + (OLD + RUN) * largest);     /* [CONV_BATCH][size], by how far back */
+    float *x = w + CONV_BATCH * largest;                                    /* [size] */
+    Place *place = reinterpret_cast<Place *>(x + largest);
     asm volatile("griddepcontrol.wait;" ::: "memory");
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     if (unit >= H + 2 * G) return;
-    if (lane < n) {
-        int slot;
-        const int len = length_of(a, row0 + lane, slot);
-        place[lane] = len ? place_of(a.conv, row0 + lane) : Place{-1, 0, 0};
-    }
-    __syncwarp();
     const bool query = unit < H, key = !query && unit < H + G;
     const int kvh = query ? 0 : key ? unit - H : unit - H - G, size = query || key ? a.dim : a.vdim;
     const int ch0 = query ? a.off_q + unit * a.dim : key ? a.off_k + kvh * a.dim : a.off_v + kvh * a.vdim;
-    if (a.keep)
-        for (int r = 0; r < n; r++)
-            if (place[r].pos >= 0)
-                for (int i = 2 * lane; i < size; i += 64) keep2<T>(a.conv, row0 + r, place[r], ch0 + i);
-    if (query && !a.q) return;
-    float *x = sm + warp * RUN * a.dim;
-    for (int i = 2 * lane; i < size; i += 64) {
-        conv_run<T, RUN>(a.conv, row0, n, place, ch0 + i, [&](int r, float2 y) {
-            if (query || key) *reinterpret_cast<float2 *>(x + r * a.dim + i) = y;
-            else if (r < n && place[r].pos >= 0) store2(cache_row<T>(a, place[r].slot, kvh, place[r].pos) + a.dim + i, y.x, y.y);
-        });
+    const T *proj = (const T *)a.conv.proj + ch0;
+    const int per = size / PER, first = row0 - OLD;
+#pragma unroll 4
+    for (int i = lane; i < (OLD + n) * per; i += 32) {
+        const int r = i / per, c = (i - r * per) * PER;
+        cp_async16(smem_u32(tile + r * size + c), proj + (size_t)max(first + r, 0) * a.conv.ldp + c, first + r >= 0);
     }
-    if (!query && !key) return;
+    for (int i = lane; i < CONV_BATCH * size / 4; i += 32) {
+        const int back = 4 * i / size, c = 4 * i - back * size;
+        const bool on = back < a.conv.taps;
+        cp_async16(smem_u32(w + 4 * i), a.conv.w + (size_t)(on ? a.conv.taps - 1 - back : 0) * a.conv.width + ch0 + c, on);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    bool elsewhere = false;
+    if (lane < n) {
+        int slot;
+        const int len = length_of(a, row0 + lane, slot);
+        const Place at = len ? place_of(a.conv, row0 + lane) : Place{-1, 0, 0};
+        place[lane] = at;
+        elsewhere = at.before < a.conv.taps - 1 || a.conv.taps > CONV_BATCH; /* some tap is not a row of the pass */
+    }
+    const uint32_t special = __ballot_sync(0xffffffffu, elsewhere);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncwarp();
     const int half = a.rot / 2;
-    for (int i = lane; i < half; i += 32) { /* in place: a pair belongs to one lane */
-        float c[RUN], s[RUN];
+    const float inv_count = 1.f / (float)a.norm_count;
+#pragma unroll 1
+    for (int r = 0; r < n; r++) {
+        const Place at = place[r];
+        if (at.pos < 0) continue;
+        if (a.keep)
+            for (int i = 2 * lane; i < size; i += 64) keep2<T>(a.conv, row0 + r, at, ch0 + i);
+        if (query && !a.q) continue;
+        T *out = query ? (T *)a.q + ((size_t)(row0 + r) * H + unit) * a.dim : cache_row<T>(a, at.slot, kvh, at.pos) + (key ? 0 : a.dim);
+        for (int i = 4 * lane; i < size; i += 128) {
+            float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (special >> r & 1) {
+                const float2 u = conv2<T>(a.conv, row0 + r, at, ch0 + i), v = conv2<T>(a.conv, row0 + r, at, ch0 + i + 2);
+                y = make_float4(u.x, u.y, v.x, v.y);
+            } else {
 #pragma unroll
-        for (int r = 0; r < RUN; r++) {
-            const size_t at = (size_t)(r < n && place[r].pos >= 0 ? place[r].pos : 0) * half + i;
-            c[r] = a.cos[at], s[r] = a.sin[at];
+                for (int back = 0; back < CONV_BATCH; back++) {
+                    const float4 f = *reinterpret_cast<const float4 *>(w + back * size + i), v = load4(tile + (r + OLD - back) * size + i);
+                    y.x = fmaf(f.x, v.x, y.x), y.y = fmaf(f.y, v.y, y.y), y.z = fmaf(f.z, v.z, y.z), y.w = fmaf(f.w, v.w, y.w);
+                }
+            }
+            if (query || key) *reinterpret_cast<float4 *>(x + i) = y;
+            else store4(out + i, y);
         }
-#pragma unroll
-        for (int r = 0; r < RUN; r++) {
-            float *p = x + r * a.dim + i;
-            const float u = p[0], v = p[half];
-            p[0] = u * c[r] - v * s[r];
-            p[half] = v * c[r] + u * s[r];
+        if (!query && !key) continue;
+        __syncwarp();
+        for (int i = lane; i < half; i += 32) { /* in place: a pair belongs to one lane */
+            const float c = a.cos[(size_t)at.pos * half + i], s = a.sin[(size_t)at.pos * half + i], u = x[i], v = x[i + half];
+            x[i] = u * c - v * s;
+            x[i + half] = v * c + u * s;
         }
-    }
-    __syncwarp();
-#pragma unroll
-    for (int r = 0; r < RUN; r++) {
+        __syncwarp();
         float sum = 0.f;
-        for (int i = 2 * lane; i < a.dim; i += 64) {
-            const float2 v = *reinterpret_cast<const float2 *>(x + r * a.dim + i);
-            sum = fmaf(v.x, v.x, fmaf(v.y, v.y, sum));
+        for (int i = 4 * lane; i < size; i += 128) {
+            const float4 v = *reinterpret_cast<const float4 *>(x + i);
+            sum = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, sum))));
         }
         for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-        if (r >= n || place[r].pos < 0) continue;
-        const float f = 1.f / sqrtf(sum / (float)a.norm_count + a.eps);
-        T *out = query ? (T *)a.q + ((size_t)(row0 + r) * H + unit) * a.dim : cache_row<T>(a, place[r].slot, kvh, place[r].pos);
-        for (int i = 2 * lane; i < a.dim; i += 64) {
-            const float2 v = *reinterpret_cast<const float2 *>(x + r * a.dim + i);
-            store2(out + i, v.x * f, v.y * f);
+        const float f = sizeof(T) == 2 ? rsqrtf(fmaf(sum, inv_count, a.eps)) : 1.f / sqrtf(sum / (float)a.norm_count + a.eps);
+        for (int i = 4 * lane; i < size; i += 128) {
+            const float4 v = *reinterpret_cast<const float4 *>(x + i);
+            store4(out + i, make_float4(v.x * f, v.y * f, v.z * f, v.w * f));
         }
+        __syncwarp();
     }
 }
 
@@ -216,9 +249,6 @@ __device__ __forceinline__ void ldsm4(uint32_t *r, uint32_t addr) {
 __device__ __forceinline__ void ldsm4_t(uint32_t *r, uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void *src, bool on) { /* 16 bytes, zeros when off */
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
 }
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
@@ -649,11 +679,11 @@ int check(const ncb_gqa &g) {
         g.table_len <= 0)
         return NCB_ERR_ARG;
     const int W = g.conv.width;
-    if (g.off_q < 0 || g.off_q % 2 || g.off_q + g.heads * g.dim > W || g.off_g < 0 || g.off_g + g.heads > g.conv.ldp) return NCB_ERR_ARG;
-    if (g.own_kv && (g.off_k < 0 || g.off_k % 2 || g.off_k + g.kv_heads * g.dim > W || g.off_v < 0 || g.off_v % 2 || g.off_v + g.kv_heads * g.vdim > W))
+    if (g.off_q < 0 || g.off_q % 4 || g.off_q + g.heads * g.dim > W || g.off_g < 0 || g.off_g + g.heads > g.conv.ldp) return NCB_ERR_ARG;
+    if (g.own_kv && (g.off_k < 0 || g.off_k % 4 || g.off_k + g.kv_heads * g.dim > W || g.off_v < 0 || g.off_v % 4 || g.off_v + g.kv_heads * g.vdim > W))
         return NCB_ERR_ARG;
     if (!g.kv || (g.rot && (!g.cos || !g.sin))) return NCB_ERR_ARG;
-    return ((uintptr_t)g.q | (uintptr_t)g.kv | (uintptr_t)g.parts | (uintptr_t)g.out) % 16 || g.ldo % 2 ? NCB_ERR_ALIGN : NCB_OK;
+    return ((uintptr_t)g.q | (uintptr_t)g.kv | (uintptr_t)g.parts | (uintptr_t)g.out) % 16 || g.ldo % 2 || g.conv.ldp % 4 ? NCB_ERR_ALIGN : NCB_OK;
 }
 int check_parts(const ncb_gqa &g) {
     if (!g.parts || g.chunk_tiles <= 0 || g.max_chunks <= 0 || g.max_len <= 0 || g.conv.rows > 65535 ||
@@ -670,12 +700,16 @@ int gqa_rows(const ncb_gqa *g, int f32, void *stream) {
     if (!g) return NCB_ERR_ARG;
     const int rc = check(*g);
     if (rc != NCB_OK || g->conv.rows == 0) return rc;
-    const size_t smem = (size_t)(THREADS / 32) * RUN * (g->dim * 4 + sizeof(Place));
+    const size_t one = (rows_smem(g->dim > g->vdim ? g->dim : g->vdim, f32 ? 4 : 2) + 15) / 16 * 16;
+    const int warps = 4 * one <= 200 * 1024 ? 4 : 1;
+    const size_t smem = warps * one;
     if (smem > 200 * 1024) return NCB_ERR_UNSUPPORTED;
+    if (((uintptr_t)g->conv.proj | (uintptr_t)g->conv.w) % 16 || g->conv.ldp % 8 || g->conv.width % 8 || g->off_q % 8 || (g->own_kv && (g->off_k | g->off_v) % 8))
+        return NCB_ERR_ALIGN;
     const int units = g->heads + (g->own_kv ? 2 * g->kv_heads : 0);
-    const dim3 grid((units + THREADS / 32 - 1) / (THREADS / 32), (unsigned)((g->conv.rows + RUN - 1) / RUN));
-    return f32 ? launch(k_gqa_rows<float>, grid, THREADS, smem, 1, (cudaStream_t)stream, *g)
-               : launch(k_gqa_rows<bf16>, grid, THREADS, smem, 1, (cudaStream_t)stream, *g);
+    const dim3 grid((units + warps - 1) / warps, (unsigned)((g->conv.rows + RUN - 1) / RUN));
+    return f32 ? launch(k_gqa_rows<float>, grid, 32 * warps, smem, 1, (cudaStream_t)stream, *g)
+               : launch(k_gqa_rows<bf16>, grid, 32 * warps, smem, 1, (cudaStream_t)stream, *g);
 }
 
 /* 1 if gqa_split in bf16 takes these (padded) sizes with q NULL. */

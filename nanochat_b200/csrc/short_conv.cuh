@@ -59,38 +59,18 @@ template <typename T> __device__ __forceinline__ float2 conv2(const ncb_conv &c,
     }
     return y;
 }
-/* The same of the n (at most N) rows from row0, whose places are place[0 .. n), given to put(row - row0, y): each projected
- * value is loaded once where the taps before a row are rows of the pass. put() is also called, with anything, for rows past n. */
-template <typename T, int N, typename F> __device__ __forceinline__ void conv_run(const ncb_conv &c, int row0, int n, const Place *place, int ch, F put) {
-    constexpr int OLD = CONV_BATCH - 1;
-    if (n <= 0) {
-#pragma unroll 1
-        for (int i = 0; i < N; i++) put(i, make_float2(0.f, 0.f));
-        return;
-    }
-    const T *u = (const T *)c.proj + (ptrdiff_t)row0 * c.ldp + ch;
-    float2 x[N + OLD], w[CONV_BATCH]; /* w[back]: zero past the taps */
-#pragma unroll
-    for (int i = 0; i < N + OLD; i++) { /* (loads of rows that are not needed go to one that is) */
-        const int r = i - OLD;
-        x[i] = load2<T>(u + (ptrdiff_t)(r < n && row0 + r >= 0 ? r : 0) * c.ldp);
-    }
-#pragma unroll
-    for (int back = 0; back < CONV_BATCH; back++) {
-        w[back] = *reinterpret_cast<const float2 *>(c.w + (size_t)max(c.taps - 1 - back, 0) * c.width + ch);
-        if (back >= c.taps) w[back] = make_float2(0.f, 0.f);
-    }
-#pragma unroll
-    for (int i = 0; i < N; i++) {
-        float2 y = make_float2(0.f, 0.f);
-#pragma unroll
-        for (int back = 0; back < CONV_BATCH; back++) y.x = fmaf(w[back].x, x[i + OLD - back].x, y.x), y.y = fmaf(w[back].y, x[i + OLD - back].y, y.y);
-        put(i, y);
-    }
-    const bool all = c.taps > CONV_BATCH;
-#pragma unroll 1
-    for (int i = 0; i < min(n, N); i++) /* the sequences' first rows in the pass */
-        if (all || place[i].before < c.taps - 1) put(i, place[i].pos < 0 ? make_float2(0.f, 0.f) : conv2<T>(c, row0 + i, place[i], ch));
+/* Four neighbouring values. */
+__device__ __forceinline__ float4 load4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
+__device__ __forceinline__ float4 load4(const bf16 *p) {
+    const uint2 v = *reinterpret_cast<const uint2 *>(p);
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xffff0000u));
+}
+__device__ __forceinline__ void store4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+__device__ __forceinline__ void store4(bf16 *p, float4 v) {
+    uint2 o;
+    reinterpret_cast<__nv_bfloat162 &>(o.x) = __floats2bfloat162_rn(v.x, v.y);
+    reinterpret_cast<__nv_bfloat162 &>(o.y) = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2 *>(p) = o;
 }
 /* Keeps channels ch, ch + 1 of the row in the ring. A row on its own may do so at once: it reads the other taps' places. */
 template <typename T> __device__ __forceinline__ void keep2(const ncb_conv &c, int row, const Place &at, int ch) {

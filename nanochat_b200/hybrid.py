@@ -93,7 +93,7 @@ class HybridConfig:
         """Device bytes one more slot costs: its rows and states in every layer's cache and its rows of a decode step."""
         cache = sum(MIXERS[s.kind].cache_bytes(s.mixer, self.max_len, self.itemsize) for s in self.layers)
         columns = up(self.width, 128)
-        rows = 16 * columns + 8 * up(self.vocab, 64) + 8 * (cache_pages(self.max_len) * 64 + 1)
+        rows = (16 + 4 * max(self.streams - 1, 0)) * columns + 8 * up(self.vocab, 64) + 8 * (cache_pages(self.max_len) * 64 + 1)
         return cache + rows
 
 

@@ -193,9 +193,9 @@ def test_structures_match_the_header():
     text = re.sub(r"/\*.*?\*/", "", (ROOT / "include" / "nanochat_b200.h").read_text(), flags=re.S)
     for cls, name in ((native.GemmRs, "ncb_gemm_rs"), (native.Latent, "ncb_latent"), (native.Gla, "ncb_gla")):
         body = re.search(r"typedef struct \{([^}]*)\} " + name + ";", text).group(1)
-        fields = [f for decl in body.split(";") if decl.strip()
+        fields = [f for decl in re.sub(r"\[[^]]*\]", "", body).split(";") if decl.strip()
                   for f in re.findall(r"(\w+)\s*(?:,|$)", decl.strip() + ",")]
-        assert fields == [f for f, _ in cls._fields_], name
+        assert fields == [f.rstrip("_") for f, _ in cls._fields_], name
 
 
 def test_row_plans():
