@@ -31,16 +31,20 @@ namespace cg = cooperative_groups;
 
 namespace {
 
+constexpr float LOG2E = 1.4426950408889634f, LN2 = 0.6931471805599453f;
+
 __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
 /* The activation of the convolutions: at the precision of what they are kept in. */
-template <typename T> __device__ __forceinline__ float silu(float z) { return sizeof(T) == 2 ? __fdividef(z, 1.f + __expf(-z)) : z / (1.f + expf(-z)); }
+template <typename T> __device__ __forceinline__ float silu(float z) { return sizeof(T) == 2 ? __fdividef(z, 1.f + ex2(-z * LOG2E)) : z / (1.f + expf(-z)); }
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 /* exp(-a_exp softplus(z)). The second form is a few ulps away from the first: log(1 + e) as a series where 1 + e loses e's bits. */
 template <typename T> __device__ __forceinline__ float decay_of(float z, float a_exp) { return expf(-a_exp * softplus(z)); }
 template <> __device__ __forceinline__ float decay_of<bf16>(float z, float a_exp) {
-    const float e = __expf(-fabsf(z));
+    const float e = ex2(-fabsf(z) * LOG2E);
     const float series = e * fmaf(e, fmaf(e, fmaf(e, fmaf(e, 0.2f, -0.25f), 1.f / 3.f), -0.5f), 1.f);
-    return __expf(-a_exp * (fmaxf(z, 0.f) + (e < 0.03125f ? series : __logf(1.f + e))));
+    float log2;
+    asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(log2) : "f"(1.f + e));
+    return ex2(-a_exp * LOG2E * (fmaxf(z, 0.f) + (e < 0.03125f ? series : log2 * LN2)));
 }
 constexpr float UNIT_EPS = 1e-6f;
 
@@ -296,11 +300,11 @@ __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
         : "l"(reinterpret_cast<uint64_t &>(a)), "l"(reinterpret_cast<uint64_t &>(b)), "l"(reinterpret_cast<uint64_t &>(c)));
     return r;
 }
-/* v[0 .. 63] summed over the warp by halving: lane l ends up with the sums of values 2 l and 2 l + 1 in v[0], v[1]. */
+/* v[0 .. 63] summed over each half of the warp by halving: lane l of a half ends up with the sums of values 4 l .. 4 l + 3. */
 __device__ __forceinline__ void reduce64(float (&v)[64], int lane) {
 #pragma unroll
-    for (int step = 0; step < 5; step++) {
-        const int n = 32 >> step, off = 16 >> step;
+    for (int step = 0; step < 4; step++) {
+        const int n = 32 >> step, off = 8 >> step;
         const bool upper = lane & off;
 #pragma unroll
         for (int i = 0; i < n; i++) {
@@ -339,7 +343,7 @@ __host__ __device__ inline ChunkSmem chunk_smem(int C, int D, int V, int taps, i
     const int fp32 = 3 * C * D * 4, later = 2 * C * (VALUES + 8) * 2 + 2 * C * (C + 8) * 2 + C * (C + 4) * 4;
     s.al = 2 * C * D * 4;
     s.terms = fp32 > later ? fp32 : later;
-    const int rows = (C + taps - 1) * (2 * D + (V < VALUES ? V : VALUES)) * 2, staged = rows + C * (rank_a + 8) * 2, terms = 6 * C * (D + 8) * 2;
+    const int rows = (C + (taps > CONV_BATCH ? taps : CONV_BATCH) - 1) * (2 * D + (V < VALUES ? V : VALUES)) * 2, staged = rows + C * (rank_a + 8) * 2, terms = 6 * C * (D + 8) * 2;
     s.low = s.terms + rows;
     s.A = s.terms + (staged > terms ? staged : terms);
     s.G = s.A + C * (C + 4) * 4;
@@ -392,50 +396,63 @@ template <int MT, int CHUNK_THREADS> __global__ void __launch_bounds__(CHUNK_THR
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     if (n == 0) return;
     const bf16 *proj = (const bf16 *)a.conv.proj;
-    /* `count` channels from ch of the chunk's rows and the taps - 1 positions before it, to columns c0 .. of rows of ld values;
-     * rows past the chunk are its last one, positions before 0 are zeros */
-    auto stage_rows = [&](bf16 *dst, int ld, int c0, int ch, int count) {
-        const int per = count / 8;
-        for (int i = tid; i < (C + taps - 1) * per; i += CHUNK_THREADS) {
-            const int r = i / per, c = (i - r * per) * 8, t = r - (taps - 1);
-            bf16 *to = dst + r * ld + c0 + c;
-            if (start.pos + t < 0) {
-                *reinterpret_cast<uint4 *>(to) = make_uint4(0u, 0u, 0u, 0u);
-                continue;
-            }
-            const bf16 *from = t >= -start.before ? proj + (ptrdiff_t)(first + min(t, n - 1)) * a.conv.ldp
-                                                  : (const bf16 *)a.conv.ring + ((size_t)start.slot * taps + (start.pos + t) % taps) * a.conv.width;
-            cp_async16(smem_addr(to), from + ch + c);
+    /* Fields of the chunk's rows and of the `old` positions before it, a warp per row: n_field runs of `count` channels from
+     * ch[field]. Rows past the chunk are its last one; positions before 0 and those that no tap reaches are zeros. */
+    const int old = max(taps, CONV_BATCH) - 1;
+    auto stage_rows = [&](bf16 *dst, int ld, int n_fields, const int *ch, const int *count) {
+        for (int r = warp; r < C + old; r += CHUNK_WARPS) {
+            const int t = r - old;
+            const bool zero = start.pos + t < 0 || t <= -taps;
+            const bf16 *from = t >= -start.before || zero ? proj + (ptrdiff_t)(first + (zero ? 0 : min(t, n - 1))) * a.conv.ldp
+                                                          : (const bf16 *)a.conv.ring + ((size_t)start.slot * taps + (start.pos + t) % taps) * a.conv.width;
+            bf16 *to = dst + r * ld;
+#pragma unroll
+            for (int f = 0; f < 3; f++)
+                if (f < n_fields) {
+                    for (int c = 8 * lane; c < count[f]; c += 256) {
+                        if (zero) *reinterpret_cast<uint4 *>(to + c) = make_uint4(0u, 0u, 0u, 0u);
+                        else cp_async16(smem_addr(to + c), from + ch[f] + c);
+                    }
+                    to += count[f];
+                }
         }
     };
-    /* 8 tokens of a pair of channels from staged rows (x: the first token's oldest tap), convolved and activated */
+    /* 8 tokens of a pair of channels from staged rows (x: `old` rows before the first), convolved and activated */
     auto convolve = [&](const bf16 *x, int ld, int ch, float2 (&y)[8]) {
+        float2 w[CONV_BATCH], v[8 + CONV_BATCH - 1];
+        const float *wp = a.conv.w + (size_t)(taps - 1) * a.conv.width + ch;
 #pragma unroll
-        for (int t = 0; t < 8; t++) y[t] = make_float2(0.f, 0.f);
-#pragma unroll 4
-        for (int j = 0; j < taps; j++) {
-            const float2 w = *reinterpret_cast<const float2 *>(a.conv.w + (size_t)j * a.conv.width + ch);
+        for (int back = 0; back < CONV_BATCH; back++)
+            w[back] = back < taps ? *reinterpret_cast<const float2 *>(wp - (ptrdiff_t)back * a.conv.width) : make_float2(0.f, 0.f);
+        const bf16 *near = x + (old - (CONV_BATCH - 1)) * ld;
 #pragma unroll
-            for (int t = 0; t < 8; t++) {
-                const float2 v = load2<bf16>(x + (t + j) * ld);
-                y[t].x = fmaf(w.x, v.x, y[t].x), y[t].y = fmaf(w.y, v.y, y[t].y);
-            }
+        for (int i = 0; i < 8 + CONV_BATCH - 1; i++) {
+            const uint32_t b = *reinterpret_cast<const uint32_t *>(near + i * ld);
+            v[i] = make_float2(__uint_as_float(b << 16), __uint_as_float(b & 0xffff0000u));
+        }
+#pragma unroll
+        for (int t = 0; t < 8; t++) {
+            y[t] = mul2(w[0], v[t + CONV_BATCH - 1]);
+#pragma unroll
+            for (int back = 1; back < CONV_BATCH; back++) y[t] = fma2(w[back], v[t + CONV_BATCH - 1 - back], y[t]);
+        }
+#pragma unroll 1
+        for (int back = CONV_BATCH; back < taps; back++) { /* a longer convolution */
+            const float2 f = *reinterpret_cast<const float2 *>(wp - (ptrdiff_t)back * a.conv.width);
+#pragma unroll
+            for (int t = 0; t < 8; t++) y[t] = fma2(f, load2<bf16>(x + (old + t - back) * ld), y[t]);
         }
 #pragma unroll
         for (int t = 0; t < 8; t++) y[t] = make_float2(silu<bf16>(y[t].x), silu<bf16>(y[t].y));
     };
-    stage_rows(rows, wide, 0, a.off_q + kh * D, D);
-    stage_rows(rows, wide, D, a.off_k + kh * D, D);
-    stage_rows(rows, wide, 2 * D, a.off_v + h * V, nv0);
-    const int sl = a.rank_a + 8;
     {
-        const int per = a.rank_a / 8;
-        for (int i = tid; i < C * per; i += CHUNK_THREADS) {
-            const int t = i / per, c = i - t * per;
-            cp_async16(smem_addr(low + t * sl + c * 8), proj + (size_t)(first + min(t, n - 1)) * a.conv.ldp + a.off_a + c * 8);
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
+        const int ch[3] = {a.off_q + kh * D, a.off_k + kh * D, a.off_v + h * V}, count[3] = {D, D, nv0};
+        stage_rows(rows, wide, 3, ch, count);
     }
+    const int sl = a.rank_a + 8;
+    for (int t = warp; t < C; t += CHUNK_WARPS)
+        for (int c = 8 * lane; c < a.rank_a; c += 256) cp_async16(smem_addr(low + t * sl + c), proj + (size_t)(first + min(t, n - 1)) * a.conv.ldp + a.off_a + c);
+    asm volatile("cp.async.commit_group;" ::: "memory");
     for (int i = tid; i < C * SA; i += CHUNK_THREADS) A[i] = 0.f;
     if (tid < C) beta[tid] = tid < n ? sigmoid(to_f(proj[(size_t)(first + tid) * a.conv.ldp + a.off_b + h])) : 0.f;
     asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -520,23 +537,35 @@ template <int MT, int CHUNK_THREADS> __global__ void __launch_bounds__(CHUNK_THR
                 if (t + j * CHUNK_WARPS < C) q[(t + j * CHUNK_WARPS) * D + d] *= x[j], k[(t + j * CHUNK_WARPS) * D + d] *= y[j];
     }
     __syncthreads();
-    for (int i = tid; i < MT * D; i += CHUNK_THREADS) { /* per sub-chunk: q, k with the decays since its start, k with those to its end */
-        const int sub = i / D, d = i - sub * D;
-        float f = 1.f;
+    for (int i = tid; i < MT * D; i += CHUNK_THREADS) { /* (pair of channels, sub-chunk, direction) */
+        const int d = 2 * (i % (D / 2)), sub = i / (D / 2) % MT;
+        const float2 *x = reinterpret_cast<const float2 *>(q + sub * SUB * D + d), *y = reinterpret_cast<const float2 *>(k + sub * SUB * D + d),
+                     *f = reinterpret_cast<const float2 *>(al + sub * SUB * D + d);
+        const int ld = D / 2, ls = sd / 2, low = C * sd / 2;
+        float2 p = make_float2(1.f, 1.f);
+        if (i < MT * (D / 2)) { /* q, k with the decays since the sub-chunk's start */
+            uint32_t *qo = reinterpret_cast<uint32_t *>(qs + sub * SUB * sd + d), *ko = reinterpret_cast<uint32_t *>(ks + sub * SUB * sd + d);
 #pragma unroll 4
-        for (int t = 0; t < SUB; t++) {
-            const int r = sub * SUB + t;
-            f *= al[r * D + d];
-            split1(q[r * D + d] * f, qs + r * sd + d, qs + (C + r) * sd + d);
-            split1(k[r * D + d] * f, ks + r * sd + d, ks + (C + r) * sd + d);
-        }
-        G[i] = f;
-        f = 1.f;
+            for (int t = 0; t < SUB; t++) {
+                p = mul2(p, f[t * ld]);
+                const float2 a = mul2(x[t * ld], p), b = mul2(y[t * ld], p);
+                uint32_t hi, lo;
+                split2(a.x, a.y, hi, lo);
+                qo[t * ls] = hi, qo[low + t * ls] = lo;
+                split2(b.x, b.y, hi, lo);
+                ko[t * ls] = hi, ko[low + t * ls] = lo;
+            }
+            *reinterpret_cast<float2 *>(G + sub * D + d) = p;
+        } else { /* k with the decays to its end */
+            uint32_t *ko = reinterpret_cast<uint32_t *>(kd + sub * SUB * sd + d);
 #pragma unroll 4
-        for (int t = SUB - 1; t >= 0; t--) {
-            const int r = sub * SUB + t;
-            split1(k[r * D + d] * f, kd + r * sd + d, kd + (C + r) * sd + d);
-            f *= al[r * D + d];
+            for (int t = SUB - 1; t >= 0; t--) {
+                const float2 b = mul2(y[t * ld], p);
+                uint32_t hi, lo;
+                split2(b.x, b.y, hi, lo);
+                ko[t * ls] = hi, ko[low + t * ls] = lo;
+                p = mul2(p, f[t * ld]);
+            }
         }
     }
     __syncthreads();
@@ -582,16 +611,16 @@ template <int MT, int CHUNK_THREADS> __global__ void __launch_bounds__(CHUNK_THR
             for (int e = 0; e < 4; e++)
                 put(keys, i * SUB + g + (e >> 1) * 8, j * SUB + c * 8 + t2 + (e & 1), acc[0][c][e] + acc[1][c][e] + acc[2][c][e]);
     }
-    for (int task = CHUNK_WARPS - 1 - warp; task < MT * 8; task += CHUNK_WARPS) { /* inside a sub-chunk: (q or k, sub-chunk, four s) */
-        const bool keys = task & 1;
-        const int i0 = (task >> 3) * SUB, s0 = (task >> 1) % 4 * 4;
+    for (int task = CHUNK_WARPS - 1 - warp; task < MT * 4; task += CHUNK_WARPS) { /* inside a sub-chunk: (sub-chunk, four s), k in half a warp, q in the other */
+        const bool keys = lane < 16;
+        const int i0 = (task >> 2) * SUB, s0 = task % 4 * 4;
         const float *x = keys ? k : q;
         float2 sums[2][SUB]; /* [pair of s][t - s0]: what lies before s is never used */
 #pragma unroll
         for (int e = 0; e < 2 * SUB; e++) sums[e / SUB][e % SUB] = make_float2(0.f, 0.f);
         if (i0 < n)
 #pragma unroll 1
-            for (int d = lane; d < D; d += 32) {
+            for (int d = lane & 15; d < D; d += 16) {
                 const float *kp = k + (i0 + s0) * D + d, *xp = x + (i0 + s0) * D + d, *ap = al + (i0 + s0) * D + d;
                 float2 f[2] = {make_float2(kp[0], kp[D]), make_float2(kp[2 * D], kp[3 * D])};
 #pragma unroll
@@ -610,8 +639,8 @@ template <int MT, int CHUNK_THREADS> __global__ void __launch_bounds__(CHUNK_THR
         for (int e = 0; e < 2 * SUB; e++) acc[e / SUB * 2 * SUB + e % SUB] = sums[e / SUB][e % SUB].x, acc[(e / SUB * 2 + 1) * SUB + e % SUB] = sums[e / SUB][e % SUB].y;
         reduce64(acc, lane);
 #pragma unroll
-        for (int e = 0; e < 2; e++) {
-            const int s = s0 + (2 * lane + e) / 16, t = s0 + (2 * lane + e) % 16;
+        for (int e = 0; e < 4; e++) {
+            const int at = 4 * (lane & 15) + e, s = s0 + at / 16, t = s0 + at % 16;
             if (t < SUB && (keys ? t > s : t >= s)) put(keys, i0 + t, i0 + s, acc[e]);
         }
     }
@@ -674,7 +703,8 @@ template <int MT, int CHUNK_THREADS> __global__ void __launch_bounds__(CHUNK_THR
     for (int v0 = 0; v0 < V; v0 += VALUES) {
         const int nv = min(VALUES, V - v0);
         if (v0) { /* more values: their rows where qs was */
-            stage_rows(rows, nv, 0, a.off_v + h * V + v0, nv);
+            const int ch[3] = {a.off_v + h * V + v0, 0, 0}, count[3] = {nv, 0, 0};
+            stage_rows(rows, nv, 1, ch, count);
             asm volatile("cp.async.commit_group;" ::: "memory");
             asm volatile("cp.async.wait_group 0;" ::: "memory");
             __syncthreads();
