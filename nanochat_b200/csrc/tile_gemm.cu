@@ -28,7 +28,7 @@
 namespace {
 
 constexpr int BM = 128;          /* rows per tile = MMA M */
-constexpr int THREADS = 192;     /* producer warp, MMA warp, four epilogue warps */
+constexpr int THREADS = 192;     /* producer warp, MMA warp, four epilogue warps (eight for several streams: threads_of) */
 constexpr int A_BYTES = BM * KBLK * 2;
 
 constexpr int TURN_FLOATS = 32 * 33; /* per epilogue warp: see stream_columns */
@@ -36,6 +36,10 @@ constexpr int TURN_FLOATS = 32 * 33; /* per epilogue warp: see stream_columns */
 enum { EPI_STORE = 0, EPI_RESID = 1, EPI_RELU2 = 2, EPI_F32 = 3, EPI_GEGLU = 5, EPI_STREAM = 6, EPI_STREAMS = 7, EPI_SWIGLU = 8 };
 
 constexpr bool writes_stream(int epi) { return epi == EPI_STREAM || epi == EPI_STREAMS; }
+/* The update of several streams is bound by what its loads have in flight: twice as many warps share the columns of a tile. */
+__host__ __device__ constexpr int epilogue_warps(int epi) { return epi == EPI_STREAMS ? 8 : 4; }
+constexpr int threads_of(int epi) { return THREADS + 32 * (epilogue_warps(epi) - 4); }
+constexpr int turn_bytes(int epi) { return writes_stream(epi) ? epilogue_warps(epi) * TURN_FLOATS * 4 : 0; }
 
 template <int BN> struct Tile {
     static constexpr int B_BYTES = BN * KBLK * 2;
@@ -43,7 +47,7 @@ template <int BN> struct Tile {
     static constexpr int STAGES = BN == 256 ? 4 : 6;               /* 192 KB of ring either way */
     static constexpr int RING_BYTES = STAGES * STAGE_BYTES;
     /* 1024: the ring is aligned by hand; 256: barriers; then the stream update's staging */
-    static constexpr int smem_bytes(int epi) { return 1024 + RING_BYTES + 256 + (writes_stream(epi) ? 4 * TURN_FLOATS * 4 : 0); }
+    static constexpr int smem_bytes(int epi) { return 1024 + RING_BYTES + 256 + turn_bytes(epi); }
     static constexpr int TMEM_COLS = 2 * BN;                       /* two accumulators */
 };
 
@@ -219,7 +223,7 @@ static __device__ __forceinline__ void streams_columns(const TileArgs &a, int m,
 }
 
 template <int BN, int EPI>
-__global__ void __launch_bounds__(THREADS, 1) k_tile_gemm(const __grid_constant__ CUtensorMap map_x,
+__global__ void __launch_bounds__(threads_of(EPI), 1) k_tile_gemm(const __grid_constant__ CUtensorMap map_x,
                                                           const __grid_constant__ CUtensorMap map_w,
                                                           const __grid_constant__ CUtensorMap map_w_half, const TileArgs a) {
     using T = Tile<BN>;
@@ -248,7 +252,7 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm(const __grid_constant_
         }
         for (int b = 0; b < 2; b++) {
             mbar_init(acc_full(b), 1);
-            mbar_init(acc_empty(b), 4); /* one arrival per epilogue warp */
+            mbar_init(acc_empty(b), epilogue_warps(EPI)); /* one arrival per epilogue warp */
         }
         *failed = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -326,9 +330,9 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm(const __grid_constant_
                 umma_commit(acc_full(buf));
             }
         }
-    } else { /* epilogue warps 2..5: tensor-memory lanes 32 (warp % 4) .. + 31 */
-        const int quarter = warp & 3;
-        float *turn = reinterpret_cast<float *>(tail + 256) + quarter * TURN_FLOATS; /* EPI_STREAM only */
+    } else { /* epilogue warps 2..5 (2..9): tensor-memory lanes 32 (warp % 4) .. + 31 */
+        const int quarter = warp & 3, share = (warp - 2) >> 2; /* eight warps: every other 32 columns each */
+        float *turn = reinterpret_cast<float *>(tail + 256) + (quarter + 4 * share) * TURN_FLOATS; /* EPI_STREAM, EPI_STREAMS only */
         uint32_t it = 0;
         for (int u = blockIdx.x; u < units; u += gridDim.x, it++) {
             const uint32_t buf = it & 1;
@@ -344,7 +348,7 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm(const __grid_constant_
             const int row = m0 + quarter * 32 + lane;
             const bool live = row < a.rows;
 #pragma unroll 1
-            for (int c = 0; c < un.width / 32; c++) {
+            for (int c = share; c < un.width / 32; c += epilogue_warps(EPI) / 4) {
                 float v[32];
                 tmem_load32(tmem + ((uint32_t)(quarter * 32) << 16) + buf * BN + c * 32, v);
                 if (EPI == EPI_STREAM) {
@@ -393,7 +397,7 @@ constexpr bool PAIR_BY_DEFAULT = true;
  * tiles fit one round (64). Of an MMA's NMMA W rows each block stages NMMA / 2. */
 template <int NMMA, int NSUB, int EPI> struct Pair {
     static constexpr int WIDTH = NMMA * NSUB;
-    static constexpr int TURN_BYTES = writes_stream(EPI) ? 4 * TURN_FLOATS * 4 : 0; /* the stream update's staging */
+    static constexpr int TURN_BYTES = turn_bytes(EPI); /* the stream update's staging */
     static constexpr int SUB_BYTES = (NMMA / 2) * KBLK * 2;        /* this block's W rows of one MMA */
     static constexpr int B_BYTES = NSUB * SUB_BYTES;
     static constexpr int STAGE_BYTES = A_BYTES + B_BYTES;          /* 32 KB (256 wide) or 36 KB (320 wide) */
@@ -453,7 +457,7 @@ template <int WIDTH> static __device__ __forceinline__ Unit pair_unit_of(int u, 
 }
 
 template <int NMMA, int NSUB, int EPI>
-__global__ void __launch_bounds__(THREADS, 1) k_tile_gemm_pair(const __grid_constant__ CUtensorMap map_x,
+__global__ void __launch_bounds__(threads_of(EPI), 1) k_tile_gemm_pair(const __grid_constant__ CUtensorMap map_x,
                                                                const __grid_constant__ CUtensorMap map_w,
                                                                const __grid_constant__ CUtensorMap map_w_half, const TileArgs a) {
     using P = Pair<NMMA, NSUB, EPI>;
@@ -487,7 +491,7 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm_pair(const __grid_cons
         }
         for (int b = 0; b < 2; b++) {
             mbar_init(acc_full(b), 1);
-            mbar_init(acc_empty(b), 8); /* four epilogue warps in each block */
+            mbar_init(acc_empty(b), 2 * epilogue_warps(EPI)); /* the epilogue warps of each block */
         }
         *failed = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -579,9 +583,9 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm_pair(const __grid_cons
                 umma_commit_pair(acc_full(buf));
             }
         }
-    } else { /* epilogue warps 2..5 of both blocks: this block's tensor-memory lanes 32 (warp % 4) .. + 31 */
-        const int quarter = warp & 3;
-        float *turn = reinterpret_cast<float *>(tail + 256) + quarter * TURN_FLOATS; /* EPI_STREAM only */
+    } else { /* epilogue warps 2..5 (2..9) of both blocks: this block's tensor-memory lanes 32 (warp % 4) .. + 31 */
+        const int quarter = warp & 3, share = (warp - 2) >> 2; /* eight warps: every other 32 columns each */
+        float *turn = reinterpret_cast<float *>(tail + 256) + (quarter + 4 * share) * TURN_FLOATS; /* EPI_STREAM, EPI_STREAMS only */
         uint32_t it = 0;
         for (int u = pair; u < units; u += n_pairs, it++) {
             const uint32_t buf = acc_of(it);
@@ -597,7 +601,7 @@ __global__ void __launch_bounds__(THREADS, 1) k_tile_gemm_pair(const __grid_cons
             const int row = m0 + quarter * 32 + lane;
             const bool live = row < a.rows;
 #pragma unroll 1
-            for (int c = 0; c < un.width / 32; c++) {
+            for (int c = share; c < un.width / 32; c += epilogue_warps(EPI) / 4) {
                 float v[32];
                 tmem_load32(tmem + ((uint32_t)(quarter * 32) << 16) + buf * WIDTH + c * 32, v);
                 if (EPI == EPI_STREAM) {
@@ -654,7 +658,7 @@ int launch(const CUtensorMap &map_x, const CUtensorMap &map_w, const CUtensorMap
     a.split_from = (BN == 256 && tiles > sms && rest > 0 && 2 * rest <= sms) ? tiles - rest : tiles;
     cudaLaunchConfig_t config = {};
     config.gridDim = dim3(tiles < sms ? tiles : sms);
-    config.blockDim = dim3(THREADS);
+    config.blockDim = dim3(threads_of(EPI));
     config.dynamicSmemBytes = Tile<BN>::smem_bytes(EPI);
     config.stream = stream;
     cudaLaunchAttribute attribute[1];
@@ -741,7 +745,7 @@ int launch_pair(const CUtensorMap &map_x, const CUtensorMap &map_w, const CUtens
     a.split_from = (NSUB == 1 && tiles > pairs && rest > 0 && 2 * rest <= pairs) ? tiles - rest : tiles;
     cudaLaunchConfig_t config = {};
     config.gridDim = dim3(2 * (tiles < pairs ? tiles : pairs));
-    config.blockDim = dim3(THREADS);
+    config.blockDim = dim3(threads_of(EPI));
     config.dynamicSmemBytes = P::SMEM_BYTES;
     config.stream = stream;
     cudaLaunchAttribute attribute[2];
