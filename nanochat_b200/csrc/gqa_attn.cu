@@ -79,9 +79,9 @@ template <typename T> __device__ __forceinline__ void head_row(const ncb_gqa &a,
 constexpr int RUN = 16; /* consecutive rows a warp of k_gqa_rows works on */
 
 /* Shared memory per warp of k_gqa_rows: the projected rows with the taps before them, the convolution's weights (CONV_BATCH of
- * them, zero past the taps), a head's row, the rows' places. */
+ * them, zero past the taps), two of a head's rows, the rows' places. */
 __host__ __device__ inline size_t rows_smem(int size, int itemsize) {
-    return (size_t)(RUN + CONV_BATCH - 1) * size * itemsize + (size_t)CONV_BATCH * size * 4 + (size_t)size * 4 + RUN * sizeof(Place) + 8;
+    return (size_t)(RUN + CONV_BATCH - 1) * size * itemsize + (size_t)CONV_BATCH * size * 4 + (size_t)2 * size * 4 + RUN * sizeof(Place) + 8;
 }
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void *src, bool on) { /* 16 bytes, zeros when off */
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
@@ -90,7 +90,7 @@ __device__ __forceinline__ void cp_async16(uint32_t dst, const void *src, bool o
 /* Grid (units / warps rounded up, rows / RUN rounded up), a warp per unit and run of rows: the query heads, then with own_kv the
  * key and the value heads. q NULL: the query heads only keep their ring. A loop over the rows with a short body: the kernel has
  * many warps, and what is unrolled far has to be fetched by each of them. */
-template <typename T> __global__ void __launch_bounds__(THREADS) k_gqa_rows(const ncb_gqa a) {
+template <typename T> __global__ void __launch_bounds__(THREADS, 7) k_gqa_rows(const ncb_gqa a) {
     extern __shared__ __align__(128) uint8_t raw[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, unit = blockIdx.x * (blockDim.x >> 5) + warp;
     const int H = a.heads, G = a.own_kv ? a.kv_heads : 0, row0 = blockIdx.y * RUN, n = (int)min((long long)RUN, a.conv.rows - row0);
@@ -99,8 +99,8 @@ template <typename T> __global__ void __launch_bounds__(THREADS) k_gqa_rows(cons
     uint8_t *mine = raw + warp * ((rows_smem(largest, sizeof(T)) + 15) / 16 * 16);
     T *tile = reinterpret_cast<T *>(mine);                                  /* [OLD + RUN][size] */
     float *w = reinterpret_cast<float *>(tile + (OLD + RUN) * largest);     /* [CONV_BATCH][size], by how far back */
-    float *x = w + CONV_BATCH * largest;                                    /* [size] */
-    Place *place = reinterpret_cast<Place *>(x + largest);
+    float *x = w + CONV_BATCH * largest;                                    /* [2][size] */
+    Place *place = reinterpret_cast<Place *>(x + 2 * largest);
     asm volatile("griddepcontrol.wait;" ::: "memory");
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     if (unit >= H + 2 * G) return;
@@ -133,13 +133,95 @@ template <typename T> __global__ void __launch_bounds__(THREADS) k_gqa_rows(cons
     __syncwarp();
     const int half = a.rot / 2;
     const float inv_count = 1.f / (float)a.norm_count;
+    auto norm_scale = [&](float sum) { return sizeof(T) == 2 ? rsqrtf(fmaf(sum, inv_count, a.eps)) : 1.f / sqrtf(sum / (float)a.norm_count + a.eps); };
+    if (a.keep)
+        for (int r = 0; r < n; r++)
+            if (place[r].pos >= 0)
+                for (int i = 2 * lane; i < size; i += 64) keep2<T>(a.conv, row0 + r, place[r], ch0 + i);
+    if (query && !a.q) return;
+    if (size <= 128) { /* four channels per lane: two rows at a time, weights and older taps in registers */
+        const int i = 4 * lane;
+        const bool on = i < size;
+        /* lane r: where row r goes (NULL: nowhere) and its position */
+        int pos = -1;
+        T *to = nullptr;
+        if (lane < n) {
+            const Place at = place[lane];
+            pos = at.pos;
+            if (pos >= 0) to = query ? (T *)a.q + ((size_t)(row0 + lane) * H + unit) * a.dim : cache_row<T>(a, at.slot, kvh, pos) + (key ? 0 : a.dim);
+        }
+        float4 f[CONV_BATCH], v[OLD + 2];
+#pragma unroll
+        for (int back = 0; back < CONV_BATCH; back++) f[back] = on ? load4(w + back * size + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int j = 0; j < OLD; j++) v[j] = on ? load4(tile + j * size + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 1
+        for (int r = 0; r < n; r += 2) {
+            T *out[2];
+            float4 y[2];
+#pragma unroll
+            for (int e = 0; e < 2; e++) {
+                out[e] = reinterpret_cast<T *>(__shfl_sync(0xffffffffu, reinterpret_cast<unsigned long long>(to), r + e));
+                v[OLD + e] = on ? load4(tile + (min(r + e, n - 1) + OLD) * size + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+                y[e] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+                for (int back = 0; back < CONV_BATCH; back++) {
+                    const float4 c = f[back], u = v[OLD + e - back];
+                    y[e].x = fmaf(c.x, u.x, y[e].x), y[e].y = fmaf(c.y, u.y, y[e].y), y[e].z = fmaf(c.z, u.z, y[e].z), y[e].w = fmaf(c.w, u.w, y[e].w);
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < OLD; j++) v[j] = v[j + 2];
+            if (special >> r & 3)
+                for (int e = 0; e < 2; e++)
+                    if ((special >> (r + e) & 1) && out[e] && on) {
+                        const float2 lo = conv2<T>(a.conv, row0 + r + e, place[r + e], ch0 + i), hi = conv2<T>(a.conv, row0 + r + e, place[r + e], ch0 + i + 2);
+                        const float4 z = make_float4(lo.x, lo.y, hi.x, hi.y);
+                        if (e) y[1] = z;
+                        else y[0] = z;
+                    }
+            if (!query && !key) {
+#pragma unroll
+                for (int e = 0; e < 2; e++)
+                    if (out[e] && on) store4(out[e] + i, y[e]);
+                continue;
+            }
+            if (half) {
+                if (on) *reinterpret_cast<float4 *>(x + i) = y[0], *reinterpret_cast<float4 *>(x + size + i) = y[1];
+                __syncwarp();
+                const int p0 = max(__shfl_sync(0xffffffffu, pos, r), 0), p1 = max(__shfl_sync(0xffffffffu, pos, r + 1), 0);
+                for (int j = lane; j < 2 * half; j += 32) { /* in place: a pair belongs to one lane */
+                    const bool second = j >= half;
+                    const int d = second ? j - half : j;
+                    const size_t at = (size_t)(second ? p1 : p0) * half + d;
+                    float *row = x + (second ? size : 0) + d;
+                    const float c = a.cos[at], s = a.sin[at], u = row[0], z = row[half];
+                    row[0] = u * c - z * s;
+                    row[half] = z * c + u * s;
+                }
+                __syncwarp();
+                if (on) y[0] = load4(x + i), y[1] = load4(x + size + i);
+            }
+            /* both rows' sums of squares in one reduction: a half of the warp each */
+            float sq[2];
+#pragma unroll
+            for (int e = 0; e < 2; e++) sq[e] = fmaf(y[e].x, y[e].x, fmaf(y[e].y, y[e].y, fmaf(y[e].z, y[e].z, y[e].w * y[e].w)));
+            float sum = (lane & 16 ? sq[1] : sq[0]) + __shfl_xor_sync(0xffffffffu, lane & 16 ? sq[0] : sq[1], 16);
+#pragma unroll
+            for (int o = 8; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+            const float scale = norm_scale(sum);
+#pragma unroll
+            for (int e = 0; e < 2; e++) {
+                const float g = __shfl_sync(0xffffffffu, scale, 16 * e);
+                if (out[e] && on) store4(out[e] + i, make_float4(y[e].x * g, y[e].y * g, y[e].z * g, y[e].w * g));
+            }
+        }
+        return;
+    }
 #pragma unroll 1
     for (int r = 0; r < n; r++) {
         const Place at = place[r];
         if (at.pos < 0) continue;
-        if (a.keep)
-            for (int i = 2 * lane; i < size; i += 64) keep2<T>(a.conv, row0 + r, at, ch0 + i);
-        if (query && !a.q) continue;
         T *out = query ? (T *)a.q + ((size_t)(row0 + r) * H + unit) * a.dim : cache_row<T>(a, at.slot, kvh, at.pos) + (key ? 0 : a.dim);
         for (int i = 4 * lane; i < size; i += 128) {
             float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -170,7 +252,7 @@ template <typename T> __global__ void __launch_bounds__(THREADS) k_gqa_rows(cons
             sum = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, sum))));
         }
         for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-        const float f = sizeof(T) == 2 ? rsqrtf(fmaf(sum, inv_count, a.eps)) : 1.f / sqrtf(sum / (float)a.norm_count + a.eps);
+        const float f = norm_scale(sum);
         for (int i = 4 * lane; i < size; i += 128) {
             const float4 v = *reinterpret_cast<const float4 *>(x + i);
             store4(out + i, make_float4(v.x * f, v.y * f, v.z * f, v.w * f));
